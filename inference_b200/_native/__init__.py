@@ -13,6 +13,7 @@ from pathlib import Path
 _DIR = Path(__file__).resolve().parent
 _KERNELS = None
 _HOST = None
+_TEXT_ONLY = False
 
 
 class NativeLibraryMissing(RuntimeError):
@@ -32,10 +33,20 @@ def _load(name: str, builder: str):
     return ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
 
 
+def prefer_text_kernels() -> None:
+    """For programs that only decode text: when the full kernel library has not been built, build and load the text
+    decoders' units alone."""
+    global _TEXT_ONLY
+    _TEXT_ONLY = True
+
+
 def kernels() -> ctypes.CDLL:
     global _KERNELS
     if _KERNELS is None:
-        _KERNELS = _load("libswb200_kernels.so", "build_kernels")
+        if _TEXT_ONLY and not (_DIR / "libswb200_kernels.so").exists():
+            _KERNELS = _load("libswb200_text.so", "build_text")
+        else:
+            _KERNELS = _load("libswb200_kernels.so", "build_kernels")
         _declare_kernels(_KERNELS)
     return _KERNELS
 
@@ -79,6 +90,25 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
     sig("swb_rope_kv_write", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
                               c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                               c_void_p])
+    sig("swb_rope_kv_write_ex", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
+                                 c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                 c_int, c_void_p])
+    sig("swb_stream_norm", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p,
+                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                            c_float, c_int, c_void_p])
+    sig("swb_stream_embed", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int,
+                             c_int, c_int, c_void_p])
+    sig("swb_moe_table_plan", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_void_p])
+    sig("swb_gemm_grouped_rows", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                  c_int, c_int, c_void_p])
+    sig("swb_gemm_f32", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                         c_int, c_void_p])
+    sig("swb_attn_simple", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p])
+    sig("swb_attn_ext", [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_int, c_int, c_int,
+                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
+                         c_int, c_int, c_void_p, c_size_t, c_void_p])
     sig("swb_gated_act_mul", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_embedding", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
     sig("swb_gated_residual", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p])

@@ -3,11 +3,14 @@
 `libswb200_kernels.so` holds every CUDA kernel, compiled by nvcc for sm_100a only; `libswb200_host.so`
 holds the C++ host policy (scheduler, paging, prefix index, speculative math, sampler, constraint,
 checkpoint readers). Both are plain C-ABI shared objects loaded with ctypes, so they carry no
-dependency on the PyTorch headers and rebuild in seconds.
+dependency on the PyTorch headers and rebuild in seconds. `libswb200_text.so` holds the kernel units of the text
+decoders alone, for programs that build on first use and need no others.
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import contextlib
+import fcntl
 import os
 import shutil
 import subprocess
@@ -28,6 +31,21 @@ NVCC_FLAGS = [
     "-I", str(CSRC / "include"), "-I", str(CSRC / "kernels"),
 ]
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-I", str(CSRC / "include"), "-I", str(CSRC / "host")]
+
+
+# kernel units of the paged text decoders (bf16 and 32-bit), their sampling and step metadata
+TEXT_UNITS = ("api_gemm", "argmax_static", "attention", "attention_decode_tma", "attention_tcgen05", "decode_meta", "f32_ops",
+              "gemm_decode_cluster", "gemm_tcgen05", "llm_ops", "moe_routed", "sample_device", "sampling", "status",
+              "stream_ops")
+
+
+@contextlib.contextmanager
+def _build_lock():
+    """One build at a time per checkout (several processes may find the library missing)."""
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
 
 
 def _newer(src: Path, dst: Path, deps: list[Path]) -> bool:
@@ -61,17 +79,26 @@ def _compile_all(srcs: list[Path], headers: list[Path], compiler: list[str], tag
 
 
 def build_kernels(force: bool = False, verbose_ptxas: bool = False) -> Path:
-    srcs = sorted((CSRC / "kernels").glob("*.cu"))
+    return _build_kernel_lib(sorted((CSRC / "kernels").glob("*.cu")), OUT / "libswb200_kernels.so", force, verbose_ptxas)
+
+
+def build_text(force: bool = False) -> Path:
+    return _build_kernel_lib([CSRC / "kernels" / f"{u}.cu" for u in TEXT_UNITS], OUT / "libswb200_text.so", force)
+
+
+def _build_kernel_lib(srcs: list[Path], lib: Path, force: bool, verbose_ptxas: bool = False) -> Path:
     headers = (sorted((CSRC / "kernels").glob("*.cuh")) + sorted((CSRC / "kernels").glob("*.h")) +
                sorted((CSRC / "include").glob("*.h")))
     flags = list(NVCC_FLAGS)
     if verbose_ptxas:
         flags += ["-Xptxas", "-v"]
         os.environ["SWB_BUILD_VERBOSE"] = "1"
-    objs = _compile_all(srcs, headers, [NVCC, *flags], "k", force or verbose_ptxas)
-    lib = OUT / "libswb200_kernels.so"
-    if force or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
-        _run([NVCC, "-shared", "-o", str(lib), *map(str, objs), "-lcudart"])
+    with _build_lock():
+        objs = _compile_all(srcs, headers, [NVCC, *flags], "k", force or verbose_ptxas)
+        if force or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in objs):
+            tmp = lib.with_suffix(f".{os.getpid()}.tmp")
+            _run([NVCC, "-shared", "-o", str(tmp), *map(str, objs), "-lcudart"])
+            os.replace(tmp, lib)
     return lib
 
 

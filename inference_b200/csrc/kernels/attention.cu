@@ -516,6 +516,7 @@ int swb_attn_paged(const void* q, long long q_stride_tok, int q_stride_head, voi
   p.softcap = softcap;
   p.causal = causal;
   p.num_splits = 1;
+  p.k_dim = p.v_dim = HD;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (mode == 0) {
     dim3 grid((max_q_len + 63) / 64, Hq, num_seqs);
@@ -597,6 +598,67 @@ int swb_attn_paged_prefill_tc(const void* q, long long q_stride_tok, int q_strid
                                    num_seqs, max_q_len, max_q_len, Hq, Hkv, scale, reinterpret_cast<cudaStream_t>(stream),
                                    nullptr, 0, 0, 0, 0, 0, causal, cu_q, total_tokens, 128, kv_lens, block_table,
                                    max_blocks, block_size, num_blocks);
+}
+
+// Attention with per-tensor head widths, chunked masking and sinks over the paged cache (kcache [num_blocks, Hkv,
+// block_size, D], vcache [num_blocks, Hkv, block_size, Dv], contiguous) or, with block_table == nullptr, over fresh keys
+// and values in strided rows of one flat token axis (prefill only). q [total_tokens, Hq, D] rows of stride q_stride_tok
+// (heads contiguous), out [total_tokens, Hq, Dv]. chunk > 0: query i sees key j <= i only if floor(i / chunk) ==
+// floor(j / chunk), positions counted from the sequence's start. sink (nullable fp32 [Hq]): exp(sink[h]) joins the softmax
+// denominator. Widths: multiples of 8 up to 128. mode 0 = prefill (tcgen05 kernel, sequences from cu_q), 1 = decode
+// (TMA-fed kernel, block_size 16, max_q_len * Hq / Hkv <= 16, uniform q_len when cu_q is null). Returns -3 when the
+// problem is outside the two kernels' reach.
+int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long k_stride_tok, const void* v,
+                 long long v_stride_tok, void* out, long long out_stride_tok, const int* block_table, int max_blocks,
+                 int block_size, int num_blocks, const int* cu_q, const int* kv_lens, int num_seqs, int max_q_len,
+                 int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink, int mode,
+                 int num_splits, void* workspace, size_t workspace_bytes, void* stream) {
+  using namespace swb;
+  if (num_seqs <= 0 || total_tokens <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (Hkv <= 0 || Hq % Hkv != 0 || max_q_len <= 0) return -3;
+  if (mode == 0)
+    return attn_ext_tcgen05_launch(q, q_stride_tok, k, k_stride_tok, v, v_stride_tok, out, out_stride_tok, num_seqs,
+                                   max_q_len, total_tokens, Hq, Hkv, D, Dv, scale, chunk, sink, cu_q, kv_lens,
+                                   block_table, max_blocks, block_size, num_blocks, st);
+  if (D < 8 || Dv < 8 || D > HD || Dv > HD || (D % 8) || (Dv % 8) || block_size != 16 || !block_table || !kv_lens ||
+      num_blocks <= 0 || max_q_len * (Hq / Hkv) > 16 || !(scale > 0.f) || chunk < 0 || (q_stride_tok % 8))
+    return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -3;
+  AttnParams p{};
+  p.q = reinterpret_cast<const bf16*>(q);
+  p.q_stride_tok = q_stride_tok;
+  p.q_stride_head = D;
+  p.out = reinterpret_cast<bf16*>(out);
+  p.out_stride_tok = out_stride_tok;
+  p.k = reinterpret_cast<const bf16*>(k);
+  p.v = reinterpret_cast<const bf16*>(v);
+  p.block_table = block_table;
+  p.max_blocks = max_blocks;
+  p.block_size = block_size;
+  p.cu_q = cu_q;
+  p.kv_lens = kv_lens;
+  p.uniform_q_len = max_q_len;
+  p.num_seqs = num_seqs;
+  p.Hq = Hq;
+  p.Hkv = Hkv;
+  p.G = Hq / Hkv;
+  p.scale = scale;
+  p.causal = 1;
+  p.k_dim = D;
+  p.v_dim = Dv;
+  p.chunk = chunk;
+  p.sink = sink;
+  if (num_splits < 1) num_splits = 1;
+  if (num_splits > 32) num_splits = 32;
+  p.num_splits = num_splits;
+  if (num_splits > 1) {
+    if (!workspace || workspace_bytes < swb_attn_decode_workspace_bytes(num_seqs, Hkv, num_splits)) return -5;
+    p.part_o = reinterpret_cast<float*>(reinterpret_cast<char*>(workspace) + attn_counter_bytes(num_seqs, Hkv));
+    p.part_ml = p.part_o + (size_t)num_seqs * Hkv * num_splits * 16 * HD;
+    p.split_counters = reinterpret_cast<int*>(workspace);
+  }
+  return attn_decode_tma_launch(p, num_blocks, st);
 }
 
 // 0: pick the tcgen05 kernel whenever it supports the problem; 1: always the mma.sync kernel (comparison runs).

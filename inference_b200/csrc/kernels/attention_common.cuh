@@ -35,6 +35,10 @@ struct AttnParams {
   float* part_ml;
   int cluster_merge;     // the splits of a (sequence, kv head) are one thread-block cluster (num_splits <= 8)
   int* split_counters;   // [num_seqs * Hkv] zero between launches: in-kernel merge by the last split to arrive (TMA kernel)
+  // TMA decode kernel only
+  int k_dim, v_dim;      // head widths of q / k and of v / out (multiples of 8, <= HD)
+  int chunk;             // > 0: a query sees only keys of its own chunk, floor(i / chunk) == floor(j / chunk)
+  const float* sink;     // optional [Hq]: exp(sink[h]) joins the softmax denominator
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, uint32_t src_bytes) {
@@ -86,4 +90,9 @@ int attn_dense_tcgen05_launch(const void* q, long long q_stride_tok, int q_strid
                               int col_offset = 0, int causal = 0, const int* cu_q = nullptr, int total_tokens = 0,
                               int head_dim = 128, const int* kv_lens = nullptr, const int* block_table = nullptr,
                               int max_blocks = 0, int block_size = 0, int num_blocks = 0);
+int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, long long k_stride_tok, const void* v,
+                            long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
+                            int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
+                            const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
+                            int num_blocks, cudaStream_t stream);
 }  // namespace swb

@@ -1,4 +1,5 @@
-// Decode attention over the paged KV cache with TMA-fed, warp-specialised CTAs (block_size 16, head_dim 128).
+// Decode attention over the paged KV cache with TMA-fed, warp-specialised CTAs (block_size 16, head widths up to 128:
+// columns past the width of q / k or v are zero fill of the tensor maps, whole 64-column halves past it are not fetched).
 //
 // One CTA per (KV split, kv head, sequence). Warp 4 is the producer: for every 64-token tile it looks up
 // the four 16-token blocks in the block table and issues one tiled TMA copy per (block, K|V, 64-column
@@ -40,6 +41,17 @@ __device__ __forceinline__ uint32_t tma_tile_off(int tok, int c) {
 // Q rows are written by ordinary stores with the simple XOR swizzle of the other kernels.
 __device__ __forceinline__ uint32_t q_off(int r, int c) { return (uint32_t)(r * 256 + ((c ^ (r & 7)) << 4)); }
 
+// 1 / softmax denominator of a row with running max M (log2 units) and sum L relative to it; the numerators are relative
+// to M as well. A sink adds exp(sink) to the denominator; one far above every score makes the weights vanish.
+__device__ __forceinline__ float softmax_inv(const AttnParams& p, int head, float M, float L) {
+  if (p.sink) {
+    const float sk = p.sink[head] * 1.4426950408889634f;
+    const float top = fmaxf(sk, M), e = exp2f(M - top);
+    return e / (L * e + exp2f(sk - top));
+  }
+  return L > 0.f ? 1.f / L : 0.f;
+}
+
 __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                               const __grid_constant__ CUtensorMap tmap_v,
                                                               const AttnParams p) {
@@ -76,16 +88,20 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   const int kv_len = p.kv_lens[seq];
   const int nrows = min(16, q_len * p.G);
   const int causal_shift = kv_len - q_len;
+  // chunked attention starts at the tile that holds the first key of the first query's chunk
+  const int tile_lo = p.chunk > 0 ? max(causal_shift, 0) / p.chunk * p.chunk / KV_TILE : 0;
   const int total_tiles = (kv_len + KV_TILE - 1) / KV_TILE;
-  const int per = (total_tiles + p.num_splits - 1) / p.num_splits;
-  const int t0 = split * per;
+  const int per = (total_tiles - tile_lo + p.num_splits - 1) / p.num_splits;
+  const int t0 = tile_lo + split * per;
   const int n_tiles = max(0, min(total_tiles, t0 + per) - t0);
+  const int k_steps = (p.k_dim + 15) >> 4, v_steps = (p.v_dim + 15) >> 4;   // 16-column MMA steps that hold data
+  const int k_halves = (p.k_dim + 63) >> 6, v_halves = (p.v_dim + 63) >> 6;
 
   // Q rows -> shared (row r = query token r / G, head kvh * G + r % G), zero rows past nrows
   for (int idx = threadIdx.x; idx < 256; idx += blockDim.x) {
     const int row = idx >> 4, c = idx & 15;
     uint4 val = make_uint4(0, 0, 0, 0);
-    if (row < nrows) {
+    if (row < nrows && c * 8 < p.k_dim) {
       const int qtok = row / p.G, hg = row % p.G;
       val = *reinterpret_cast<const uint4*>(p.q + (size_t)(q_start + qtok) * p.q_stride_tok +
                                             (size_t)(kvh * p.G + hg) * p.q_stride_head + c * 8);
@@ -113,7 +129,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         outstanding &= ~(1u << stage);
         uint8_t* sK = ring + stage * STAGE_BYTES;
         uint8_t* sV = sK + TILE_BYTES;
-        mbar_arrive_expect_tx(&bar_full[stage], STAGE_BYTES);
+        mbar_arrive_expect_tx(&bar_full[stage], (uint32_t)(k_halves + v_halves) * 4 * 2048);
         const int tok0 = (t0 + j) * KV_TILE;
 #pragma unroll
         for (int b = 0; b < 4; ++b) {
@@ -122,9 +138,9 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           const int blk = tstart < kv_len ? __ldg(&table[tstart >> 4]) : first_block;
           const int row0 = (blk * p.Hkv + kvh) * 16;
           tma_load_2d(sK + (b * 2 + 0) * 2048, &tmap_k, &bar_full[stage], 0, row0);
-          tma_load_2d(sK + (b * 2 + 1) * 2048, &tmap_k, &bar_full[stage], 64, row0);
+          if (k_halves > 1) tma_load_2d(sK + (b * 2 + 1) * 2048, &tmap_k, &bar_full[stage], 64, row0);
           tma_load_2d(sV + (b * 2 + 0) * 2048, &tmap_v, &bar_full[stage], 0, row0);
-          tma_load_2d(sV + (b * 2 + 1) * 2048, &tmap_v, &bar_full[stage], 64, row0);
+          if (v_halves > 1) tma_load_2d(sV + (b * 2 + 1) * 2048, &tmap_v, &bar_full[stage], 64, row0);
         }
         outstanding |= 1u << stage;
         issue_phase = (issue_phase & ~(1u << stage)) | (phase << stage);
@@ -162,6 +178,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       for (int i = 0; i < 2; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
       for (int kk = 0; kk < 8; ++kk) {
+        if (kk >= k_steps) break;
         const int mi = lane >> 3;
         const int tok = warp * 16 + (mi >> 1) * 8 + (lane & 7);
         uint32_t b0, b1, b2, b3;
@@ -178,7 +195,9 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           const int col = tok_base + nt * 8 + t4 * 2 + (e & 1);
           const int row = g + ((e >> 1) ? 8 : 0);
           const int qtok = row / p.G;
-          const bool ok = (col < kv_len) && (!p.causal || col <= qtok + causal_shift);
+          const int qpos = qtok + causal_shift;
+          const bool ok = (col < kv_len) && (!p.causal || col <= qpos) &&
+                          (p.chunk <= 0 || col >= qpos / p.chunk * p.chunk);
           s[nt][e] = ok ? val : -INFINITY;
         }
       }
@@ -215,6 +234,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         a[3] = pack_bf16(s[1][2], s[1][3]);
 #pragma unroll
         for (int dp = 0; dp < 8; ++dp) {
+          if (dp >= v_steps) break;
           const int mi = lane >> 3;
           const int tok = warp * 16 + (mi & 1) * 8 + (lane & 7);
           uint32_t b0, b1, b2, b3;
@@ -271,9 +291,10 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       }
       const int qtok = row / p.G, hg = row % p.G;
       if (p.num_splits == 1) {
-        const float inv = L > 0.f ? 1.f / L : 0.f;
-        p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * HD + d] =
-            __float2bfloat16(acc * inv);
+        const float inv = softmax_inv(p, kvh * p.G + hg, M, L);
+        if (d < p.v_dim)
+          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] =
+              __float2bfloat16(acc * inv);
       } else {
         const size_t base = (((size_t)seq * p.Hkv + kvh) * p.num_splits + split) * 16 + row;
         p.part_o[base * HD + d] = acc;
@@ -336,11 +357,11 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         sSc[row * 32 + sp] = sc;
         L += sc * sL[row * 32 + sp];
       }
-      const float inv = L > 0.f ? 1.f / L : 0.f;
+      const float inv = softmax_inv(p, kvh * p.G + row % p.G, M, L);
       for (int sp = 0; sp < S; ++sp) sSc[row * 32 + sp] *= inv;
     }
     __syncthreads();
-    if (threadIdx.x < 128) {
+    if ((int)threadIdx.x < p.v_dim) {
       const int d = threadIdx.x;
       if (small) {
 #pragma unroll
@@ -351,7 +372,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
             for (int sp = 0; sp < 8; ++sp)
               if (sp < S) acc += sSc[row * 32 + sp] * po[row][sp];
             const int qtok = row / p.G, hg = row % p.G;
-            p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * HD + d] = __float2bfloat16(acc);
+            p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] = __float2bfloat16(acc);
           }
         }
       } else {
@@ -361,7 +382,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           for (int sp = 0; sp < S; ++sp)
             acc += sSc[row * 32 + sp] * __ldcg(p.part_o + (base0 + (size_t)sp * 16 + row) * HD + d);
           const int qtok = row / p.G, hg = row % p.G;
-          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * HD + d] = __float2bfloat16(acc);
+          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] = __float2bfloat16(acc);
         }
       }
     }
@@ -384,9 +405,9 @@ int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t str
   }
   CUtensorMap tk, tv;
   const int rows = num_blocks * p.Hkv * 16;
-  int rc = make_tmap_bf16_2d(&tk, p.k, rows, HD, HD, 16);
+  int rc = make_tmap_bf16_2d(&tk, p.k, rows, p.k_dim, p.k_dim, 16);
   if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tv, p.v, rows, HD, HD, 16);
+  rc = make_tmap_bf16_2d(&tv, p.v, rows, p.v_dim, p.v_dim, 16);
   if (rc) return rc;
   dim3 grid(p.num_splits, p.Hkv, p.num_seqs);
   if (p.num_splits > 1 && p.num_splits <= 8 && p.split_counters) {

@@ -75,6 +75,10 @@ struct FaParams {
   const int* kv_lens;
   const int* block_table;
   int max_blocks, block_size;
+  // Extended problems (the EXT instantiations only):
+  int chunk;           // > 0: query i sees key j <= i only if floor(i / chunk) == floor(j / chunk), positions of the sequence
+  const float* sink;   // optional [Hq]: exp(sink[h]) joins the softmax denominator (no key, no value, not scaled)
+  int v_dim;           // width of the v heads and of the output heads (<= HD; the tile is zero filled beyond it)
 };
 
 __device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, uint64_t* bar, int c0, int c1, int c2,
@@ -159,7 +163,9 @@ struct Barriers {
 
 // 168 registers per thread is the cap for ten warps: two of the four scheduler partitions hold three warps, and a
 // partition's file is 16 K registers (a build with 200 registers per thread does not launch).
-template <int HD>
+// EXT adds chunked masking, attention sinks and head widths below the tile width HD (q . k and P V then run over zero
+// columns that the tensor maps fill in).
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_v, const FaParams p) {
@@ -182,7 +188,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   if (q_base >= q_len || kv_len <= 0) return;   // uniform for the whole CTA, before any barrier or TMEM allocation
   const int kv_head = head / (p.Hq / p.Hkv);
   const int kv_end = p.causal ? min(kv_len, q_base + p.tiles * BM + coff) : kv_len;
-  const int n_tiles = (kv_end + BN - 1) / BN;
+  // first key tile that any row of this CTA sees (rows are ascending, so the first row's chunk starts lowest)
+  const int j0 = (EXT && p.chunk > 0) ? (q_base + coff) / p.chunk * p.chunk / BN : 0;
+  const int n_tiles = (kv_end + BN - 1) / BN - j0;
   volatile int* abort_flag = &bars->abort;
 
   if (threadIdx.x == 0) {
@@ -232,7 +240,8 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const int* pages = paged ? p.block_table + (long long)blockIdx.z * p.max_blocks : nullptr;
       const int per_tile = paged ? BN / p.block_size : 1, last_page = paged ? (kv_len - 1) / p.block_size : 0;
       const uint32_t page_bytes = paged ? (uint32_t)p.block_size * 128u : 0u;
-      auto load_tile = [&](uint32_t dst_off, const CUtensorMap* map, uint64_t* bar, int j) {
+      auto load_tile = [&](uint32_t dst_off, const CUtensorMap* map, uint64_t* bar, int jrel) {
+        const int j = jrel + j0;
         if (!paged) {
           for (int a = 0; a < ATOMS; ++a)
             tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * 64, kv_head, tok0 + j * BN, batch);
@@ -340,11 +349,20 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       tmem_ld_wait();
       // keys past the sequence (zero fill, or the next sequence of a packed batch) and, when causal, keys after the
       // query position never contribute
-      if ((j + 1) * BN > kv_len || (p.causal && (j + 1) * BN > q_base + q * BM + coff)) {
+      const int key0 = (j + j0) * BN;
+      if (key0 + BN > kv_len || (p.causal && key0 + BN > q_base + q * BM + coff)) {
         const int last_key = p.causal ? min(kv_len - 1, row + coff) : kv_len - 1;
 #pragma unroll
         for (int i = 0; i < BN; ++i)
-          if (j * BN + i > last_key) s[i] = __float_as_uint(-INFINITY);
+          if (key0 + i > last_key) s[i] = __float_as_uint(-INFINITY);
+      }
+      if constexpr (EXT) {   // keys of earlier chunks; only tiles below the last row's chunk start can hold any
+        if (p.chunk > 0 && key0 < (q_base + q * BM + BM - 1 + coff) / p.chunk * p.chunk) {
+          const int first_key = (row + coff) / p.chunk * p.chunk;
+#pragma unroll
+          for (int i = 0; i < BN; ++i)
+            if (key0 + i < first_key) s[i] = __float_as_uint(-INFINITY);
+        }
       }
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
 #pragma unroll
@@ -374,7 +392,8 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           }
         }
       }
-      const float neg_m = -m_used * p.scale_log2;
+      // a row whose chunk starts beyond this tile has seen no key yet: its exponentials are all zero
+      const float neg_m = (EXT && m_used == -INFINITY) ? 0.f : -m_used * p.scale_log2;
       float l0 = 0.f, l1 = 0.f;
       // (Measured alternatives for this loop, all slower on B200: every 4th / 2nd exponential as a cubic on the FMA pipe
       // -8 % / -17 %; pairs of exponentials as one bf16x2 special-function operation -6 %; three-input max with
@@ -397,7 +416,14 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     if (ok && my_tiles > 0) ok = mbar_wait(&bars->o_final, 0, abort_flag, 32 + q);
     if (ok && my_tiles > 0) {
       tc_fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if constexpr (EXT) {
+        if (p.sink) {   // join the sink in a frame whose largest exponent is zero
+          const float sk = p.sink[head] * 1.4426950408889634f, mm = m_used * p.scale_log2;
+          const float top = fmaxf(sk, mm), e = ex2(mm - top);
+          inv = e / (l * e + ex2(sk - top));
+        }
+      }
       // Stage this warp's 32 rows x HD columns in the (now idle) Q region, then write every row's HD * 2 bytes with
       // HD / 8 lanes x 16 bytes: contiguous runs for local stores and for stores that cross NVLink alike.
       // 16-byte chunk c of row r sits at c ^ (r & 7).
@@ -425,7 +451,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         const int grow = row0 + r;
         if (grow < q_len) {
           const uint4 val = *reinterpret_cast<const uint4*>(slab + r * ROW_BYTES + ((ch ^ (r & 7)) << 4));
-          bf16* dst = p.out + ((long long)batch * p.q_len + tok0 + grow) * p.out_stride_tok + (long long)head * HD;
+          if (EXT && ch * 8 >= p.v_dim) continue;
+          bf16* dst = p.out + ((long long)batch * p.q_len + tok0 + grow) * p.out_stride_tok +
+                      (long long)head * (EXT ? p.v_dim : HD);
           if (p.scatter.enabled) {
             const OutScatter& sc = p.scatter;
             const int g2 = grow - sc.split;
@@ -524,6 +552,37 @@ int make_tmap_heads(CUtensorMap* out, const void* ptr, int hd, int heads, int to
 int g_force_tiles = 0;   // 0: choose per problem; 1 / 2: fixed query tiles per CTA (comparison runs)
 void attn_dense_tcgen05_set_tiles(int tiles) { g_force_tiles = tiles; }
 
+namespace {
+
+template <int HD, bool EXT>
+int launch_fa(dim3 grid, cudaStream_t stream, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
+              const FaParams& p) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !configured[dev]) {
+    cudaError_t e = cudaFuncSetAttribute(attn_dense_tcgen05_kernel<HD, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)FaCfg<HD>::SMEM_BYTES);
+    if (e != cudaSuccess) return -(int)e;
+    configured[dev] = true;
+  }
+  return launch_kernel(attn_dense_tcgen05_kernel<HD, EXT>, grid, dim3(THREADS), FaCfg<HD>::SMEM_BYTES, stream, tq, tk, tv, p);
+}
+
+int launch_tiles(int hd, bool ext, int q_len, int Hq, int batch, cudaStream_t stream, const CUtensorMap& tq,
+                 const CUtensorMap& tk, const CUtensorMap& tv, FaParams& p) {
+  // one-tile CTAs when that shortens the schedule: a one-tile CTA takes ~0.85 of a two-tile CTA's time (measured)
+  const int sms = 148;
+  const long c2 = (long)((q_len + 2 * BM - 1) / (2 * BM)) * Hq * batch, c1 = (long)((q_len + BM - 1) / BM) * Hq * batch;
+  const double t2 = (double)((c2 + sms - 1) / sms), t1 = 0.85 * (double)((c1 + sms - 1) / sms);
+  p.tiles = (g_force_tiles == 1 || g_force_tiles == 2) ? g_force_tiles : (t1 < t2 ? 1 : 2);
+  const dim3 grid((q_len + p.tiles * BM - 1) / (p.tiles * BM), Hq, batch);
+  if (ext) return hd == 64 ? launch_fa<64, true>(grid, stream, tq, tk, tv, p) : launch_fa<128, true>(grid, stream, tq, tk, tv, p);
+  return hd == 64 ? launch_fa<64, false>(grid, stream, tq, tk, tv, p) : launch_fa<128, false>(grid, stream, tq, tk, tv, p);
+}
+
+}  // namespace
+
 // Returns 1 when the tcgen05 kernel handles this problem, 0 otherwise.
 int attn_dense_tcgen05_supported(const void* q, const void* k, const void* v, long long q_stride_tok, int q_stride_head,
                                  long long kv_stride_tok, int kv_stride_head, long long out_stride_tok, int D,
@@ -558,18 +617,6 @@ int attn_dense_tcgen05_launch(const void* q, long long q_stride_tok, int q_strid
   rc = make_tmap_heads(&tv, v, head_dim, Hkv, map_kv_tokens, paged ? num_blocks : map_batch, kv_stride_head,
                        kv_stride_tok, kv_stride_tok * map_kv_tokens, paged ? block_size : 0);
   if (rc) return rc;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_dense_tcgen05_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)FaCfg<128>::SMEM_BYTES);
-    if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_dense_tcgen05_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                               (int)FaCfg<64>::SMEM_BYTES);
-    if (e != cudaSuccess) return -(int)e;
-    configured[dev] = true;
-  }
   FaParams p{};
   p.out = reinterpret_cast<bf16*>(out);
   p.out_stride_tok = out_stride_tok;
@@ -594,15 +641,51 @@ int attn_dense_tcgen05_launch(const void* q, long long q_stride_tok, int q_strid
     p.scatter.n1 = n1;
     p.scatter.col_offset = col_offset;
   }
-  // one-tile CTAs when that shortens the schedule: a one-tile CTA takes ~0.85 of a two-tile CTA's time (measured)
-  const int sms = 148;
-  const long c2 = (long)((q_len + 2 * BM - 1) / (2 * BM)) * Hq * batch, c1 = (long)((q_len + BM - 1) / BM) * Hq * batch;
-  const double t2 = (double)((c2 + sms - 1) / sms), t1 = 0.85 * (double)((c1 + sms - 1) / sms);
-  p.tiles = (g_force_tiles == 1 || g_force_tiles == 2) ? g_force_tiles : (t1 < t2 ? 1 : 2);
-  dim3 grid((q_len + p.tiles * BM - 1) / (p.tiles * BM), Hq, batch);
-  if (head_dim == 64)
-    return launch_kernel(attn_dense_tcgen05_kernel<64>, grid, dim3(THREADS), FaCfg<64>::SMEM_BYTES, stream, tq, tk, tv, p);
-  return launch_kernel(attn_dense_tcgen05_kernel<128>, grid, dim3(THREADS), FaCfg<128>::SMEM_BYTES, stream, tq, tk, tv, p);
+  return launch_tiles(head_dim, false, q_len, Hq, batch, stream, tq, tk, tv, p);
+}
+
+// Attention over queries and keys of any head widths up to 128 (multiples of 8), with chunked masking and sinks: the
+// packed fresh-prefill form (k / v strided rows of one flat token axis) or, with block_table, the paged form (caches
+// [num_blocks, Hkv, block_size, D] and [num_blocks, Hkv, block_size, Dv]). Causal; sequences from cu_q.
+int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, long long k_stride_tok, const void* v,
+                            long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
+                            int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
+                            const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
+                            int num_blocks, cudaStream_t stream) {
+  const bool paged = block_table != nullptr;
+  if (D < 8 || Dv < 8 || D > 128 || Dv > 128 || (D % 8) || (Dv % 8) || !cu_q || Hq % Hkv || !(scale > 0.f) || chunk < 0) return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
+       reinterpret_cast<uintptr_t>(out)) & 15)
+    return -3;
+  if ((q_stride_tok | out_stride_tok) % 8) return -3;
+  if (paged ? (!kv_lens || block_size < 8 || block_size % 8 || BN % block_size || num_blocks <= 0 || max_blocks <= 0)
+            : ((k_stride_tok | v_stride_tok) % 8 != 0))
+    return -3;
+  CUtensorMap tq, tk, tv;
+  int rc = make_tmap_heads(&tq, q, D, Hq, total_tokens, 1, D, q_stride_tok, q_stride_tok * total_tokens);
+  if (rc) return rc;
+  rc = make_tmap_heads(&tk, k, D, Hkv, total_tokens, paged ? num_blocks : 1, D, k_stride_tok, k_stride_tok * total_tokens,
+                       paged ? block_size : 0);
+  if (rc) return rc;
+  rc = make_tmap_heads(&tv, v, Dv, Hkv, total_tokens, paged ? num_blocks : 1, Dv, v_stride_tok, v_stride_tok * total_tokens,
+                       paged ? block_size : 0);
+  if (rc) return rc;
+  FaParams p{};
+  p.out = reinterpret_cast<bf16*>(out);
+  p.out_stride_tok = out_stride_tok;
+  p.Hq = Hq;
+  p.Hkv = Hkv;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.causal = 1;
+  p.cu_q = cu_q;
+  p.kv_lens = kv_lens;
+  p.block_table = block_table;
+  p.max_blocks = max_blocks;
+  p.block_size = block_size;
+  p.chunk = chunk;
+  p.sink = sink;
+  p.v_dim = Dv;
+  return launch_tiles(D > 64 || Dv > 64 ? 128 : 64, true, max_q_len, Hq, num_seqs, stream, tq, tk, tv, p);
 }
 
 }  // namespace swb

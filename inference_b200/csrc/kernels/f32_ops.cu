@@ -1,0 +1,192 @@
+// 32-bit mode and unrestricted shapes: an fp32 GEMM (dense or grouped rows) and a paged attention kernel for any head
+// widths, both on the ordinary FMA pipes with true fp32 products. They serve models that run in float32 (numerical
+// checks), and the attention kernel also serves bf16 models whose head widths the tensor-core kernels do not cover.
+#include "common.cuh"
+#include "gemm_tcgen05.cuh"
+
+namespace swb {
+
+SWB_REGISTER_STATUS_UNIT(f32_ops);
+
+namespace {
+
+__device__ __forceinline__ float to_f(float x) { return x; }
+__device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ void from_f(float& d, float x) { d = x; }
+__device__ __forceinline__ void from_f(bf16& d, float x) { d = __float2bfloat16(x); }
+
+constexpr int TM = 64, TN = 64, TK = 16;
+
+// out[r, n] = act(sum_k a[src ? src[r] : r, k] w[e, n, k]); 64 x 64 tile, 4 x 4 per thread. Grouped: blockIdx.z = expert.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ a, int lda, const int* __restrict__ src,
+                                                       const int* __restrict__ offsets, const float* __restrict__ w, int ldw,
+                                                       float* out, int ldo, int T, int N, int K, int act) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sa[TK][TM + 4], sw[TK][TN + 4];
+  const int lo = offsets ? offsets[blockIdx.z] : 0, hi = offsets ? offsets[blockIdx.z + 1] : T;
+  const int r0 = lo + blockIdx.y * TM, n0 = blockIdx.x * TN;
+  if (r0 >= hi) return;
+  const float* we = w + (size_t)blockIdx.z * N * ldw;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;   // 64 rows x 16 columns, four per thread
+  const int arow = r0 + lr;
+  const float* ap = arow < hi ? a + (size_t)(src ? src[arow] : arow) * lda : nullptr;
+  const float* wp = n0 + lr < N ? we + (size_t)(n0 + lr) * ldw : nullptr;
+  for (int k0 = 0; k0 < K; k0 += TK) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int k = k0 + lk + j;
+      sa[lk + j][lr] = (ap && k < K) ? ap[k] : 0.f;
+      sw[lk + j][lr] = (wp && k < K) ? wp[k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < TK; ++k) {
+      float x[4], y[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = sa[k][ty * 4 + i], y[i] = sw[k][tx * 4 + i];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = r0 + ty * 4 + i;
+    if (r >= hi) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (act == SWB_ACT_RELU2) v = relu2_f(v);
+      else if (act == SWB_ACT_SILU) v = silu_f(v);
+      else if (act == SWB_ACT_GELU_TANH) v = gelu_tanh_f(v);
+      out[(size_t)r * ldo + n] = v;
+    }
+  }
+}
+
+constexpr int AW = 4;          // warps per CTA: keys are dealt out to them
+constexpr int MAX_PER_LANE = 16;   // head widths up to 512
+
+// One CTA per (query token, head). Each warp runs an online softmax over its share of the visible keys; lanes split the
+// head dimension. The sink joins the denominator when the four partial results are merged.
+template <typename E>
+__global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restrict__ q, long long q_stride_tok,
+                                                              const E* __restrict__ kc, const E* __restrict__ vc, E* out,
+                                                              long long out_stride_tok, const int* __restrict__ block_table,
+                                                              int max_blocks, int block_size, const int* __restrict__ cu_q,
+                                                              const int* __restrict__ kv_lens, int num_seqs, int uniform_q,
+                                                              int Hq, int Hkv, int D, int Dv, float scale, int chunk,
+                                                              const float* __restrict__ sink) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, head = blockIdx.y, kvh = head / (Hq / Hkv);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int seq = 0;
+  if (cu_q) {                    // the last sequence whose first token is not after t (empty sequences are skipped over)
+    int lo = 0, hi = num_seqs - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu_q[mid] <= t) lo = mid;
+      else hi = mid - 1;
+    }
+    seq = lo;
+  } else {
+    seq = t / uniform_q;
+  }
+  const int q0 = cu_q ? cu_q[seq] : seq * uniform_q, q_len = cu_q ? cu_q[seq + 1] - q0 : uniform_q;
+  const int pos = kv_lens[seq] - q_len + (t - q0);
+  const int first = chunk > 0 ? pos / chunk * chunk : 0;
+  const int* table = block_table + (size_t)seq * max_blocks;
+  const E* qr = q + (size_t)t * q_stride_tok + (size_t)head * D;
+  float qv[MAX_PER_LANE], o[MAX_PER_LANE];
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) {
+    const int d = lane + i * 32;
+    qv[i] = d < D ? to_f(qr[d]) : 0.f;
+    o[i] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int j = first + warp; j <= pos; j += AW) {
+    const size_t row = ((size_t)table[j / block_size] * Hkv + kvh) * block_size + j % block_size;
+    const E* kr = kc + row * D;
+    const E* vr = vc + row * Dv;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) {
+      const int d = lane + i * 32;
+      if (d < D) s = fmaf(qv[i], to_f(kr[d]), s);
+    }
+    s = warp_sum(s) * scale;
+    const float mn = fmaxf(m, s), f = expf(m - mn), e = expf(s - mn);
+    l = l * f + e;
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < MAX_PER_LANE; ++i) {
+      const int d = lane + i * 32;
+      if (d < Dv) o[i] = fmaf(e, to_f(vr[d]), o[i] * f);
+    }
+  }
+  __shared__ float so[AW][32 * MAX_PER_LANE], sm[AW], sl[AW];
+#pragma unroll
+  for (int i = 0; i < MAX_PER_LANE; ++i) so[warp][lane + i * 32] = o[i];
+  if (lane == 0) sm[warp] = m, sl[warp] = l;
+  __syncthreads();
+  float top = sink ? sink[head] : -INFINITY;
+  for (int w = 0; w < AW; ++w) top = fmaxf(top, sm[w]);
+  float den = sink ? expf(sink[head] - top) : 0.f;
+  for (int w = 0; w < AW; ++w) den += sl[w] * expf(sm[w] - top);
+  for (int d = threadIdx.x; d < Dv; d += AW * 32) {
+    float v = 0.f;
+    for (int w = 0; w < AW; ++w) v = fmaf(so[w][d], expf(sm[w] - top), v);
+    from_f(out[(size_t)t * out_stride_tok + (size_t)head * Dv + d], v / den);
+  }
+}
+
+}  // namespace
+}  // namespace swb
+
+extern "C" {
+
+// fp32 GEMM without reduced-precision modes. Dense: offsets null, groups 1. Grouped: w [groups, N, ldw], rows of group g
+// are [offsets[g], offsets[g + 1]), at most T rows in all; src (nullable) names the row of `a` for each row.
+int swb_gemm_f32(const float* a, int lda, const int* src, const int* offsets, int groups, const float* w, int ldw, float* out,
+                 int ldo, int T, int N, int K, int act, void* stream) {
+  using namespace swb;
+  if (T <= 0 || N <= 0 || K <= 0) return 0;
+  if (groups < 1 || (groups > 1 && !offsets) || gemm_act_pairs(act)) return -3;
+  return launch_kernel(gemm_f32_kernel, dim3((N + TN - 1) / TN, (T + TM - 1) / TM, groups), dim3(256), 0,
+                       reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act);
+}
+
+// Paged attention for any head widths up to 512 in fp32 arithmetic; elements fp32 or bf16 (fp32 flag). Arguments as in
+// swb_attn_ext; causal, sequences from cu_q or uniform lengths of uniform_q tokens.
+int swb_attn_simple(const void* q, long long q_stride_tok, const void* k, const void* v, void* out, long long out_stride_tok,
+                    const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
+                    int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk,
+                    const float* sink, int fp32, void* stream) {
+  using namespace swb;
+  if (total_tokens <= 0 || num_seqs <= 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv || D < 1 || Dv < 1 || D > 32 * MAX_PER_LANE || Dv > 32 * MAX_PER_LANE || block_size <= 0 ||
+      !block_table || !kv_lens || chunk < 0 || (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)))
+    return -3;
+  const dim3 grid((unsigned)total_tokens, Hq), block(AW * 32);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (fp32)
+    return launch_kernel(attn_simple_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(q), q_stride_tok,
+                         reinterpret_cast<const float*>(k), reinterpret_cast<const float*>(v), reinterpret_cast<float*>(out),
+                         out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D,
+                         Dv, scale, chunk, sink);
+  return launch_kernel(attn_simple_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(q), q_stride_tok,
+                       reinterpret_cast<const bf16*>(k), reinterpret_cast<const bf16*>(v), reinterpret_cast<bf16*>(out),
+                       out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv,
+                       scale, chunk, sink);
+}
+
+}  // extern "C"

@@ -151,6 +151,7 @@ __device__ __forceinline__ unsigned long long ssq_fixed(float ss) {
 __device__ __forceinline__ float act_apply(float x, int act) {
   if (act == SWB_ACT_SILU) return silu_f(x);
   if (act == SWB_ACT_GELU_TANH) return gelu_tanh_f(x);
+  if (act == SWB_ACT_RELU2) return relu2_f(x);
   return x;
 }
 
@@ -561,7 +562,7 @@ gemm_decode_cluster_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
               acc[2 * j + 1] += t.y;
             }
           }
-          if (p.act >= SWB_ACT_SWIGLU_PAIRS) {
+          if (gemm_act_pairs(p.act)) {
             // rows come in (gate, up) pairs: four gated outputs, one 8-byte store
             const int a1 = p.act == SWB_ACT_SWIGLU_PAIRS ? SWB_ACT_SILU : SWB_ACT_GELU_TANH;
             uint2 o;
@@ -604,7 +605,7 @@ gemm_decode_cluster_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
               }
             }
           }
-        } else if (p.act >= SWB_ACT_SWIGLU_PAIRS) {
+        } else if (gemm_act_pairs(p.act)) {
           const int a1 = p.act == SWB_ACT_SWIGLU_PAIRS ? SWB_ACT_SILU : SWB_ACT_GELU_TANH;
           for (int j = 0; j + 1 < nvalid; j += 2) {
             const float gte = acc[j] + (p.bias ? __bfloat162float(p.bias[feat + j]) : 0.f);

@@ -105,6 +105,7 @@ struct SegIter {
 __device__ __forceinline__ float apply_act(float x, int act) {
   if (act == SWB_ACT_SILU) return silu_f(x);
   if (act == SWB_ACT_GELU_TANH) return gelu_tanh_f(x);
+  if (act == SWB_ACT_RELU2) return relu2_f(x);
   return x;
 }
 
@@ -760,7 +761,7 @@ int gemm_bf16_launch(const GemmArgs& a, cudaStream_t stream) {
   if (a.conv_c > 0) {
     // implicit 3x3 convolution: tokens-as-M only; a 128-pixel tile is a run of one image row or whole rows
     const long hw = (long)a.conv_h * a.conv_w;
-    if (a.scatter || a.group_of_mtile || a.ssq_in || a.ssq_out || (a.peer && a.peer->mode) || a.act >= SWB_ACT_SWIGLU_PAIRS)
+    if (a.scatter || a.group_of_mtile || a.ssq_in || a.ssq_out || (a.peer && a.peer->mode) || gemm_act_pairs(a.act))
       return -3;
     if (a.conv_n <= 0 || a.conv_h <= 0 || a.conv_w <= 0 || (a.conv_c % BK) != 0 || a.K != 9 * a.conv_c ||
         (long)a.T != hw * a.conv_n || (hw % BM) != 0 || !((a.conv_w % BM) == 0 || (BM % a.conv_w) == 0))
@@ -779,7 +780,7 @@ int gemm_bf16_launch(const GemmArgs& a, cudaStream_t stream) {
                                   !gemm_bf16_gated_supported(a.T, a.N & ~1, a.K)))
     return -3;
   // gated-pair epilogues exist in the decode cluster kernel only (bf16 output, no residual)
-  const bool pairs = a.act >= SWB_ACT_SWIGLU_PAIRS;
+  const bool pairs = gemm_act_pairs(a.act);
   if (pairs && (a.scatter || a.group_of_mtile || a.residual || a.out_fp32 || (a.N & 1) || a.force_mode == 0 ||
                 a.force_mode == 1 || !gemm_bf16_gated_supported(a.T, a.N, a.K)))
     return -3;

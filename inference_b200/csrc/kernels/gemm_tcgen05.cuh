@@ -10,8 +10,10 @@ namespace swb {
 
 // 3 / 4: gated pairs. Output features come in (gate, up) row pairs of the weight: out[t, f] = silu|gelu(acc[2f]) * acc[2f+1],
 // so the output is half as wide as the weight has rows (SwiGLU / GeGLU fused into the gate-up projection).
+// 5: square of relu (ungated).
 enum GemmAct : int { SWB_ACT_NONE = 0, SWB_ACT_SILU = 1, SWB_ACT_GELU_TANH = 2, SWB_ACT_SWIGLU_PAIRS = 3,
-                     SWB_ACT_GEGLU_PAIRS = 4 };
+                     SWB_ACT_GEGLU_PAIRS = 4, SWB_ACT_RELU2 = 5 };
+__host__ __device__ inline bool gemm_act_pairs(int act) { return act == SWB_ACT_SWIGLU_PAIRS || act == SWB_ACT_GEGLU_PAIRS; }
 
 // The first SWB_GEMM_COUNTER_BYTES of a GEMM workspace hold per-tile arrival counters (zero between
 // launches: the caller zeroes them once, the kernel restores zero); fp32 split-K partials follow.

@@ -177,18 +177,26 @@ __global__ void __launch_bounds__(THREADS) layernorm_mod_kernel(const bf16* __re
   }
 }
 
+__device__ __forceinline__ float elem_to_f(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ float elem_to_f(float x) { return x; }
+__device__ __forceinline__ void elem_from_f(bf16& d, float x) { d = __float2bfloat16(x); }
+__device__ __forceinline__ void elem_from_f(float& d, float x) { d = x; }
+
 // Per (token, head) warp: optional per-head RMSNorm (q_norm / k_norm), rotary embedding from a
 // precomputed fp32 cos/sin table [max_pos, rot_dim/2], then: q heads are written back in place, k and v
 // heads are written into the paged cache (layout [block, kv_head, block_size, head_dim]) at slot_mapping[t].
 // interleaved = 0: NeoX half-split pairs (i, i + rot_dim/2); 1: GPT-J pairs (2i, 2i+1).
+// E is the element type of the projection buffer and the cache (bf16, or float for the 32-bit mode); EPL elements per
+// lane bound the head width to 32 * EPL; v heads may have a width Dv of their own.
+template <typename E, int EPL>
 __global__ void __launch_bounds__(256) rope_kv_write_kernel(
-    bf16* qkv, int ld_qkv, const int* __restrict__ positions, const long long* __restrict__ slot_mapping,
+    E* qkv, int ld_qkv, const int* __restrict__ positions, const long long* __restrict__ slot_mapping,
     const float* __restrict__ cos_tab, const float* __restrict__ sin_tab, int rot_dim, int interleaved,
     const bf16* __restrict__ q_norm_w, const bf16* __restrict__ k_norm_w, float norm_eps, float norm_w_offset,
-    bf16* kcache, bf16* vcache, int block_size, int T, int Hq, int Hkv, int D) {
+    E* kcache, E* vcache, int block_size, int T, int Hq, int Hkv, int Dqk, int Dv) {
   pdl_launch_dependents();
   pdl_wait(TL_ROPE_KV);
-  __shared__ float rope_smem[8 * 256];
+  __shared__ float rope_smem[8 * 32 * EPL];
   const int warps_per_block = blockDim.x >> 5;
   const int lane = threadIdx.x & 31;
   const long long gw = (long long)blockIdx.x * warps_per_block + (threadIdx.x >> 5);
@@ -196,18 +204,20 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
   if (gw >= (long long)T * heads) return;
   const int t = (int)(gw / heads);
   const int h = (int)(gw % heads);
-  bf16* src = qkv + (size_t)t * ld_qkv + (size_t)h * D;
   const bool is_q = h < Hq;
   const bool is_k = !is_q && h < Hq + Hkv;
+  const int D = (is_q || is_k) ? Dqk : Dv;
+  E* src = qkv + (size_t)t * ld_qkv +
+           ((is_q || is_k) ? (size_t)h * Dqk : (size_t)(Hq + Hkv) * Dqk + (size_t)(h - Hq - Hkv) * Dv);
   const int pos = positions[t];
-  const int epl = (D + 31) / 32;  // elements per lane, <= 8 (D <= 256)
-  float v[8];
+  const int epl = (D + 31) / 32;  // elements per lane, <= EPL
+  float v[EPL];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
+  for (int i = 0; i < EPL; ++i) {
     const int d = lane + i * 32;
-    v[i] = (i < epl && d < D) ? __bfloat162float(src[d]) : 0.f;
+    v[i] = (i < epl && d < D) ? elem_to_f(src[d]) : 0.f;
   }
-  bf16* dst = src;
+  E* dst = src;
   if (!is_q && (is_k ? kcache : vcache) != nullptr) {
     // with a cache the k / v heads go to their slot (in-place otherwise: dense attention reads qkv directly)
     const long long slot = slot_mapping ? slot_mapping[t] : -1;
@@ -217,7 +227,7 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
       const long long blk = slot / block_size;
       const int off = (int)(slot % block_size);
       const int kvh = is_k ? (h - Hq) : (h - Hq - Hkv);
-      bf16* base = is_k ? kcache : vcache;
+      E* base = is_k ? kcache : vcache;
       dst = base + (((size_t)blk * Hkv + kvh) * block_size + off) * (size_t)D;
     }
   }
@@ -226,11 +236,11 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
     if (nw) {
       float ss = 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
+      for (int i = 0; i < EPL; ++i) ss += v[i] * v[i];
       ss = warp_sum(ss);
       const float inv = rsqrtf(ss / (float)D + norm_eps);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < EPL; ++i) {
         const int d = lane + i * 32;
         if (i < epl && d < D) {
           // round through bf16 like an unfused norm would before the rotation
@@ -243,15 +253,15 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
     const float* sn = sin_tab + (size_t)pos * half;
     if (!interleaved) {
       // partner of element d (< rot_dim) is d +/- half; exchange through this warp's shared-memory row
-      float* row = rope_smem + (threadIdx.x >> 5) * 256;
+      float* row = rope_smem + (threadIdx.x >> 5) * (32 * EPL);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < EPL; ++i) {
         const int d = lane + i * 32;
         if (i < epl && d < D) row[d] = v[i];
       }
       __syncwarp();
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < EPL; ++i) {
         const int d = lane + i * 32;
         if (i < epl && d < rot_dim) {
           const bool lo = d < half;
@@ -263,7 +273,7 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
       }
     } else {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < EPL; ++i) {
         const int d = lane + i * 32;
         const float partner = __shfl_xor_sync(0xffffffffu, v[i], 1);
         if (i < epl && d < rot_dim) {
@@ -276,16 +286,16 @@ __global__ void __launch_bounds__(256) rope_kv_write_kernel(
   }
   if (dst) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < EPL; ++i) {
       const int d = lane + i * 32;
-      if (i < epl && d < D) dst[d] = __float2bfloat16(v[i]);
+      if (i < epl && d < D) elem_from_f(dst[d], v[i]);
     }
   }
   if (is_k && dst != src) {   // the rotated key also stays in the projection buffer
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < EPL; ++i) {
       const int d = lane + i * 32;
-      if (i < epl && d < D) src[d] = __float2bfloat16(v[i]);
+      if (i < epl && d < D) elem_from_f(src[d], v[i]);
     }
   }
 }
@@ -521,31 +531,53 @@ int swb_layernorm_mod(const void* x, int ldx, const void* scale, const void* shi
   });
 }
 
+// fp32 = 1: qkv and both caches hold floats (q_norm_w / k_norm_w stay bf16). Dv: width of the v heads and of the v cache.
+int swb_rope_kv_write_ex(void* qkv, int ld_qkv, const int* positions, const long long* slot_mapping,
+                         const float* cos_tab, const float* sin_tab, int rot_dim, int interleaved, const void* q_norm_w,
+                         const void* k_norm_w, float norm_eps, float norm_w_offset, void* kcache, void* vcache,
+                         int block_size, int T, int Hq, int Hkv, int D, int Dv, int fp32, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (D > 512 || Dv > 512 || rot_dim > D || (rot_dim & 1)) return -3;
+  const int wpb = 8;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const bf16* qn = reinterpret_cast<const bf16*>(q_norm_w);
+  const bf16* kn = reinterpret_cast<const bf16*>(k_norm_w);
+  if (!fp32 && D == 128 && Dv == 128 && rot_dim == 128 && (ld_qkv % 2) == 0 && (reinterpret_cast<uintptr_t>(qkv) & 3) == 0) {
+    const int heads_active = Hq + Hkv + (vcache ? Hkv : 0);   // V stays where it is unless it goes to a cache
+    const long long nblk = ((long long)T * heads_active + wpb - 1) / wpb;
+    auto kern = interleaved ? rope_kv_write_d128_kernel<true> : rope_kv_write_d128_kernel<false>;
+    launch_rc = launch_kernel(kern, dim3((unsigned)nblk), dim3(wpb * 32), 0, st, reinterpret_cast<bf16*>(qkv), ld_qkv,
+                              positions, slot_mapping, cos_tab, sin_tab, qn, kn, norm_eps, norm_w_offset,
+                              reinterpret_cast<bf16*>(kcache), reinterpret_cast<bf16*>(vcache), block_size, T, Hq, Hkv,
+                              heads_active);
+    return last_err();
+  }
+  const long long warps = (long long)T * (Hq + 2 * Hkv);
+  const dim3 grid((unsigned)((warps + wpb - 1) / wpb)), block(wpb * 32);
+  const bool wide = D > 256 || Dv > 256;
+  if (fp32) {
+    auto kern = wide ? rope_kv_write_kernel<float, 16> : rope_kv_write_kernel<float, 8>;
+    launch_rc = launch_kernel(kern, grid, block, 0, st, reinterpret_cast<float*>(qkv), ld_qkv, positions, slot_mapping,
+                              cos_tab, sin_tab, rot_dim, interleaved, qn, kn, norm_eps, norm_w_offset,
+                              reinterpret_cast<float*>(kcache), reinterpret_cast<float*>(vcache), block_size, T, Hq, Hkv, D,
+                              Dv);
+  } else {
+    auto kern = wide ? rope_kv_write_kernel<bf16, 16> : rope_kv_write_kernel<bf16, 8>;
+    launch_rc = launch_kernel(kern, grid, block, 0, st, reinterpret_cast<bf16*>(qkv), ld_qkv, positions, slot_mapping,
+                              cos_tab, sin_tab, rot_dim, interleaved, qn, kn, norm_eps, norm_w_offset,
+                              reinterpret_cast<bf16*>(kcache), reinterpret_cast<bf16*>(vcache), block_size, T, Hq, Hkv, D,
+                              Dv);
+  }
+  return last_err();
+}
+
 int swb_rope_kv_write(void* qkv, int ld_qkv, const int* positions, const long long* slot_mapping,
                       const float* cos_tab, const float* sin_tab, int rot_dim, int interleaved, const void* q_norm_w,
                       const void* k_norm_w, float norm_eps, float norm_w_offset, void* kcache, void* vcache,
                       int block_size, int T, int Hq, int Hkv, int D, void* stream) {
-  using namespace swb;
-  if (T <= 0) return 0;
-  if (D > 256 || rot_dim > D || (rot_dim & 1)) return -3;
-  const int wpb = 8;
-  if (D == 128 && rot_dim == 128 && (ld_qkv % 2) == 0 && (reinterpret_cast<uintptr_t>(qkv) & 3) == 0) {
-    const int heads_active = Hq + Hkv + (vcache ? Hkv : 0);   // V stays where it is unless it goes to a cache
-    const long long nblk = ((long long)T * heads_active + wpb - 1) / wpb;
-    auto kern = interleaved ? rope_kv_write_d128_kernel<true> : rope_kv_write_d128_kernel<false>;
-    launch_rc = launch_kernel(kern, dim3((unsigned)nblk), dim3(wpb * 32), 0, reinterpret_cast<cudaStream_t>(stream),
-                              reinterpret_cast<bf16*>(qkv), ld_qkv, positions, slot_mapping, cos_tab, sin_tab,
-                              reinterpret_cast<const bf16*>(q_norm_w), reinterpret_cast<const bf16*>(k_norm_w),
-                              norm_eps, norm_w_offset, reinterpret_cast<bf16*>(kcache), reinterpret_cast<bf16*>(vcache),
-                              block_size, T, Hq, Hkv, heads_active);
-    return last_err();
-  }
-  const long long warps = (long long)T * (Hq + 2 * Hkv);
-  const long long blocks = (warps + wpb - 1) / wpb;
-  launch_rc = launch_kernel(rope_kv_write_kernel, dim3((unsigned)blocks), dim3(wpb * 32), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<bf16*>(qkv), ld_qkv, positions, slot_mapping, cos_tab, sin_tab, rot_dim, interleaved,
-      reinterpret_cast<const bf16*>(q_norm_w), reinterpret_cast<const bf16*>(k_norm_w), norm_eps, norm_w_offset,
-      reinterpret_cast<bf16*>(kcache), reinterpret_cast<bf16*>(vcache), block_size, T, Hq, Hkv, D);
-  return last_err();
+  return swb_rope_kv_write_ex(qkv, ld_qkv, positions, slot_mapping, cos_tab, sin_tab, rot_dim, interleaved, q_norm_w,
+                              k_norm_w, norm_eps, norm_w_offset, kcache, vcache, block_size, T, Hq, Hkv, D, D, 0, stream);
 }
 
 int swb_gated_act_mul(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, void* stream) {

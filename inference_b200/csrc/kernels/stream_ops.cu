@@ -1,0 +1,247 @@
+// Kernels around a 32-bit residual stream: embedding into the stream and the fused step between two sublayers.
+//
+// stream_norm_kernel is that step in one pass over a row:
+//     x   += norm1(branch)            branch = a projection output row, or the mean of a token's expert output rows
+//     out  = norm2(x) * out_scale     or the stream itself, for a projection that reads it un-normalised
+// A layer with norms before and after each sublayer then needs one such launch per sublayer. Both norms are layer norms
+// (mean removed, weight and bias) or RMS norms, computed in fp32 on the row held in registers, two passes (mean, then
+// squared deviations). The output is stored once per token, or to every row of an expert-sorted buffer that the token's
+// routing names, so the gather in front of a grouped GEMM costs no launch of its own.
+// Rows are padded to a multiple of 8 columns; padding columns of the stream, the weights and the outputs are zero and do
+// not enter the statistics.
+#include "common.cuh"
+
+namespace swb {
+
+SWB_REGISTER_STATUS_UNIT(stream_ops);
+
+namespace {
+
+struct StreamNormParams {
+  float* x;                  // [T, ldx] residual stream
+  int ldx;
+  const long long* rows;     // optional: process row rows[i] of x as output row i (then no branch)
+  const void* branch;        // optional bf16 / fp32 [*, ld_branch]
+  int ld_branch, branch_fp32;
+  const int* branch_rows;    // optional [T, branch_top]: the branch is the weighted sum of these rows
+  int branch_top;
+  float branch_weight;
+  const float *w1, *b1;      // norm of the branch (b1 optional; w1 null: the branch is added as it is)
+  const float *w2, *b2;      // norm of the stream (w2 null: the stream itself is stored)
+  void* out;                 // optional bf16 / fp32 [*, ldo]
+  int ldo, out_fp32;
+  const int* out_rows;       // optional [T, out_top]: the output row goes to all of these rows
+  int out_top;
+  int H, Hp;
+  float eps, out_scale;
+  int center;                // 1: layer norm, 0: RMS norm
+};
+
+__device__ __forceinline__ float4 load4(const void* base, size_t off, int fp32) {
+  if (fp32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(base) + off);
+  const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(base) + off);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(void* base, size_t off, int fp32, float4 v) {
+  if (fp32) {
+    *reinterpret_cast<float4*>(reinterpret_cast<float*>(base) + off) = v;
+    return;
+  }
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(base) + off) =
+      make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+// Sum over the block; `red` alternates between two slots so that one barrier per reduction is enough.
+template <int THREADS>
+__device__ __forceinline__ float block_total(float v, float* red) {
+  v = warp_sum(v);
+  if constexpr (THREADS == 32) return v;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < THREADS / 32 ? red[lane] : 0.f);
+}
+
+// v <- norm(v) * w + b over the first H columns of the row (thread t owns float4 columns t, t + THREADS, ...)
+template <int THREADS, int VPT>
+__device__ __forceinline__ void norm_row(float4* v, const float* __restrict__ w, const float* __restrict__ b, int H, int nvec,
+                                         float eps, int center, float* red) {
+  float mean = 0.f;
+  if (center) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);   // padding columns hold zeros
+    mean = block_total<THREADS>(s, red) / (float)H;
+    red += 32;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * THREADS) * 4;
+    v[i].x -= mean, v[i].y -= mean, v[i].z -= mean, v[i].w -= mean;
+    if (c < H) ss += v[i].x * v[i].x;
+    if (c + 1 < H) ss += v[i].y * v[i].y;
+    if (c + 2 < H) ss += v[i].z * v[i].z;
+    if (c + 3 < H) ss += v[i].w * v[i].w;
+  }
+  const float r = rsqrtf(block_total<THREADS>(ss, red) / (float)H + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c4 = threadIdx.x + i * THREADS;
+    if (c4 < nvec) {
+      const float4 ww = __ldg(reinterpret_cast<const float4*>(w) + c4);
+      const float4 bb = b ? __ldg(reinterpret_cast<const float4*>(b) + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[i] = make_float4(v[i].x * r * ww.x + bb.x, v[i].y * r * ww.y + bb.y, v[i].z * r * ww.z + bb.z,
+                         v[i].w * r * ww.w + bb.w);
+    }
+  }
+}
+
+template <int THREADS, int VPT>
+__global__ void __launch_bounds__(THREADS) stream_norm_kernel(const StreamNormParams p) {
+  pdl_launch_dependents();
+  pdl_wait(TL_RMSNORM);
+  __shared__ float red[4 * 32];
+  const int row = blockIdx.x;
+  const int nvec = p.Hp / 4;
+  float* xr = p.x + (size_t)(p.rows ? p.rows[row] : row) * p.ldx;
+  float4 x[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    x[i] = c < nvec ? *reinterpret_cast<const float4*>(xr + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if (p.branch) {
+    float4 v[VPT];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int terms = p.branch_rows ? p.branch_top : 1;
+    for (int k = 0; k < terms; ++k) {
+      const size_t br = p.branch_rows ? (size_t)p.branch_rows[row * p.branch_top + k] : (size_t)row;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * THREADS;
+        if (c < nvec) {
+          const float4 y = load4(p.branch, br * p.ld_branch + c * 4, p.branch_fp32);
+          v[i].x += y.x, v[i].y += y.y, v[i].z += y.z, v[i].w += y.w;
+        }
+      }
+    }
+    if (p.branch_rows) {
+#pragma unroll
+      for (int i = 0; i < VPT; ++i)
+        v[i].x *= p.branch_weight, v[i].y *= p.branch_weight, v[i].z *= p.branch_weight, v[i].w *= p.branch_weight;
+    }
+    if (p.w1) norm_row<THREADS, VPT>(v, p.w1, p.b1, p.H, nvec, p.eps, p.center, red);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * THREADS;
+      if (c < nvec) {
+        x[i].x += v[i].x, x[i].y += v[i].y, x[i].z += v[i].z, x[i].w += v[i].w;
+        *reinterpret_cast<float4*>(xr + c * 4) = x[i];
+      }
+    }
+  }
+  if (!p.out) return;
+  if (p.w2) norm_row<THREADS, VPT>(x, p.w2, p.b2, p.H, nvec, p.eps, p.center, red + 64);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c < nvec) {
+      x[i].x *= p.out_scale, x[i].y *= p.out_scale, x[i].z *= p.out_scale, x[i].w *= p.out_scale;
+      if (!p.out_rows) {
+        store4(p.out, (size_t)row * p.ldo + c * 4, p.out_fp32, x[i]);
+      } else {
+        for (int k = 0; k < p.out_top; ++k)
+          store4(p.out, (size_t)p.out_rows[row * p.out_top + k] * p.ldo + c * 4, p.out_fp32, x[i]);
+      }
+    }
+  }
+}
+
+// x[t] = table[ids[t]] as fp32; optional copies of the row in the activation type (out_a / out_b, strides ld_a / ld_b).
+// Ids outside [0, vocab) read as a zero row.
+__global__ void __launch_bounds__(256) stream_embed_kernel(const long long* __restrict__ ids, const void* table, int table_fp32,
+                                                           int vocab, float* x, int ldx, void* out_a, int ld_a, void* out_b,
+                                                           int ld_b, int out_fp32, int T, int Hp) {
+  pdl_launch_dependents();
+  pdl_wait(TL_EMBED);
+  const int nvec = Hp / 4;
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (long long)T * nvec) return;
+  const int t = (int)(idx / nvec), c = (int)(idx % nvec) * 4;
+  const long long id = ids[t];
+  const float4 v = (id >= 0 && id < vocab) ? load4(table, (size_t)id * Hp + c, table_fp32) : make_float4(0.f, 0.f, 0.f, 0.f);
+  *reinterpret_cast<float4*>(x + (size_t)t * ldx + c) = v;
+  if (out_a) store4(out_a, (size_t)t * ld_a + c, out_fp32, v);
+  if (out_b) store4(out_b, (size_t)t * ld_b + c, out_fp32, v);
+}
+
+template <int THREADS, int VPT>
+int launch_sn(const StreamNormParams& p, int T, cudaStream_t s) {
+  return launch_kernel(stream_norm_kernel<THREADS, VPT>, dim3((unsigned)T), dim3(THREADS), 0, s, p);
+}
+
+}  // namespace
+}  // namespace swb
+
+extern "C" {
+
+// See StreamNormParams. All pointers 16-byte aligned (8 for bf16 rows), strides multiples of 4 elements, Hp a multiple of
+// 8 up to 32768, H <= Hp.
+int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch, int ld_branch, int branch_fp32,
+                    const int* branch_rows, int branch_top, float branch_weight, const float* w1, const float* b1,
+                    const float* w2, const float* b2, void* out, int ldo, int out_fp32, const int* out_rows, int out_top,
+                    int T, int H, int Hp, float eps, float out_scale, int center, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (H <= 0 || H > Hp || (Hp % 8) || (ldx % 4) || (branch && (ld_branch % 4)) || (out && (ldo % 4)) || (rows && branch) ||
+      (branch_rows && branch_top <= 0) || (out_rows && out_top <= 0))
+    return -3;
+  StreamNormParams p{};
+  p.x = reinterpret_cast<float*>(x);
+  p.ldx = ldx;
+  p.rows = rows;
+  p.branch = branch;
+  p.ld_branch = ld_branch;
+  p.branch_fp32 = branch_fp32;
+  p.branch_rows = branch_rows;
+  p.branch_top = branch_top;
+  p.branch_weight = branch_weight;
+  p.w1 = w1, p.b1 = b1, p.w2 = w2, p.b2 = b2;
+  p.out = out;
+  p.ldo = ldo;
+  p.out_fp32 = out_fp32;
+  p.out_rows = out_rows;
+  p.out_top = out_top;
+  p.H = H, p.Hp = Hp;
+  p.eps = eps;
+  p.out_scale = out_scale;
+  p.center = center;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const int nvec = Hp / 4;
+  if (nvec <= 128) return launch_sn<128, 1>(p, T, s);
+  if (nvec <= 256) return launch_sn<256, 1>(p, T, s);
+  if (nvec <= 512) return launch_sn<256, 2>(p, T, s);
+  if (nvec <= 1024) return launch_sn<256, 4>(p, T, s);
+  if (nvec <= 2048) return launch_sn<512, 4>(p, T, s);
+  if (nvec <= 4096) return launch_sn<1024, 4>(p, T, s);
+  if (nvec <= 8192) return launch_sn<1024, 8>(p, T, s);
+  return -3;
+}
+
+int swb_stream_embed(const long long* ids, const void* table, int table_fp32, int vocab, void* x, int ldx, void* out_a,
+                     int ld_a, void* out_b, int ld_b, int out_fp32, int T, int Hp, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if ((Hp % 8) || (ldx % 4) || (out_a && (ld_a % 4)) || (out_b && (ld_b % 4))) return -3;
+  const long long n = (long long)T * (Hp / 4);
+  return launch_kernel(stream_embed_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0,
+                       reinterpret_cast<cudaStream_t>(stream), ids, table, table_fp32, vocab,
+                       reinterpret_cast<float*>(x), ldx, out_a, ld_a, out_b, ld_b, out_fp32, T, Hp);
+}
+
+}  // extern "C"

@@ -26,6 +26,9 @@ class DecodeBackend(Protocol):
         """Appends new_tokens[i] to seqs[i]; returns per-sequence fp32 logits on the host-visible device:
         [vocab] (last position) or [len_i, vocab] when all_positions."""
     def forward_greedy(self, seqs: list[Any], new_tokens: list[list[int]]) -> list[int]: ...
+    def forward_at(self, seqs: list[Any], new_tokens: list[list[int]], want: list[list[int]]) -> torch.Tensor | None:
+        """Appends new_tokens[i] to seqs[i] in one step; fp32 logits at the places want[i] within new_tokens[i], in order
+        [sum of len(want[i]), vocab], or None when nothing is wanted."""
     def truncate(self, seq: Any, length: int) -> None: ...
     def fork(self, seq: Any, n_tokens: int) -> Any:
         """A new sequence sharing the first n_tokens tokens of seq's cache (copy-on-write where supported)."""
@@ -101,6 +104,14 @@ class GpuBackend:
             return [int(x) for x in self.runner.decode(seqs, [t[0] for t in new_tokens]).tolist()]
         return [int(x) for x in self.runner.prefill(seqs, new_tokens, embed_overrides=ov, mrope_overrides=mr).tolist()]
 
+    def forward_at(self, seqs, new_tokens, want):
+        if self._is_decode(seqs, new_tokens):
+            rows = [i for i, w in enumerate(want) for _ in w]
+            logits = self.runner.decode(seqs, [t[0] for t in new_tokens], want_logits=True)
+            return logits[rows] if rows else None
+        logits = self.runner.prefill(seqs, new_tokens, want=want)
+        return logits if any(want) else None
+
     def truncate(self, seq, length):
         seq.truncate(length)
 
@@ -157,6 +168,10 @@ class OracleBackend:
 
     def forward_greedy(self, seqs, new_tokens):
         return [int(torch.argmax(l)) for l in self.forward(seqs, new_tokens)]
+
+    def forward_at(self, seqs, new_tokens, want):
+        rows = [lg[w] for lg, w in zip(self.forward(seqs, new_tokens, all_positions=True), want) if w]
+        return torch.cat(rows, dim=0) if rows else None
 
     def truncate(self, seq, length):
         seq.cache.truncate(length)

@@ -7,6 +7,8 @@ allocator policy (copy-on-write prefix sharing), so a block id is valid across a
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 
 from ..policy.paging import BlockAllocator
@@ -34,6 +36,43 @@ class PagedKvPool:
                           elem: int = 2) -> int:
         per_block = num_layers * 2 * kv_heads * block_size * head_dim * elem
         return max(1, bytes_budget // per_block)
+
+
+@dataclass(frozen=True)
+class KvGeometry:
+    """K / V shape of one cache-owning layer run."""
+    kv_heads: int
+    k_dim: int
+    v_dim: int
+
+
+class LayeredKvPool:
+    """Paged pool of a model whose layers differ in head count or head width, or run more than once: every run owns a K
+    tensor [blocks, kv_heads, block_size, k_dim] and a V tensor [blocks, kv_heads, block_size, v_dim]. Block ids are
+    shared by all runs (one allocator), so sequences, forks and rollbacks work as on the uniform pool."""
+
+    def __init__(self, geometry: list[KvGeometry], num_blocks: int, block_size: int = 16,
+                 device: torch.device | str = "cuda", dtype: torch.dtype = torch.bfloat16):
+        self.geometry, self.num_layers = list(geometry), len(geometry)
+        self.num_blocks, self.block_size = num_blocks, block_size
+
+        def pages(g: KvGeometry, dim: int) -> torch.Tensor:
+            return torch.zeros((num_blocks, g.kv_heads, block_size, dim), dtype=dtype, device=device)
+        self.data = [(pages(g, g.k_dim), pages(g, g.v_dim)) for g in geometry]
+        self.allocator = BlockAllocator(num_blocks)
+
+    @property
+    def bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for kv in self.data for t in kv)
+
+    def copy_block(self, src: int, dst: int) -> None:
+        for kv in self.data:
+            for t in kv:
+                t[dst].copy_(t[src])
+
+    @staticmethod
+    def block_bytes(geometry: list[KvGeometry], block_size: int = 16, elem: int = 2) -> int:
+        return sum(g.kv_heads * block_size * (g.k_dim + g.v_dim) * elem for g in geometry)
 
 
 class PagedSequence:

@@ -40,11 +40,13 @@ class LlmEngine:
         self.model = model
         self.cfg = cfg or EngineConfig()
         c, m = self.cfg, model.cfg
-        if c.kv_bytes is not None:
+        if c.kv_bytes is not None and hasattr(model, "kv_block_bytes"):
+            nblocks = max(1, c.kv_bytes // model.kv_block_bytes(c.block_size))
+        elif c.kv_bytes is not None:
             nblocks = PagedKvPool.blocks_for_budget(c.kv_bytes, m.num_layers, model.hkv, m.head_dim, c.block_size)
         else:
             nblocks = c.max_batch * ((c.max_seq_len + c.block_size - 1) // c.block_size) + 8
-        if hasattr(model, "make_pool"):      # pipeline-sharded model: one KV tensor per stage device, shared block ids
+        if hasattr(model, "make_pool"):      # pipeline-sharded or layer-by-layer model: its own KV tensors, shared block ids
             self.pool = model.make_pool(nblocks, c.block_size)
         else:
             self.pool = PagedKvPool(m.num_layers, nblocks, model.hkv, m.head_dim, c.block_size, device=model.device)

@@ -23,6 +23,7 @@ from ..io import gguf_quants as gq
 from ..io.safetensors_io import load_dir
 from ..models.config import Architecture, ModelConfig
 from ..models.oracle import OracleLlama
+from ..models.registry import gpu_supported
 from ..policy.sampler import SamplingParams
 from .backend import DecodeBackend, GpuBackend, OracleBackend
 from .decode import GenerationConfig, generate
@@ -52,11 +53,6 @@ def _read_json(p: Path) -> dict:
         return json.loads(p.read_text())
     except (OSError, json.JSONDecodeError):
         return {}
-
-
-def _supported_on_gpu(cfg: ModelConfig) -> bool:
-    return (cfg.head_dim == 128 and cfg.mla is None and
-            cfg.architecture not in (Architecture.QWEN35, Architecture.DEEPSEEK_V2))
 
 
 def probe_config(spec: LoadSpec) -> ModelConfig | None:
@@ -303,25 +299,11 @@ def _build_backend(cfg: ModelConfig, weights: dict, backend_name: str, comm=None
                             device="cuda" if on_gpu else "cpu")
         return OracleBackend(model, max_context=qcfg.max_position_embeddings or 8192)
     if backend_name == BACKEND_GPU:
-        if not torch.cuda.is_available():
-            raise LoadError("the b200 backend needs a CUDA device (use the cpu runtime bundle on hosts without one)")
-        if not _supported_on_gpu(cfg):
-            raise Unsupported(f"{cfg.architecture.value} (head_dim {cfg.head_dim}) is not served by the sm_100a "
-                              "decoder; load it through the cpu-llama provider")
-        from ..models.llama import LlamaGpu
-        from .kv_pool import PagedKvPool
-        from .runner import ModelRunner
+        from .loading import gpu_backend
 
-        dev = comm.device if comm is not None else torch.device("cuda", torch.cuda.current_device())
-        model = LlamaGpu(cfg, comm=comm, device=dev).load_state_dict(weights)
-        ctx = min(cfg.max_position_embeddings or 8192, 32768)
-        max_batch = 16
-        free, _total = torch.cuda.mem_get_info(dev)
-        per_block = cfg.num_layers * 2 * model.hkv * 16 * cfg.head_dim * 2
-        want = max_batch * ((ctx + 15) // 16) + 64
-        nblocks = max(64, min(want, int(free * 0.6) // per_block))
-        pool = PagedKvPool(cfg.num_layers, nblocks, model.hkv, cfg.head_dim, 16, device=dev)
-        return GpuBackend(ModelRunner(model, pool, max_batch=max_batch, max_seq_len=ctx))
+        return gpu_backend(cfg, weights, comm)
+    if cfg.architecture is Architecture.ZOBUNEX:
+        raise Unsupported(f"{cfg.architecture.value} runs on the b200 backend only")
     return OracleBackend(OracleLlama(cfg, weights, dtype=torch.float32, device="cpu"),
                          max_context=cfg.max_position_embeddings or 8192)
 
@@ -469,7 +451,7 @@ class Qwen3VlProvider(LlamaProvider):
         if on_gpu and not torch.cuda.is_available():
             raise LoadError("the b200 backend needs a CUDA device (use the cpu runtime bundle on hosts without one)")
         dev, dtype = ("cuda", torch.bfloat16) if on_gpu else ("cpu", torch.float32)
-        if on_gpu and _supported_on_gpu(cfg) and os.environ.get("SWB_QWEN3_VL_DECODER", "paged") != "oracle":
+        if on_gpu and gpu_supported(cfg) and os.environ.get("SWB_QWEN3_VL_DECODER", "paged") != "oracle":
             # the paged sm_100a decoder: per-token three-axis rotary table and DeepStack taps ride on the prefill step
             backend = _build_backend(cfg, text, backend_name, comm)
         else:
@@ -595,11 +577,12 @@ def _can_load_gpu(spec: LoadSpec) -> bool:
     if _can_load_qwen3_vl(spec):            # a snapshot with a vision tower belongs to the vision-language provider
         return False
     cfg = probe_config(spec)
-    return cfg is not None and (_supported_on_gpu(cfg) or cfg.architecture is Architecture.QWEN35)
+    return cfg is not None and (gpu_supported(cfg) or cfg.architecture is Architecture.QWEN35)
 
 
 def _can_load_cpu(spec: LoadSpec) -> bool:
-    return not _can_load_qwen3_vl(spec) and probe_config(spec) is not None
+    cfg = probe_config(spec)
+    return not _can_load_qwen3_vl(spec) and cfg is not None and cfg.architecture is not Architecture.ZOBUNEX
 
 
 B200_LLAVA = TextLlmRegistration(lambda: _descriptor_vision("b200-llava", BACKEND_GPU),

@@ -13,23 +13,9 @@ import os
 
 import torch
 
-from ..models.llama import LlamaGpu, StepInputs
+from ..models.llama import LlamaGpu, StepInputs, splits_for as _splits_for
 from ..utils import tracing
 from .kv_pool import PagedKvPool, PagedSequence
-
-
-def _splits_for(batch: int, kv_heads: int, max_kv: int, sms: int = 148) -> int:
-    """KV splits of the decode attention: enough CTAs for `SWB_ATTN_CTAS_PER_SM` (default 2) per SM, never below one
-    64-key tile per split."""
-    import os
-
-    tiles = max(1, (max_kv + 63) // 64)
-    per_sm = max(0.25, float(os.environ.get("SWB_ATTN_CTAS_PER_SM", "2")))
-    want = max(1, int(per_sm * sms) // max(1, batch * kv_heads))
-    s = 1
-    while s * 2 <= min(want, tiles, 32):
-        s *= 2
-    return s
 
 
 def _bucket(batch: int, max_batch: int) -> int:
@@ -58,6 +44,9 @@ class ModelRunner:
         self.model, self.pool = model, pool
         self.max_batch, self.max_seq_len = max_batch, max_seq_len
         self.max_blocks = (max_seq_len + pool.block_size - 1) // pool.block_size
+        # models whose layers differ in KV heads or visible keys choose their splits themselves (one per layer)
+        self._splits = getattr(model, "decode_splits", None) or \
+            (lambda batch, max_kv: _splits_for(batch, model.hkv, max_kv))
         self.use_graphs = use_graphs and not getattr(model, "eager_only", False)   # mixture-of-experts routing is device side, so those models capture too
         dev = model.device
         model.ensure_rope(max_seq_len + 64)
@@ -95,14 +84,15 @@ class ModelRunner:
     # ---- prefill (eager, ragged) ------------------------------------------------------------------
     def prefill(self, seqs: list[PagedSequence], new_tokens: list[list[int]], *, want_logits: bool = False,
                 all_positions: bool = False, embed_overrides: list[tuple[list[int], torch.Tensor] | None] | None = None,
-                mrope_overrides: list | None = None):
+                mrope_overrides: list | None = None, want: list[list[int]] | None = None):
         """Appends new_tokens[i] to seqs[i] (any mix of lengths, including chunked / prefix-seeded sequences)
         and returns greedy next tokens [num_seqs] (or fp32 logits when want_logits). embed_overrides[i] =
         (positions within new_tokens[i], vectors [len(positions), hidden]) replaces those tokens' embeddings (the
         image placeholders of a vision-language prompt). mrope_overrides[i] = (positions [3, len(new_tokens[i])], next
         position, rows within new_tokens[i], taps) gives those tokens three-axis rotary positions and adds taps[l] to
         the residual stream at `rows` after decoder layer l; the sequence's later tokens continue at `next position`
-        (kept on the sequence as `rope_delta`)."""
+        (kept on the sequence as `rope_delta`). want[i] = places within new_tokens[i]: returns the fp32 logits of exactly
+        these places, sequence by sequence [sum of len(want[i]), vocab]."""
         dev = self.model.device
         ids, pos, slots, cu, kvl, rows = [], [], [], [0], [], []
         fresh = all(s.length == 0 for s in seqs)     # no earlier context: attention can read K / V from the QKV buffer
@@ -116,6 +106,8 @@ class ModelRunner:
             cu.append(cu[-1] + len(toks))
             kvl.append(s.length)
             rows.append(cu[-1] - 1)
+        if want is not None:
+            rows = [cu[i] + w for i, places in enumerate(want) for w in places]
         maxb = max(len(s.blocks) for s in seqs)
         table = torch.zeros((len(seqs), maxb), dtype=torch.int32)
         for i, s in enumerate(seqs):
@@ -130,7 +122,7 @@ class ModelRunner:
             block_table=table.to(dev), kv_lens=torch.tensor(kvl, dtype=torch.int32, device=dev),
             cu_q=None if decode else torch.tensor(cu, dtype=torch.int32, device=dev), max_q_len=max_q,
             num_seqs=len(seqs), decode=decode, fresh_prefill=fresh and not decode,
-            attn_splits=_splits_for(len(seqs), self.model.hkv, max(kvl)) if decode else 1,
+            attn_splits=self._splits(len(seqs), max(kvl)) if decode else 1,
             logits_rows=None if all_positions else torch.tensor(rows, dtype=torch.int64, device=dev))
         if embed_overrides is not None:
             er, ev = [], []
@@ -146,7 +138,7 @@ class ModelRunner:
         with tracing.span("runner.prefill", tokens=len(ids), seqs=len(seqs)):
             hidden = self.model.forward_hidden(inp, self.pool.data)
             self.launches_last = self.model.launches
-            if want_logits or all_positions:
+            if want_logits or all_positions or want is not None:
                 return self.model.logits(hidden)
             return self.model.greedy_tokens(hidden)
 
@@ -235,7 +227,7 @@ class ModelRunner:
                                               self._table.data_ptr(), stream_ptr())
         check(rc, "swb_decode_meta_unpack")
 
-    def _decode_body(self, B: int, splits: int, want_logits: bool, feedback: bool = False):
+    def _decode_body(self, B: int, splits, want_logits: bool, feedback: bool = False):
         self._unpack_meta(B, skip_ids=feedback, multi=feedback and self.model.device.type == "cuda")
         cap = self.decode_split if 0 < self.decode_split < B else B
         parts = []
@@ -281,7 +273,7 @@ class ModelRunner:
             self._meta_copy_done = torch.cuda.Event()
             self._meta_copy_done.record()
         self.h2d_bytes_last = self._host_meta.numel() * 4
-        splits = _splits_for(Bp, self.model.hkv, max_kv)
+        splits = self._splits(Bp, max_kv)
         key = (Bp, splits, want_logits)
         if not self.use_graphs or self.model.device.type != "cuda":
             toks, logits = self._decode_body(Bp, splits, want_logits)
@@ -326,7 +318,7 @@ class ModelRunner:
             max_kv = self._fill_decode_meta(seqs, tokens if k == 0 else [0] * B)
             host_all[k].copy_(self._host_meta)
         self.h2d_bytes_last = host_all.numel() * 4
-        splits = _splits_for(B, self.model.hkv, max_kv)
+        splits = self._splits(B, max_kv)
         first = torch.tensor(tokens, dtype=torch.int64)
         if dev.type != "cuda" or not self.use_graphs:
             out = torch.empty((n_steps, B), dtype=torch.int64, device=dev)

@@ -26,9 +26,14 @@ class Architecture(enum.Enum):
     DEEPSEEK_V2 = "deepseek_v2"  # multi-head latent attention + fine-grained MoE + YaRN
     QWEN35 = "qwen3_5"       # hybrid Gated-DeltaNet / gated full attention
     QWEN3_VL = "qwen3_vl"    # VLM-wrapped Qwen3 decoder with interleaved M-RoPE
+    ZOBUNEX = "zobunex"      # listed layers with a loop, chunked sink attention, sandwich layer norms, token-routed experts
 
     @staticmethod
     def from_config(cfg: dict[str, Any]) -> "Architecture":
+        if isinstance(cfg.get("architecture"), str):        # configs that list their layers name the design itself
+            if cfg["architecture"].lower() == "zobunex":
+                return Architecture.ZOBUNEX
+            raise Unsupported(f"unsupported architecture {cfg['architecture']!r}")
         archs = cfg.get("architectures")
         arch = archs[0] if isinstance(archs, list) and archs and isinstance(archs[0], str) else None
         model_type = cfg.get("model_type") if isinstance(cfg.get("model_type"), str) else None
@@ -125,6 +130,113 @@ class RopeSpec:
     interleaved: bool
 
 
+@dataclass(frozen=True)
+class AttentionSpec:
+    """One attention mixer: `rot_dims` leading dimensions of q and k are rotated, `chunk` > 0 limits a query to the keys of
+    its own run of `chunk` positions, `scale` multiplies the scores."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int
+    rot_dims: int
+    rot_base: float
+
+    @property
+    def groups(self) -> int:
+        return self.heads // self.kv_heads
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    experts: int
+    top: int
+    ff: int
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: AttentionSpec
+    mlp: ExpertsSpec | None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class StackConfig:
+    """A decoder described layer by layer, with an optional range of layers that runs several times in a row."""
+    layers: tuple[LayerSpec, ...]
+    loop: LoopSpec | None
+    logit_scale: float
+
+    def runs(self) -> list[tuple[int, bool]]:
+        """(layer, first layer of a loop pass) in execution order; every run owns a cache."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return [(i, False) for i in range(n)]
+        out = [(i, False) for i in range(lp.start)]
+        for _ in range(lp.times):
+            out += [(i, i == lp.start) for i in range(lp.start, lp.stop)]
+        return out + [(i, False) for i in range(lp.stop, n)]
+
+    @staticmethod
+    def from_json(top: dict[str, Any]) -> "StackConfig":
+        def need(d: Any, key: str, where: str) -> Any:
+            if not isinstance(d, dict) or d.get(key) is None:
+                raise ConfigError(f"config.json missing `{where}{key}`")
+            return d[key]
+
+        def count(d: Any, key: str, where: str, low: int = 1) -> int:
+            v = need(d, key, where)
+            if isinstance(v, bool) or not isinstance(v, (int, float)) or int(v) != v or v < low:
+                raise ConfigError(f"config.json: `{where}{key}` must be an integer >= {low}, not {v!r}")
+            return int(v)
+
+        def real(d: Any, key: str, where: str) -> float:
+            v = need(d, key, where)
+            if isinstance(v, bool) or not isinstance(v, (int, float)):
+                raise ConfigError(f"config.json: `{where}{key}` must be a number, not {v!r}")
+            return float(v)
+
+        layers = []
+        for i, lay in enumerate(need(top, "layers", "")):
+            at = f"layers[{i}]."
+            if need(lay, "type", at) != "attention":
+                raise Unsupported(f"config.json: `{at}type` {lay['type']!r}")
+            m, mw = need(lay, "mixer", at), at + "mixer."
+            rot, mask = m.get("rot"), m.get("mask")
+            spec = AttentionSpec(count(m, "heads", mw), count(m, "kv_heads", mw), count(m, "dim", mw), count(m, "vdim", mw),
+                                 real(m, "scale", mw), count(mask, "size", mw + "mask.") if mask else 0,
+                                 count(rot, "dims", mw + "rot.", 0) if rot else 0, real(rot, "base", mw + "rot.") if rot else 1.0)
+            if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim:
+                raise ConfigError(f"config.json: `{mw}` heads / kv_heads / rot.dims do not fit together")
+            mlp, f = None, lay.get("mlp")
+            if f is not None:
+                fw = at + "mlp."
+                if need(f, "kind", fw) != "moe":
+                    raise Unsupported(f"config.json: `{fw}kind` {f['kind']!r}")
+                r = need(f, "router", fw)
+                mlp = ExpertsSpec(count(r, "experts", fw + "router."), count(r, "top", fw + "router."),
+                                  count(need(f, "expert", fw), "ff", fw + "expert."))
+            layers.append(LayerSpec(spec, mlp))
+        if not layers:
+            raise ConfigError("config.json: `layers` is empty")
+        loop, lp = None, top.get("loop")
+        if lp:
+            loop = LoopSpec(count(lp, "start", "loop.", 0), count(lp, "stop", "loop.", 0), count(lp, "times", "loop."))
+            if loop.start > loop.stop or loop.stop > len(layers):
+                raise ConfigError("config.json: `loop` does not lie within the layers")
+            if loop.start == loop.stop:
+                loop = None
+        return StackConfig(tuple(layers), loop, real(top, "logit_scale", "") if top.get("logit_scale") is not None else 1.0)
+
+
 @dataclass
 class ModelConfig:
     hidden_size: int
@@ -150,12 +262,15 @@ class ModelConfig:
     mla: MlaConfig | None = None
     yarn: YarnConfig | None = None
     mrope_section: tuple[int, int, int] | None = None
+    stack: StackConfig | None = None
     raw: dict[str, Any] = field(default_factory=dict, repr=False)
 
     # ---- parsing ---------------------------------------------------------------------------
     @staticmethod
     def from_json(top: dict[str, Any]) -> "ModelConfig":
         arch = Architecture.from_config(top)
+        if arch is Architecture.ZOBUNEX:
+            return ModelConfig._from_stack(top, arch)
         v = top.get("text_config", top) if arch is Architecture.QWEN3_VL else top
 
         def integer(key: str) -> int | None:
@@ -245,6 +360,24 @@ class ModelConfig:
             raw=dict(top))
 
     @staticmethod
+    def _from_stack(top: dict[str, Any], arch: Architecture) -> "ModelConfig":
+        """A config that lists its layers; the flat fields hold the largest value over the layers."""
+        stack = StackConfig.from_json(top)
+        norm = top.get("norm") if isinstance(top.get("norm"), dict) else {}
+        for key, v in (("width", top.get("width")), ("vocab", top.get("vocab")), ("norm.eps", norm.get("eps"))):
+            if isinstance(v, bool) or not isinstance(v, (int, float)) or v <= 0:
+                raise ConfigError(f"config.json: `{key}` must be a positive number, not {v!r}")
+        mix = [lay.mixer for lay in stack.layers]
+        ffs = [lay.mlp.ff for lay in stack.layers if lay.mlp is not None]
+        mpe = top.get("max_position_embeddings")
+        return ModelConfig(
+            hidden_size=int(top["width"]), intermediate_size=max(ffs, default=0), num_layers=len(stack.layers),
+            num_heads=max(m.heads for m in mix), num_kv_heads=max(m.kv_heads for m in mix),
+            head_dim=max(max(m.dim, m.vdim) for m in mix), vocab_size=int(top["vocab"]), rms_norm_eps=float(norm["eps"]),
+            tie_word_embeddings=True, architecture=arch, max_position_embeddings=int(mpe) if isinstance(mpe, int) else 0,
+            stack=stack, raw=dict(top))
+
+    @staticmethod
     def from_dir(path: str | Path) -> "ModelConfig":
         p = Path(path)
         p = p / "config.json" if p.is_dir() else p
@@ -256,6 +389,8 @@ class ModelConfig:
     def to_json(self) -> dict[str, Any]:
         """A minimal HF-style config.json that round-trips through from_json."""
         d: dict[str, Any] = dict(self.raw) if self.raw else {}
+        if self.stack is not None:
+            return d
         d.update({
             "hidden_size": self.hidden_size, "intermediate_size": self.intermediate_size,
             "num_hidden_layers": self.num_layers, "num_attention_heads": self.num_heads,
@@ -276,6 +411,8 @@ class ModelConfig:
     # ---- derived quantities ----------------------------------------------------------------
     @property
     def groups(self) -> int:
+        if self.stack is not None:
+            return max(lay.mixer.groups for lay in self.stack.layers)
         return self.num_heads // self.num_kv_heads
 
     @property

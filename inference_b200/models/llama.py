@@ -34,7 +34,7 @@ class StepInputs:
     max_q_len: int
     num_seqs: int
     decode: bool = False               # q_len * gqa_group <= 16 for every sequence
-    attn_splits: int = 1
+    attn_splits: int | tuple[int, ...] = 1   # KV splits of the decode attention (one per layer when layers differ)
     logits_rows: torch.Tensor | None = None  # int64 rows of the hidden state to project; None => all rows
     fresh_prefill: bool = False        # every sequence starts at position 0 (context == this step's tokens)
     embed_rows: torch.Tensor | None = None    # int64 [R]: rows of the flat batch whose embedding is replaced ...
@@ -43,6 +43,18 @@ class StepInputs:
     #                                           this step: replaces the position-indexed table (three-axis rotary phases)
     deepstack: tuple[torch.Tensor, list[torch.Tensor]] | None = None   # (int64 rows [R], taps): taps[l] [R, H] is added
     #                                           to the residual stream at those rows after decoder layer l (Qwen3-VL)
+
+
+def splits_for(batch: int, kv_heads: int, max_kv: int, sms: int = 148) -> int:
+    """KV splits of the decode attention: enough CTAs for `SWB_ATTN_CTAS_PER_SM` (default 2) per SM, never below one
+    64-key tile per split."""
+    tiles = max(1, (max_kv + 63) // 64)
+    per_sm = max(0.25, float(os.environ.get("SWB_ATTN_CTAS_PER_SM", "2")))
+    want = max(1, int(per_sm * sms) // max(1, batch * kv_heads))
+    s = 1
+    while s * 2 <= min(want, tiles, 32):
+        s *= 2
+    return s
 
 
 @dataclass

@@ -6,7 +6,8 @@ import torch
 from .._native import kernels
 from .runtime import check, ptr, require_cuda, stream_ptr
 
-ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "swiglu_pairs": 3, "geglu_pairs": 4}
+ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "swiglu_pairs": 3, "geglu_pairs": 4, "relu2": 5}
+_PAIRS = (3, 4)     # gated pairs halve the width
 _WORKSPACES: dict[tuple[int, int], torch.Tensor] = {}
 WORKSPACE_BYTES = 64 * 1024 + (96 << 20)
 
@@ -33,7 +34,7 @@ def gemm_bf16(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = N
     assert a.stride(1) == 1 and w.stride(1) == 1
     T, K = a.shape
     N = w.shape[0]
-    n_out = N // 2 if ACT[act] >= 3 else N      # gated pairs halve the width
+    n_out = N // 2 if ACT[act] in _PAIRS else N
     if out is None:
         out = torch.empty((T, n_out), dtype=out_dtype, device=a.device)
     assert out.shape == (T, n_out) and out.stride(1) == 1 and out.dtype in (torch.bfloat16, torch.float32)
@@ -99,7 +100,7 @@ def gemm_bf16_normed(a: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | No
     require_cuda(a, w)
     T, K = a.shape
     N = w.shape[0]
-    n_out = N // 2 if ACT[act] >= 3 else N
+    n_out = N // 2 if ACT[act] in _PAIRS else N
     if out is None:
         out = torch.empty((T, n_out), dtype=torch.bfloat16, device=a.device)
     assert out.shape == (T, n_out) and out.dtype == torch.bfloat16 and a.stride(1) == 1 and w.stride(1) == 1
@@ -142,3 +143,22 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *
     lead = x.shape[:-1]
     y = gemm_bf16(x.reshape(-1, x.shape[-1]), w, bias=bias, **kw)
     return y.reshape(*lead, w.shape[0])
+
+
+def gemm_f32(a: torch.Tensor, w: torch.Tensor, *, act: str | None = None, out: torch.Tensor | None = None,
+             offsets: torch.Tensor | None = None, src: torch.Tensor | None = None, rows: int | None = None) -> torch.Tensor:
+    """True 32-bit product (no TF32): out[T, N] = act(a[T, K] @ w[N, K]^T). Grouped: w [G, N, K], offsets int32 [G + 1] on
+    the device, rows [offsets[g], offsets[g + 1]) use w[g] and read a[src[r]] (r itself without src); `rows` bounds them."""
+    require_cuda(a, w)
+    assert a.dtype == torch.float32 and w.dtype == torch.float32 and a.stride(1) == 1 and w.is_contiguous()
+    G = w.shape[0] if offsets is not None else 1
+    N, K = w.shape[-2:]
+    T = rows if rows is not None else a.shape[0]
+    assert a.shape[1] == K and (w.dim() == 3) == (offsets is not None)
+    if out is None:
+        out = torch.empty((T, N), dtype=torch.float32, device=a.device)
+    assert out.shape == (T, N) and out.dtype == torch.float32 and out.stride(1) == 1
+    rc = kernels().swb_gemm_f32(a.data_ptr(), a.stride(0), ptr(src), ptr(offsets), G, w.data_ptr(), K, out.data_ptr(),
+                                out.stride(0), T, N, K, ACT[act], stream_ptr())
+    check(rc, "swb_gemm_f32")
+    return out

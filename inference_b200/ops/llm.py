@@ -64,21 +64,28 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: torc
                   cos: torch.Tensor, sin: torch.Tensor, kcache: torch.Tensor | None, vcache: torch.Tensor | None,
                   n_heads: int, n_kv_heads: int, head_dim: int, *, rot_dim: int | None = None,
                   interleaved: bool = False, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
-                  norm_eps: float = 1e-6, norm_w_offset: float = 0.0, block_size: int = 16) -> None:
-    """In place on qkv [T, (Hq + 2 Hkv) * D]: per-head q/k RMSNorm (optional), RoPE on q and k; k and v are
-    also written to the paged cache [blocks, Hkv, block_size, D] at slot_mapping (int64; -1 = skip)."""
+                  norm_eps: float = 1e-6, norm_w_offset: float = 0.0, block_size: int = 16,
+                  v_dim: int | None = None) -> None:
+    """In place on qkv [T, (Hq + Hkv) * D + Hkv * v_dim]: per-head q/k RMSNorm (optional), RoPE on q and k; k and v are
+    also written to the paged cache [blocks, Hkv, block_size, D | v_dim] at slot_mapping (int64; -1 = skip). bf16, or
+    fp32 throughout (projection and caches). v_dim defaults to D."""
     require_cuda(qkv, positions, cos, sin)
     T = qkv.shape[0]
-    assert qkv.stride(1) == 1 and positions.dtype == torch.int32
+    vd = head_dim if v_dim is None else v_dim
+    assert qkv.stride(1) == 1 and positions.dtype == torch.int32 and qkv.dtype in (torch.bfloat16, torch.float32)
+    assert qkv.shape[1] >= (n_heads + n_kv_heads) * head_dim + n_kv_heads * vd
+    for c in (kcache, vcache):
+        assert c is None or c.dtype == qkv.dtype
     assert cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous()
     if slot_mapping is not None:
         assert slot_mapping.dtype == torch.int64
     rd = rot_dim if rot_dim is not None else head_dim
     assert cos.shape[-1] == rd // 2
-    rc = kernels().swb_rope_kv_write(qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), ptr(slot_mapping),
-                                     cos.data_ptr(), sin.data_ptr(), rd, 1 if interleaved else 0, ptr(q_norm),
-                                     ptr(k_norm), norm_eps, norm_w_offset, ptr(kcache), ptr(vcache), block_size, T,
-                                     n_heads, n_kv_heads, head_dim, stream_ptr())
+    rc = kernels().swb_rope_kv_write_ex(qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), ptr(slot_mapping),
+                                        cos.data_ptr(), sin.data_ptr(), rd, 1 if interleaved else 0, ptr(q_norm),
+                                        ptr(k_norm), norm_eps, norm_w_offset, ptr(kcache), ptr(vcache), block_size, T,
+                                        n_heads, n_kv_heads, head_dim, vd, 1 if qkv.dtype == torch.float32 else 0,
+                                        stream_ptr())
     check(rc, "swb_rope_kv_write")
 
 
