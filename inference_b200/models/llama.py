@@ -327,13 +327,23 @@ class LlamaGpu:
             self.lm_head = rnd(self.vocab_local, H)
         sandwich = cfg.architecture.sandwich_norms
         self.layers = []
+        P = self.comm.world
         for _ in range(cfg.num_layers):
+            moe = None
+            if cfg.moe is not None:
+                E, f = cfg.moe.num_experts, cfg.moe.moe_intermediate_size // P
+                fs = cfg.moe.shared_expert_intermediate_size // P
+                router = torch.empty(E, H, dtype=torch.bfloat16, device=dev).normal_(0.0, std, generator=ge)
+                moe = MoeWeights(router=router, gate_up=rnd(E, 2 * f, H), down=rnd(E, H, f),
+                                 shared_gate_up=rnd(2 * fs, H) if fs else None, shared_down=rnd(H, fs) if fs else None,
+                                 shared_gate=None)
+            ffn = 8 if moe is not None else self.ffn        # sparse layers keep no dense FFN
             self.layers.append(LayerWeights(
                 ln1=ones(H), qkv=rnd((self.hq + 2 * self.hkv) * D, H), qkv_bias=None,
                 q_norm=torch.ones(D, dtype=torch.bfloat16, device=dev) if cfg.architecture.has_qk_norm else None,
                 k_norm=torch.ones(D, dtype=torch.bfloat16, device=dev) if cfg.architecture.has_qk_norm else None,
                 o=rnd(H, self.hq * D), post_attn_ln=ones(H) if sandwich else None, ln2=ones(H),
-                gate_up=rnd(2 * self.ffn, H), down=rnd(H, self.ffn), post_mlp_ln=ones(H) if sandwich else None))
+                gate_up=rnd(2 * ffn, H), down=rnd(H, ffn), post_mlp_ln=ones(H) if sandwich else None, moe=moe))
         self.fold_norms()
         return self
 

@@ -208,3 +208,40 @@ def test_restatement_sees_chunk_edges_and_sinks():
     assert torch.allclose(a[0], manual)
     assert not torch.allclose(a, ref.attention(q, k, v, at, 0.5, 36, torch.zeros(2, dtype=torch.float64)), atol=1e-3)
     assert not torch.allclose(a, ref.attention(q, k, v, at, 0.5, 37, None), atol=1e-3)
+
+
+def _drop(cfg, w, name, value):
+    return cfg, {k: (torch.full_like(t, value) if k.endswith(name) else t) for k, t in w.items()}
+
+
+def _chunks(cfg, w, by):
+    for lay in cfg["layers"]:
+        lay["mixer"]["mask"]["size"] += by
+    return cfg, w
+
+
+def _swap_loop(cfg, w):
+    W = cfg["width"]
+    return cfg, {**w, "loop.in": torch.cat([w["loop.in"][:, W:], w["loop.in"][:, :W]], 1)}
+
+
+def _one_pass_less(cfg, w):
+    cfg["loop"]["times"] -= 1
+    return cfg, w
+
+
+def _next_row(cfg, w):
+    return cfg, {k: (t.roll(1, 0) if k.endswith("table") else t) for k, t in w.items()}
+
+
+@pytest.mark.parametrize("mistake", [lambda c, w: _drop(c, w, ".sink", -60.0), lambda c, w: _chunks(c, w, 1),
+                                     lambda c, w: _chunks(c, w, -1), lambda c, w: _drop(c, w, "norm1b.b", 0.0), _swap_loop,
+                                     _one_pass_less, _next_row])
+def test_test_models_are_sensitive_to_mistakes(mistake):
+    """A mistake planted in the restatement moves the logits of the test models far beyond the tolerances of the GPU tests
+    (3e-2 in bf16)."""
+    tokens = torch.randint(0, 321, (139,), generator=torch.Generator().manual_seed(2)).tolist()
+    cfg, w = ref.model_a(), ref.random_weights(ref.model_a(), seed=ord("a"))
+    good = ref.run(cfg, w, tokens)[0]
+    bad = ref.run(*mistake(copy.deepcopy(cfg), w), tokens)[0]
+    assert float((good - bad).square().mean().sqrt() / good.square().mean().sqrt()) > 0.15

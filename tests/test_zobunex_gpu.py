@@ -427,7 +427,7 @@ def test_greedy_generation_loops(dtype):
     for chunk in (0, 16):
         reqs = [ContinuousRequest(p, 12) for p in prompts]
         runs.append([r.tokens for r in generate_continuous(b, reqs, ContinuousConfig(max_batch=3, prefill_chunk=chunk))])
-    cache = PrefixCache(b, capacity=4)
+    cache = PrefixCache(b, capacity=8)
     runs.append([generate_cached(b, cache, p, cfg).tokens for p in prompts])
     runs.append([generate_cached(b, cache, p, cfg).tokens for p in prompts])       # every prompt again, from cached pages
     assert cache.stats.hits > 0
