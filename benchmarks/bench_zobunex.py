@@ -209,6 +209,7 @@ def kernel_rows(size, emit):
     # ---- experts --------------------------------------------------------------------------------------------------------
     from inference_b200.models import ModelConfig
     from inference_b200.models.llama import LlamaGpu, MoeWeights
+    from inference_b200.models.zobunex import ZobunexGpu
     m = MoeWeights(rnd(E, W, std=0.02), rnd(E, 2 * ff, W, std=0.02), rnd(E, W, ff, std=0.02), None, None, None)
     like = LlamaGpu.__new__(LlamaGpu)
     like.cfg = ModelConfig.from_json(llama_config(size))
@@ -217,7 +218,7 @@ def kernel_rows(size, emit):
     table = torch.rand((V, E), generator=gen, device=dev).topk(top, 1).indices.int()[None].contiguous()
     for T in (1, 8, 64, 256, 1024, 8192):
         ids = torch.randint(0, V, (T,), generator=gen, device=dev)
-        padded = T * top > 16 * E
+        padded = T * top > ZobunexGpu.rows_per_expert_small * E
         plan = ops.table_routing(ids, table, E, padded=padded)[0]
         hx = rnd(T, W)
         h = rnd(plan.rows, W) if padded else hx

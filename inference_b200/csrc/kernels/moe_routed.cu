@@ -24,7 +24,8 @@ __global__ void __launch_bounds__(1024) moe_table_plan_kernel(const long long* _
                                                               const int* __restrict__ tables, int vocab, int top, int E,
                                                               int pad, int* dest, int* src, int* offsets, int* active,
                                                               int* tile_group, int rows_cap) {
-  pdl_launch_dependents();
+  // No early trigger here: the kernels of the step start after this grid has finished, so the grouped kernels may read the
+  // plan before they wait for the rows they multiply. (Prefetching the weight rows into L2 there as well was slower.)
   pdl_wait();
   extern __shared__ int sm[];
   int* count = sm;          // [E] pairs per expert, then the write cursor
@@ -200,13 +201,14 @@ __device__ __forceinline__ void grouped_pass(const GroupedRowsParams& p, const b
 template <int MT>
 __global__ void __launch_bounds__(GR_WARPS * 32) grouped_rows_kernel(const GroupedRowsParams p) {
   pdl_launch_dependents();
-  pdl_wait();
   __shared__ float red[GR_WARPS * 32 * (16 * MT + 1)];
   const int e = p.active[blockIdx.y];
-  if (e < 0) return;
-  const int lo = p.offsets[e], hi = p.offsets[e + 1];
   const int f0 = blockIdx.x * (16 * MT);
-  const bf16* wrow = p.w + (size_t)e * p.N * p.K;
+  const bf16* wrow = p.w + (size_t)max(e, 0) * p.N * p.K;
+  int lo = 0, hi = 0;
+  if (e >= 0) lo = p.offsets[e], hi = p.offsets[e + 1];
+  pdl_wait();
+  if (e < 0) return;
   for (int r = lo; r < hi; r += 32) {
     const int n = min(32, hi - r);
     if (n <= 8) grouped_pass<MT, 1>(p, wrow, f0, r, n, red);

@@ -4,8 +4,8 @@
 //     x   += norm1(branch)            branch = a projection output row, or the mean of a token's expert output rows
 //     out  = norm2(x) * out_scale     or the stream itself, for a projection that reads it un-normalised
 // A layer with norms before and after each sublayer then needs one such launch per sublayer. Both norms are layer norms
-// (mean removed, weight and bias) or RMS norms, computed in fp32 on the row held in registers, two passes (mean, then
-// squared deviations). The output is stored once per token, or to every row of an expert-sorted buffer that the token's
+// (mean removed, weight and bias) or RMS norms, computed in fp32 on the row held in registers (squared deviations from the
+// mean, never a difference of large sums). The output is stored once per token, or to every row of an expert-sorted buffer that the token's
 // routing names, so the gather in front of a grouped GEMM costs no launch of its own.
 // Rows are padded to a multiple of 8 columns; padding columns of the stream, the weights and the outputs are zero and do
 // not enter the statistics.
@@ -65,29 +65,63 @@ __device__ __forceinline__ float block_total(float v, float* red) {
   return warp_sum(lane < THREADS / 32 ? red[lane] : 0.f);
 }
 
+// Mean and sum of squared deviations of a row whose threads hold N values each: every thread takes those of its own
+// values, then equal-sized groups are merged pairwise (M2 = M2a + M2b + (mean_a - mean_b)^2 n / 2), so one barrier serves
+// both and no large sums cancel.
+template <int THREADS, int N>
+__device__ __forceinline__ float2 block_moments(const float* v, float* red) {
+  float m = 0.f, q = 0.f, n = (float)N;
+#pragma unroll
+  for (int i = 0; i < N; ++i) m += v[i];
+  m *= 1.f / N;
+#pragma unroll
+  for (int i = 0; i < N; ++i) q += (v[i] - m) * (v[i] - m);
+  auto merge = [&](int o) {
+    const float mo = __shfl_xor_sync(0xffffffffu, m, o), qo = __shfl_xor_sync(0xffffffffu, q, o), d = m - mo;
+    q += qo + d * d * (0.5f * n);
+    m = 0.5f * (m + mo);
+    n *= 2.f;
+  };
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) merge(o);
+  constexpr int WARPS = THREADS / 32;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (lane == 0) red[warp] = m, red[32 + warp] = q;
+  __syncthreads();
+  m = red[lane % WARPS], q = red[32 + lane % WARPS];
+#pragma unroll
+  for (int o = WARPS / 2; o > 0; o >>= 1) merge(o);
+  return make_float2(m, q);
+}
+
 // v <- norm(v) * w + b over the first H columns of the row (thread t owns float4 columns t, t + THREADS, ...)
 template <int THREADS, int VPT>
 __device__ __forceinline__ void norm_row(float4* v, const float* __restrict__ w, const float* __restrict__ b, int H, int nvec,
                                          float eps, int center, float* red) {
-  float mean = 0.f;
-  if (center) {
+  float mean = 0.f, ss = 0.f;
+  const bool full = center && H == THREADS * VPT * 4;     // every thread holds the same number of columns
+  if (full) {
+    const float2 mq = block_moments<THREADS, VPT * 4>(reinterpret_cast<const float*>(v), red);
+    mean = mq.x, ss = mq.y;
+  } else if (center) {
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);   // padding columns hold zeros
     mean = block_total<THREADS>(s, red) / (float)H;
     red += 32;
   }
-  float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (threadIdx.x + i * THREADS) * 4;
     v[i].x -= mean, v[i].y -= mean, v[i].z -= mean, v[i].w -= mean;
+    if (full) continue;
     if (c < H) ss += v[i].x * v[i].x;
     if (c + 1 < H) ss += v[i].y * v[i].y;
     if (c + 2 < H) ss += v[i].z * v[i].z;
     if (c + 3 < H) ss += v[i].w * v[i].w;
   }
-  const float r = rsqrtf(block_total<THREADS>(ss, red) / (float)H + eps);
+  if (!full) ss = block_total<THREADS>(ss, red);
+  const float r = rsqrtf(ss / (float)H + eps);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c4 = threadIdx.x + i * THREADS;

@@ -107,7 +107,6 @@ class ZobunexGpu:
     # ---- weights ----------------------------------------------------------------------------------------------
     def load_state_dict(self, weights: dict[str, torch.Tensor]) -> "ZobunexGpu":
         W, V = self.width, self.cfg.vocab_size
-        left = set(weights)
 
         def get(name: str, *shape: int) -> torch.Tensor:
             if name not in weights:
@@ -115,7 +114,6 @@ class ZobunexGpu:
             t = weights[name]
             if tuple(t.shape) != shape:
                 raise LoadError(f"tensor {name} has shape {tuple(t.shape)}, expected {shape}")
-            left.discard(name)
             return t
 
         def norm(name: str) -> NormWeights:
@@ -140,8 +138,6 @@ class ZobunexGpu:
                 self._set_experts(lay, e, [get(f"{p}e{x}.up", e.ff, W) for x in range(e.experts)],
                                   [get(f"{p}e{x}.down", W, e.ff) for x in range(e.experts)], table, tables)
             self.layers.append(lay)
-        if left:
-            raise LoadError(f"unexpected tensors: {', '.join(sorted(left)[:4])}" + (" ..." if len(left) > 4 else ""))
         self._stack_tables(tables)
         return self
 
@@ -236,7 +232,7 @@ class ZobunexGpu:
             self.launches += 1
         return plans
 
-    rows_per_expert_small = 16
+    rows_per_expert_small = 4      # measured on B200: above it the padded tiles win although most of their rows are empty
 
     def _attention(self, lay: _Layer, h: torch.Tensor, inp: StepInputs, kv, splits: int) -> torch.Tensor:
         m, T = lay.spec, h.shape[0]

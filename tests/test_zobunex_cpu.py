@@ -108,7 +108,7 @@ def test_weight_errors():
         return ZobunexGpu(_cfg(), device=torch.device("cpu")).load_state_dict(w)
     good = ref.random_weights(ref.model_a())
     load(good)
-    for name, t in (("l0.mix.sink", None), ("loop.in", torch.zeros(3, 3)), ("l9.extra", torch.zeros(1)),
+    for name, t in (("l0.mix.sink", None), ("loop.in", torch.zeros(3, 3)), ("l2.norm2b.b", None),
                     ("l0.mlp.table", good["l0.mlp.table"] + 5)):
         w = dict(good)
         if t is None:

@@ -29,7 +29,8 @@ def rnd(*shape, seed=0, dtype=torch.float32, std=1.0):
 
 
 # ---- mechanisms alone -----------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("H,Hp", [(160, 160), (90, 96), (1, 8), (1030, 1032), (4096, 4096), (9000, 9000)])
+@pytest.mark.parametrize("H,Hp", [(160, 160), (90, 96), (1, 8), (512, 512), (1030, 1032), (1024, 1024), (2048, 2048), (4096, 4096),
+                                  (8192, 8192), (9000, 9000), (16384, 16384)])
 @pytest.mark.parametrize("center", [True, False])
 def test_stream_norm_joins_norms_and_writes(H, Hp, center):
     from inference_b200 import ops
