@@ -43,8 +43,9 @@ __device__ __forceinline__ uint32_t q_off(int r, int c) { return (uint32_t)(r * 
 
 // 1 / softmax denominator of a row with running max M (log2 units) and sum L relative to it; the numerators are relative
 // to M as well. A sink adds exp(sink) to the denominator; one far above every score makes the weights vanish.
+template <bool EXT>
 __device__ __forceinline__ float softmax_inv(const AttnParams& p, int head, float M, float L) {
-  if (p.sink) {
+  if (EXT && p.sink) {
     const float sk = p.sink[head] * 1.4426950408889634f;
     const float top = fmaxf(sk, M), e = exp2f(M - top);
     return e / (L * e + exp2f(sk - top));
@@ -52,6 +53,8 @@ __device__ __forceinline__ float softmax_inv(const AttnParams& p, int head, floa
   return L > 0.f ? 1.f / L : 0.f;
 }
 
+// EXT: chunked masking and sinks. FULL: q / k and v are HD wide (their loop bounds are then constants).
+template <bool EXT, bool FULL>
 __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                               const __grid_constant__ CUtensorMap tmap_v,
                                                               const AttnParams p) {
@@ -89,19 +92,20 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   const int nrows = min(16, q_len * p.G);
   const int causal_shift = kv_len - q_len;
   // chunked attention starts at the tile that holds the first key of the first query's chunk
-  const int tile_lo = p.chunk > 0 ? max(causal_shift, 0) / p.chunk * p.chunk / KV_TILE : 0;
+  const int tile_lo = (EXT && p.chunk > 0) ? max(causal_shift, 0) / p.chunk * p.chunk / KV_TILE : 0;
   const int total_tiles = (kv_len + KV_TILE - 1) / KV_TILE;
   const int per = (total_tiles - tile_lo + p.num_splits - 1) / p.num_splits;
   const int t0 = tile_lo + split * per;
   const int n_tiles = max(0, min(total_tiles, t0 + per) - t0);
-  const int k_steps = (p.k_dim + 15) >> 4, v_steps = (p.v_dim + 15) >> 4;   // 16-column MMA steps that hold data
-  const int k_halves = (p.k_dim + 63) >> 6, v_halves = (p.v_dim + 63) >> 6;
+  const int k_dim = FULL ? HD : p.k_dim, v_dim = FULL ? HD : p.v_dim;
+  const int k_steps = (k_dim + 15) >> 4, v_steps = (v_dim + 15) >> 4;   // 16-column MMA steps that hold data
+  const int k_halves = (k_dim + 63) >> 6, v_halves = (v_dim + 63) >> 6;
 
   // Q rows -> shared (row r = query token r / G, head kvh * G + r % G), zero rows past nrows
   for (int idx = threadIdx.x; idx < 256; idx += blockDim.x) {
     const int row = idx >> 4, c = idx & 15;
     uint4 val = make_uint4(0, 0, 0, 0);
-    if (row < nrows && c * 8 < p.k_dim) {
+    if (row < nrows && c * 8 < k_dim) {
       const int qtok = row / p.G, hg = row % p.G;
       val = *reinterpret_cast<const uint4*>(p.q + (size_t)(q_start + qtok) * p.q_stride_tok +
                                             (size_t)(kvh * p.G + hg) * p.q_stride_head + c * 8);
@@ -197,7 +201,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           const int qtok = row / p.G;
           const int qpos = qtok + causal_shift;
           const bool ok = (col < kv_len) && (!p.causal || col <= qpos) &&
-                          (p.chunk <= 0 || col >= qpos / p.chunk * p.chunk);
+                          (!EXT || p.chunk <= 0 || col >= qpos / p.chunk * p.chunk);
           s[nt][e] = ok ? val : -INFINITY;
         }
       }
@@ -291,9 +295,9 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       }
       const int qtok = row / p.G, hg = row % p.G;
       if (p.num_splits == 1) {
-        const float inv = softmax_inv(p, kvh * p.G + hg, M, L);
-        if (d < p.v_dim)
-          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] =
+        const float inv = softmax_inv<EXT>(p, kvh * p.G + hg, M, L);
+        if (d < v_dim)
+          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] =
               __float2bfloat16(acc * inv);
       } else {
         const size_t base = (((size_t)seq * p.Hkv + kvh) * p.num_splits + split) * 16 + row;
@@ -357,11 +361,11 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         sSc[row * 32 + sp] = sc;
         L += sc * sL[row * 32 + sp];
       }
-      const float inv = softmax_inv(p, kvh * p.G + row % p.G, M, L);
+      const float inv = softmax_inv<EXT>(p, kvh * p.G + row % p.G, M, L);
       for (int sp = 0; sp < S; ++sp) sSc[row * 32 + sp] *= inv;
     }
     __syncthreads();
-    if ((int)threadIdx.x < p.v_dim) {
+    if ((int)threadIdx.x < v_dim) {
       const int d = threadIdx.x;
       if (small) {
 #pragma unroll
@@ -372,7 +376,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
             for (int sp = 0; sp < 8; ++sp)
               if (sp < S) acc += sSc[row * 32 + sp] * po[row][sp];
             const int qtok = row / p.G, hg = row % p.G;
-            p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] = __float2bfloat16(acc);
+            p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] = __float2bfloat16(acc);
           }
         }
       } else {
@@ -382,7 +386,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           for (int sp = 0; sp < S; ++sp)
             acc += sSc[row * 32 + sp] * __ldcg(p.part_o + (base0 + (size_t)sp * 16 + row) * HD + d);
           const int qtok = row / p.G, hg = row % p.G;
-          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * p.v_dim + d] = __float2bfloat16(acc);
+          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] = __float2bfloat16(acc);
         }
       }
     }
@@ -394,14 +398,17 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 
 // Launches the TMA decode kernel; kcache / vcache are one layer's [blocks, Hkv, 16, 128] tensors.
 int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t stream) {
-  static bool configured[64] = {false};
+  const bool ext = p.chunk > 0 || p.sink != nullptr, full = p.k_dim == HD && p.v_dim == HD;
+  const int which = full ? (ext ? 1 : 0) : 2;
+  auto kernel = which == 0 ? attn_decode_tma_kernel<false, true>
+                           : which == 1 ? attn_decode_tma_kernel<true, true> : attn_decode_tma_kernel<true, false>;
+  static bool configured[3][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e =
-        cudaFuncSetAttribute(attn_decode_tma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+  if (dev >= 0 && dev < 64 && !configured[which][dev]) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
     if (e != cudaSuccess) return -(int)e;
-    configured[dev] = true;
+    configured[which][dev] = true;
   }
   CUtensorMap tk, tv;
   const int rows = num_blocks * p.Hkv * 16;
@@ -432,10 +439,10 @@ int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t str
     }
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, attn_decode_tma_kernel, tk, tv, pc);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, tk, tv, pc);
     return e == cudaSuccess ? 0 : -(int)e;
   }
-  return launch_kernel(attn_decode_tma_kernel, grid, dim3(160), SMEM_BYTES, stream, tk, tv, p);
+  return launch_kernel(kernel, grid, dim3(160), SMEM_BYTES, stream, tk, tv, p);
 }
 
 }  // namespace swb

@@ -239,7 +239,7 @@ def test_chunk_attention_prefill(H, G, D, Dv, mode, chunk):
     assert _attention_case(torch.bfloat16, H, G, D, Dv, chunk, lens, q_lens, mode) < OP_TOL[torch.bfloat16]
 
 
-@pytest.mark.parametrize("chunk", [16, 37, 120, 128, 300])
+@pytest.mark.parametrize("chunk", [16, 37, 90, 128, 300])
 @pytest.mark.parametrize("plant", [-17, -1, 0, 1])
 @pytest.mark.parametrize("mode", ["fresh", "paged", "decode"])
 def test_chunk_edges_carry_the_weight(chunk, plant, mode):
