@@ -95,9 +95,9 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
                                  c_int, c_void_p])
     sig("swb_stream_norm", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p,
                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                            c_float, c_int, c_void_p])
+                            c_float, c_int, c_int, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_void_p])
     sig("swb_stream_embed", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int,
-                             c_int, c_int, c_void_p])
+                             c_float, c_int, c_int, c_void_p])
     sig("swb_moe_table_plan", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_void_p, c_int, c_void_p])
     sig("swb_gemm_grouped_rows", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
@@ -105,7 +105,18 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
     sig("swb_gemm_f32", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                          c_int, c_void_p])
     sig("swb_attn_simple", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p,
-                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p])
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p])
+    sig("swb_head_product_simple", [c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int,
+                                    c_int, c_int, c_int, c_int, c_void_p])
+    sig("swb_latent_prep", [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    sig("swb_delta_prep", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    sig("swb_delta_scan", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                           c_void_p, c_void_p])
+    sig("swb_delta_post", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p,
+                           c_int, c_void_p, c_int, c_void_p])
+    sig("swb_poly_norm", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p])
     sig("swb_attn_ext", [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_int, c_int, c_int,
                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
                          c_int, c_int, c_void_p, c_size_t, c_void_p])
@@ -154,7 +165,7 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
                                       c_int, c_int, c_int, c_void_p])
     sig("swb_gemm_peer_max_ctas", [])
     sig("swb_decode_meta_unpack", [c_void_p, c_ll, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                                   c_void_p, c_void_p, c_void_p])
+                                   c_void_p, c_void_p, c_void_p, c_void_p])
     sig("swb_decode_step_tail", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     sig("swb_gemm_bf16_grouped", [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                   c_int, c_void_p])

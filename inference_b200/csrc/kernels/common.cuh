@@ -324,6 +324,24 @@ __device__ __forceinline__ float relu2_f(float x) {
   return r * r;
 }
 
+// Sequence of flat token t: the last one whose first token is not after t (empty sequences are skipped over), or t / uniform.
+__device__ __forceinline__ int seq_of_token(const int* cu_q, int num_seqs, int uniform, int t) {
+  if (!cu_q) return t / uniform;
+  int lo = 0, hi = num_seqs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= t) lo = mid;
+    else hi = mid - 1;
+  }
+  return lo;
+}
+
+// element conversions of kernels that run in bf16 or fp32
+__device__ __forceinline__ float to_f(float x) { return x; }
+__device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
+__device__ __forceinline__ void from_f(float& d, float x) { d = x; }
+__device__ __forceinline__ void from_f(bf16& d, float x) { d = __float2bfloat16(x); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -9,11 +9,11 @@ namespace swb {
 SWB_REGISTER_STATUS_UNIT(decode_meta);
 namespace {
 
-// meta rows: [ids MB][positions MB][slots MB][kv lens MB][block table MB * mb], int32.
+// meta rows: [ids MB][positions MB][slots MB][kv lens MB][state slots MB, only with `states`][block table MB * mb], int32.
 __global__ void __launch_bounds__(256) decode_meta_unpack_kernel(const int* __restrict__ meta_all, long long n_meta,
                                                                  const int* __restrict__ step_ptr, int MB, int B,
                                                                  int mb, long long* ids, int* pos, long long* slots,
-                                                                 int* kvl, int* table) {
+                                                                 int* kvl, int* states, int* table) {
   pdl_launch_dependents();
   pdl_wait(TL_META);
   const int step = step_ptr ? *step_ptr : 0;
@@ -21,13 +21,14 @@ __global__ void __launch_bounds__(256) decode_meta_unpack_kernel(const int* __re
   const int n_table = B * mb;
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n_table + B; i += gridDim.x * blockDim.x) {
     if (i < n_table) {
-      table[i] = m[4 * MB + i];
+      table[i] = m[(states ? 5 : 4) * MB + i];
     } else {
       const int r = i - n_table;
       if (ids) ids[r] = m[r];
       pos[r] = m[MB + r];
       slots[r] = m[2 * MB + r];
       kvl[r] = m[3 * MB + r];
+      if (states) states[r] = m[4 * MB + r];
     }
   }
 }
@@ -53,7 +54,7 @@ __global__ void __launch_bounds__(128) decode_step_tail_kernel(const long long* 
 extern "C" {
 
 int swb_decode_meta_unpack(const void* meta_all, long long n_meta, const void* step_ptr, int MB, int B, int mb,
-                           void* ids, void* pos, void* slots, void* kvl, void* table, void* stream) {
+                           void* ids, void* pos, void* slots, void* kvl, void* states, void* table, void* stream) {
   using namespace swb;
   if (B <= 0 || B > MB || mb <= 0) return -3;
   const int n = B * mb + B;
@@ -61,7 +62,8 @@ int swb_decode_meta_unpack(const void* meta_all, long long n_meta, const void* s
   return launch_kernel(decode_meta_unpack_kernel, dim3(grid), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
                        reinterpret_cast<const int*>(meta_all), n_meta, reinterpret_cast<const int*>(step_ptr), MB, B,
                        mb, reinterpret_cast<long long*>(ids), reinterpret_cast<int*>(pos),
-                       reinterpret_cast<long long*>(slots), reinterpret_cast<int*>(kvl), reinterpret_cast<int*>(table));
+                       reinterpret_cast<long long*>(slots), reinterpret_cast<int*>(kvl), reinterpret_cast<int*>(states),
+                       reinterpret_cast<int*>(table));
 }
 
 int swb_decode_step_tail(const void* tokens, void* ids, void* out_all, void* step_ptr, int B, void* stream) {

@@ -10,11 +10,6 @@ SWB_REGISTER_STATUS_UNIT(f32_ops);
 
 namespace {
 
-__device__ __forceinline__ float to_f(float x) { return x; }
-__device__ __forceinline__ float to_f(bf16 x) { return __bfloat162float(x); }
-__device__ __forceinline__ void from_f(float& d, float x) { d = x; }
-__device__ __forceinline__ void from_f(bf16& d, float x) { d = __float2bfloat16(x); }
-
 constexpr int TM = 64, TN = 64, TK = 16;
 
 // out[r, n] = act(sum_k a[src ? src[r] : r, k] w[e, n, k]); 64 x 64 tile, 4 x 4 per thread. Grouped: blockIdx.z = expert.
@@ -72,42 +67,31 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 }
 
 constexpr int AW = 4;          // warps per CTA: keys are dealt out to them
-constexpr int MAX_PER_LANE = 16;   // head widths up to 512
+constexpr int MAX_PER_LANE = 32;   // head widths up to 1024
 
 // One CTA per (query token, head). Each warp runs an online softmax over its share of the visible keys; lanes split the
 // head dimension. The sink joins the denominator when the four partial results are merged.
-template <typename E>
+template <typename E, int PL>
 __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restrict__ q, long long q_stride_tok,
                                                               const E* __restrict__ kc, const E* __restrict__ vc, E* out,
                                                               long long out_stride_tok, const int* __restrict__ block_table,
                                                               int max_blocks, int block_size, const int* __restrict__ cu_q,
                                                               const int* __restrict__ kv_lens, int num_seqs, int uniform_q,
-                                                              int Hq, int Hkv, int D, int Dv, float scale, int chunk,
+                                                              int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
                                                               const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, head = blockIdx.y, kvh = head / (Hq / Hkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  int seq = 0;
-  if (cu_q) {                    // the last sequence whose first token is not after t (empty sequences are skipped over)
-    int lo = 0, hi = num_seqs - 1;
-    while (lo < hi) {
-      const int mid = (lo + hi + 1) >> 1;
-      if (cu_q[mid] <= t) lo = mid;
-      else hi = mid - 1;
-    }
-    seq = lo;
-  } else {
-    seq = t / uniform_q;
-  }
+  const int seq = seq_of_token(cu_q, num_seqs, uniform_q, t);
   const int q0 = cu_q ? cu_q[seq] : seq * uniform_q, q_len = cu_q ? cu_q[seq + 1] - q0 : uniform_q;
   const int pos = kv_lens[seq] - q_len + (t - q0);
   const int first = chunk > 0 ? pos / chunk * chunk : 0;
   const int* table = block_table + (size_t)seq * max_blocks;
   const E* qr = q + (size_t)t * q_stride_tok + (size_t)head * D;
-  float qv[MAX_PER_LANE], o[MAX_PER_LANE];
+  float qv[PL], o[PL];
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) {
+  for (int i = 0; i < PL; ++i) {
     const int d = lane + i * 32;
     qv[i] = d < D ? to_f(qr[d]) : 0.f;
     o[i] = 0.f;
@@ -116,10 +100,10 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
   for (int j = first + warp; j <= pos; j += AW) {
     const size_t row = ((size_t)table[j / block_size] * Hkv + kvh) * block_size + j % block_size;
     const E* kr = kc + row * D;
-    const E* vr = vc + row * Dv;
+    const E* vr = vc + row * v_row;
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
+    for (int i = 0; i < PL; ++i) {
       const int d = lane + i * 32;
       if (d < D) s = fmaf(qv[i], to_f(kr[d]), s);
     }
@@ -128,14 +112,14 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
     l = l * f + e;
     m = mn;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
+    for (int i = 0; i < PL; ++i) {
       const int d = lane + i * 32;
       if (d < Dv) o[i] = fmaf(e, to_f(vr[d]), o[i] * f);
     }
   }
-  __shared__ float so[AW][32 * MAX_PER_LANE], sm[AW], sl[AW];
+  __shared__ float so[AW][32 * PL], sm[AW], sl[AW];
 #pragma unroll
-  for (int i = 0; i < MAX_PER_LANE; ++i) so[warp][lane + i * 32] = o[i];
+  for (int i = 0; i < PL; ++i) so[warp][lane + i * 32] = o[i];
   if (lane == 0) sm[warp] = m, sl[warp] = l;
   __syncthreads();
   float top = sink ? sink[head] : -INFINITY;
@@ -147,6 +131,60 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
     for (int w = 0; w < AW; ++w) v = fmaf(so[w][d], expf(sm[w] - top), v);
     from_f(out[(size_t)t * out_stride_tok + (size_t)head * Dv + d], v / den);
   }
+}
+
+// out[t, h, n] = sigmoid(gate[t, h]) * sum_k a[t, h, k] w[h, n, k] with free strides of w, for 8 tokens per CTA (gate optional).
+constexpr int HP_T = 8, HP_K = 128;
+template <typename E>
+__global__ void __launch_bounds__(64) head_product_kernel(const E* __restrict__ a, long long a_tok, int a_head,
+                                                          const E* __restrict__ w, long long w_head, int w_n, int w_k, E* out,
+                                                          long long out_tok, int out_head, const E* gate, long long gate_tok, int T,
+                                                          int N, int K) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sa[HP_T][HP_K];
+  const int n = blockIdx.x * 64 + threadIdx.x, h = blockIdx.y, t0 = blockIdx.z * HP_T;
+  const E* wr = w + h * w_head + (long long)min(n, N - 1) * w_n;
+  float acc[HP_T] = {};
+  for (int k0 = 0; k0 < K; k0 += HP_K) {
+    __syncthreads();
+    for (int i = threadIdx.x; i < HP_T * HP_K; i += 64) {
+      const int r = i / HP_K, k = i % HP_K;
+      sa[r][k] = (t0 + r < T && k0 + k < K) ? to_f(a[(t0 + r) * a_tok + (long long)h * a_head + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+    const int m = min(HP_K, K - k0);
+    for (int k = 0; k < m; ++k) {
+      const float x = to_f(wr[(long long)(k0 + k) * w_k]);
+#pragma unroll
+      for (int r = 0; r < HP_T; ++r) acc[r] = fmaf(x, sa[r][k], acc[r]);
+    }
+  }
+  if (n >= N) return;
+#pragma unroll
+  for (int r = 0; r < HP_T; ++r) {
+    if (t0 + r >= T) break;
+    float v = acc[r];
+    if (gate) v /= 1.f + expf(-to_f(gate[(t0 + r) * gate_tok + h]));
+    from_f(out[(t0 + r) * out_tok + (long long)h * out_head + n], v);
+  }
+}
+
+template <typename E>
+int launch_attn_simple(const E* q, long long q_stride_tok, const E* k, const E* v, E* out, long long out_stride_tok,
+                       const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
+                       int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
+                       const float* sink, cudaStream_t s) {
+  const dim3 grid((unsigned)total_tokens, Hq), block(AW * 32);
+  auto go = [&](auto kernel) {
+    return launch_kernel(kernel, grid, block, 0, s, q, q_stride_tok, k, v, out, out_stride_tok, block_table, max_blocks, block_size,
+                         cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv, v_row, scale, chunk, sink);
+  };
+  const int widest = max(D, Dv);
+  if (widest <= 128) return go(attn_simple_kernel<E, 4>);
+  if (widest <= 320) return go(attn_simple_kernel<E, 10>);
+  if (widest <= 640) return go(attn_simple_kernel<E, 20>);
+  return go(attn_simple_kernel<E, MAX_PER_LANE>);
 }
 
 }  // namespace
@@ -165,28 +203,46 @@ int swb_gemm_f32(const float* a, int lda, const int* src, const int* offsets, in
                        reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act);
 }
 
-// Paged attention for any head widths up to 512 in fp32 arithmetic; elements fp32 or bf16 (fp32 flag). Arguments as in
-// swb_attn_ext; causal, sequences from cu_q or uniform lengths of uniform_q tokens.
+// Paged attention for any head widths up to 1024 in fp32 arithmetic; elements fp32 or bf16 (fp32 flag). Arguments as in
+// swb_attn_ext; causal, sequences from cu_q or uniform lengths of uniform_q tokens. v_row: elements between the value rows of
+// consecutive tokens of a page (0: Dv), so that values may be the leading columns of wider rows.
 int swb_attn_simple(const void* q, long long q_stride_tok, const void* k, const void* v, void* out, long long out_stride_tok,
                     const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
-                    int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk,
+                    int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
                     const float* sink, int fp32, void* stream) {
   using namespace swb;
   if (total_tokens <= 0 || num_seqs <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || D < 1 || Dv < 1 || D > 32 * MAX_PER_LANE || Dv > 32 * MAX_PER_LANE || block_size <= 0 ||
-      !block_table || !kv_lens || chunk < 0 || (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)))
+      !block_table || !kv_lens || chunk < 0 || (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)) ||
+      (v_row && v_row < Dv))
     return -3;
-  const dim3 grid((unsigned)total_tokens, Hq), block(AW * 32);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (!v_row) v_row = Dv;
+  if (fp32)
+    return launch_attn_simple(reinterpret_cast<const float*>(q), q_stride_tok, reinterpret_cast<const float*>(k),
+                              reinterpret_cast<const float*>(v), reinterpret_cast<float*>(out), out_stride_tok, block_table,
+                              max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, total_tokens, Hq, Hkv, D, Dv, v_row, scale,
+                              chunk, sink, s);
+  return launch_attn_simple(reinterpret_cast<const bf16*>(q), q_stride_tok, reinterpret_cast<const bf16*>(k),
+                            reinterpret_cast<const bf16*>(v), reinterpret_cast<bf16*>(out), out_stride_tok, block_table, max_blocks,
+                            block_size, cu_q, kv_lens, num_seqs, uniform_q, total_tokens, Hq, Hkv, D, Dv, v_row, scale, chunk, sink, s);
+}
+
+// Per-head products of any sizes and strides (elements): out[t, h, n] = sigmoid(gate[t, h]) sum_k a[t, h, k] w[h, n, k].
+int swb_head_product_simple(const void* a, long long a_tok, int a_head, const void* w, long long w_head, int w_n, int w_k, void* out,
+                            long long out_tok, int out_head, const void* gate, long long gate_tok, int T, int H, int N, int K, int fp32,
+                            void* stream) {
+  using namespace swb;
+  if (T <= 0 || H <= 0 || N <= 0 || K <= 0) return 0;
+  const dim3 grid((N + 63) / 64, H, (T + HP_T - 1) / HP_T), block(64);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (fp32)
-    return launch_kernel(attn_simple_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(q), q_stride_tok,
-                         reinterpret_cast<const float*>(k), reinterpret_cast<const float*>(v), reinterpret_cast<float*>(out),
-                         out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D,
-                         Dv, scale, chunk, sink);
-  return launch_kernel(attn_simple_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(q), q_stride_tok,
-                       reinterpret_cast<const bf16*>(k), reinterpret_cast<const bf16*>(v), reinterpret_cast<bf16*>(out),
-                       out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv,
-                       scale, chunk, sink);
+    return launch_kernel(head_product_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(a), a_tok, a_head,
+                         reinterpret_cast<const float*>(w), w_head, w_n, w_k, reinterpret_cast<float*>(out), out_tok, out_head,
+                         reinterpret_cast<const float*>(gate), gate_tok, T, N, K);
+  return launch_kernel(head_product_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(a), a_tok, a_head,
+                       reinterpret_cast<const bf16*>(w), w_head, w_n, w_k, reinterpret_cast<bf16*>(out), out_tok, out_head,
+                       reinterpret_cast<const bf16*>(gate), gate_tok, T, N, K);
 }
 
 }  // extern "C"

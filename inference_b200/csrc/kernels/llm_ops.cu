@@ -415,6 +415,103 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const bf16* __restri
   *reinterpret_cast<uint4*>(out + (size_t)t * ldo + v * 8) = pack8(o);
 }
 
+// out = a N(z) + b N(z^2) + c N(z^3) + e with the powers taken element by element and N(y) = y / sqrt(mean(y^2) + eps) over
+// a row's F values; coef = (a, b, c, e). One CTA per row, statistics in fp32. Rows of at most THREADS * VPT * 8 values stay in
+// registers (VPT > 0), longer ones are read twice.
+template <typename E>
+__device__ __forceinline__ void load_row8(const E* p, float* v) {
+  if constexpr (sizeof(E) == 2) {
+    unpack8(*reinterpret_cast<const uint4*>(p), v);
+  } else {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+  }
+}
+template <typename E>
+__device__ __forceinline__ void store_row8(E* p, const float* v) {
+  if constexpr (sizeof(E) == 2) {
+    *reinterpret_cast<uint4*>(p) = pack8(v);
+  } else {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
+template <typename E, int THREADS, int VPT>
+__global__ void __launch_bounds__(THREADS) poly_norm_kernel(const E* __restrict__ z, int ldz, E* out, int ldo, int F, int Fp,
+                                                            const float* __restrict__ coef, float eps) {
+  pdl_launch_dependents();
+  pdl_wait(TL_GATED_ACT);
+  __shared__ float red[3][THREADS / 32];
+  const E* zr = z + (size_t)blockIdx.x * ldz;
+  const int nvec = Fp / 8, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float keep[VPT > 0 ? VPT : 1][8];
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto add = [&](const float* v) {       // padding columns hold zeros
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float q = v[j] * v[j];
+      s2 += q;
+      s4 = fmaf(q, q, s4);
+      s6 = fmaf(q * q, q, s6);
+    }
+  };
+  if constexpr (VPT > 0) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * THREADS;
+      if (c < nvec) load_row8(zr + c * 8, keep[i]);
+      else
+#pragma unroll
+        for (int j = 0; j < 8; ++j) keep[i][j] = 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) add(keep[i]);
+  } else {
+    for (int c = threadIdx.x; c < nvec; c += THREADS) {
+      load_row8(zr + c * 8, keep[0]);
+      add(keep[0]);
+    }
+  }
+  s2 = warp_sum(s2), s4 = warp_sum(s4), s6 = warp_sum(s6);
+  if (lane == 0) red[0][warp] = s2, red[1][warp] = s4, red[2][warp] = s6;
+  __syncthreads();
+  s2 = s4 = s6 = 0.f;
+#pragma unroll
+  for (int w = 0; w < THREADS / 32; ++w) s2 += red[0][w], s4 += red[1][w], s6 += red[2][w];
+  const float n = (float)F;
+  const float a = coef[0] * rsqrtf(s2 / n + eps), b = coef[1] * rsqrtf(s4 / n + eps), c3 = coef[2] * rsqrtf(s6 / n + eps), e = coef[3];
+  E* orow = out + (size_t)blockIdx.x * ldo;
+  auto put = [&](int c, float* v) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = fmaf(fmaf(fmaf(c3, v[j], b), v[j], a), v[j], e);
+    store_row8(orow + c * 8, v);
+  };
+  if constexpr (VPT > 0) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * THREADS;
+      if (c < nvec) put(c, keep[i]);
+    }
+  } else {
+    for (int c = threadIdx.x; c < nvec; c += THREADS) {
+      load_row8(zr + c * 8, keep[0]);
+      put(c, keep[0]);
+    }
+  }
+}
+
+template <typename E>
+int launch_poly_norm(const E* z, int ldz, E* out, int ldo, int T, int F, int Fp, const float* coef, float eps, cudaStream_t s) {
+  const int nvec = Fp / 8;
+  const dim3 grid((unsigned)T);
+  if (nvec <= 256) return launch_kernel(poly_norm_kernel<E, 256, 1>, grid, dim3(256), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  if (nvec <= 512) return launch_kernel(poly_norm_kernel<E, 256, 2>, grid, dim3(256), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  if (nvec <= 1024) return launch_kernel(poly_norm_kernel<E, 512, 2>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  if (nvec <= 2048) return launch_kernel(poly_norm_kernel<E, 512, 4>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  return launch_kernel(poly_norm_kernel<E, 512, 0>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+}
+
 __global__ void __launch_bounds__(256) embedding_kernel(const long long* __restrict__ ids, const bf16* __restrict__ table,
                                                        bf16* out, int T, int H, int vocab_start, int vocab_end,
                                                        float scale) {
@@ -580,6 +677,16 @@ int swb_rope_kv_write(void* qkv, int ld_qkv, const int* positions, const long lo
                               k_norm_w, norm_eps, norm_w_offset, kcache, vcache, block_size, T, Hq, Hkv, D, D, 0, stream);
 }
 
+// Fp: padded row width (a multiple of 8), F <= Fp values enter the statistics; fp32 selects the element type of z and out.
+int swb_poly_norm(const void* z, int ldz, void* out, int ldo, int T, int F, int Fp, const float* coef, float eps, int fp32,
+                  void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (F <= 0 || F > Fp || (Fp % 8) || (ldz % 8) || (ldo % 8) || !coef) return -3;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (fp32) return launch_poly_norm(reinterpret_cast<const float*>(z), ldz, reinterpret_cast<float*>(out), ldo, T, F, Fp, coef, eps, s);
+  return launch_poly_norm(reinterpret_cast<const bf16*>(z), ldz, reinterpret_cast<bf16*>(out), ldo, T, F, Fp, coef, eps, s);
+}
 int swb_gated_act_mul(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;

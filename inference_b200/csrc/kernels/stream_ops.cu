@@ -7,6 +7,9 @@
 // (mean removed, weight and bias) or RMS norms, computed in fp32 on the row held in registers (squared deviations from the
 // mean, never a difference of large sums). The output is stored once per token, or to every row of an expert-sorted buffer that the token's
 // routing names, so the gather in front of a grouped GEMM costs no launch of its own.
+// The EXT instantiations add what some designs need on top: RMS norms over equal groups of columns, a stream that is read
+// from another buffer than it is written to, and the depth average, in which the joined stream is filed as one more result
+// and x becomes a weighted sum of all results so far.
 // Rows are padded to a multiple of 8 columns; padding columns of the stream, the weights and the outputs are zero and do
 // not enter the statistics.
 #include "common.cuh"
@@ -35,6 +38,13 @@ struct StreamNormParams {
   int H, Hp;
   float eps, out_scale;
   int center;                // 1: layer norm, 0: RMS norm
+  // EXT only
+  int groups;                // RMS norms over `groups` equal parts of the H columns
+  const float* x_in;         // optional: the stream is read here (row stride ldx) and written to x
+  float* hist;               // optional depth average: results 0 .. n_hist - 1, [T, ldx] each, `hist_stride` apart
+  long long hist_stride;
+  int n_hist;
+  const float* mix;          // [n_hist + 1]: x <- sum_j mix[j] hist[j] + mix[n_hist] x; the joined x becomes hist[n_hist]
 };
 
 __device__ __forceinline__ float4 load4(const void* base, size_t off, int fp32) {
@@ -134,19 +144,75 @@ __device__ __forceinline__ void norm_row(float4* v, const float* __restrict__ w,
   }
 }
 
+// RMS norm in groups of gs columns. Groups of whole 128-column chunks (the columns of one warp and one i) sum per chunk;
+// other sizes sum through a row of squares in shared memory. `part` holds Hp / 4 + H / gs floats at least (Hp + H / gs then).
 template <int THREADS, int VPT>
+__device__ __forceinline__ void group_norm_row(float4* v, const float* __restrict__ w, int H, int nvec, int groups, float eps,
+                                               float* part) {
+  const int gs = H / groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();                                   // an earlier norm may still be reading `part`
+  if (gs % 128 == 0) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const float q = warp_sum((v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w));
+      if (lane == 0) part[warp + i * (THREADS / 32)] = q;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c4 = threadIdx.x + i * THREADS;
+      if (c4 >= nvec) continue;
+      const int g = c4 * 4 / gs, per = gs / 128;
+      float ss = 0.f;
+      if (g < groups)
+        for (int k = 0; k < per; ++k) ss += part[g * per + k];
+      const float r = rsqrtf(ss / (float)gs + eps);
+      const float4 ww = __ldg(reinterpret_cast<const float4*>(w) + c4);
+      v[i] = make_float4(v[i].x * r * ww.x, v[i].y * r * ww.y, v[i].z * r * ww.z, v[i].w * r * ww.w);
+    }
+    return;
+  }
+  float* sums = part + nvec * 4;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c4 = threadIdx.x + i * THREADS;
+    if (c4 < nvec)
+      reinterpret_cast<float4*>(part)[c4] = make_float4(v[i].x * v[i].x, v[i].y * v[i].y, v[i].z * v[i].z, v[i].w * v[i].w);
+  }
+  __syncthreads();
+  for (int g = warp; g < groups; g += THREADS / 32) {
+    float ss = 0.f;
+    for (int c = lane; c < gs; c += 32) ss += part[g * gs + c];
+    ss = warp_sum(ss);
+    if (lane == 0) sums[g] = rsqrtf(ss / (float)gs + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c4 = threadIdx.x + i * THREADS, c = c4 * 4;
+    if (c4 >= nvec) continue;
+    const float4 ww = __ldg(reinterpret_cast<const float4*>(w) + c4);
+    auto r = [&](int k) { return sums[min((c + k) / gs, groups - 1)]; };
+    v[i] = make_float4(v[i].x * r(0) * ww.x, v[i].y * r(1) * ww.y, v[i].z * r(2) * ww.z, v[i].w * r(3) * ww.w);
+  }
+}
+
+template <int THREADS, int VPT, bool EXT>
 __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const StreamNormParams p) {
   pdl_launch_dependents();
   pdl_wait(TL_RMSNORM);
   __shared__ float red[4 * 32];
+  extern __shared__ float part[];      // EXT: scratch of the group norms
   const int row = blockIdx.x;
   const int nvec = p.Hp / 4;
-  float* xr = p.x + (size_t)(p.rows ? p.rows[row] : row) * p.ldx;
+  const size_t xo = (size_t)(p.rows ? p.rows[row] : row) * p.ldx;
+  float* xr = p.x + xo;
+  const float* xi = (EXT && p.x_in) ? p.x_in + xo : xr;
   float4 x[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * THREADS;
-    x[i] = c < nvec ? *reinterpret_cast<const float4*>(xr + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    x[i] = c < nvec ? *reinterpret_cast<const float4*>(xi + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   if (p.branch) {
     float4 v[VPT];
@@ -169,18 +235,51 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const StreamNormPa
       for (int i = 0; i < VPT; ++i)
         v[i].x *= p.branch_weight, v[i].y *= p.branch_weight, v[i].z *= p.branch_weight, v[i].w *= p.branch_weight;
     }
-    if (p.w1) norm_row<THREADS, VPT>(v, p.w1, p.b1, p.H, nvec, p.eps, p.center, red);
+    if (p.w1) {
+      if (EXT && p.groups > 1) group_norm_row<THREADS, VPT>(v, p.w1, p.H, nvec, p.groups, p.eps, part);
+      else norm_row<THREADS, VPT>(v, p.w1, p.b1, p.H, nvec, p.eps, p.center, red);
+    }
+    float* to = (EXT && p.hist) ? p.hist + p.n_hist * p.hist_stride + xo : xr;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int c = threadIdx.x + i * THREADS;
       if (c < nvec) {
         x[i].x += v[i].x, x[i].y += v[i].y, x[i].z += v[i].z, x[i].w += v[i].w;
-        *reinterpret_cast<float4*>(xr + c * 4) = x[i];
+        *reinterpret_cast<float4*>(to + c * 4) = x[i];
+      }
+    }
+  }
+  if constexpr (EXT) {
+    if (p.hist) {
+      const float own = __ldg(p.mix + p.n_hist);
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) x[i].x *= own, x[i].y *= own, x[i].z *= own, x[i].w *= own;
+#pragma unroll 4
+      for (int j = 0; j < p.n_hist; ++j) {
+        const float m = __ldg(p.mix + j);
+        const float* h = p.hist + j * p.hist_stride + xo;
+#pragma unroll
+        for (int i = 0; i < VPT; ++i) {
+          const int c = threadIdx.x + i * THREADS;
+          if (c < nvec) {
+            const float4 y = *reinterpret_cast<const float4*>(h + c * 4);
+            x[i].x = fmaf(m, y.x, x[i].x), x[i].y = fmaf(m, y.y, x[i].y);
+            x[i].z = fmaf(m, y.z, x[i].z), x[i].w = fmaf(m, y.w, x[i].w);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * THREADS;
+        if (c < nvec) *reinterpret_cast<float4*>(xr + c * 4) = x[i];
       }
     }
   }
   if (!p.out) return;
-  if (p.w2) norm_row<THREADS, VPT>(x, p.w2, p.b2, p.H, nvec, p.eps, p.center, red + 64);
+  if (p.w2) {
+    if (EXT && p.groups > 1) group_norm_row<THREADS, VPT>(x, p.w2, p.H, nvec, p.groups, p.eps, part);
+    else norm_row<THREADS, VPT>(x, p.w2, p.b2, p.H, nvec, p.eps, p.center, red + 64);
+  }
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * THREADS;
@@ -196,11 +295,11 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const StreamNormPa
   }
 }
 
-// x[t] = table[ids[t]] as fp32; optional copies of the row in the activation type (out_a / out_b, strides ld_a / ld_b).
+// x[t] = scale * table[ids[t]] as fp32; optional copies of the row in the activation type (out_a / out_b, strides ld_a / ld_b).
 // Ids outside [0, vocab) read as a zero row.
 __global__ void __launch_bounds__(256) stream_embed_kernel(const long long* __restrict__ ids, const void* table, int table_fp32,
                                                            int vocab, float* x, int ldx, void* out_a, int ld_a, void* out_b,
-                                                           int ld_b, int out_fp32, int T, int Hp) {
+                                                           int ld_b, int out_fp32, float scale, int T, int Hp) {
   pdl_launch_dependents();
   pdl_wait(TL_EMBED);
   const int nvec = Hp / 4;
@@ -208,7 +307,8 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const long long* __re
   if (idx >= (long long)T * nvec) return;
   const int t = (int)(idx / nvec), c = (int)(idx % nvec) * 4;
   const long long id = ids[t];
-  const float4 v = (id >= 0 && id < vocab) ? load4(table, (size_t)id * Hp + c, table_fp32) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v = (id >= 0 && id < vocab) ? load4(table, (size_t)id * Hp + c, table_fp32) : make_float4(0.f, 0.f, 0.f, 0.f);
+  v.x *= scale, v.y *= scale, v.z *= scale, v.w *= scale;
   *reinterpret_cast<float4*>(x + (size_t)t * ldx + c) = v;
   if (out_a) store4(out_a, (size_t)t * ld_a + c, out_fp32, v);
   if (out_b) store4(out_b, (size_t)t * ld_b + c, out_fp32, v);
@@ -216,7 +316,16 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const long long* __re
 
 template <int THREADS, int VPT>
 int launch_sn(const StreamNormParams& p, int T, cudaStream_t s) {
-  return launch_kernel(stream_norm_kernel<THREADS, VPT>, dim3((unsigned)T), dim3(THREADS), 0, s, p);
+  if (p.groups <= 1 && !p.x_in && !p.hist)
+    return launch_kernel(stream_norm_kernel<THREADS, VPT, false>, dim3((unsigned)T), dim3(THREADS), 0, s, p);
+  size_t smem = 0;
+  if (p.groups > 1) smem = (p.H / p.groups) % 128 == 0 ? THREADS / 32 * VPT * sizeof(float) : (size_t)(p.Hp + p.groups) * sizeof(float);
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(stream_norm_kernel<THREADS, VPT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               (int)smem);
+    if (e != cudaSuccess) return -(int)e;
+  }
+  return launch_kernel(stream_norm_kernel<THREADS, VPT, true>, dim3((unsigned)T), dim3(THREADS), smem, s, p);
 }
 
 }  // namespace
@@ -229,9 +338,13 @@ extern "C" {
 int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch, int ld_branch, int branch_fp32,
                     const int* branch_rows, int branch_top, float branch_weight, const float* w1, const float* b1,
                     const float* w2, const float* b2, void* out, int ldo, int out_fp32, const int* out_rows, int out_top,
-                    int T, int H, int Hp, float eps, float out_scale, int center, void* stream) {
+                    int T, int H, int Hp, float eps, float out_scale, int center, int groups, const void* x_in, void* hist,
+                    long long hist_stride, int n_hist, const float* mix, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
+  if (groups < 1 || H % groups || (groups > 1 && (center || b1 || b2)) || (hist && (!mix || !branch || n_hist < 0 || (hist_stride % 4))) ||
+      (rows && (x_in || hist)))
+    return -3;
   if (H <= 0 || H > Hp || (Hp % 8) || (ldx % 4) || (branch && (ld_branch % 4)) || (out && (ldo % 4)) || (rows && branch) ||
       (branch_rows && branch_top <= 0) || (out_rows && out_top <= 0))
     return -3;
@@ -255,6 +368,12 @@ int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch,
   p.eps = eps;
   p.out_scale = out_scale;
   p.center = center;
+  p.groups = groups;
+  p.x_in = reinterpret_cast<const float*>(x_in);
+  p.hist = reinterpret_cast<float*>(hist);
+  p.hist_stride = hist_stride;
+  p.n_hist = n_hist;
+  p.mix = mix;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int nvec = Hp / 4;
   if (nvec <= 128) return launch_sn<128, 1>(p, T, s);
@@ -268,14 +387,14 @@ int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch,
 }
 
 int swb_stream_embed(const long long* ids, const void* table, int table_fp32, int vocab, void* x, int ldx, void* out_a,
-                     int ld_a, void* out_b, int ld_b, int out_fp32, int T, int Hp, void* stream) {
+                     int ld_a, void* out_b, int ld_b, int out_fp32, float scale, int T, int Hp, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
   if ((Hp % 8) || (ldx % 4) || (out_a && (ld_a % 4)) || (out_b && (ld_b % 4))) return -3;
   const long long n = (long long)T * (Hp / 4);
   return launch_kernel(stream_embed_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0,
                        reinterpret_cast<cudaStream_t>(stream), ids, table, table_fp32, vocab,
-                       reinterpret_cast<float*>(x), ldx, out_a, ld_a, out_b, ld_b, out_fp32, T, Hp);
+                       reinterpret_cast<float*>(x), ldx, out_a, ld_a, out_b, ld_b, out_fp32, scale, T, Hp);
 }
 
 }  // extern "C"

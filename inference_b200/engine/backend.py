@@ -11,6 +11,7 @@ from typing import Any, Protocol
 
 import torch
 
+from ..contracts.errors import Unsupported
 from ..models.oracle import ContiguousKvCache, OracleLlama
 from .kv_pool import PagedSequence
 from .runner import ModelRunner
@@ -88,6 +89,10 @@ class GpuBackend:
         if ov is None and mr is None and not all_positions and self._is_decode(seqs, new_tokens):
             logits = self.runner.decode(seqs, [t[0] for t in new_tokens], want_logits=True)
             return [logits[i] for i in range(len(seqs))]
+        if all_positions:
+            for s, t in zip(seqs, new_tokens):
+                if len(t) > 1:                 # a verify step: its last tokens may be taken back
+                    self._checkpoint(s)
         logits = self.runner.prefill(seqs, new_tokens, want_logits=True, all_positions=all_positions,
                                      embed_overrides=ov, mrope_overrides=mr)
         if not all_positions:
@@ -112,11 +117,46 @@ class GpuBackend:
         logits = self.runner.prefill(seqs, new_tokens, want=want)
         return logits if any(want) else None
 
+    def _checkpoint(self, seq: PagedSequence) -> None:
+        """Keeps a copy of a recurrent state before a step that may be rolled back, when a slot is free for it."""
+        if not seq.stateful or seq.length == 0:
+            return
+        pool = self.runner.pool
+        if seq.checkpoint is None:
+            if pool.slots.free_blocks() == 0:
+                return
+            seq.checkpoint = (seq.length, pool.slots.alloc())
+        seq.checkpoint = (seq.length, seq.checkpoint[1])
+        pool.copy_state(seq.state_slot, seq.checkpoint[1])
+
     def truncate(self, seq, length):
-        seq.truncate(length)
+        """Recurrent layers go back to the checkpoint in front of the last verify step (to the start without one) and run
+        the kept tokens again."""
+        if not seq.stateful or length in (0, seq.length):
+            seq.truncate(length)
+            return
+        if seq.tokens is None:
+            raise Unsupported("rollback of a recurrent state whose tokens were chosen on the device")
+        again, base = seq.tokens[:length], 0
+        if seq.checkpoint is not None and seq.checkpoint[0] <= length:
+            base = seq.checkpoint[0]
+            self.runner.pool.copy_state(seq.checkpoint[1], seq.state_slot)
+        seq.truncate(base)
+        if again[base:]:
+            self.runner.prefill([seq], [again[base:]], want=[[]])
 
     def fork(self, seq, n_tokens):
-        bs = self.runner.pool.block_size
+        """Recurrent layers: only a sequence as it stands can be shared (its state is copied into a slot of its own); other
+        lengths, or no free slot, give an empty sequence."""
+        pool, bs = self.runner.pool, self.runner.pool.block_size
+        if seq.stateful:
+            if n_tokens != seq.length or n_tokens == 0 or pool.slots.free_blocks() == 0:
+                return PagedSequence(pool)
+            f = PagedSequence.seeded(pool, list(seq.blocks), n_tokens)
+            f.state_slot = pool.slots.alloc()
+            f.tokens = None if seq.tokens is None else list(seq.tokens)
+            pool.copy_state(seq.state_slot, f.state_slot)
+            return f
         whole = (n_tokens // bs) * bs
         f = PagedSequence.seeded(self.runner.pool, seq.shareable_prefix_blocks(whole), whole)
         if getattr(seq, "rope_delta", 0):

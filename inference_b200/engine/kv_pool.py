@@ -7,6 +7,7 @@ allocator policy (copy-on-write prefix sharing), so a block id is valid across a
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -40,39 +41,77 @@ class PagedKvPool:
 
 @dataclass(frozen=True)
 class KvGeometry:
-    """K / V shape of one cache-owning layer run."""
+    """K / V pages of one cache-owning layer run."""
     kv_heads: int
     k_dim: int
     v_dim: int
 
+    def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
+        return [(self.kv_heads, block_size, self.k_dim), (self.kv_heads, block_size, self.v_dim)]
+
+
+@dataclass(frozen=True)
+class LatentGeometry:
+    """Pages of a latent-attention layer: one row of `width` numbers per token, shared by all heads."""
+    width: int
+
+    def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
+        return [(block_size, self.width)]
+
+
+@dataclass(frozen=True)
+class StateGeometry:
+    """Recurrent layer: per sequence a fp32 state and a window of recent inputs in the activation type; no pages."""
+    state: tuple[int, ...]
+    window: tuple[int, ...]
+
+    def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
+        return []
+
 
 class LayeredKvPool:
-    """Paged pool of a model whose layers differ in head count or head width, or run more than once: every run owns a K
-    tensor [blocks, kv_heads, block_size, k_dim] and a V tensor [blocks, kv_heads, block_size, v_dim]. Block ids are
-    shared by all runs (one allocator), so sequences, forks and rollbacks work as on the uniform pool."""
+    """Paged pool of a model whose layers differ in what they keep, or run more than once: every run owns its page tensors
+    [blocks, ...] (K and V, or latent rows). Block ids are shared by all runs (one allocator), so sequences, forks and
+    rollbacks work as on the uniform pool. Recurrent layers own tensors [state_slots, ...] instead; a sequence holds one slot
+    for all of them from its first token to its release. A slot needs no clearing: the kernels take the state of a sequence
+    as zero at position 0."""
 
-    def __init__(self, geometry: list[KvGeometry], num_blocks: int, block_size: int = 16,
-                 device: torch.device | str = "cuda", dtype: torch.dtype = torch.bfloat16):
+    def __init__(self, geometry: list[KvGeometry | LatentGeometry | StateGeometry], num_blocks: int, block_size: int = 16,
+                 device: torch.device | str = "cuda", dtype: torch.dtype = torch.bfloat16, state_slots: int = 0):
         self.geometry, self.num_layers = list(geometry), len(geometry)
         self.num_blocks, self.block_size = num_blocks, block_size
+        self.has_state = any(isinstance(g, StateGeometry) for g in geometry)
+        if self.has_state and state_slots < 1:
+            raise ValueError("a pool with recurrent layers needs state slots")
 
-        def pages(g: KvGeometry, dim: int) -> torch.Tensor:
-            return torch.zeros((num_blocks, g.kv_heads, block_size, dim), dtype=dtype, device=device)
-        self.data = [(pages(g, g.k_dim), pages(g, g.v_dim)) for g in geometry]
+        def tensors(g) -> tuple[torch.Tensor, ...]:
+            if isinstance(g, StateGeometry):
+                return (torch.zeros((state_slots, *g.state), dtype=torch.float32, device=device),
+                        torch.zeros((state_slots, *g.window), dtype=dtype, device=device))
+            return tuple(torch.zeros((num_blocks, *s), dtype=dtype, device=device) for s in g.page_shapes(block_size))
+        self.data = [tensors(g) for g in geometry]
         self.allocator = BlockAllocator(num_blocks)
+        self.slots = BlockAllocator(state_slots) if self.has_state else None
 
     @property
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size() for kv in self.data for t in kv)
 
     def copy_block(self, src: int, dst: int) -> None:
-        for kv in self.data:
-            for t in kv:
-                t[dst].copy_(t[src])
+        for g, kv in zip(self.geometry, self.data):
+            if not isinstance(g, StateGeometry):
+                for t in kv:
+                    t[dst].copy_(t[src])
+
+    def copy_state(self, src: int, dst: int) -> None:
+        for g, kv in zip(self.geometry, self.data):
+            if isinstance(g, StateGeometry):
+                for t in kv:
+                    t[dst].copy_(t[src])
 
     @staticmethod
-    def block_bytes(geometry: list[KvGeometry], block_size: int = 16, elem: int = 2) -> int:
-        return sum(g.kv_heads * block_size * (g.k_dim + g.v_dim) * elem for g in geometry)
+    def block_bytes(geometry, block_size: int = 16, elem: int = 2) -> int:
+        return sum(math.prod(s) for g in geometry for s in g.page_shapes(block_size)) * elem
 
 
 class PagedSequence:
@@ -87,6 +126,10 @@ class PagedSequence:
         self.uid = PagedSequence._next_uid  # never reused; with `epoch` it keys cached device block tables
         PagedSequence._next_uid += 1
         self.epoch = 0   # bumped whenever an already-published block id changes (COW unshare, truncate)
+        self.state_slot = -1                    # recurrent layers: slot of this sequence's state (held while length > 0)
+        self.tokens: list[int] | None = []      # recurrent layers: what was fed, to rebuild the state of a rollback; None
+        #                                         once tokens were chosen on the device
+        self.checkpoint: tuple[int, int] | None = None   # (length, slot): copy of the state before the last verify step
 
     @classmethod
     def seeded(cls, pool: PagedKvPool, blocks: list[int], length: int) -> "PagedSequence":
@@ -102,6 +145,8 @@ class PagedSequence:
         """Make room for n_tokens more tokens and return their flat cache slots (block * bs + offset)."""
         bs = self.pool.block_size
         slots = []
+        if self.state_slot < 0 and self.stateful:
+            self.state_slot = self.pool.slots.alloc()
         for _ in range(n_tokens):
             bi, off = divmod(self.length, bs)
             if bi == len(self.blocks):
@@ -118,8 +163,23 @@ class PagedSequence:
             self.length += 1
         return slots
 
+    @property
+    def stateful(self) -> bool:
+        return getattr(self.pool, "has_state", False)
+
+    def fed(self, tokens: list[int] | None) -> None:
+        """Remembers the tokens of a step (None: they are known to the device only)."""
+        if self.stateful:
+            self.tokens = None if tokens is None or self.tokens is None else self.tokens + tokens
+
+    def drop_checkpoint(self) -> None:
+        if self.checkpoint is not None:
+            self.pool.slots.release(self.checkpoint[1])
+            self.checkpoint = None
+
     def truncate(self, length: int) -> None:
-        """Roll back to `length` tokens (speculative rejection); frees blocks past the boundary."""
+        """Roll back to `length` tokens (speculative rejection); frees blocks past the boundary. A recurrent state cannot
+        run backwards: there the caller restores or rebuilds it for `length` tokens (`GpuBackend.truncate`)."""
         bs = self.pool.block_size
         keep = (length + bs - 1) // bs
         for b in self.blocks[keep:]:
@@ -127,6 +187,8 @@ class PagedSequence:
         self.blocks = self.blocks[:keep]
         self.length = length
         self.epoch += 1
+        if self.stateful and self.tokens is not None:
+            self.tokens = self.tokens[:length]
 
     def shareable_prefix_blocks(self, n_tokens: int) -> list[int]:
         """Blocks fully covered by the first n_tokens tokens (only whole blocks are shareable)."""
@@ -137,3 +199,8 @@ class PagedSequence:
             self.pool.allocator.release(b)
         self.blocks = []
         self.length = 0
+        self.drop_checkpoint()
+        if self.state_slot >= 0:
+            self.pool.slots.release(self.state_slot)
+            self.state_slot = -1
+        self.tokens = []

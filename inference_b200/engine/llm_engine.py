@@ -41,13 +41,14 @@ class LlmEngine:
         self.cfg = cfg or EngineConfig()
         c, m = self.cfg, model.cfg
         if c.kv_bytes is not None and hasattr(model, "kv_block_bytes"):
-            nblocks = max(1, c.kv_bytes // model.kv_block_bytes(c.block_size))
+            nblocks = max(1, c.kv_bytes // max(1, model.kv_block_bytes(c.block_size)))
         elif c.kv_bytes is not None:
             nblocks = PagedKvPool.blocks_for_budget(c.kv_bytes, m.num_layers, model.hkv, m.head_dim, c.block_size)
         else:
             nblocks = c.max_batch * ((c.max_seq_len + c.block_size - 1) // c.block_size) + 8
         if hasattr(model, "make_pool"):      # pipeline-sharded or layer-by-layer model: its own KV tensors, shared block ids
-            self.pool = model.make_pool(nblocks, c.block_size)
+            extra = {"state_slots": c.max_batch} if getattr(model, "recurrent", False) else {}
+            self.pool = model.make_pool(nblocks, c.block_size, **extra)
         else:
             self.pool = PagedKvPool(m.num_layers, nblocks, model.hkv, m.head_dim, c.block_size, device=model.device)
         self.runner = ModelRunner(model, self.pool, max_batch=c.max_batch, max_seq_len=c.max_seq_len,

@@ -15,8 +15,9 @@ BLOCK = 16
 
 def gpu_backend(cfg: ModelConfig, weights: dict[str, torch.Tensor], comm=None, *, dtype: torch.dtype = torch.bfloat16,
                 max_batch: int = 16, max_context: int | None = None, kv_tokens: int | None = None) -> GpuBackend:
-    """kv_tokens: the pool holds exactly that many tokens (rounded up to pages); None sizes it for max_batch full contexts,
-    at most 60 % of the free memory."""
+    """kv_tokens: the pool holds exactly that many tokens (rounded up to pages) and, for recurrent layers, the states of
+    max_batch sequences; None sizes it for max_batch full contexts, at most 60 % of the free memory, and twice max_batch
+    states (cached prefixes and checkpoints of speculative steps hold some)."""
     if not torch.cuda.is_available():
         raise LoadError("the b200 backend needs a CUDA device (use the cpu runtime bundle on hosts without one)")
     dev = comm.device if comm is not None else torch.device("cuda", torch.cuda.current_device())
@@ -29,7 +30,8 @@ def gpu_backend(cfg: ModelConfig, weights: dict[str, torch.Tensor], comm=None, *
         free, _total = torch.cuda.mem_get_info(dev)
         per_block = model.kv_block_bytes(BLOCK) if own_pool else cfg.num_layers * 2 * model.hkv * BLOCK * cfg.head_dim * 2
         want = max_batch * ((ctx + BLOCK - 1) // BLOCK) + 64
-        nblocks = max(64, min(want, int(free * 0.6) // per_block))
-    pool = model.make_pool(nblocks, BLOCK) if own_pool else \
+        nblocks = max(64, min(want, int(free * 0.6) // max(1, per_block)))
+    extra = {"state_slots": max_batch * (2 if kv_tokens is None else 1)} if getattr(model, "recurrent", False) else {}
+    pool = model.make_pool(nblocks, BLOCK, **extra) if own_pool else \
         PagedKvPool(cfg.num_layers, nblocks, model.hkv, cfg.head_dim, BLOCK, device=dev)
     return GpuBackend(ModelRunner(model, pool, max_batch=max_batch, max_seq_len=ctx))

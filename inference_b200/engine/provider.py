@@ -302,7 +302,7 @@ def _build_backend(cfg: ModelConfig, weights: dict, backend_name: str, comm=None
         from .loading import gpu_backend
 
         return gpu_backend(cfg, weights, comm)
-    if cfg.architecture is Architecture.ZOBUNEX:
+    if cfg.stack is not None:
         raise Unsupported(f"{cfg.architecture.value} runs on the b200 backend only")
     return OracleBackend(OracleLlama(cfg, weights, dtype=torch.float32, device="cpu"),
                          max_context=cfg.max_position_embeddings or 8192)
@@ -582,7 +582,7 @@ def _can_load_gpu(spec: LoadSpec) -> bool:
 
 def _can_load_cpu(spec: LoadSpec) -> bool:
     cfg = probe_config(spec)
-    return not _can_load_qwen3_vl(spec) and cfg is not None and cfg.architecture is not Architecture.ZOBUNEX
+    return not _can_load_qwen3_vl(spec) and cfg is not None and cfg.stack is None
 
 
 B200_LLAVA = TextLlmRegistration(lambda: _descriptor_vision("b200-llava", BACKEND_GPU),

@@ -51,17 +51,20 @@ class ModelRunner:
         dev = model.device
         model.ensure_rope(max_seq_len + 64)
         # static decode-step buffers; one packed int64 staging area so a step is a single H2D copy
-        self._n_meta = max_batch * 4 + max_batch * self.max_blocks
+        self._stateful = getattr(pool, "has_state", False)
+        fixed = 5 if self._stateful else 4
+        self._n_meta = max_batch * fixed + max_batch * self.max_blocks
         self._host_meta = torch.zeros(self._n_meta, dtype=torch.int32).pin_memory() if dev.type == "cuda" else \
             torch.zeros(self._n_meta, dtype=torch.int32)
         self._host_np = self._host_meta.numpy()
-        self._host_table_np = self._host_np[4 * max_batch:].reshape(max_batch, self.max_blocks)
+        self._host_table_np = self._host_np[fixed * max_batch:].reshape(max_batch, self.max_blocks)
         self._row_state: list[tuple[int, int, int]] = [(0, 0, 0)] * max_batch  # (uid, epoch, blocks written)
         self._dev_meta = torch.zeros(self._n_meta, dtype=torch.int32, device=dev)
         self._ids = torch.zeros(max_batch, dtype=torch.int64, device=dev)
         self._pos = torch.zeros(max_batch, dtype=torch.int32, device=dev)
         self._slots = torch.zeros(max_batch, dtype=torch.int64, device=dev)
         self._kvl = torch.zeros(max_batch, dtype=torch.int32, device=dev)
+        self._states = torch.full((max_batch,), -1, dtype=torch.int32, device=dev) if self._stateful else None
         self._table = torch.zeros((max_batch, self.max_blocks), dtype=torch.int32, device=dev)
         self._host_tokens = torch.zeros(max_batch, dtype=torch.int64).pin_memory() if dev.type == "cuda" else \
             torch.zeros(max_batch, dtype=torch.int64)
@@ -123,7 +126,12 @@ class ModelRunner:
             cu_q=None if decode else torch.tensor(cu, dtype=torch.int32, device=dev), max_q_len=max_q,
             num_seqs=len(seqs), decode=decode, fresh_prefill=fresh and not decode,
             attn_splits=self._splits(len(seqs), max(kvl)) if decode else 1,
-            logits_rows=None if all_positions else torch.tensor(rows, dtype=torch.int64, device=dev))
+            logits_rows=None if all_positions else torch.tensor(rows, dtype=torch.int64, device=dev),
+            spans=[(len(t), n) for t, n in zip(new_tokens, kvl)])
+        if self._stateful:
+            inp.state_slots = torch.tensor([s.state_slot for s in seqs], dtype=torch.int32, device=dev)
+            for s, toks in zip(seqs, new_tokens):
+                s.fed(toks)
         if embed_overrides is not None:
             er, ev = [], []
             for i, ov in enumerate(embed_overrides):
@@ -170,7 +178,8 @@ class ModelRunner:
     # ---- decode (graph-captured, one token per sequence) ---------------------------------------------
     def _fill_decode_meta(self, seqs: list[PagedSequence], tokens: list[int], pad_to: int = 0) -> int:
         """Writes the step metadata of the live rows; rows len(seqs)..pad_to-1 become copies of row 0 (same
-        token, position, slot and block table), so they recompute row 0 and store identical K / V bytes."""
+        token, position, slot and block table), so they recompute row 0 and store identical K / V bytes; they own no
+        recurrent state (slot -1)."""
         MB = self.max_batch
         h, table = self._host_np, self._host_table_np
         if self._meta_copy_done is not None:
@@ -186,6 +195,8 @@ class ModelRunner:
             h[MB + i] = p + getattr(s, "rope_delta", 0)
             h[2 * MB + i] = slot
             h[3 * MB + i] = p + 1
+            if self._stateful:
+                h[4 * MB + i] = s.state_slot
             if p + 1 > max_kv:
                 max_kv = p + 1
             owner, epoch, written = self._row_state[i]
@@ -200,6 +211,8 @@ class ModelRunner:
             nb0 = len(seqs[0].blocks)
             for i in range(len(seqs), pad_to):
                 h[i], h[MB + i], h[2 * MB + i], h[3 * MB + i] = h[0], h[MB], h[2 * MB], h[3 * MB]
+                if self._stateful:
+                    h[4 * MB + i] = -1
                 table[i, :nb0] = table[0, :nb0]
                 self._row_state[i] = (-1, -1, 0)
         return max_kv
@@ -215,7 +228,10 @@ class ModelRunner:
             self._pos[:B].copy_(m[MB:MB + B])
             self._slots[:B].copy_(m[2 * MB:2 * MB + B])
             self._kvl[:B].copy_(m[3 * MB:3 * MB + B])
-            self._table[:B].copy_(m[4 * MB:4 * MB + B * mb].view(B, mb))
+            t0 = (5 if self._stateful else 4) * MB
+            if self._stateful:
+                self._states[:B].copy_(m[4 * MB:4 * MB + B])
+            self._table[:B].copy_(m[t0:t0 + B * mb].view(B, mb))
             return
         from .._native import kernels
         from ..ops.runtime import check, stream_ptr
@@ -224,6 +240,7 @@ class ModelRunner:
         rc = kernels().swb_decode_meta_unpack(src.data_ptr(), self._n_meta, self._step.data_ptr() if multi else None,
                                               MB, B, mb, None if skip_ids else self._ids.data_ptr(),
                                               self._pos.data_ptr(), self._slots.data_ptr(), self._kvl.data_ptr(),
+                                              self._states.data_ptr() if self._stateful else None,
                                               self._table.data_ptr(), stream_ptr())
         check(rc, "swb_decode_meta_unpack")
 
@@ -235,7 +252,8 @@ class ModelRunner:
             r1 = min(B, r0 + cap)
             inp = StepInputs(input_ids=self._ids[r0:r1], positions=self._pos[r0:r1], slot_mapping=self._slots[r0:r1],
                              block_table=self._table[r0:r1], kv_lens=self._kvl[r0:r1], cu_q=None, max_q_len=1,
-                             num_seqs=r1 - r0, decode=True, attn_splits=splits, logits_rows=None)
+                             num_seqs=r1 - r0, decode=True, attn_splits=splits, logits_rows=None,
+                             state_slots=self._states[r0:r1] if self._stateful else None)
             part = self.model.forward_hidden(inp, self.pool.data)
             # the model may hand back a view of a workspace that the next sub-step reuses
             parts.append(part.clone() if cap < B else part)
@@ -268,6 +286,9 @@ class ModelRunner:
         B = len(seqs)
         Bp = _bucket(B, self.max_batch) if self.pad_batches else B
         max_kv = self._fill_decode_meta(seqs, tokens, Bp)
+        if self._stateful:
+            for s, t in zip(seqs, tokens):
+                s.fed([t])
         self._dev_meta.copy_(self._host_meta, non_blocking=True)
         if want_logits and self.model.device.type == "cuda":
             self._meta_copy_done = torch.cuda.Event()
@@ -317,6 +338,8 @@ class ModelRunner:
         for k in range(n_steps):
             max_kv = self._fill_decode_meta(seqs, tokens if k == 0 else [0] * B)
             host_all[k].copy_(self._host_meta)
+        for s in seqs:
+            s.fed(None)
         self.h2d_bytes_last = host_all.numel() * 4
         splits = self._splits(B, max_kv)
         first = torch.tensor(tokens, dtype=torch.int64)
@@ -351,7 +374,12 @@ class ModelRunner:
         return self._multi_out[:n_steps * B].view(n_steps, B).clone()
 
     def _capture(self, B: int, splits: int, want_logits: bool, feedback: bool = False) -> _DecodeGraph:
-        # warm-up on a side stream (sets kernel attributes, fills the tensor-map cache), then capture
+        # warm-up on a side stream (sets kernel attributes, fills the tensor-map cache), then capture. Repeating a step
+        # rewrites the same cache rows but would advance a recurrent state, so the warm-up runs without one.
+        meta, states = self._multi_meta[0] if feedback else self._dev_meta, None
+        if self._stateful:
+            states = meta[4 * self.max_batch:5 * self.max_batch].clone()
+            meta[4 * self.max_batch:5 * self.max_batch].fill_(-1)
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):
@@ -360,6 +388,8 @@ class ModelRunner:
                     self._step.zero_()      # every warm-up run reads the same (first) row of the step table
                 self._decode_body(B, splits, want_logits, feedback)
         torch.cuda.current_stream().wait_stream(s)
+        if states is not None:
+            meta[4 * self.max_batch:5 * self.max_batch].copy_(states)
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()
         fused = self.model.comm.fused

@@ -27,12 +27,14 @@ class Architecture(enum.Enum):
     QWEN35 = "qwen3_5"       # hybrid Gated-DeltaNet / gated full attention
     QWEN3_VL = "qwen3_vl"    # VLM-wrapped Qwen3 decoder with interleaved M-RoPE
     ZOBUNEX = "zobunex"      # listed layers with a loop, chunked sink attention, sandwich layer norms, token-routed experts
+    GUNEDRA = "gunedra"      # listed layers: latent attention and channel-wise delta rule, output norms, depth averages
 
     @staticmethod
     def from_config(cfg: dict[str, Any]) -> "Architecture":
         if isinstance(cfg.get("architecture"), str):        # configs that list their layers name the design itself
-            if cfg["architecture"].lower() == "zobunex":
-                return Architecture.ZOBUNEX
+            for a in LISTED:
+                if cfg["architecture"].lower() == a.value:
+                    return a
             raise Unsupported(f"unsupported architecture {cfg['architecture']!r}")
         archs = cfg.get("architectures")
         arch = archs[0] if isinstance(archs, list) and archs and isinstance(archs[0], str) else None
@@ -75,6 +77,9 @@ class Architecture(enum.Enum):
     @property
     def sandwich_norms(self) -> bool:
         return self in (Architecture.GEMMA2, Architecture.GLM4)
+
+
+LISTED = (Architecture.ZOBUNEX, Architecture.GUNEDRA)     # designs whose config lists the layers one by one
 
 
 @dataclass(frozen=True)
@@ -149,6 +154,42 @@ class AttentionSpec:
 
 
 @dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Latent attention: keys and values of every head are projections of one cached vector of `kv_rank` numbers per token;
+    `rot_dim` further query / key dimensions are rotated, their key part is shared by the heads."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+
+    @property
+    def kv_heads(self) -> int:
+        return 1
+
+    @property
+    def groups(self) -> int:
+        return self.heads
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """Gated delta rule with a decay per head and key channel: a [dim, vdim] state per head, short convolutions of `conv`
+    taps in front of q, k and v."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    @property
+    def groups(self) -> int:
+        return 1
+
+
+@dataclass(frozen=True)
 class ExpertsSpec:
     experts: int
     top: int
@@ -156,9 +197,14 @@ class ExpertsSpec:
 
 
 @dataclass(frozen=True)
+class DenseSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec
-    mlp: ExpertsSpec | None
+    mixer: AttentionSpec | LatentAttentionSpec | ChannelDeltaSpec
+    mlp: ExpertsSpec | DenseSpec | None
 
 
 @dataclass(frozen=True)
@@ -168,12 +214,79 @@ class LoopSpec:
     times: int
 
 
+def _need(d: Any, key: str, where: str) -> Any:
+    if not isinstance(d, dict) or d.get(key) is None:
+        raise ConfigError(f"config.json missing `{where}{key}`")
+    return d[key]
+
+
+def _count(d: Any, key: str, where: str, low: int = 1) -> int:
+    v = _need(d, key, where)
+    if isinstance(v, bool) or not isinstance(v, (int, float)) or int(v) != v or v < low:
+        raise ConfigError(f"config.json: `{where}{key}` must be an integer >= {low}, not {v!r}")
+    return int(v)
+
+
+def _real(d: Any, key: str, where: str) -> float:
+    v = _need(d, key, where)
+    if isinstance(v, bool) or not isinstance(v, (int, float)):
+        raise ConfigError(f"config.json: `{where}{key}` must be a number, not {v!r}")
+    return float(v)
+
+
+def _attention_spec(m: Any, at: str) -> AttentionSpec:
+    rot, mask = m.get("rot"), m.get("mask")
+    spec = AttentionSpec(_count(m, "heads", at), _count(m, "kv_heads", at), _count(m, "dim", at), _count(m, "vdim", at),
+                         _real(m, "scale", at), _count(mask, "size", at + "mask.") if mask else 0,
+                         _count(rot, "dims", at + "rot.", 0) if rot else 0, _real(rot, "base", at + "rot.") if rot else 1.0)
+    if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim:
+        raise ConfigError(f"config.json: `{at}` heads / kv_heads / rot.dims do not fit together")
+    return spec
+
+
+def _latent_spec(m: Any, at: str) -> LatentAttentionSpec:
+    rot = _need(m, "rot", at)
+    spec = LatentAttentionSpec(_count(m, "heads", at), _count(m, "dim", at), _count(m, "rot_dim", at), _count(m, "vdim", at),
+                               _count(m, "kv_rank", at), _real(m, "scale", at), _real(rot, "base", at + "rot."))
+    if spec.rot_dim % 2 or _count(rot, "dims", at + "rot.") != spec.rot_dim:
+        raise ConfigError(f"config.json: `{at}rot.dims` must equal `rot_dim`, an even number")
+    return spec
+
+
+def _channel_delta_spec(m: Any, at: str) -> ChannelDeltaSpec:
+    spec = ChannelDeltaSpec(_count(m, "heads", at), _count(m, "kv_heads", at), _count(m, "dim", at), _count(m, "vdim", at),
+                            _count(m, "conv", at))
+    if spec.heads % spec.kv_heads:
+        raise ConfigError(f"config.json: `{at}kv_heads` does not divide `heads`")
+    return spec
+
+
+def _experts_spec(f: Any, at: str) -> ExpertsSpec:
+    r = _need(f, "router", at)
+    return ExpertsSpec(_count(r, "experts", at + "router."), _count(r, "top", at + "router."),
+                       _count(_need(f, "expert", at), "ff", at + "expert."))
+
+
+def _dense_spec(f: Any, at: str) -> DenseSpec:
+    return DenseSpec(_count(f, "ff", at))
+
+
+# what a design's layers may consist of: readers by layer type and by feed-forward kind
+_LAYER_PARTS = {
+    Architecture.ZOBUNEX: ({"attention": _attention_spec}, {"moe": _experts_spec}),
+    Architecture.GUNEDRA: ({"latent_attention": _latent_spec, "channel_delta": _channel_delta_spec}, {"dense": _dense_spec}),
+}
+
+
 @dataclass(frozen=True)
 class StackConfig:
     """A decoder described layer by layer, with an optional range of layers that runs several times in a row."""
     layers: tuple[LayerSpec, ...]
     loop: LoopSpec | None
     logit_scale: float
+    embed_scale: float = 1.0       # the embedding rows enter the stream times this
+    residual_mult: float = 1.0     # every sublayer's result joins the stream times this
+    norm_groups: int = 1           # the stream norms take the root mean square of this many equal parts separately
 
     def runs(self) -> list[tuple[int, bool]]:
         """(layer, first layer of a loop pass) in execution order; every run owns a cache."""
@@ -186,55 +299,36 @@ class StackConfig:
         return out + [(i, False) for i in range(lp.stop, n)]
 
     @staticmethod
-    def from_json(top: dict[str, Any]) -> "StackConfig":
-        def need(d: Any, key: str, where: str) -> Any:
-            if not isinstance(d, dict) or d.get(key) is None:
-                raise ConfigError(f"config.json missing `{where}{key}`")
-            return d[key]
-
-        def count(d: Any, key: str, where: str, low: int = 1) -> int:
-            v = need(d, key, where)
-            if isinstance(v, bool) or not isinstance(v, (int, float)) or int(v) != v or v < low:
-                raise ConfigError(f"config.json: `{where}{key}` must be an integer >= {low}, not {v!r}")
-            return int(v)
-
-        def real(d: Any, key: str, where: str) -> float:
-            v = need(d, key, where)
-            if isinstance(v, bool) or not isinstance(v, (int, float)):
-                raise ConfigError(f"config.json: `{where}{key}` must be a number, not {v!r}")
-            return float(v)
-
+    def from_json(top: dict[str, Any], arch: Architecture) -> "StackConfig":
+        mixers, ffs = _LAYER_PARTS[arch]
         layers = []
-        for i, lay in enumerate(need(top, "layers", "")):
+        for i, lay in enumerate(_need(top, "layers", "")):
             at = f"layers[{i}]."
-            if need(lay, "type", at) != "attention":
+            if _need(lay, "type", at) not in mixers:
                 raise Unsupported(f"config.json: `{at}type` {lay['type']!r}")
-            m, mw = need(lay, "mixer", at), at + "mixer."
-            rot, mask = m.get("rot"), m.get("mask")
-            spec = AttentionSpec(count(m, "heads", mw), count(m, "kv_heads", mw), count(m, "dim", mw), count(m, "vdim", mw),
-                                 real(m, "scale", mw), count(mask, "size", mw + "mask.") if mask else 0,
-                                 count(rot, "dims", mw + "rot.", 0) if rot else 0, real(rot, "base", mw + "rot.") if rot else 1.0)
-            if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim:
-                raise ConfigError(f"config.json: `{mw}` heads / kv_heads / rot.dims do not fit together")
+            spec = mixers[lay["type"]](_need(lay, "mixer", at), at + "mixer.")
             mlp, f = None, lay.get("mlp")
             if f is not None:
-                fw = at + "mlp."
-                if need(f, "kind", fw) != "moe":
-                    raise Unsupported(f"config.json: `{fw}kind` {f['kind']!r}")
-                r = need(f, "router", fw)
-                mlp = ExpertsSpec(count(r, "experts", fw + "router."), count(r, "top", fw + "router."),
-                                  count(need(f, "expert", fw), "ff", fw + "expert."))
+                if _need(f, "kind", at + "mlp.") not in ffs:
+                    raise Unsupported(f"config.json: `{at}mlp.kind` {f['kind']!r}")
+                mlp = ffs[f["kind"]](f, at + "mlp.")
             layers.append(LayerSpec(spec, mlp))
         if not layers:
             raise ConfigError("config.json: `layers` is empty")
+        if arch is Architecture.GUNEDRA:
+            groups, width = _count(_need(top, "norm", ""), "groups", "norm."), _count(top, "width", "")
+            if width % groups:
+                raise ConfigError("config.json: `norm.groups` does not divide `width`")
+            return StackConfig(tuple(layers), None, 1.0, _real(_need(top, "embedding", ""), "scale", "embedding."),
+                               _real(top, "residual_mult", ""), groups)
         loop, lp = None, top.get("loop")
         if lp:
-            loop = LoopSpec(count(lp, "start", "loop.", 0), count(lp, "stop", "loop.", 0), count(lp, "times", "loop."))
+            loop = LoopSpec(_count(lp, "start", "loop.", 0), _count(lp, "stop", "loop.", 0), _count(lp, "times", "loop."))
             if loop.start > loop.stop or loop.stop > len(layers):
                 raise ConfigError("config.json: `loop` does not lie within the layers")
             if loop.start == loop.stop:
                 loop = None
-        return StackConfig(tuple(layers), loop, real(top, "logit_scale", "") if top.get("logit_scale") is not None else 1.0)
+        return StackConfig(tuple(layers), loop, _real(top, "logit_scale", "") if top.get("logit_scale") is not None else 1.0)
 
 
 @dataclass
@@ -269,7 +363,7 @@ class ModelConfig:
     @staticmethod
     def from_json(top: dict[str, Any]) -> "ModelConfig":
         arch = Architecture.from_config(top)
-        if arch is Architecture.ZOBUNEX:
+        if arch in LISTED:
             return ModelConfig._from_stack(top, arch)
         v = top.get("text_config", top) if arch is Architecture.QWEN3_VL else top
 
@@ -362,7 +456,7 @@ class ModelConfig:
     @staticmethod
     def _from_stack(top: dict[str, Any], arch: Architecture) -> "ModelConfig":
         """A config that lists its layers; the flat fields hold the largest value over the layers."""
-        stack = StackConfig.from_json(top)
+        stack = StackConfig.from_json(top, arch)
         norm = top.get("norm") if isinstance(top.get("norm"), dict) else {}
         for key, v in (("width", top.get("width")), ("vocab", top.get("vocab")), ("norm.eps", norm.get("eps"))):
             if isinstance(v, bool) or not isinstance(v, (int, float)) or v <= 0:

@@ -43,6 +43,10 @@ class StepInputs:
     #                                           this step: replaces the position-indexed table (three-axis rotary phases)
     deepstack: tuple[torch.Tensor, list[torch.Tensor]] | None = None   # (int64 rows [R], taps): taps[l] [R, H] is added
     #                                           to the residual stream at those rows after decoder layer l (Qwen3-VL)
+    state_slots: torch.Tensor | None = None    # int32 [num_seqs]: slot of each sequence's recurrent state (-1 = do not
+    #                                           touch any: a padding row); None for models without recurrent layers
+    spans: list[tuple[int, int]] | None = None # host copy of (new tokens, context length) per sequence; None in a decode
+    #                                           step (one token each, lengths change under a captured graph)
 
 
 def splits_for(batch: int, kv_heads: int, max_kv: int, sms: int = 148) -> int:

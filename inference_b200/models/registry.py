@@ -9,7 +9,7 @@ from .config import Architecture, ModelConfig
 
 def gpu_supported(cfg: ModelConfig) -> bool:
     """True when a paged sm_100a decoder exists for this configuration."""
-    if cfg.architecture is Architecture.ZOBUNEX:
+    if cfg.stack is not None:
         return True
     return (cfg.head_dim == 128 and cfg.mla is None and
             cfg.architecture not in (Architecture.QWEN35, Architecture.DEEPSEEK_V2))
@@ -24,6 +24,10 @@ def gpu_model(cfg: ModelConfig, comm=None, device: torch.device | None = None, d
         from .zobunex import ZobunexGpu
 
         return ZobunexGpu(cfg, comm=comm, device=device, dtype=dtype)
+    if cfg.architecture is Architecture.GUNEDRA:
+        from .gunedra import GunedraGpu
+
+        return GunedraGpu(cfg, comm=comm, device=device, dtype=dtype)
     if dtype != torch.bfloat16:
         raise Unsupported(f"{cfg.architecture.value}: the sm_100a decoder computes in bfloat16")
     from .llama import LlamaGpu

@@ -1,0 +1,100 @@
+"""What the decoders whose config lists its layers share: construction, rotary tables, padded weights, projections, logits."""
+from __future__ import annotations
+
+import torch
+
+from .. import ops
+from ..contracts.errors import LoadError, Unsupported
+from ..engine.kv_pool import LayeredKvPool
+from ..parallel.comm import Communicator, single
+from .config import ModelConfig
+
+
+def up8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+class StackDecoder:
+    """One GPU, bf16 or true 32-bit (numerical checks). Widths that are not multiples of eight are padded with zero rows /
+    columns at load time, which changes no result."""
+    name = "stack"
+    recurrent = False      # the cache pool needs state slots
+
+    def __init__(self, cfg: ModelConfig, comm: Communicator | None = None, device: torch.device | None = None,
+                 dtype: torch.dtype = torch.bfloat16):
+        if cfg.stack is None:
+            raise Unsupported(f"{self.name} needs a config that lists its layers")
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise Unsupported(f"dtype {dtype}: bfloat16 or float32")
+        self.comm = comm or single(device)
+        if self.comm.is_parallel:
+            raise Unsupported(f"{self.name} runs on one GPU; tensor parallelism is not built for it")
+        self.cfg, self.stack, self.dtype = cfg, cfg.stack, dtype
+        self.device = device or self.comm.device
+        self.width, self.hp = cfg.hidden_size, up8(cfg.hidden_size)
+        self.layers: list = []
+        self.embed = self.final = None
+        self._rope: dict[tuple[int, float], tuple[torch.Tensor, torch.Tensor]] = {}
+        self.max_positions = 0
+        self.launches = 0
+
+    # ---- cache geometry -----------------------------------------------------------------------------------------
+    def kv_geometry(self) -> list:
+        raise NotImplementedError
+
+    def kv_block_bytes(self, block_size: int = 16) -> int:
+        return LayeredKvPool.block_bytes(self.kv_geometry(), block_size, self.dtype.itemsize)
+
+    def make_pool(self, num_blocks: int, block_size: int = 16, state_slots: int = 0) -> LayeredKvPool:
+        return LayeredKvPool(self.kv_geometry(), num_blocks, block_size, device=self.device, dtype=self.dtype, state_slots=state_slots)
+
+    # ---- rotary tables --------------------------------------------------------------------------------------------
+    def rotations(self) -> set[tuple[int, float]]:
+        """(rotated dimensions, base) of every layer that rotates."""
+        raise NotImplementedError
+
+    def ensure_rope(self, max_positions: int) -> None:
+        if max_positions <= self.max_positions:
+            return
+        for dims, base in self.rotations():
+            i = torch.arange(dims // 2, dtype=torch.float64)
+            ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * (base ** (-2.0 * i / max(dims, 1)))[None, :]
+            self._rope[(dims, base)] = (ang.cos().float().to(self.device).contiguous(),
+                                        ang.sin().float().to(self.device).contiguous())
+        self.max_positions = max_positions
+
+    # ---- weights ----------------------------------------------------------------------------------------------------
+    @staticmethod
+    def tensor(weights: dict[str, torch.Tensor], name: str, *shape: int | None) -> torch.Tensor:
+        """A tensor by name, its shape checked (None: any extent)."""
+        if name not in weights:
+            raise LoadError(f"missing tensor {name}")
+        t = weights[name]
+        if len(t.shape) != len(shape) or any(b is not None and a != b for a, b in zip(t.shape, shape)):
+            raise LoadError(f"tensor {name} has shape {tuple(t.shape)}, expected {shape}")
+        return t
+
+    def _mat(self, t: torch.Tensor) -> torch.Tensor:
+        """A matrix whose columns are stream columns: padded to the padded width, in the compute type, on the device."""
+        return torch.nn.functional.pad(t.to(self.device, self.dtype), (0, self.hp - self.width)).contiguous()
+
+    def _fp32(self, t: torch.Tensor, pad_to: int | None = None) -> torch.Tensor:
+        t = t.to(self.device, torch.float32)
+        return torch.nn.functional.pad(t, (0, (pad_to or t.shape[-1]) - t.shape[-1])).contiguous()
+
+    # ---- forward ----------------------------------------------------------------------------------------------------
+    def _linear(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
+                out: torch.Tensor | None = None) -> torch.Tensor:
+        self.launches += 1
+        if self.dtype == torch.float32:
+            return ops.gemm_f32(a, w, out=out)
+        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16)
+
+    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        if hidden.shape[0] == 0:
+            return torch.empty((0, self.cfg.vocab_size), dtype=torch.float32, device=self.device)
+        return self._linear(hidden, self.embed, torch.float32)
+
+    def greedy_tokens(self, hidden: torch.Tensor) -> torch.Tensor:
+        self.launches += 1
+        return ops.argmax(self.logits(hidden))

@@ -26,15 +26,12 @@ import torch
 
 from .. import ops
 from ..contracts.errors import LoadError, Unsupported
-from ..engine.kv_pool import KvGeometry, LayeredKvPool
+from ..engine.kv_pool import KvGeometry
 from ..ops import Branch, NormWeights
-from ..parallel.comm import Communicator, single
+from ..parallel.comm import Communicator
 from .config import AttentionSpec, ExpertsSpec, ModelConfig
 from .llama import StepInputs, splits_for
-
-
-def _up8(n: int) -> int:
-    return (n + 7) // 8 * 8
+from .stack import StackDecoder, up8 as _up8
 
 
 @dataclass
@@ -56,65 +53,37 @@ class _Layer:
     table: tuple[tuple[int, int], int] | None = None   # (routing group, index in it)
 
 
-class ZobunexGpu:
+class ZobunexGpu(StackDecoder):
+    name = "Zobunex"
+
     def __init__(self, cfg: ModelConfig, comm: Communicator | None = None, device: torch.device | None = None,
                  dtype: torch.dtype = torch.bfloat16):
-        if cfg.stack is None:
-            raise Unsupported("ZobunexGpu needs a config that lists its layers")
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise Unsupported(f"dtype {dtype}: bfloat16 or float32")
-        self.comm = comm or single(device)
-        if self.comm.is_parallel:
-            raise Unsupported("Zobunex runs on one GPU; tensor parallelism is not built for it")
-        self.cfg, self.stack, self.dtype = cfg, cfg.stack, dtype
-        self.device = device or self.comm.device
-        self.width, self.hp = cfg.hidden_size, _up8(cfg.hidden_size)
+        super().__init__(cfg, comm, device, dtype)
         self.runs = self.stack.runs()
         self.loops = self.stack.loop is not None
         self.layers: list[_Layer] = []
         self.tables: dict[tuple[int, int], torch.Tensor] = {}   # (experts, top) -> int32 [layers of the group, vocab, top]
-        self.embed = self.loop_in = self.final = None
-        self._rope: dict[tuple[int, float], tuple[torch.Tensor, torch.Tensor]] = {}
-        self.max_positions = 0
-        self.launches = 0
+        self.loop_in = None
 
     # ---- cache geometry and scheduling hooks ----------------------------------------------------------------
     def kv_geometry(self) -> list[KvGeometry]:
         lays = self.stack.layers
         return [KvGeometry(lays[i].mixer.kv_heads, _up8(lays[i].mixer.dim), _up8(lays[i].mixer.vdim)) for i, _ in self.runs]
 
-    def kv_block_bytes(self, block_size: int = 16) -> int:
-        return LayeredKvPool.block_bytes(self.kv_geometry(), block_size, self.dtype.itemsize)
-
-    def make_pool(self, num_blocks: int, block_size: int = 16) -> LayeredKvPool:
-        return LayeredKvPool(self.kv_geometry(), num_blocks, block_size, device=self.device, dtype=self.dtype)
-
     def decode_splits(self, batch: int, max_kv: int) -> tuple[int, ...]:
         """KV splits per layer: a chunked layer never reads more than one chunk (plus the rest of its first tile)."""
         return tuple(splits_for(batch, m.kv_heads, min(max_kv, m.chunk + 63) if m.chunk else max_kv)
                      for m in (lay.mixer for lay in self.stack.layers))
 
-    def ensure_rope(self, max_positions: int) -> None:
-        if max_positions <= self.max_positions:
-            return
-        for dims, base in {(lay.mixer.rot_dims, lay.mixer.rot_base) for lay in self.stack.layers}:
-            i = torch.arange(dims // 2, dtype=torch.float64)
-            ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * (base ** (-2.0 * i / max(dims, 1)))[None, :]
-            self._rope[(dims, base)] = (ang.cos().float().to(self.device).contiguous(),
-                                        ang.sin().float().to(self.device).contiguous())
-        self.max_positions = max_positions
+    def rotations(self) -> set[tuple[int, float]]:
+        return {(lay.mixer.rot_dims, lay.mixer.rot_base) for lay in self.stack.layers}
 
     # ---- weights ----------------------------------------------------------------------------------------------
     def load_state_dict(self, weights: dict[str, torch.Tensor]) -> "ZobunexGpu":
         W, V = self.width, self.cfg.vocab_size
 
         def get(name: str, *shape: int) -> torch.Tensor:
-            if name not in weights:
-                raise LoadError(f"missing tensor {name}")
-            t = weights[name]
-            if tuple(t.shape) != shape:
-                raise LoadError(f"tensor {name} has shape {tuple(t.shape)}, expected {shape}")
-            return t
+            return self.tensor(weights, name, *shape)
 
         def norm(name: str) -> NormWeights:
             return self._norm(get(name, W), get(name + ".b", W))
@@ -168,13 +137,8 @@ class ZobunexGpu:
         self._stack_tables(tables)
         return self
 
-    def _mat(self, t: torch.Tensor) -> torch.Tensor:
-        """A matrix whose columns are stream columns: padded to the padded width, in the compute type, on the device."""
-        return torch.nn.functional.pad(t.to(self.device, self.dtype), (0, self.hp - self.width)).contiguous()
-
     def _norm(self, w: torch.Tensor, b: torch.Tensor) -> NormWeights:
-        pad = (0, self.hp - self.width)
-        return NormWeights(*(torch.nn.functional.pad(t.to(self.device, torch.float32), pad).contiguous() for t in (w, b)))
+        return NormWeights(self._fp32(w, self.hp), self._fp32(b, self.hp))
 
     def _loop_matrix(self, w: torch.Tensor) -> torch.Tensor:
         W, out = self.width, torch.zeros((self.hp, 2 * self.hp), dtype=self.dtype, device=self.device)
@@ -215,13 +179,6 @@ class ZobunexGpu:
         return sum(t.nbytes for t in ts)
 
     # ---- forward ------------------------------------------------------------------------------------------------
-    def _linear(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
-                out: torch.Tensor | None = None) -> torch.Tensor:
-        self.launches += 1
-        if self.dtype == torch.float32:
-            return ops.gemm_f32(a, w, out=out)
-        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16)
-
     def _route(self, ids: torch.Tensor) -> dict:
         """Expert routing of every layer of this step. Steps with few rows per expert use dense segments (weight-streaming
         kernel), larger ones segments padded to the tile of the grouped tcgen05 GEMM."""
@@ -300,12 +257,3 @@ class ZobunexGpu:
             advance(None, None)
         return advance(self.final, torch.empty((inp.logits_rows.numel(), hp), dtype=self.dtype, device=dev),
                        rows=inp.logits_rows, out_scale=scale)
-
-    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        if hidden.shape[0] == 0:
-            return torch.empty((0, self.cfg.vocab_size), dtype=torch.float32, device=self.device)
-        return self._linear(hidden, self.embed, torch.float32)
-
-    def greedy_tokens(self, hidden: torch.Tensor) -> torch.Tensor:
-        self.launches += 1
-        return ops.argmax(self.logits(hidden))

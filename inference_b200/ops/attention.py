@@ -176,7 +176,7 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
             return out
     rc = kernels().swb_attn_simple(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), out.data_ptr(),
                                    out.stride(0), block_table.data_ptr(), block_table.stride(0), bs, ptr(cu_q),
-                                   kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq, Hkv, D, Dv, scale, chunk, ptr(sink),
+                                   kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq, Hkv, D, Dv, 0, scale, chunk, ptr(sink),
                                    1 if q.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_attn_simple")
     return out

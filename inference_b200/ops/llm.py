@@ -105,6 +105,20 @@ def gated_act_mul(gate_up: torch.Tensor, act: str = "silu", out: torch.Tensor | 
     return out.reshape(*gate_up.shape[:-1], F)
 
 
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, width: int | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """out = a N(z) + b N(z^2) + c N(z^3) + e for rows z [T, Fp] (bf16 / fp32), coef fp32 (a, b, c, e), powers element by element
+    and N(y) = y / sqrt(mean(y^2) + eps) over the first `width` columns (the rest hold zeros). fp32 statistics."""
+    require_cuda(z, coef)
+    T, Fp = z.shape
+    assert z.stride(1) == 1 and z.dtype in (torch.bfloat16, torch.float32) and coef.dtype == torch.float32 and coef.numel() == 4
+    if out is None:
+        out = torch.empty((T, Fp), dtype=z.dtype, device=z.device)
+    rc = kernels().swb_poly_norm(z.data_ptr(), z.stride(0), out.data_ptr(), out.stride(0), T, width or Fp, Fp, coef.data_ptr(), eps,
+                                 1 if z.dtype == torch.float32 else 0, stream_ptr())
+    check(rc, "swb_poly_norm")
+    return out
+
+
 def embedding(ids: torch.Tensor, table: torch.Tensor, *, scale: float = 1.0, vocab_start: int = 0,
               out: torch.Tensor | None = None) -> torch.Tensor:
     require_cuda(ids, table)
