@@ -95,4 +95,9 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
                             int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
                             const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
                             int num_blocks, cudaStream_t stream);
+int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok,
+                               const void* k2, long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok,
+                               int num_seqs, int max_q_len, int total_tokens, int H, int d1, int d2, int Dv, float scale,
+                               const float* sink, const void* gate, long long gate_stride, const int* cu_q, const int* seqs,
+                               const int* cu_k, cudaStream_t stream);
 }  // namespace swb

@@ -31,21 +31,23 @@ namespace {
 
 constexpr int BM = 128;          // query rows per tile (two tiles per CTA)
 constexpr int BN = 128;          // keys per tile
-constexpr int KV_STAGES = 2;
+constexpr int MAX_STAGES = 2;
 constexpr int THREADS = 320;
 constexpr uint32_t ATOM_BYTES = BM * 64 * 2;       // 16 KB: 128 rows of one 64-column swizzle atom
-// Head dim 128 (two swizzle atoms per tile) or 64 (one atom: half the shared memory and half the MMA work of the padded path).
-template <int HD>
+// Tile widths of q / k (QK) and of v (VD). 128 is two swizzle atoms per tile, 64 one atom (half the shared memory and half the
+// MMA work of the padded path); q and k of latent attention take up to three, which leaves room for one V stage.
+template <int QK, int VD>
 struct FaCfg {
-  static_assert(HD == 64 || HD == 128, "head dim 64 or 128");
-  static constexpr int ATOMS = HD / 64;
-  static constexpr uint32_t TILE_BYTES = BM * HD * 2;
+  static_assert((QK == 64 || QK == 128 || QK == 192) && (VD == 64 || VD == 128), "tile widths");
+  static constexpr int ATOMS = QK / 64, V_ATOMS = VD / 64;
+  static constexpr int K_STAGES = 2, V_STAGES = QK == 192 ? 1 : 2;
+  static constexpr uint32_t TILE_BYTES = BM * QK * 2, V_TILE_BYTES = BM * VD * 2;
   static constexpr uint32_t SMEM_Q = 0;                                   // 2 tiles
-  static constexpr uint32_t SMEM_K = 2 * TILE_BYTES;                      // KV_STAGES tiles
-  static constexpr uint32_t SMEM_V = SMEM_K + KV_STAGES * TILE_BYTES;
-  static constexpr uint32_t SMEM_BAR = SMEM_V + KV_STAGES * TILE_BYTES;
+  static constexpr uint32_t SMEM_K = 2 * TILE_BYTES;
+  static constexpr uint32_t SMEM_V = SMEM_K + K_STAGES * TILE_BYTES;
+  static constexpr uint32_t SMEM_BAR = SMEM_V + V_STAGES * V_TILE_BYTES;
   static constexpr size_t SMEM_BYTES = SMEM_BAR + 256 + 1024 /*alignment slack*/;
-  static constexpr int ROW_BYTES = HD * 2;                                // one output row of one head
+  static constexpr int ROW_BYTES = VD * 2;                                // one output row of one head
   static constexpr int CHUNKS = ROW_BYTES / 16;                           // 16-byte chunks per row
 };
 constexpr uint32_t TMEM_COLS = 512;
@@ -78,7 +80,14 @@ struct FaParams {
   // Extended problems (the EXT instantiations only):
   int chunk;           // > 0: query i sees key j <= i only if floor(i / chunk) == floor(j / chunk), positions of the sequence
   const float* sink;   // optional [Hq]: exp(sink[h]) joins the softmax denominator (no key, no value, not scaled)
-  int v_dim;           // width of the v heads and of the output heads (<= HD; the tile is zero filled beyond it)
+  int v_dim;           // width of the v heads and of the output heads (<= VD; the tile is zero filled beyond it)
+  // Latent attention (LAT): q and k in two parts, k's second part shared by the heads; keys and values are rows
+  // [cu_k[z], cu_k[z + 1]) of one flat axis (null: those of the queries), the queries the last positions of them.
+  const int* seqs;     // optional: sequence of blockIdx.z (cu_q is indexed by it, cu_k by blockIdx.z)
+  const int* cu_k;
+  const bf16* gate;    // optional [tokens, >= Hq] logits: head outputs are scaled by their sigmoid
+  long long gate_stride;
+  int first_atoms;     // 64-column atoms of the first part; the second takes the rest of the tile
 };
 
 __device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, uint64_t* bar, int c0, int c1, int c2,
@@ -152,8 +161,8 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
 
 struct Barriers {
   uint64_t q_full;
-  uint64_t k_full[KV_STAGES], k_empty[KV_STAGES];
-  uint64_t v_full[KV_STAGES], v_empty[KV_STAGES];
+  uint64_t k_full[MAX_STAGES], k_empty[MAX_STAGES];
+  uint64_t v_full[MAX_STAGES], v_empty[MAX_STAGES];
   uint64_t s_full[2];   // MMA -> softmax q: S_q of the current key tile is complete
   uint64_t p_full[2];   // softmax q -> MMA: P_q is in TMEM (128 arrivals)
   uint64_t o_final;     // every MMA of the CTA has completed
@@ -163,14 +172,16 @@ struct Barriers {
 
 // 168 registers per thread is the cap for ten warps: two of the four scheduler partitions hold three warps, and a
 // partition's file is 16 K registers (a build with 200 registers per thread does not launch).
-// EXT adds chunked masking, attention sinks and head widths below the tile width HD (q . k and P V then run over zero
-// columns that the tensor maps fill in).
-template <int HD, bool EXT>
+// EXT adds chunked masking, attention sinks and head widths below the tile widths (q . k and P V then run over zero
+// columns that the tensor maps fill in). LAT adds what latent attention needs: two-part q / k, key ranges, output gates.
+template <int QK, int VD, bool EXT, bool LAT>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                          const __grid_constant__ CUtensorMap tmap_v, const FaParams p) {
-  using C = FaCfg<HD>;
-  constexpr uint32_t TILE_BYTES = C::TILE_BYTES, SMEM_Q = C::SMEM_Q, SMEM_K = C::SMEM_K, SMEM_V = C::SMEM_V, SMEM_BAR = C::SMEM_BAR;
+                          const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_q2,
+                          const __grid_constant__ CUtensorMap tmap_k2, const FaParams p) {
+  using C = FaCfg<QK, VD>;
+  constexpr int K_STAGES = C::K_STAGES, V_STAGES = C::V_STAGES, V_ATOMS = C::V_ATOMS;
+  constexpr uint32_t TILE_BYTES = C::TILE_BYTES, V_TILE_BYTES = C::V_TILE_BYTES, SMEM_Q = C::SMEM_Q, SMEM_K = C::SMEM_K, SMEM_V = C::SMEM_V, SMEM_BAR = C::SMEM_BAR;
   constexpr int ATOMS = C::ATOMS, ROW_BYTES = C::ROW_BYTES, CHUNKS = C::CHUNKS;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -179,11 +190,13 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   const int q_base = blockIdx.x * (p.tiles * BM);
   const int head = blockIdx.y;
   // packed variable-length batch: this CTA's sequence covers tokens [tok0, tok0 + q_len) of one flat token axis
-  const int tok0 = p.cu_q ? p.cu_q[blockIdx.z] : 0;
-  const int q_len = p.cu_q ? p.cu_q[blockIdx.z + 1] - tok0 : p.q_len;
-  const bool paged = p.block_table != nullptr;
-  const int kv_len = paged ? p.kv_lens[blockIdx.z] : (p.cu_q ? q_len : p.kv_len);
-  const int coff = paged ? max(kv_len - q_len, 0) : 0;   // position of query 0 among the sequence's keys
+  const int seq = (LAT && p.seqs) ? p.seqs[blockIdx.z] : blockIdx.z;
+  const int tok0 = p.cu_q ? p.cu_q[seq] : 0;
+  const int q_len = p.cu_q ? p.cu_q[seq + 1] - tok0 : p.q_len;
+  const bool paged = !LAT && p.block_table != nullptr, ranged = LAT && p.cu_k;
+  const int key0_row = ranged ? p.cu_k[blockIdx.z] : tok0;
+  const int kv_len = paged ? p.kv_lens[blockIdx.z] : ranged ? p.cu_k[blockIdx.z + 1] - key0_row : (p.cu_q ? q_len : p.kv_len);
+  const int coff = paged || ranged ? max(kv_len - q_len, 0) : 0;   // position of query 0 among the sequence's keys
   const int batch = p.cu_q ? 0 : blockIdx.z;
   if (q_base >= q_len || kv_len <= 0) return;   // uniform for the whole CTA, before any barrier or TMEM allocation
   const int kv_head = head / (p.Hq / p.Hkv);
@@ -195,7 +208,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
 
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
-    for (int s = 0; s < KV_STAGES; ++s) {
+    for (int s = 0; s < MAX_STAGES; ++s) {
       mbar_init(&bars->k_full[s], 1);
       mbar_init(&bars->k_empty[s], 1);
       mbar_init(&bars->v_full[s], 1);
@@ -213,6 +226,10 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     tma_prefetch_desc(&tmap_q);
     tma_prefetch_desc(&tmap_k);
     tma_prefetch_desc(&tmap_v);
+    if constexpr (LAT) {
+      tma_prefetch_desc(&tmap_q2);
+      tma_prefetch_desc(&tmap_k2);
+    }
   }
   if (warp == 9) {
     tmem_alloc(&bars->tmem_base, TMEM_COLS);
@@ -230,9 +247,11 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     if (lane == 0) {
       mbar_arrive_expect_tx(&bars->q_full, p.tiles * TILE_BYTES);
       for (int q = 0; q < p.tiles; ++q)
-        for (int a = 0; a < ATOMS; ++a)
-          tma_load_4d(smem + SMEM_Q + q * TILE_BYTES + a * ATOM_BYTES, &tmap_q, &bars->q_full, a * 64, head,
-                      tok0 + q_base + q * BM, batch);
+        for (int a = 0; a < ATOMS; ++a) {
+          const bool second = LAT && a >= p.first_atoms;
+          tma_load_4d(smem + SMEM_Q + q * TILE_BYTES + a * ATOM_BYTES, second ? &tmap_q2 : &tmap_q, &bars->q_full,
+                      (second ? a - p.first_atoms : a) * 64, head, tok0 + q_base + q * BM, batch);
+        }
       bool ok = true;
       int issued_k = 0, issued_v = 0;
       // paged: a tile is BN / block_size pages, each a box of block_size rows that lands at its place in the swizzled
@@ -240,54 +259,57 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const int* pages = paged ? p.block_table + (long long)blockIdx.z * p.max_blocks : nullptr;
       const int per_tile = paged ? BN / p.block_size : 1, last_page = paged ? (kv_len - 1) / p.block_size : 0;
       const uint32_t page_bytes = paged ? (uint32_t)p.block_size * 128u : 0u;
-      auto load_tile = [&](uint32_t dst_off, const CUtensorMap* map, uint64_t* bar, int jrel) {
+      auto load_tile = [&](uint32_t dst_off, const CUtensorMap* map, uint64_t* bar, int jrel, int atoms, bool is_k) {
         const int j = jrel + j0;
         if (!paged) {
-          for (int a = 0; a < ATOMS; ++a)
-            tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * 64, kv_head, tok0 + j * BN, batch);
+          for (int a = 0; a < atoms; ++a) {
+            if (LAT && is_k && a >= p.first_atoms)
+              tma_load_4d(smem + dst_off + a * ATOM_BYTES, &tmap_k2, bar, (a - p.first_atoms) * 64, 0, key0_row + j * BN, batch);
+            else
+              tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * 64, kv_head, key0_row + j * BN, batch);
+          }
           return;
         }
         for (int g = 0; g < per_tile; ++g) {
           const int page = pages[min(j * per_tile + g, last_page)];
-          for (int a = 0; a < ATOMS; ++a)
+          for (int a = 0; a < atoms; ++a)
             tma_load_4d(smem + dst_off + a * ATOM_BYTES + g * page_bytes, map, bar, a * 64, 0, kv_head, page);
         }
       };
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int s = j % KV_STAGES;
-        const uint32_t ph = (j / KV_STAGES) & 1;
-        ok = mbar_wait(&bars->k_empty[s], ph ^ 1, abort_flag, 10);
+        const int s = j % K_STAGES, sv = j % V_STAGES;
+        ok = mbar_wait(&bars->k_empty[s], ((j / K_STAGES) & 1) ^ 1, abort_flag, 10);
         if (!ok) break;
         mbar_arrive_expect_tx(&bars->k_full[s], TILE_BYTES);
-        load_tile(SMEM_K + s * TILE_BYTES, &tmap_k, &bars->k_full[s], j);
+        load_tile(SMEM_K + s * TILE_BYTES, &tmap_k, &bars->k_full[s], j, ATOMS, true);
         issued_k = j + 1;
-        ok = mbar_wait(&bars->v_empty[s], ph ^ 1, abort_flag, 11);
+        ok = mbar_wait(&bars->v_empty[sv], ((j / V_STAGES) & 1) ^ 1, abort_flag, 11);
         if (!ok) break;
-        mbar_arrive_expect_tx(&bars->v_full[s], TILE_BYTES);
-        load_tile(SMEM_V + s * TILE_BYTES, &tmap_v, &bars->v_full[s], j);
+        mbar_arrive_expect_tx(&bars->v_full[sv], V_TILE_BYTES);
+        load_tile(SMEM_V + sv * V_TILE_BYTES, &tmap_v, &bars->v_full[sv], j, V_ATOMS, false);
         issued_v = j + 1;
       }
       if (!ok) {
         // drain: every copy this thread started must land before the CTA's shared memory is released
         volatile int never = 0;
         mbar_wait(&bars->q_full, 0, &never, 12);
-        for (int j = max(0, issued_k - KV_STAGES); j < issued_k; ++j)
-          mbar_wait(&bars->k_full[j % KV_STAGES], (j / KV_STAGES) & 1, &never, 13);
-        for (int j = max(0, issued_v - KV_STAGES); j < issued_v; ++j)
-          mbar_wait(&bars->v_full[j % KV_STAGES], (j / KV_STAGES) & 1, &never, 14);
+        for (int j = max(0, issued_k - K_STAGES); j < issued_k; ++j)
+          mbar_wait(&bars->k_full[j % K_STAGES], (j / K_STAGES) & 1, &never, 13);
+        for (int j = max(0, issued_v - V_STAGES); j < issued_v; ++j)
+          mbar_wait(&bars->v_full[j % V_STAGES], (j / V_STAGES) & 1, &never, 14);
       }
     }
   } else if (warp == 9) {
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t IDESC_QK = umma_idesc_bf16_f32(BM, BN);
-      constexpr uint32_t IDESC_PV = umma_idesc_bf16_f32(BM, HD) | (1u << 16);   // B is MN-major
+      constexpr uint32_t IDESC_PV = umma_idesc_bf16_f32(BM, VD) | (1u << 16);   // B is MN-major
       const uint32_t col_s[2] = {COL_S0, COL_S1}, col_o[2] = {COL_O0, COL_O1};
       const uint32_t q_addr = smem_u32(smem + SMEM_Q), k_addr = smem_u32(smem + SMEM_K),
                      v_addr = smem_u32(smem + SMEM_V);
       auto issue_qk = [&](int q, int s) {
 #pragma unroll
-        for (int k = 0; k < HD / 16; ++k) {
+        for (int k = 0; k < QK / 16; ++k) {
           const uint32_t off = (k >> 2) * ATOM_BYTES + (k & 3) * 32;
           umma_f16_ss(tmem + col_s[q], umma_desc_kmajor_sw128(q_addr + q * TILE_BYTES + off),
                       umma_desc_kmajor_sw128(k_addr + s * TILE_BYTES + off), IDESC_QK, k > 0);
@@ -303,8 +325,8 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         umma_commit(&bars->k_empty[0]);
       }
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int s = j % KV_STAGES, sn = (j + 1) % KV_STAGES;
-        const uint32_t ph = (j / KV_STAGES) & 1, phn = ((j + 1) / KV_STAGES) & 1;
+        const int s = j % V_STAGES, sn = (j + 1) % K_STAGES;
+        const uint32_t ph = (j / V_STAGES) & 1, phn = ((j + 1) / K_STAGES) & 1;
         ok = mbar_wait(&bars->v_full[s], ph, abort_flag, 22);
         if (ok && j + 1 < n_tiles) ok = mbar_wait(&bars->k_full[sn], phn, abort_flag, 23);
         for (int q = 0; q < p.tiles && ok; ++q) {
@@ -314,7 +336,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
 #pragma unroll
           for (int k = 0; k < BN / 16; ++k)
             umma_f16_ts(tmem + col_o[q], tmem + col_s[q] + k * 8,
-                        umma_desc_mnmajor_sw128(v_addr + s * TILE_BYTES + k * 2048), IDESC_PV, (j > 0) || (k > 0));
+                        umma_desc_mnmajor_sw128(v_addr + s * V_TILE_BYTES + k * 2048), IDESC_PV, (j > 0) || (k > 0));
           const bool last_q = (q == p.tiles - 1);
           if (last_q) umma_commit(&bars->v_empty[s]);
           if (j + 1 < n_tiles) {
@@ -382,7 +404,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
         if (j > 0) {   // O holds nothing before the first PV
 #pragma unroll
-          for (int c = 0; c < HD / 32; ++c) {
+          for (int c = 0; c < VD / 32; ++c) {
             uint32_t o[32];
             tmem_ld_x32(t_o + c * 32, o);
             tmem_ld_wait();
@@ -424,12 +446,18 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           inv = e / (l * e + ex2(sk - top));
         }
       }
-      // Stage this warp's 32 rows x HD columns in the (now idle) Q region, then write every row's HD * 2 bytes with
-      // HD / 8 lanes x 16 bytes: contiguous runs for local stores and for stores that cross NVLink alike.
+      if constexpr (LAT) {
+        if (p.gate && row < q_len) {
+          const float z = __bfloat162float(p.gate[(long long)(tok0 + row) * p.gate_stride + head]);
+          inv *= 1.f / (1.f + ex2(-1.4426950408889634f * z));
+        }
+      }
+      // Stage this warp's 32 rows x VD columns in the (now idle) Q region, then write every row's VD * 2 bytes with
+      // VD / 8 lanes x 16 bytes: contiguous runs for local stores and for stores that cross NVLink alike.
       // 16-byte chunk c of row r sits at c ^ (r & 7).
       uint8_t* slab = smem + SMEM_Q + warp * (32 * ROW_BYTES);
 #pragma unroll
-      for (int c = 0; c < HD / 32; ++c) {
+      for (int c = 0; c < VD / 32; ++c) {
         uint32_t o[32];
         tmem_ld_x32(t_o + c * 32, o);
         tmem_ld_wait();
@@ -453,13 +481,13 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           const uint4 val = *reinterpret_cast<const uint4*>(slab + r * ROW_BYTES + ((ch ^ (r & 7)) << 4));
           if (EXT && ch * 8 >= p.v_dim) continue;
           bf16* dst = p.out + ((long long)batch * p.q_len + tok0 + grow) * p.out_stride_tok +
-                      (long long)head * (EXT ? p.v_dim : HD);
+                      (long long)head * (EXT ? p.v_dim : VD);
           if (p.scatter.enabled) {
             const OutScatter& sc = p.scatter;
             const int g2 = grow - sc.split;
             const int rk = grow < sc.split ? grow / sc.n0 : g2 / sc.n1;
             const int local = grow < sc.split ? grow % sc.n0 : sc.n0 + g2 % sc.n1;
-            dst = sc.peer[rk] + (long long)local * p.out_stride_tok + sc.col_offset + head * HD;
+            dst = sc.peer[rk] + (long long)local * p.out_stride_tok + sc.col_offset + head * VD;
           }
           *reinterpret_cast<uint4*>(dst + ch * 8) = val;
         }
@@ -554,31 +582,40 @@ void attn_dense_tcgen05_set_tiles(int tiles) { g_force_tiles = tiles; }
 
 namespace {
 
-template <int HD, bool EXT>
-int launch_fa(dim3 grid, cudaStream_t stream, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
-              const FaParams& p) {
+struct FaMaps {
+  CUtensorMap q, k, v, q2, k2;     // q2 / k2: second parts of latent attention
+};
+
+template <int QK, int VD, bool EXT, bool LAT>
+int launch_fa(dim3 grid, cudaStream_t stream, const FaMaps& m, const FaParams& p) {
   static bool configured[64] = {false};
+  auto kernel = attn_dense_tcgen05_kernel<QK, VD, EXT, LAT>;
+  constexpr size_t SMEM = FaCfg<QK, VD>::SMEM_BYTES;
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_dense_tcgen05_kernel<HD, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)FaCfg<HD>::SMEM_BYTES);
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);
     if (e != cudaSuccess) return -(int)e;
     configured[dev] = true;
   }
-  return launch_kernel(attn_dense_tcgen05_kernel<HD, EXT>, grid, dim3(THREADS), FaCfg<HD>::SMEM_BYTES, stream, tq, tk, tv, p);
+  return launch_kernel(kernel, grid, dim3(THREADS), SMEM, stream, m.q, m.k, m.v, m.q2, m.k2, p);
 }
 
-int launch_tiles(int hd, bool ext, int q_len, int Hq, int batch, cudaStream_t stream, const CUtensorMap& tq,
-                 const CUtensorMap& tk, const CUtensorMap& tv, FaParams& p) {
+enum class FaKind { DENSE, EXT, LATENT };
+
+// qk: tile width of q and k
+int launch_tiles(int qk, FaKind kind, int q_len, int Hq, int batch, cudaStream_t stream, const FaMaps& m, FaParams& p) {
   // one-tile CTAs when that shortens the schedule: a one-tile CTA takes ~0.85 of a two-tile CTA's time (measured)
   const int sms = 148;
   const long c2 = (long)((q_len + 2 * BM - 1) / (2 * BM)) * Hq * batch, c1 = (long)((q_len + BM - 1) / BM) * Hq * batch;
   const double t2 = (double)((c2 + sms - 1) / sms), t1 = 0.85 * (double)((c1 + sms - 1) / sms);
   p.tiles = (g_force_tiles == 1 || g_force_tiles == 2) ? g_force_tiles : (t1 < t2 ? 1 : 2);
   const dim3 grid((q_len + p.tiles * BM - 1) / (p.tiles * BM), Hq, batch);
-  if (ext) return hd == 64 ? launch_fa<64, true>(grid, stream, tq, tk, tv, p) : launch_fa<128, true>(grid, stream, tq, tk, tv, p);
-  return hd == 64 ? launch_fa<64, false>(grid, stream, tq, tk, tv, p) : launch_fa<128, false>(grid, stream, tq, tk, tv, p);
+  if (kind == FaKind::LATENT)
+    return qk == 192 ? launch_fa<192, 128, true, true>(grid, stream, m, p) : launch_fa<128, 128, true, true>(grid, stream, m, p);
+  if (kind == FaKind::EXT)
+    return qk == 64 ? launch_fa<64, 64, true, false>(grid, stream, m, p) : launch_fa<128, 128, true, false>(grid, stream, m, p);
+  return qk == 64 ? launch_fa<64, 64, false, false>(grid, stream, m, p) : launch_fa<128, 128, false, false>(grid, stream, m, p);
 }
 
 }  // namespace
@@ -605,16 +642,16 @@ int attn_dense_tcgen05_launch(const void* q, long long q_stride_tok, int q_strid
   if (paged && (head_dim != 128 || !cu_q || !kv_lens || block_size < 8 || block_size % 8 || BN % block_size ||
                 num_blocks <= 0 || max_blocks <= 0 || peers))
     return -3;
-  CUtensorMap tq, tk, tv;
+  FaMaps m{};
   // packed batches address one flat token axis (batch = the number of sequences only sizes the grid)
   const int map_q_tokens = cu_q ? total_tokens : q_len, map_kv_tokens = cu_q ? total_tokens : kv_len;
   const int map_batch = cu_q ? 1 : batch;
-  int rc = make_tmap_heads(&tq, q, head_dim, Hq, map_q_tokens, map_batch, q_stride_head, q_stride_tok, q_stride_tok * map_q_tokens);
+  int rc = make_tmap_heads(&m.q, q, head_dim, Hq, map_q_tokens, map_batch, q_stride_head, q_stride_tok, q_stride_tok * map_q_tokens);
   if (rc) return rc;
-  rc = make_tmap_heads(&tk, k, head_dim, Hkv, map_kv_tokens, paged ? num_blocks : map_batch, kv_stride_head,
+  rc = make_tmap_heads(&m.k, k, head_dim, Hkv, map_kv_tokens, paged ? num_blocks : map_batch, kv_stride_head,
                        kv_stride_tok, kv_stride_tok * map_kv_tokens, paged ? block_size : 0);
   if (rc) return rc;
-  rc = make_tmap_heads(&tv, v, head_dim, Hkv, map_kv_tokens, paged ? num_blocks : map_batch, kv_stride_head,
+  rc = make_tmap_heads(&m.v, v, head_dim, Hkv, map_kv_tokens, paged ? num_blocks : map_batch, kv_stride_head,
                        kv_stride_tok, kv_stride_tok * map_kv_tokens, paged ? block_size : 0);
   if (rc) return rc;
   FaParams p{};
@@ -641,7 +678,7 @@ int attn_dense_tcgen05_launch(const void* q, long long q_stride_tok, int q_strid
     p.scatter.n1 = n1;
     p.scatter.col_offset = col_offset;
   }
-  return launch_tiles(head_dim, false, q_len, Hq, batch, stream, tq, tk, tv, p);
+  return launch_tiles(head_dim, FaKind::DENSE, q_len, Hq, batch, stream, m, p);
 }
 
 // Attention over queries and keys of any head widths up to 128 (multiples of 8), with chunked masking and sinks: the
@@ -661,13 +698,13 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
   if (paged ? (!kv_lens || block_size < 8 || block_size % 8 || BN % block_size || num_blocks <= 0 || max_blocks <= 0)
             : ((k_stride_tok | v_stride_tok) % 8 != 0))
     return -3;
-  CUtensorMap tq, tk, tv;
-  int rc = make_tmap_heads(&tq, q, D, Hq, total_tokens, 1, D, q_stride_tok, q_stride_tok * total_tokens);
+  FaMaps m{};
+  int rc = make_tmap_heads(&m.q, q, D, Hq, total_tokens, 1, D, q_stride_tok, q_stride_tok * total_tokens);
   if (rc) return rc;
-  rc = make_tmap_heads(&tk, k, D, Hkv, total_tokens, paged ? num_blocks : 1, D, k_stride_tok, k_stride_tok * total_tokens,
+  rc = make_tmap_heads(&m.k, k, D, Hkv, total_tokens, paged ? num_blocks : 1, D, k_stride_tok, k_stride_tok * total_tokens,
                        paged ? block_size : 0);
   if (rc) return rc;
-  rc = make_tmap_heads(&tv, v, Dv, Hkv, total_tokens, paged ? num_blocks : 1, Dv, v_stride_tok, v_stride_tok * total_tokens,
+  rc = make_tmap_heads(&m.v, v, Dv, Hkv, total_tokens, paged ? num_blocks : 1, Dv, v_stride_tok, v_stride_tok * total_tokens,
                        paged ? block_size : 0);
   if (rc) return rc;
   FaParams p{};
@@ -685,7 +722,46 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
   p.chunk = chunk;
   p.sink = sink;
   p.v_dim = Dv;
-  return launch_tiles(D > 64 || Dv > 64 ? 128 : 64, true, max_q_len, Hq, num_seqs, stream, tq, tk, tv, p);
+  return launch_tiles(D > 64 || Dv > 64 ? 128 : 64, FaKind::EXT, max_q_len, Hq, num_seqs, stream, m, p);
+}
+
+// Latent attention on expanded keys and values, causal: q [total_tokens] rows of H heads of [d1 | d2] (stride q_stride_tok), k
+// and v rows of one flat axis of key_rows rows (heads of d1 and Dv columns), k2 [key_rows] rows of d2 columns shared by the
+// heads. cu_k [num_seqs + 1]: each sequence's key rows, ending with those of its queries (null: the queries' own rows). seqs:
+// the sequences of this launch (null: all). gate: logits [total_tokens, >= H] or null.
+int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok,
+                               const void* k2, long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok,
+                               int num_seqs, int max_q_len, int total_tokens, int H, int d1, int d2, int Dv, float scale,
+                               const float* sink, const void* gate, long long gate_stride, const int* cu_q, const int* seqs,
+                               const int* cu_k, cudaStream_t stream) {
+  if (d1 < 8 || d2 < 8 || Dv < 8 || d1 > 128 || d2 > 64 || Dv > 128 || ((d1 | d2 | Dv) % 8) || !cu_q || !(scale > 0.f)) return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
+       reinterpret_cast<uintptr_t>(k2) | reinterpret_cast<uintptr_t>(out)) & 15)
+    return -3;
+  if ((q_stride_tok | kv_stride_tok | k2_stride_tok | out_stride_tok) % 8) return -3;
+  FaMaps m{};
+  const bf16* qb = reinterpret_cast<const bf16*>(q);
+  int rc = make_tmap_heads(&m.q, qb, d1, H, total_tokens, 1, d1 + d2, q_stride_tok, q_stride_tok * total_tokens);
+  if (!rc) rc = make_tmap_heads(&m.q2, qb + d1, d2, H, total_tokens, 1, d1 + d2, q_stride_tok, q_stride_tok * total_tokens);
+  if (!rc) rc = make_tmap_heads(&m.k, k, d1, H, key_rows, 1, d1, kv_stride_tok, kv_stride_tok * key_rows);
+  if (!rc) rc = make_tmap_heads(&m.k2, k2, d2, 1, key_rows, 1, d2, k2_stride_tok, k2_stride_tok * key_rows);
+  if (!rc) rc = make_tmap_heads(&m.v, v, Dv, H, key_rows, 1, Dv, kv_stride_tok, kv_stride_tok * key_rows);
+  if (rc) return rc;
+  FaParams p{};
+  p.out = reinterpret_cast<bf16*>(out);
+  p.out_stride_tok = out_stride_tok;
+  p.Hq = p.Hkv = H;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.causal = 1;
+  p.cu_q = cu_q;
+  p.sink = sink;
+  p.v_dim = Dv;
+  p.seqs = seqs;
+  p.cu_k = cu_k;
+  p.gate = reinterpret_cast<const bf16*>(gate);
+  p.gate_stride = gate_stride;
+  p.first_atoms = (d1 + 63) / 64;
+  return launch_tiles(p.first_atoms == 1 ? 128 : 192, FaKind::LATENT, max_q_len, H, num_seqs, stream, m, p);
 }
 
 }  // namespace swb

@@ -1,7 +1,17 @@
 // Latent attention: a token's keys and values of all heads are projections of one cached row [c | k_rot], c the normed latent
 // (rank numbers) and k_rot the rotated key part shared by the heads.
-//   latent_prep   norm of c, rotation of k_rot and of every head's rotated query part, cache write.
+//   latent_prep     norm of c, rotation of k_rot and of every head's rotated query part, cache write.
+//   latent_decode   attention in the latent space for steps with few tokens per sequence. The queries were taken through the
+//                   key projection, so all heads read the same cached rows, which serve as keys (all columns) and as values
+//                   (the latent columns). Everything is computed transposed on the tensor cores: S^T = K Q^T puts 128 keys on
+//                   the rows of the MMA and the (few) query rows on its columns, O^T = C^T P^T the latent columns on the rows;
+//                   C^T is the very tile that served as K, read as an MN-major operand. A page row is fetched once per 16 or
+//                   32 query rows. Partial results of KV splits stay un-normalised in fp32.
+//   head_mma        per-head products with the key and value projections around it; the value side merges the splits, adds
+//                   the sink to the denominator and applies the output gate.
+#include "attention_common.cuh"
 #include "common.cuh"
+#include "gemm_tcgen05.cuh"
 
 namespace swb {
 
@@ -18,7 +28,8 @@ struct LatentPrepParams {
   const int* positions;
   const long long* slots;    // row of the cache, < 0: none
   void* cache;               // [rows, rk + rp]
-  void* q_abs;               // optional [T, H, rk + rp]: receives the rotated query part at column rk
+  void* q_abs;               // optional [rows, H, rk + rp]: receives the rotated query part at column rk
+  const int* q_row;          // optional [T]: row of q_abs of each token, < 0: none
   int T, H, dn, rot, rp, rank, rk;
 };
 
@@ -47,6 +58,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
     c[i] = x;
     if (dst) dst[i] = x;
   }
+  const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t;
   const float* cs = p.cos + (size_t)pos * (p.rot / 2);
   const float* sn = p.sin + (size_t)pos * (p.rot / 2);
   for (int i = threadIdx.x; i < (p.H + 1) * half; i += 256) {       // pairs of the heads' queries, then of the shared key
@@ -59,9 +71,527 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
       from_f(y[1], v * a + u * b);
       x[0] = y[0], x[1] = y[1];
     }
-    E* to = h < p.H ? (p.q_abs ? reinterpret_cast<E*>(p.q_abs) + ((size_t)t * p.H + h) * width : nullptr) : dst;
+    E* to = h < p.H ? (q_row >= 0 ? reinterpret_cast<E*>(p.q_abs) + ((size_t)q_row * p.H + h) * width : nullptr) : dst;
     if (to) to[p.rk + 2 * k] = y[0], to[p.rk + 2 * k + 1] = y[1];
   }
+}
+
+// Cached rows of several sequences side by side: out row cu_k[s] + i is row i of sequence s (16-byte pieces).
+__global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table,
+                                                            int max_blocks, int block_size, const int* __restrict__ seqs,
+                                                            const int* __restrict__ cu_k, int num_seqs, int rows, int pieces, uint4* out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < (long long)rows * pieces; i += (long long)gridDim.x * 256) {
+    const int r = (int)(i / pieces), c = (int)(i % pieces);
+    const int z = seq_of_token(cu_k, num_seqs, 1, r), k = r - cu_k[z], s = seqs ? seqs[z] : z;
+    const int page = block_table[(size_t)s * max_blocks + k / block_size];
+    out[i] = cache[((size_t)page * block_size + k % block_size) * pieces + c];
+  }
+}
+
+// ---- attention in the latent space ---------------------------------------------------------------------------------
+constexpr int DEC_KEYS = 128;                      // keys per tile: the rows of the S^T MMA
+constexpr uint32_t DEC_ATOM = DEC_KEYS * 128;      // 128 rows of one 64-column swizzle atom
+constexpr int DEC_MAX_PAIRS = 16;                  // ring slots of two atoms
+constexpr int DEC_THREADS = 192;                   // warps 0-3 softmax, warp 4 TMA, warp 5 MMA
+
+struct LatentDecodeParams {
+  const int* block_table;
+  int max_blocks, block_size;
+  const int* cu_q;           // [num_seqs + 1] or null (uniform_q tokens each)
+  const int* kv_lens;
+  int uniform_q, H, num_splits, rows_total;
+  float scale_log2;
+  float* part_o;             // [splits, rows_total, rk]
+  float* part_ml;            // [splits, rows_total, 2]: running max (log2 units), sum relative to it
+  int rk, latent_atoms, pairs, rot_atoms, rot_steps, ring_pairs, ring_rots;
+};
+
+struct DecBarriers {
+  uint64_t q_full, s_full, p_full, o_final;
+  uint64_t pair_full[DEC_MAX_PAIRS], pair_empty[DEC_MAX_PAIRS];
+  uint64_t rot_full[2], rot_empty[2];
+  uint32_t tmem_base;
+  int abort;
+};
+
+// A tile [keys][64 columns per atom] as the A operand of O^T += C^T P^T: rows are the MMA's K dimension, the second atom holds
+// columns 64..127 of the 128 MMA rows.
+__device__ __forceinline__ uint64_t dec_desc_mnmajor(uint32_t smem_addr) {
+  uint64_t d = 0;
+  d |= (uint64_t)((smem_addr & 0x3FFFF) >> 4);
+  d |= (uint64_t)(DEC_ATOM >> 4) << 16;
+  d |= (uint64_t)(1024 >> 4) << 32;
+  d |= (uint64_t)1 << 46;
+  d |= (uint64_t)2 << 61;
+  return d;
+}
+__device__ __forceinline__ void tmem_ld_cols16(uint32_t taddr, float* v) {
+  uint32_t r[16];
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr)
+      : "memory");
+#pragma unroll
+  for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tmem_st_cols16(uint32_t taddr, const float* v) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr),
+      "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]),
+      "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15])
+      : "memory");
+}
+template <int NB>
+__device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, float* v) {
+#pragma unroll
+  for (int c = 0; c < NB; c += 16) tmem_ld_cols16(taddr + c, v + c);
+  tmem_ld_wait();
+#pragma unroll
+  for (int c = 0; c < NB; ++c) asm volatile("" : "+f"(v[c]));      // uses stay behind the wait
+}
+
+// Barrier of the four softmax warps that also agrees on whether everyone is still fine.
+__device__ __forceinline__ bool softmax_sync(bool ok) {
+  uint32_t all;
+  asm volatile(
+      "{\n.reg .pred p, q;\nsetp.ne.b32 p, %1, 0;\nbarrier.cta.red.and.pred q, 1, 128, p;\nselp.u32 %0, 1, 0, q;\n}\n"
+      : "=r"(all)
+      : "r"((uint32_t)ok)
+      : "memory");
+  return all != 0;
+}
+
+// Reduces v[c] over the lanes of the warp for NB columns at once; lane c (mod NB) returns column c. Destroys v.
+template <int NB, bool MAX>
+__device__ __forceinline__ float reduce_columns(float* v, int lane) {
+#pragma unroll
+  for (int o = NB / 2; o > 0; o >>= 1) {
+    const bool hi = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float keep = hi ? v[i + o] : v[i], send = hi ? v[i] : v[i + o];
+      const float got = __shfl_xor_sync(0xffffffffu, send, o);
+      v[i] = MAX ? fmaxf(keep, got) : keep + got;
+    }
+  }
+  if constexpr (NB == 16) {
+    const float got = __shfl_xor_sync(0xffffffffu, v[0], 16);
+    v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
+  }
+  return v[0];
+}
+
+template <int NB>
+__global__ void __launch_bounds__(DEC_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
+                     const LatentDecodeParams p) {
+  constexpr uint32_t Q_ATOM = NB * 128, TMEM_COLS = NB == 16 ? 128 : 256, COL_O = NB;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* s_rot = smem + p.ring_pairs * 2 * DEC_ATOM;
+  uint8_t* s_q = s_rot + p.ring_rots * p.rot_atoms * DEC_ATOM;
+  uint8_t* s_p = s_q + (p.latent_atoms + p.rot_atoms) * Q_ATOM;
+  float* red = reinterpret_cast<float*>(s_p + 2 * Q_ATOM);      // [2][4][NB]
+  DecBarriers* bars = reinterpret_cast<DecBarriers*>(red + 8 * NB);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  volatile int* abort_flag = &bars->abort;
+
+  pdl_launch_dependents();
+  pdl_wait(TL_ATTN_DECODE);
+  const int seq = blockIdx.z, split = blockIdx.x, row0 = blockIdx.y * NB;
+  const int q_start = p.cu_q ? p.cu_q[seq] : seq * p.uniform_q;
+  const int q_len = p.cu_q ? p.cu_q[seq + 1] - q_start : p.uniform_q;
+  const int nrows = min(NB, q_len * p.H - row0);
+  if (nrows <= 0) return;
+  const int kv_len = p.kv_lens[seq], base_row = q_start * p.H + row0;
+  // keys that the last row of this block sees
+  const int kv_end = min(kv_len, kv_len - q_len + (row0 + nrows - 1) / p.H + 1);
+  const int tiles = (kv_end + DEC_KEYS - 1) / DEC_KEYS, per = (tiles + p.num_splits - 1) / p.num_splits;
+  const int t0 = split * per, n_tiles = min(tiles, t0 + per) - t0;
+  if (n_tiles <= 0) {
+    for (int i = threadIdx.x; i < nrows; i += DEC_THREADS) {
+      float* ml = p.part_ml + ((size_t)split * p.rows_total + base_row + i) * 2;
+      ml[0] = -INFINITY, ml[1] = 0.f;
+    }
+    return;
+  }
+  if (threadIdx.x == 0) {
+    mbar_init(&bars->q_full, 1);
+    mbar_init(&bars->s_full, 1);
+    mbar_init(&bars->p_full, 128);
+    mbar_init(&bars->o_final, 1);
+    for (int i = 0; i < p.ring_pairs; ++i) mbar_init(&bars->pair_full[i], 1), mbar_init(&bars->pair_empty[i], 1);
+    for (int i = 0; i < p.ring_rots; ++i) mbar_init(&bars->rot_full[i], 1), mbar_init(&bars->rot_empty[i], 1);
+    bars->abort = 0;
+    mbar_fence_init();
+  }
+  if (warp == 4 && lane == 0) {
+    tma_prefetch_desc(&tmap_q);
+    tma_prefetch_desc(&tmap_kv);
+  }
+  if (warp == 5) {
+    tmem_alloc(&bars->tmem_base, TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = bars->tmem_base;
+
+  if (warp == 4) {
+    // ------------------------------------------------------------------ TMA producer
+    if (lane == 0) {
+      mbar_arrive_expect_tx(&bars->q_full, (p.latent_atoms + p.rot_atoms) * Q_ATOM);
+      for (int a = 0; a < p.latent_atoms; ++a) tma_load_2d(s_q + a * Q_ATOM, &tmap_q, &bars->q_full, a * 64, base_row);
+      for (int a = 0; a < p.rot_atoms; ++a)
+        tma_load_2d(s_q + (p.latent_atoms + a) * Q_ATOM, &tmap_q, &bars->q_full, p.rk + a * 64, base_row);
+      const int* pages = p.block_table + (size_t)seq * p.max_blocks;
+      const int per_tile = DEC_KEYS / p.block_size, last_page = (kv_len - 1) / p.block_size;
+      const uint32_t page_bytes = (uint32_t)p.block_size * 128u;
+      bool ok = true;
+      int n_pair = 0, n_rot = 0;                     // slots filled so far
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        int rows[16];                                // first cache row of each page; pages past the last repeat it (masked)
+#pragma unroll
+        for (int g = 0; g < 16; ++g) rows[g] = g < per_tile ? pages[min((t0 + j) * per_tile + g, last_page)] * p.block_size : 0;
+        auto load_atom = [&](uint8_t* dst, uint64_t* bar, int x) {
+#pragma unroll
+          for (int g = 0; g < 16; ++g)
+            if (g < per_tile) tma_load_2d(dst + g * page_bytes, &tmap_kv, bar, x, rows[g]);
+        };
+        {
+          const int sl = n_rot % p.ring_rots;
+          ok = mbar_wait(&bars->rot_empty[sl], ((n_rot / p.ring_rots) & 1) ^ 1, abort_flag, 710);
+          if (!ok) break;
+          mbar_arrive_expect_tx(&bars->rot_full[sl], p.rot_atoms * DEC_ATOM);
+          for (int a = 0; a < p.rot_atoms; ++a)
+            load_atom(s_rot + (sl * p.rot_atoms + a) * DEC_ATOM, &bars->rot_full[sl], p.rk + a * 64);
+          ++n_rot;
+        }
+        for (int i = 0; i < p.pairs; ++i) {
+          const int sl = n_pair % p.ring_pairs, atoms = min(2, p.latent_atoms - 2 * i);
+          ok = mbar_wait(&bars->pair_empty[sl], ((n_pair / p.ring_pairs) & 1) ^ 1, abort_flag, 711);
+          if (!ok) break;
+          mbar_arrive_expect_tx(&bars->pair_full[sl], atoms * DEC_ATOM);
+          for (int a = 0; a < atoms; ++a)
+            load_atom(smem + (sl * 2 + a) * DEC_ATOM, &bars->pair_full[sl], (2 * i + a) * 64);
+          ++n_pair;
+        }
+      }
+      if (!ok) {
+        // drain: every copy this thread started must land before the CTA's shared memory is released
+        volatile int never = 0;
+        mbar_wait(&bars->q_full, 0, &never, 712);
+        for (int i = max(0, n_rot - p.ring_rots); i < n_rot; ++i)
+          mbar_wait(&bars->rot_full[i % p.ring_rots], (i / p.ring_rots) & 1, &never, 713);
+        for (int i = max(0, n_pair - p.ring_pairs); i < n_pair; ++i)
+          mbar_wait(&bars->pair_full[i % p.ring_pairs], (i / p.ring_pairs) & 1, &never, 714);
+      }
+    }
+  } else if (warp == 5) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      constexpr uint32_t IDESC_S = umma_idesc_bf16_f32(DEC_KEYS, NB);
+      constexpr uint32_t IDESC_O = umma_idesc_bf16_f32(128, NB) | (1u << 15);   // A is MN-major
+      const uint32_t ring = smem_u32(smem), rot = smem_u32(s_rot), q = smem_u32(s_q), pp = smem_u32(s_p);
+      bool ok = mbar_wait(&bars->q_full, 0, abort_flag, 720);
+      int n_pair = 0, n_rot = 0;
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        const int rs = n_rot % p.ring_rots;
+        ok = mbar_wait(&bars->rot_full[rs], (n_rot / p.ring_rots) & 1, abort_flag, 721);
+        if (!ok) break;
+        tc_fence_after_sync();
+        for (int k = 0; k < p.rot_steps; ++k)
+          umma_f16_ss(tmem, umma_desc_kmajor_sw128(rot + (rs * p.rot_atoms + (k >> 2)) * DEC_ATOM + (k & 3) * 32),
+                      umma_desc_kmajor_sw128(q + (p.latent_atoms + (k >> 2)) * Q_ATOM + (k & 3) * 32), IDESC_S, k > 0);
+        umma_commit(&bars->rot_empty[rs]);
+        ++n_rot;
+        for (int i = 0; i < p.pairs && ok; ++i) {
+          const int sl = (n_pair + i) % p.ring_pairs, steps = min(2, p.latent_atoms - 2 * i) * 4;
+          ok = mbar_wait(&bars->pair_full[sl], ((n_pair + i) / p.ring_pairs) & 1, abort_flag, 722);
+          if (!ok) break;
+          tc_fence_after_sync();
+          for (int k = 0; k < steps; ++k)
+            umma_f16_ss(tmem, umma_desc_kmajor_sw128(ring + (sl * 2 + (k >> 2)) * DEC_ATOM + (k & 3) * 32),
+                        umma_desc_kmajor_sw128(q + (2 * i + (k >> 2)) * Q_ATOM + (k & 3) * 32), IDESC_S, 1);
+        }
+        if (!ok) break;
+        umma_commit(&bars->s_full);
+        ok = mbar_wait(&bars->p_full, j & 1, abort_flag, 723);
+        if (!ok) break;
+        tc_fence_after_sync();
+        for (int i = 0; i < p.pairs; ++i) {
+          const int sl = (n_pair + i) % p.ring_pairs;
+#pragma unroll
+          for (int k = 0; k < DEC_KEYS / 16; ++k)
+            umma_f16_ss(tmem + COL_O + i * NB, dec_desc_mnmajor(ring + sl * 2 * DEC_ATOM + k * 2048),
+                        umma_desc_kmajor_sw128(pp + (k >> 2) * Q_ATOM + (k & 3) * 32), IDESC_O, (j > 0) || (k > 0));
+          umma_commit(&bars->pair_empty[sl]);
+        }
+        n_pair += p.pairs;
+      }
+      umma_commit(&bars->o_final);   // also on the abort path: it only tracks MMAs already issued
+      if (!ok) {                     // TMEM must not be freed under MMAs that are still running
+        volatile int never = 0;
+        mbar_wait(&bars->o_final, 0, &never, 724);
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax: thread = key of the tile
+    const uint32_t t_lane = tmem + ((uint32_t)(warp * 32) << 16);
+    const int key = warp * 32 + lane;
+    float m[NB], l[NB];
+#pragma unroll
+    for (int n = 0; n < NB; ++n) m[n] = -INFINITY, l[n] = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      float s[NB];
+      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full, j & 1, abort_flag, 730));
+      if (ok) {
+        tc_fence_after_sync();
+        tmem_ld_cols<NB>(t_lane, s);
+        const int k0 = (t0 + j) * DEC_KEYS;
+        if (k0 + DEC_KEYS > kv_len - q_len + row0 / p.H + 1) {      // some key of the tile lies behind the first row
+#pragma unroll
+          for (int n = 0; n < NB; ++n)
+            if (k0 + key > kv_len - q_len + (row0 + n) / p.H || k0 + key >= kv_len) s[n] = -INFINITY;
+        }
+        float v[NB];
+#pragma unroll
+        for (int n = 0; n < NB; ++n) v[n] = s[n];
+        const float top = reduce_columns<NB, true>(v, lane);
+        if (lane < NB) red[((j & 1) * 4 + warp) * NB + lane] = top;
+      }
+      ok = softmax_sync(ok);
+      if (!ok) break;
+      float mn[NB];
+      bool grow = false;
+#pragma unroll
+      for (int n = 0; n < NB; n += 4) {
+        float4 a = *reinterpret_cast<const float4*>(&red[((j & 1) * 4) * NB + n]);
+#pragma unroll
+        for (int w = 1; w < 4; ++w) {
+          const float4 b = *reinterpret_cast<const float4*>(&red[((j & 1) * 4 + w) * NB + n]);
+          a.x = fmaxf(a.x, b.x), a.y = fmaxf(a.y, b.y), a.z = fmaxf(a.z, b.z), a.w = fmaxf(a.w, b.w);
+        }
+        mn[n] = fmaxf(m[n], a.x), mn[n + 1] = fmaxf(m[n + 1], a.y), mn[n + 2] = fmaxf(m[n + 2], a.z), mn[n + 3] = fmaxf(m[n + 3], a.w);
+      }
+#pragma unroll
+      for (int n = 0; n < NB; ++n) grow |= (mn[n] - m[n]) * p.scale_log2 > 8.f;
+      if (grow) {                    // the same in every thread: move all columns to their current maximum
+        float f[NB];
+#pragma unroll
+        for (int n = 0; n < NB; ++n) {
+          f[n] = mn[n] == -INFINITY ? 1.f : exp2f((m[n] - mn[n]) * p.scale_log2);
+          m[n] = mn[n];
+          l[n] *= f[n];
+        }
+        if (j > 0) {                 // the last PV has completed (s_full of this tile was committed behind it)
+          for (int i = 0; i < p.pairs; ++i) {
+            float o[NB];
+            tmem_ld_cols<NB>(t_lane + COL_O + i * NB, o);
+#pragma unroll
+            for (int n = 0; n < NB; ++n) o[n] *= f[n];
+#pragma unroll
+            for (int c = 0; c < NB; c += 16) tmem_st_cols16(t_lane + COL_O + i * NB + c, o + c);
+          }
+          asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+        }
+      }
+      uint8_t* dst = s_p + (key >> 6) * Q_ATOM + (key & 7) * 2;
+#pragma unroll
+      for (int n = 0; n < NB; ++n) {
+        const float e = exp2f(fmaf(s[n], p.scale_log2, m[n] == -INFINITY ? 0.f : -m[n] * p.scale_log2));
+        l[n] += e;
+        *reinterpret_cast<bf16*>(dst + n * 128 + ((((key & 63) >> 3) ^ (n & 7)) << 4)) = __float2bfloat16(e);
+      }
+      fence_proxy_async_smem();
+      tc_fence_before_sync();
+      mbar_arrive(&bars->p_full);
+    }
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_final, 0, abort_flag, 731));
+    float* lred = red;                               // the last tile used slot (n_tiles - 1) & 1 of the maxima: use the other
+    lred += (n_tiles & 1) * 4 * NB;
+    {
+      float v[NB];
+#pragma unroll
+      for (int n = 0; n < NB; ++n) v[n] = l[n];
+      const float sum = reduce_columns<NB, false>(v, lane);
+      if (lane < NB) lred[warp * NB + lane] = sum;
+    }
+    if (softmax_sync(ok)) {
+      tc_fence_after_sync();
+      const size_t base = (size_t)split * p.rows_total + base_row;
+#pragma unroll
+      for (int n = 0; n < NB; ++n)
+        if (threadIdx.x == n && n < nrows) {
+          float* ml = p.part_ml + (base + n) * 2;
+          ml[0] = m[n] * p.scale_log2;
+          ml[1] = lred[n] + lred[NB + n] + lred[2 * NB + n] + lred[3 * NB + n];
+        }
+      for (int i = 0; i < p.pairs; ++i) {
+        float o[NB];
+        tmem_ld_cols<NB>(t_lane + COL_O + i * NB, o);
+        const int col = i * 128 + key;
+#pragma unroll
+        for (int n = 0; n < NB; ++n)
+          if (n < nrows && col < p.rk) p.part_o[(base + n) * p.rk + col] = o[n];
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 5) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem, TMEM_COLS);
+  }
+}
+
+// ---- per-head products ----------------------------------------------------------------------------------------------
+struct HeadMmaParams {
+  const bf16* a;             // [tokens, heads, K] strided (MERGE: unused)
+  long long a_tok;
+  int a_head;
+  const bf16* w;             // [H, N, K]
+  bf16* out;                 // [tokens, heads, N] strided
+  long long out_tok;
+  int out_head;
+  const bf16* gate;          // optional [tokens, >= H] logits
+  long long gate_tok;
+  const int *rows_in, *rows_out;   // optional: token of row i in `a`, and in `out` and `gate`
+  int n, H, N, K;
+  // MERGE: a is the merged split partials
+  const float *part_o, *part_ml, *sink;
+  int num_splits, rows_total;
+};
+
+constexpr int HM_TOK = 16;   // tokens per CTA: the rows of the MMA
+
+// out[t, h, n] = gate * sum_k a[t, h, k] w[h, n, k]: four warps, NT 8-column MMA tiles each. A lane's eight consecutive k are
+// spread over two MMAs the same way for both operands, so every load is 16 bytes.
+template <int NT, bool MERGE>
+__global__ void __launch_bounds__(128) head_mma_kernel(const HeadMmaParams p) {
+  extern __shared__ __align__(16) uint8_t hm_smem[];
+  const int ld = p.K + 8;
+  bf16* sa = reinterpret_cast<bf16*>(hm_smem);                             // [16][K + 8]
+  float* wt = reinterpret_cast<float*>(hm_smem + (size_t)HM_TOK * ld * 2); // [16][32]: weight of each split
+  const int h = blockIdx.y, t0 = blockIdx.z * HM_TOK, m = min(HM_TOK, p.n - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+  const int n0 = (blockIdx.x * 4 + warp) * NT * 8;
+  pdl_launch_dependents();
+  pdl_wait();
+  auto token_in = [&](int i) { return p.rows_in ? p.rows_in[t0 + i] : t0 + i; };
+  auto token_out = [&](int i) { return p.rows_out ? p.rows_out[t0 + i] : t0 + i; };
+  if constexpr (MERGE) {
+    for (int i = threadIdx.x; i < m; i += 128) {
+      const size_t row = (size_t)token_in(i) * p.H + h;
+      const float sk = p.sink[h] * 1.4426950408889634f;
+      float top = sk, den = 0.f;
+      for (int s = 0; s < p.num_splits; ++s) top = fmaxf(top, p.part_ml[((size_t)s * p.rows_total + row) * 2]);
+      for (int s = 0; s < p.num_splits; ++s) {
+        const float* ml = p.part_ml + ((size_t)s * p.rows_total + row) * 2;
+        const float w = ml[1] > 0.f ? exp2f(ml[0] - top) : 0.f;
+        wt[i * 32 + s] = w;
+        den = fmaf(w, ml[1], den);
+      }
+      den = 1.f / (den + exp2f(sk - top));
+      for (int s = 0; s < p.num_splits; ++s) wt[i * 32 + s] *= den;
+    }
+    __syncthreads();
+    const int nv = p.K / 4;
+    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += 128) {
+      const int i = idx / nv, c = (idx % nv) * 4;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < m) {
+        const float* o = p.part_o + ((size_t)token_in(i) * p.H + h) * p.K + c;
+        for (int s = 0; s < p.num_splits; ++s) {
+          const float w = wt[i * 32 + s];
+          if (w == 0.f) continue;    // an empty split wrote nothing
+          const float4 x = *reinterpret_cast<const float4*>(o + (size_t)s * p.rows_total * p.K);
+          v.x = fmaf(w, x.x, v.x), v.y = fmaf(w, x.y, v.y), v.z = fmaf(w, x.z, v.z), v.w = fmaf(w, x.w, v.w);
+        }
+      }
+      *reinterpret_cast<uint2*>(sa + i * ld + c) = make_uint2(attn::pack_bf16(v.x, v.y), attn::pack_bf16(v.z, v.w));
+    }
+  } else {
+    const int nv = p.K / 8;
+    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += 128) {
+      const int i = idx / nv, c = (idx % nv) * 8;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (i < m) v = *reinterpret_cast<const uint4*>(p.a + token_in(i) * p.a_tok + (long long)h * p.a_head + c);
+      *reinterpret_cast<uint4*>(sa + i * ld + c) = v;
+    }
+  }
+  __syncthreads();
+  if (n0 >= p.N) return;
+  float acc[NT][4] = {};
+  const bf16* wr[NT];
+#pragma unroll
+  for (int t = 0; t < NT; ++t) wr[t] = p.w + ((size_t)h * p.N + min(n0 + t * 8 + g, p.N - 1)) * p.K + t4 * 8;
+#pragma unroll 4
+  for (int k = 0; k < p.K; k += 32) {
+    const bool in = k + t4 * 8 < p.K;
+    uint4 lo = make_uint4(0, 0, 0, 0), hi = lo, b[NT];
+    if (in) {
+      lo = *reinterpret_cast<const uint4*>(sa + g * ld + k + t4 * 8);
+      hi = *reinterpret_cast<const uint4*>(sa + (g + 8) * ld + k + t4 * 8);
+    }
+#pragma unroll
+    for (int t = 0; t < NT; ++t) b[t] = in ? __ldg(reinterpret_cast<const uint4*>(wr[t] + k)) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+      attn::mma_16816(acc[t], a0, b[t].x, b[t].y);
+      attn::mma_16816(acc[t], a1, b[t].z, b[t].w);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < NT; ++t) {
+    const int n = n0 + t * 8 + t4 * 2;
+    if (n >= p.N) continue;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int i = g + r * 8;
+      if (i >= m) continue;
+      const int tok = token_out(i);
+      float s = 1.f;
+      if (p.gate) s = 1.f / (1.f + expf(-__bfloat162float(p.gate[tok * p.gate_tok + h])));
+      *reinterpret_cast<uint32_t*>(p.out + tok * p.out_tok + (long long)h * p.out_head + n) =
+          attn::pack_bf16(acc[t][2 * r] * s, acc[t][2 * r + 1] * s);
+    }
+  }
+}
+
+template <int NT, bool MERGE>
+int launch_head_mma(const HeadMmaParams& p, cudaStream_t s) {
+  const size_t smem = (size_t)HM_TOK * (p.K + 8) * 2 + (MERGE ? HM_TOK * 32 * 4 : 0);
+  return launch_kernel(head_mma_kernel<NT, MERGE>, dim3((p.N + NT * 32 - 1) / (NT * 32), p.H, (p.n + HM_TOK - 1) / HM_TOK), dim3(128),
+                       smem, s, p);
+}
+
+template <int NB>
+int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDecodeParams p, int seqs, int max_rows, cudaStream_t s) {
+  constexpr size_t LIMIT = 227 * 1024;
+  const size_t fixed = 1024 + (size_t)(p.latent_atoms + p.rot_atoms + 2) * NB * 128 + 8 * NB * 4 + sizeof(DecBarriers);
+  const size_t pair = 2 * DEC_ATOM, rot = (size_t)p.rot_atoms * DEC_ATOM;
+  p.ring_rots = fixed + p.pairs * pair + 2 * rot <= LIMIT ? 2 : 1;
+  if (fixed + p.pairs * pair + p.ring_rots * rot > LIMIT) return -3;
+  p.ring_pairs = (int)((LIMIT - fixed - p.ring_rots * rot) / pair);
+  if (p.ring_pairs > DEC_MAX_PAIRS) p.ring_pairs = DEC_MAX_PAIRS;
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64 || !configured[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LIMIT);
+    if (e != cudaSuccess) return -(int)e;
+    if (dev >= 0 && dev < 64) configured[dev] = true;
+  }
+  const size_t smem = fixed + p.ring_pairs * pair + p.ring_rots * rot;
+  return launch_kernel(latent_decode_kernel<NB>, dim3(p.num_splits, (max_rows + NB - 1) / NB, seqs), dim3(DEC_THREADS), smem, s, tq, tk, p);
 }
 
 }  // namespace
@@ -70,15 +600,90 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
 extern "C" {
 
 int swb_latent_prep(void* buf, int ld, int col_c, const float* w, float eps, const float* cos, const float* sin, const int* positions,
-                    const long long* slots, void* cache, void* q_abs, int T, int H, int dn, int rot, int rp, int rank, int rk, int fp32,
+                    const long long* slots, void* cache, void* q_abs, const int* q_row, int T, int H, int dn, int rot, int rp, int rank, int rk, int fp32,
                     void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
   if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || (rp % 2) || rank <= 0 || rank > rk || !cache || !slots) return -3;
-  const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, T, H, dn, rot, rp, rank, rk};
+  const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot, rp, rank, rk};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return fp32 ? launch_kernel(latent_prep_kernel<float>, dim3((unsigned)T), dim3(256), 0, s, p)
               : launch_kernel(latent_prep_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, s, p);
+}
+
+// out [rows, width] bf16 <- the cached rows of num_seqs sequences (seqs: their indices in block_table, null: 0, 1, ...), those of
+// sequence s at [cu_k[s], cu_k[s + 1]). width % 8 == 0.
+int swb_latent_gather(const void* cache, const int* block_table, int max_blocks, int block_size, const int* seqs, const int* cu_k,
+                      int num_seqs, int rows, int width, void* out, void* stream) {
+  using namespace swb;
+  if (rows <= 0) return 0;
+  if (width % 8 || num_seqs <= 0 || block_size <= 0 || ((reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15)) return -3;
+  const long long n = (long long)rows * (width / 8);
+  const unsigned grid = (unsigned)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+  return launch_kernel(latent_gather_kernel, dim3(grid), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
+                       reinterpret_cast<const uint4*>(cache), block_table, max_blocks, block_size, seqs, cu_k, num_seqs, rows, width / 8,
+                       reinterpret_cast<uint4*>(out));
+}
+
+// Prefill attention on expanded keys and values; see attn_latent_tcgen05_launch.
+int swb_latent_prefill(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok, const void* k2,
+                       long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
+                       int total_tokens, int H, int d1, int d2, int Dv, float scale, const float* sink, const void* gate,
+                       long long gate_stride, const int* cu_q, const int* seqs, const int* cu_k, void* stream) {
+  using namespace swb;
+  if (num_seqs <= 0 || total_tokens <= 0) return 0;
+  if (max_q_len <= 0 || key_rows <= 0) return -3;
+  return attn_latent_tcgen05_launch(q, q_stride_tok, k, v, kv_stride_tok, k2, k2_stride_tok, key_rows, out, out_stride_tok, num_seqs,
+                                    max_q_len, total_tokens, H, d1, d2, Dv, scale, sink, gate, gate_stride, cu_q, seqs, cu_k,
+                                    reinterpret_cast<cudaStream_t>(stream));
+}
+
+// Attention of q_abs [T * H, rk + rp] over the cached rows [num_blocks * block_size, rk + rp] into split partials (see
+// LatentDecodeParams). max_q: most tokens of a sequence.
+int swb_latent_decode(const void* q_abs, const void* cache, int num_blocks, int block_size, const int* block_table, int max_blocks,
+                      const int* cu_q, const int* kv_lens, int n_seqs, int uniform_q, int max_q, int T, int H, int rk,
+                      int rp, float scale, int num_splits, float* part_o, float* part_ml, void* stream) {
+  using namespace swb;
+  if (T <= 0 || n_seqs <= 0) return 0;
+  if (rk % 64 || rk < 64 || rk > 512 || rp % 8 || rp < 8 || rp > 128 || block_size < 8 || block_size % 8 || DEC_KEYS % block_size ||
+      !(scale > 0.f) || num_splits < 1 || num_splits > 32 || H < 1 || max_q < 1 || (!cu_q && uniform_q < 1))
+    return -3;
+  if ((reinterpret_cast<uintptr_t>(q_abs) | reinterpret_cast<uintptr_t>(cache)) & 15) return -3;
+  LatentDecodeParams p{};
+  p.block_table = block_table, p.max_blocks = max_blocks, p.block_size = block_size;
+  p.cu_q = cu_q, p.kv_lens = kv_lens;
+  p.uniform_q = uniform_q, p.H = H, p.num_splits = num_splits, p.rows_total = T * H;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.part_o = part_o, p.part_ml = part_ml;
+  p.rk = rk, p.latent_atoms = rk / 64, p.pairs = (p.latent_atoms + 1) / 2, p.rot_atoms = (rp + 63) / 64, p.rot_steps = (rp + 15) / 16;
+  const int rows = max_q * H, nb = rows <= 16 ? 16 : 32;
+  CUtensorMap tq, tk;
+  int rc = make_tmap_bf16_2d(&tq, q_abs, T * H, rk + rp, rk + rp, nb);
+  if (rc) return rc;
+  rc = make_tmap_bf16_2d(&tk, cache, num_blocks * block_size, rk + rp, rk + rp, block_size);
+  if (rc) return rc;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return nb == 16 ? launch_latent_decode<16>(tq, tk, p, n_seqs, rows, s) : launch_latent_decode<32>(tq, tk, p, n_seqs, rows, s);
+}
+
+// out[t, h, n] = sigmoid(gate[t, h]) sum_k a[t, h, k] w[h, n, k] in bf16 for n tokens: row i is token rows_in[i] of a and
+// rows_out[i] of out and gate (null: i). With
+// part_o, a[t, h] are the merged split partials of swb_latent_decode with sinks (K = rk) and `a` is unused. K, N and all strides
+// are multiples of 8.
+int swb_head_mma(const void* a, long long a_tok, int a_head, const void* w, void* out, long long out_tok, int out_head, const void* gate,
+                 long long gate_tok, const int* rows_in, const int* rows_out, int n, int H, int N, int K, const float* part_o, const float* part_ml,
+                 const float* sink, int num_splits, int rows_total, void* stream) {
+  using namespace swb;
+  if (n <= 0 || H <= 0) return 0;
+  if (N < 8 || N % 8 || K < 8 || K % 8 || K > 1024 || (out_tok % 8) || (out_head % 8) || (part_o && (!part_ml || !sink || num_splits > 32)) ||
+      (!part_o && (!a || (a_tok % 8) || (a_head % 8) || (reinterpret_cast<uintptr_t>(a) & 15))) ||
+      (reinterpret_cast<uintptr_t>(w) & 15) || (reinterpret_cast<uintptr_t>(out) & 3))
+    return -3;
+  const HeadMmaParams p{reinterpret_cast<const bf16*>(a), a_tok, a_head, reinterpret_cast<const bf16*>(w), reinterpret_cast<bf16*>(out),
+                        out_tok, out_head, reinterpret_cast<const bf16*>(gate), gate_tok, rows_in, rows_out, n, H, N, K, part_o, part_ml, sink,
+                        num_splits, rows_total};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return part_o ? launch_head_mma<1, true>(p, s) : launch_head_mma<2, false>(p, s);
 }
 
 }  // extern "C"
