@@ -2,11 +2,13 @@
 //     S <- g * S          (rows of S are key channels)
 //     u  = beta (v - S^T k),   S <- S + k u^T,   o = S^T q
 // Three launches around the projections:
-//   delta_prep   short causal convolutions with silu, unit q / k, decays, step sizes (a warp per token and head);
-//   delta_scan   the recurrence. A column of S (one value channel) never meets the others, so LPC lanes own one column with
-//                DPL key channels each in registers; q, k, g stream through shared memory in blocks of tokens. Both dots run
-//                on the decayed state, o = (g S)^T q + (k . q) u, so one cross-lane reduction per token is on the critical
-//                path. Arithmetic is fp32 in token order: results do not depend on how a prompt was cut.
+//   delta_prep   short causal convolutions with silu, unit q / k, decays, step sizes. A warp takes one head over a run of
+//                tokens and keeps the convolution window in registers;
+//   delta_scan   the recurrence. A column of S (one value channel) never meets the others: sixteen lanes own NC columns, DPL key
+//                channels of each in registers, so that every q, k, g value read from shared memory serves NC columns (reading
+//                them is what bounds the kernel otherwise). Both dots run on the decayed state, o = (g S)^T q + (k . q) u, so one
+//                cross-lane reduction per token is on the critical path; it folds the 2 NC sums into different lanes on the way.
+//                Arithmetic is fp32 in token order: results do not depend on how a prompt was cut.
 //   delta_post   RMS norm over a head's value channels, weight and gate; moves the convolution windows on.
 // States and windows live in slots; a sequence's state is zero at position 0, a slot below 0 is neither read nor written.
 #include "common.cuh"
@@ -31,7 +33,7 @@ struct PrepParams {
   int ld, col_b;
   const void* decay;         // [T, ld_decay]: decay logits, H dp
   int ld_decay;
-  const float* conv;         // [2 G dp + H vp, taps]
+  const float* conv;         // [taps, 2 G dp + H vp]
   const void* window;        // [slots, taps - 1, 2 G dp + H vp]
   const float *a_log, *dt_bias;
   float *qk, *kq, *g, *v, *beta;       // [T, G, 2, dp] (k, q), [T, G], [T, H, dp], [T, H, vp], [T, H]
@@ -41,83 +43,145 @@ struct PrepParams {
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
-template <typename E>
-struct ConvIn {
-  const E* buf;
-  const E* window;           // of this sequence's slot, or null (no history)
-  int ld, C, taps, start, t; // start: flat index of the sequence's first token of this step
-  // silu(sum_j w[c, taps - 1 - j] x[t - j])
-  __device__ __forceinline__ float operator()(const float* __restrict__ conv, int c) const {
-    const float* w = conv + (size_t)c * taps;
-    float y = 0.f;
-    for (int j = 0; j < taps; ++j) {
-      const int r = t - (taps - 1 - j);
-      float x = 0.f;
-      if (r >= start) x = to_f(buf[(size_t)r * ld + c]);
-      else if (window) x = to_f(window[(size_t)(taps - 1 + r - start) * C + c]);
-      y = fmaf(w[j], x, y);
+// Four channels of the convolution at consecutive tokens. TAPS > 0: the last TAPS - 1 inputs stay in registers; 0: any number of
+// taps, every input is loaded again.
+template <typename E, int TAPS>
+struct Conv4 {
+  const E *buf, *window;     // window: of this sequence's slot, or null (no history)
+  const float* w;            // [taps, C]
+  int ld, C, taps, c, start;
+  float4 x[TAPS > 1 ? TAPS - 1 : 1], wt[TAPS > 0 ? TAPS : 1];
+
+  __device__ __forceinline__ float4 input(int t) const {
+    if (t >= start) return load_row4(buf + (size_t)t * ld + c);
+    if (window) return load_row4(window + (size_t)(taps - 1 + t - start) * C + c);
+    return make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  __device__ __forceinline__ void weights() {
+    if constexpr (TAPS > 0)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) wt[j] = *reinterpret_cast<const float4*>(w + (size_t)j * C + c);
+  }
+  __device__ __forceinline__ void begin(int t) {       // t: the first token that will be asked for
+    if constexpr (TAPS > 1)
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) x[j] = input(t - (TAPS - 1) + j);
+  }
+  static __device__ __forceinline__ void mac(float4& y, float4 a, float4 b) {
+    y.x = fmaf(a.x, b.x, y.x), y.y = fmaf(a.y, b.y, y.y), y.z = fmaf(a.z, b.z, y.z), y.w = fmaf(a.w, b.w, y.w);
+  }
+  __device__ __forceinline__ float4 next(int t) {      // silu(sum_j w[taps - 1 - j] x[t - j])
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (TAPS > 0) {
+      const float4 now = load_row4(buf + (size_t)t * ld + c);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) mac(y, wt[j], x[j]);
+      mac(y, wt[TAPS - 1], now);
+#pragma unroll
+      for (int j = 0; j + 2 < TAPS; ++j) x[j] = x[j + 1];
+      if constexpr (TAPS > 1) x[TAPS - 2] = now;
+    } else {
+      for (int j = 0; j < taps; ++j) mac(y, *reinterpret_cast<const float4*>(w + (size_t)j * C + c), input(t - (taps - 1) + j));
     }
-    return y * sigmoid_f(y);
+    y.x *= sigmoid_f(y.x), y.y *= sigmoid_f(y.y), y.z *= sigmoid_f(y.z), y.w *= sigmoid_f(y.w);
+    return y;
   }
 };
 
-// Warp task of a token: [0, G) unit q and k of a key head; [G, G + H) decays, step size; [G + H, G + 2 H) values.
-template <typename E>
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+
+// Warp task over a run of tokens: [0, G) unit q and k of a key head; [G, G + H) decays and step sizes of a head; [G + H, G + 2 H)
+// its values. NI: 128-channel pieces of a key head.
+template <typename E, int TAPS, int NI>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const PrepParams p) {
-  pdl_launch_dependents();
   pdl_wait();
   const DeltaShape& s = p.s;
   const int task = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (task >= s.G + 2 * s.H) return;
   const int nq = s.G * s.dp, C = 2 * nq + s.H * s.vp;
   const E* buf = reinterpret_cast<const E*>(p.buf);
-  for (int i = 0; i < p.tokens_per_cta; ++i) {
-    const int t = blockIdx.x * p.tokens_per_cta + i;
-    if (t >= s.T) return;
-    if (task >= s.G && task < s.G + s.H) {
-      const int h = task - s.G;
-      const float rate = -expf(p.a_log[h]);
-      const E* x = reinterpret_cast<const E*>(p.decay) + (size_t)t * p.ld_decay + h * s.dp;
-      float* g = p.g + ((size_t)t * s.H + h) * s.dp;
-      for (int c = lane; c < s.dp; c += 32) g[c] = expf(rate * softplus_f(to_f(x[c]) + p.dt_bias[h * s.dp + c]));
-      if (lane == 0) p.beta[(size_t)t * s.H + h] = sigmoid_f(to_f(buf[(size_t)t * p.ld + p.col_b + h]));
-      continue;
+  const int t_lo = blockIdx.x * p.tokens_per_cta, t_hi = min(s.T, t_lo + p.tokens_per_cta);
+  if (task >= s.G && task < s.G + s.H) {
+    const int h = task - s.G;
+    const float rate = -expf(p.a_log[h]);
+    for (int c = lane * 4; c < s.dp; c += 128) {
+      const float4 b = *reinterpret_cast<const float4*>(p.dt_bias + h * s.dp + c);
+#pragma unroll 2
+      for (int t = t_lo; t < t_hi; ++t) {
+        float4 x = load_row4(reinterpret_cast<const E*>(p.decay) + (size_t)t * p.ld_decay + h * s.dp + c);
+        x.x = expf(rate * softplus_f(x.x + b.x)), x.y = expf(rate * softplus_f(x.y + b.y));
+        x.z = expf(rate * softplus_f(x.z + b.z)), x.w = expf(rate * softplus_f(x.w + b.w));
+        *reinterpret_cast<float4*>(p.g + ((size_t)t * s.H + h) * s.dp + c) = x;
+      }
     }
-    const int seq = seq_of_token(s.cu_q, s.num_seqs, s.uniform_q, t);
-    const int start = s.cu_q ? s.cu_q[seq] : seq * s.uniform_q, slot = s.slots[seq];
-    const bool fresh = s.positions[start] == 0 || slot < 0;
-    const ConvIn<E> conv{buf, fresh ? nullptr : reinterpret_cast<const E*>(p.window) + (size_t)slot * (s.taps - 1) * C,
-                         p.ld, C, s.taps, start, t};
+    for (int t = t_lo + lane; t < t_hi; t += 32) p.beta[(size_t)t * s.H + h] = sigmoid_f(to_f(buf[(size_t)t * p.ld + p.col_b + h]));
+  } else if (task < s.G + 2 * s.H) {
+    int seq = -1, start = 0, stop = t_lo;
+    const E* window = nullptr;
+    auto enter = [&](int t) {                          // the sequence that token t starts, or lies in
+      seq = seq_of_token(s.cu_q, s.num_seqs, s.uniform_q, t);
+      start = s.cu_q ? s.cu_q[seq] : seq * s.uniform_q;
+      stop = s.cu_q ? s.cu_q[seq + 1] : start + s.uniform_q;
+      const int slot = s.slots[seq];
+      window = s.positions[start] == 0 || slot < 0 ? nullptr : reinterpret_cast<const E*>(p.window) + (size_t)slot * (s.taps - 1) * C;
+    };
     if (task < s.G) {
-      float kk = 0.f, qq = 0.f, kq = 0.f;
-      float kv[16], qv[16];            // dp <= 512
+      Conv4<E, TAPS> cq[NI], ck[NI];
+      const float q_scale = rsqrtf((float)s.dim);
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        const int c = lane + j * 32;
-        kv[j] = qv[j] = 0.f;
-        if (c < s.dp) {
-          qv[j] = conv(p.conv, task * s.dp + c);
-          kv[j] = conv(p.conv, nq + task * s.dp + c);
+      for (int i = 0; i < NI; ++i) {
+        const int c = min(lane * 4 + i * 128, s.dp - 4);
+        cq[i].buf = ck[i].buf = buf, cq[i].w = ck[i].w = p.conv, cq[i].ld = ck[i].ld = p.ld, cq[i].C = ck[i].C = C;
+        cq[i].taps = ck[i].taps = s.taps, cq[i].c = task * s.dp + c, ck[i].c = nq + task * s.dp + c;
+        cq[i].weights(), ck[i].weights();
+      }
+      for (int t = t_lo; t < t_hi; ++t) {
+        if (t >= stop || t == t_lo) {
+          enter(t);
+#pragma unroll
+          for (int i = 0; i < NI; ++i) {
+            cq[i].window = ck[i].window = window, cq[i].start = ck[i].start = start;
+            cq[i].begin(t), ck[i].begin(t);
+          }
         }
-        qq = fmaf(qv[j], qv[j], qq);
-        kk = fmaf(kv[j], kv[j], kk);
-        kq = fmaf(kv[j], qv[j], kq);
-      }
-      qq = warp_sum(qq), kk = warp_sum(kk), kq = warp_sum(kq);
-      const float rk = rsqrtf(kk + 1e-6f), rq = rsqrtf(qq + 1e-6f) * rsqrtf((float)s.dim);
-      float* out = p.qk + ((size_t)t * s.G + task) * 2 * s.dp;
+        float4 q[NI], k[NI];
+        float qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        const int c = lane + j * 32;
-        if (c < s.dp) out[c] = kv[j] * rk, out[s.dp + c] = qv[j] * rq;
+        for (int i = 0; i < NI; ++i) {
+          q[i] = cq[i].next(t), k[i] = ck[i].next(t);
+          if (lane * 4 + i * 128 >= s.dp) q[i] = k[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+          qq += dot4(q[i], q[i]), kk += dot4(k[i], k[i]), kq += dot4(k[i], q[i]);
+        }
+        qq = warp_sum(qq), kk = warp_sum(kk), kq = warp_sum(kq);
+        const float rk = rsqrtf(kk + 1e-6f), rq = rsqrtf(qq + 1e-6f) * q_scale;
+        float* out = p.qk + ((size_t)t * s.G + task) * 2 * s.dp;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int c = lane * 4 + i * 128;
+          if (c >= s.dp) continue;
+          *reinterpret_cast<float4*>(out + c) = make_float4(k[i].x * rk, k[i].y * rk, k[i].z * rk, k[i].w * rk);
+          *reinterpret_cast<float4*>(out + s.dp + c) = make_float4(q[i].x * rq, q[i].y * rq, q[i].z * rq, q[i].w * rq);
+        }
+        if (lane == 0) p.kq[(size_t)t * s.G + task] = kq * rk * rq;
       }
-      if (lane == 0) p.kq[(size_t)t * s.G + task] = kq * rk * rq;
     } else {
       const int h = task - s.G - s.H;
-      float* out = p.v + ((size_t)t * s.H + h) * s.vp;
-      for (int c = lane; c < s.vp; c += 32) out[c] = conv(p.conv, 2 * nq + h * s.vp + c);
+      for (int c = lane * 4; c < s.vp; c += 128) {
+        Conv4<E, TAPS> cv;
+        cv.buf = buf, cv.w = p.conv, cv.ld = p.ld, cv.C = C, cv.taps = s.taps, cv.c = 2 * nq + h * s.vp + c;
+        cv.weights();
+        stop = t_lo;
+        for (int t = t_lo; t < t_hi; ++t) {
+          if (t >= stop) {
+            enter(t);
+            cv.window = window, cv.start = start;
+            cv.begin(t);
+          }
+          *reinterpret_cast<float4*>(p.v + ((size_t)t * s.H + h) * s.vp + c) = cv.next(t);
+        }
+      }
     }
   }
+  pdl_launch_dependents();
 }
 
 struct ScanParams {
@@ -154,33 +218,58 @@ __device__ __forceinline__ void cp_async4(void* dst, const void* src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
-constexpr int SCAN_WARPS = 4;
+constexpr int SCAN_WARPS = 4, SCAN_LANES = 16;
+
+// DPL key channels per lane in pieces of V (2 or 4); `at(i)` is the first channel of piece i of lane `sub`.
+template <int DPL>
+struct Lane {
+  static constexpr int V = DPL % 4 ? 2 : 4, N = DPL / V;
+  static __device__ __forceinline__ int at(int i, int sub) { return (i * SCAN_LANES + sub) * V; }
+  static __device__ __forceinline__ void load(const float* p, int sub, uint64_t* v) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      if constexpr (V == 4) {
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(p + at(i, sub));
+        v[2 * i] = x.x, v[2 * i + 1] = x.y;
+      } else {
+        v[i] = *reinterpret_cast<const uint64_t*>(p + at(i, sub));
+      }
+    }
+  }
+  static __device__ __forceinline__ void store(float* p, int sub, const uint64_t* v) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      if constexpr (V == 4) *reinterpret_cast<ulonglong2*>(p + at(i, sub)) = make_ulonglong2(v[2 * i], v[2 * i + 1]);
+      else *reinterpret_cast<uint64_t*>(p + at(i, sub)) = v[i];
+    }
+  }
+};
 
 // TB tokens per staged block; layout of one token in shared memory: k [dp], q [dp], g [dp], v [COLS], (kq, beta, -, -)
-template <int DPL, int LPC, int TB>
+template <int DPL, int NC, int TB>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanParams p) {
-  constexpr int DP = DPL * LPC, COLS = SCAN_WARPS * 32 / LPC, TOK = 3 * DP + COLS + 4, N2 = DPL / 2;
+  constexpr int DP = DPL * SCAN_LANES, COLS = SCAN_WARPS * 2 * NC, TOK = 3 * DP + COLS + 4, N2 = DPL / 2;
+  constexpr bool AHEAD = DPL <= 16;                  // operands of the next token are read while this one is computed
+  using L = Lane<DPL>;
   extern __shared__ __align__(16) float sm[];        // 2 blocks of TB tokens
-  pdl_launch_dependents();
   pdl_wait();
   const DeltaShape& s = p.s;
   const int seq = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS, kvh = h / (s.H / s.G);
-  const int tid = threadIdx.x, sub = tid % LPC, lc = tid / LPC, col = c0 + lc;
+  const int tid = threadIdx.x, sub = tid % SCAN_LANES, lc = tid / SCAN_LANES * NC;   // first of this lane's NC columns
   const int start = s.cu_q ? s.cu_q[seq] : seq * s.uniform_q, n = s.cu_q ? s.cu_q[seq + 1] - start : s.uniform_q;
   if (n <= 0) return;
   const int slot = s.slots[seq];
-  const bool live = col < s.vp;
-  float* st = p.state + (((size_t)max(slot, 0) * s.H + h) * s.vp + (live ? col : 0)) * DP;
-  uint64_t S[N2];
-  if (slot >= 0 && live && s.positions[start] != 0) {
+  float* st = p.state + (((size_t)max(slot, 0) * s.H + h) * s.vp + c0 + lc) * DP;
+  const bool carried = slot >= 0 && s.positions[start] != 0;
+  uint64_t S[NC][N2];
 #pragma unroll
-    for (int i = 0; i < DPL / 4; ++i) {
-      const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(st + (i * LPC + sub) * 4);
-      S[2 * i] = v.x, S[2 * i + 1] = v.y;
+  for (int c = 0; c < NC; ++c) {
+    if (carried && c0 + lc + c < s.vp) {
+      L::load(st + c * DP, sub, S[c]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < N2; ++i) S[c][i] = 0ull;
     }
-  } else {
-#pragma unroll
-    for (int i = 0; i < N2; ++i) S[i] = 0ull;
   }
   const int ncols = min(COLS, s.vp - c0);            // vp % 8 == 0, so whole 16-byte pieces
   auto stage = [&](int b) {
@@ -206,8 +295,11 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   const int blocks = (n + TB - 1) / TB;
+  // which of the 2 NC sums this lane ends up with: dots with k (upper bit 0) or q (1), of column `mine`
+  const int mine = NC == 4 ? (sub >> 1) & 3 : NC == 2 ? (sub >> 2) & 1 : 0;
+  const bool is_q = sub & 8, writes = is_q && (sub & (NC == 4 ? 1 : NC == 2 ? 3 : 7)) == 0 && c0 + lc + mine < s.vp;
   stage(0);
-  float* orow = p.o + ((size_t)start * s.H + h) * s.vp + col;
+  float* orow = p.o + ((size_t)start * s.H + h) * s.vp + c0 + lc + mine;
   for (int b = 0; b < blocks; ++b) {
     if (b + 1 < blocks) {
       stage(b + 1);
@@ -218,40 +310,59 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
     __syncthreads();
     const float* tok = sm + (b & 1) * TB * TOK;
     const int m = min(TB, n - b * TB);
+    uint64_t k[N2], q[N2], g[N2];
+    if (AHEAD) L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
     for (int r = 0; r < m; ++r, tok += TOK, orow += (size_t)s.H * s.vp) {
-      const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(tok);
-      const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(tok + DP);
-      const ulonglong2* g4 = reinterpret_cast<const ulonglong2*>(tok + 2 * DP);
-      uint64_t ak[2] = {0ull, 0ull}, aq[2] = {0ull, 0ull}, kk[N2];
+      if (!AHEAD) L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
+      float a[2 * NC];
 #pragma unroll
-      for (int i = 0; i < DPL / 4; ++i) {
-        const ulonglong2 g = g4[i * LPC + sub], k = k4[i * LPC + sub], q = q4[i * LPC + sub];
-        S[2 * i] = mul2(S[2 * i], g.x);
-        S[2 * i + 1] = mul2(S[2 * i + 1], g.y);
-        ak[0] = fma2(S[2 * i], k.x, ak[0]);
-        ak[1] = fma2(S[2 * i + 1], k.y, ak[1]);
-        aq[0] = fma2(S[2 * i], q.x, aq[0]);
-        aq[1] = fma2(S[2 * i + 1], q.y, aq[1]);
-        kk[2 * i] = k.x, kk[2 * i + 1] = k.y;
+      for (int c = 0; c < NC; ++c) {
+        uint64_t ak = 0ull, aq = 0ull;
+#pragma unroll
+        for (int i = 0; i < N2; ++i) {
+          S[c][i] = mul2(S[c][i], g[i]);
+          ak = i ? fma2(S[c][i], k[i], ak) : mul2(S[c][i], k[i]);
+          aq = i ? fma2(S[c][i], q[i], aq) : mul2(S[c][i], q[i]);
+        }
+        a[c] = sum2(ak), a[NC + c] = sum2(aq);
       }
-      float dk = sum2(ak[0]) + sum2(ak[1]), dq = sum2(aq[0]) + sum2(aq[1]);
+      const float kq = tok[3 * DP + COLS], beta = tok[3 * DP + COLS + 1], v = tok[3 * DP + lc + mine];
+      uint64_t k_now[N2];
 #pragma unroll
-      for (int o = 1; o < LPC; o <<= 1) {
-        dk += __shfl_xor_sync(0xffffffffu, dk, o);
-        dq += __shfl_xor_sync(0xffffffffu, dq, o);
+      for (int i = 0; i < N2; ++i) k_now[i] = k[i];
+      if (AHEAD && r + 1 < m) L::load(tok + TOK, sub, k), L::load(tok + TOK + DP, sub, q), L::load(tok + TOK + 2 * DP, sub, g);
+      // fold: each step halves the number of sums a lane still carries, then plain sums over the remaining lane bits
+      int o = 8;
+#pragma unroll
+      for (int w = NC; w >= 1; w >>= 1, o >>= 1) {
+        const bool hi = sub & o;
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+          const float keep = hi ? a[i + w] : a[i], send = hi ? a[i] : a[i + w];
+          a[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
       }
-      const float u = tok[3 * DP + COLS + 1] * (tok[3 * DP + lc] - dk);
-      const uint64_t uu = dup2(u);
 #pragma unroll
-      for (int i = 0; i < N2; ++i) S[i] = fma2(kk[i], uu, S[i]);
-      if (sub == 0 && live) *orow = fmaf(tok[3 * DP + COLS], u, dq);
+      for (; o > 0; o >>= 1) a[0] += __shfl_xor_sync(0xffffffffu, a[0], o);
+      const float u_mine = beta * (v - a[0]);        // meaningful in the lanes that hold a dot with k
+      float u_out = 0.f;
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const float u = __shfl_sync(0xffffffffu, u_mine, (tid & 16) | (NC == 4 ? c << 1 : NC == 2 ? c << 2 : 0));
+        if (c == mine) u_out = u;
+        const uint64_t uu = dup2(u);
+#pragma unroll
+        for (int i = 0; i < N2; ++i) S[c][i] = fma2(k_now[i], uu, S[c][i]);
+      }
+      if (writes) *orow = fmaf(kq, u_out, a[0]);
     }
     __syncthreads();
   }
-  if (slot >= 0 && live) {
+  pdl_launch_dependents();
+  if (slot >= 0) {
 #pragma unroll
-    for (int i = 0; i < DPL / 4; ++i)
-      *reinterpret_cast<ulonglong2*>(st + (i * LPC + sub) * 4) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+    for (int c = 0; c < NC; ++c)
+      if (c0 + lc + c < s.vp) L::store(st + c * DP, sub, S[c]);
   }
 }
 
@@ -299,28 +410,41 @@ __global__ void __launch_bounds__(256) delta_post_kernel(const PostParams p) {
   const int t = (int)(id / s.H), h = (int)(id % s.H);
   const float* o = p.o + id * s.vp;
   float ss = 0.f;
-  for (int c = lane; c < s.vp; c += 32) ss = fmaf(o[c], o[c], ss);      // padding columns are zero
+  for (int c = lane * 8; c < s.vp; c += 256) {       // padding columns are zero
+    float v[8];
+    load_row8(o + c, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+  }
   const float r = rsqrtf(warp_sum(ss) / (float)s.vdim + p.eps);
   const E* gate = reinterpret_cast<const E*>(p.gate) + (size_t)t * p.ld_gate + h * s.vp;
   E* out = reinterpret_cast<E*>(p.out) + id * s.vp;
-  for (int c = lane; c < s.vp; c += 32) from_f(out[c], o[c] * r * p.w[c] * sigmoid_f(to_f(gate[c])));
+  for (int c = lane * 8; c < s.vp; c += 256) {
+    float v[8], w[8], z[8];
+    load_row8(o + c, v);
+    load_row8(p.w + c, w);
+    load_row8(gate + c, z);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= r * w[j] * sigmoid_f(z[j]);
+    store_row8(out + c, v);
+  }
 }
 
-template <int DPL, int LPC, int TB>
+template <int DPL, int NC, int TB>
 int launch_scan(const ScanParams& p, cudaStream_t st) {
-  constexpr int DP = DPL * LPC, COLS = SCAN_WARPS * 32 / LPC;
+  constexpr int DP = DPL * SCAN_LANES, COLS = SCAN_WARPS * 2 * NC;
   constexpr size_t smem = 2 * TB * (3 * DP + COLS + 4) * sizeof(float);
   if (smem > 48 * 1024) {
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-      const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DPL, LPC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DPL, NC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return -(int)e;
       if (dev >= 0 && dev < 64) configured[dev] = true;
     }
   }
-  return launch_kernel(delta_scan_kernel<DPL, LPC, TB>, dim3((p.s.vp + COLS - 1) / COLS, p.s.H, p.s.num_seqs), dim3(SCAN_WARPS * 32),
+  return launch_kernel(delta_scan_kernel<DPL, NC, TB>, dim3((p.s.vp + COLS - 1) / COLS, p.s.H, p.s.num_seqs), dim3(SCAN_WARPS * 32),
                        smem, st, p);
 }
 
@@ -340,6 +464,29 @@ DeltaShape make_shape(const int* dims, const int* cu_q, const int* positions, co
 
 extern "C" {
 
+}  // extern "C"
+namespace swb {
+namespace {
+template <typename E, int NI>
+int launch_prep(const PrepParams& p, cudaStream_t st) {
+  const dim3 grid((p.s.T + p.tokens_per_cta - 1) / p.tokens_per_cta, (p.s.G + 2 * p.s.H + 7) / 8);
+  if constexpr (NI > 2) return launch_kernel(delta_prep_kernel<E, 0, NI>, grid, dim3(256), 0, st, p);
+  else switch (p.s.taps) {
+    case 1: return launch_kernel(delta_prep_kernel<E, 1, NI>, grid, dim3(256), 0, st, p);
+    case 2: return launch_kernel(delta_prep_kernel<E, 2, NI>, grid, dim3(256), 0, st, p);
+    case 3: return launch_kernel(delta_prep_kernel<E, 3, NI>, grid, dim3(256), 0, st, p);
+    case 4: return launch_kernel(delta_prep_kernel<E, 4, NI>, grid, dim3(256), 0, st, p);
+    default: return launch_kernel(delta_prep_kernel<E, 0, NI>, grid, dim3(256), 0, st, p);
+  }
+}
+template <typename E>
+int launch_prep(const PrepParams& p, cudaStream_t st) {
+  return p.s.dp <= 128 ? launch_prep<E, 1>(p, st) : p.s.dp <= 256 ? launch_prep<E, 2>(p, st) : launch_prep<E, 4>(p, st);
+}
+}  // namespace
+}  // namespace swb
+extern "C" {
+
 // dims: host int[10] = T, num_seqs, uniform_q (cu_q null), H, G, dim, dp, vdim, vp, taps. fp32 selects the element type of
 // the projections, windows and decay logits.
 int swb_delta_prep(const int* dims, const int* cu_q, const int* positions, const int* slots, const void* buf, int ld, int col_b,
@@ -347,13 +494,11 @@ int swb_delta_prep(const int* dims, const int* cu_q, const int* positions, const
                    float* qk, float* kq, float* g, float* v, float* beta, int fp32, void* stream) {
   using namespace swb;
   PrepParams p{make_shape(dims, cu_q, positions, slots), buf, ld, col_b, decay, ld_decay, conv, window, a_log, dt_bias, qk, kq, g, v,
-               beta, dims[0] >= 2048 ? 8 : 1};
+               beta, dims[0] >= 4096 ? 16 : dims[0] >= 1024 ? 8 : dims[0] >= 256 ? 4 : 1};
   if (dims[0] <= 0) return 0;
-  if (!shape_ok(p.s)) return -3;
-  const dim3 grid((p.s.T + p.tokens_per_cta - 1) / p.tokens_per_cta, (p.s.G + 2 * p.s.H + 7) / 8);
+  if (!shape_ok(p.s) || (ld % 4) || (ld_decay % 4)) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return fp32 ? launch_kernel(delta_prep_kernel<float>, grid, dim3(256), 0, st, p)
-              : launch_kernel(delta_prep_kernel<bf16>, grid, dim3(256), 0, st, p);
+  return fp32 ? launch_prep<float>(p, st) : launch_prep<bf16>(p, st);
 }
 
 int swb_delta_scan(const int* dims, const int* cu_q, const int* positions, const int* slots, const float* qk, const float* kq,
@@ -364,13 +509,13 @@ int swb_delta_scan(const int* dims, const int* cu_q, const int* positions, const
   if (!shape_ok(p.s)) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   switch (p.s.dp) {
-    case 32: return launch_scan<8, 4, 16>(p, st);
-    case 64: return launch_scan<16, 4, 16>(p, st);
-    case 96: return launch_scan<24, 4, 16>(p, st);
-    case 128: return launch_scan<32, 4, 16>(p, st);
-    case 192: return launch_scan<24, 8, 8>(p, st);
-    case 256: return launch_scan<32, 8, 8>(p, st);
-    case 512: return launch_scan<32, 16, 4>(p, st);
+    case 32: return launch_scan<2, 4, 16>(p, st);
+    case 64: return launch_scan<4, 4, 16>(p, st);
+    case 96: return launch_scan<6, 4, 16>(p, st);
+    case 128: return launch_scan<8, 4, 16>(p, st);
+    case 192: return launch_scan<12, 4, 8>(p, st);
+    case 256: return launch_scan<16, 4, 8>(p, st);
+    case 512: return launch_scan<32, 2, 4>(p, st);
     default: return -3;
   }
 }

@@ -33,46 +33,54 @@ struct LatentPrepParams {
   int T, H, dn, rot, rp, rank, rk;
 };
 
+// One CTA per token: warp 0 norms the latent, the others rotate in groups of eight dimensions (four pairs).
 template <typename E>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams p) {
+__global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
   pdl_launch_dependents();
   pdl_wait(TL_ROPE_KV);
-  __shared__ float red[8];
-  const int t = blockIdx.x, pos = p.positions[t], half = p.rp / 2, width = p.rk + p.rp;
+  const int t = blockIdx.x, pos = p.positions[t], width = p.rk + p.rp, lane = threadIdx.x & 31;
   E* row = reinterpret_cast<E*>(p.buf) + (size_t)t * p.ld;
   E* c = row + p.col_c;
   const long long slot = p.slots[t];
   E* dst = slot >= 0 ? reinterpret_cast<E*>(p.cache) + (size_t)slot * width : nullptr;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < p.rank; i += 256) ss = fmaf(to_f(c[i]), to_f(c[i]), ss);
-  ss = warp_sum(ss);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  ss = 0.f;
+  if (threadIdx.x < 32) {
+    float ss = 0.f;
+    for (int i = lane * 8; i < p.rk; i += 256) {       // padding columns are zero
+      float v[8];
+      load_row8(c + i, v);
 #pragma unroll
-  for (int w = 0; w < 8; ++w) ss += red[w];
-  const float r = rsqrtf(ss / (float)p.rank + p.eps);
-  for (int i = threadIdx.x; i < p.rk; i += 256) {
-    E x;
-    from_f(x, i < p.rank ? to_f(c[i]) * r * p.w[i] : 0.f);
-    c[i] = x;
-    if (dst) dst[i] = x;
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+    }
+    const float r = rsqrtf(warp_sum(ss) / (float)p.rank + p.eps);
+    for (int i = lane * 8; i < p.rk; i += 256) {
+      float v[8], w[8];
+      load_row8(c + i, v);
+      load_row8(p.w + i, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= r * w[j];
+      store_row8(c + i, v);
+      if (dst) store_row8(dst + i, v);
+    }
+    return;
   }
-  const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t;
+  const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t, per = p.rp / 8;
   const float* cs = p.cos + (size_t)pos * (p.rot / 2);
   const float* sn = p.sin + (size_t)pos * (p.rot / 2);
-  for (int i = threadIdx.x; i < (p.H + 1) * half; i += 256) {       // pairs of the heads' queries, then of the shared key
-    const int h = i / half, k = i % half;
-    E* x = (h < p.H ? row + h * (p.dn + p.rp) + p.dn : c + p.rk) + 2 * k;
-    E y[2] = {x[0], x[1]};
-    if (2 * k < p.rot) {
-      const float u = to_f(x[0]), v = to_f(x[1]), a = cs[k], b = sn[k];
-      from_f(y[0], u * a - v * b);
-      from_f(y[1], v * a + u * b);
-      x[0] = y[0], x[1] = y[1];
+  for (int i = threadIdx.x - 32; i < (p.H + 1) * per; i += 96) {    // the heads' queries, then the shared key part
+    const int h = i / per, k = i % per * 8;
+    E* x = (h < p.H ? row + h * (p.dn + p.rp) + p.dn : c + p.rk) + k;
+    float v[8];
+    load_row8(x, v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (k + 2 * j >= p.rot) continue;
+      const float a = cs[k / 2 + j], b = sn[k / 2 + j], u = v[2 * j], w = v[2 * j + 1];
+      v[2 * j] = u * a - w * b;
+      v[2 * j + 1] = w * a + u * b;
     }
+    store_row8(x, v);
     E* to = h < p.H ? (q_row >= 0 ? reinterpret_cast<E*>(p.q_abs) + ((size_t)q_row * p.H + h) * width : nullptr) : dst;
-    if (to) to[p.rk + 2 * k] = y[0], to[p.rk + 2 * k + 1] = y[1];
+    if (to) store_row8(to + p.rk + k, v);
   }
 }
 
@@ -94,7 +102,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
 constexpr int DEC_KEYS = 128;                      // keys per tile: the rows of the S^T MMA
 constexpr uint32_t DEC_ATOM = DEC_KEYS * 128;      // 128 rows of one 64-column swizzle atom
 constexpr int DEC_MAX_PAIRS = 16;                  // ring slots of two atoms
-constexpr int DEC_THREADS = 192;                   // warps 0-3 softmax, warp 4 TMA, warp 5 MMA
+constexpr int DEC_THREADS = 320;                   // warps 0-3 / 4-7 softmax of half the query rows each, warp 8 TMA, warp 9 MMA
 
 struct LatentDecodeParams {
   const int* block_table;
@@ -145,22 +153,41 @@ __device__ __forceinline__ void tmem_st_cols16(uint32_t taddr, const float* v) {
       "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15])
       : "memory");
 }
+__device__ __forceinline__ void tmem_ld_cols8(uint32_t taddr, float* v) {
+  uint32_t r[8];
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+               : "r"(taddr)
+               : "memory");
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tmem_st_cols8(uint32_t taddr, const float* v) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]),
+               "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7])
+               : "memory");
+}
+template <int NB>
+__device__ __forceinline__ void tmem_st_cols(uint32_t taddr, const float* v) {
+  if constexpr (NB == 8) tmem_st_cols8(taddr, v);
+  else tmem_st_cols16(taddr, v);
+}
 template <int NB>
 __device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, float* v) {
-#pragma unroll
-  for (int c = 0; c < NB; c += 16) tmem_ld_cols16(taddr + c, v + c);
+  if constexpr (NB == 8) tmem_ld_cols8(taddr, v);
+  else tmem_ld_cols16(taddr, v);
   tmem_ld_wait();
 #pragma unroll
   for (int c = 0; c < NB; ++c) asm volatile("" : "+f"(v[c]));      // uses stay behind the wait
 }
 
-// Barrier of the four softmax warps that also agrees on whether everyone is still fine.
-__device__ __forceinline__ bool softmax_sync(bool ok) {
+// Barrier of the four warps of softmax group `id` (1 or 2) that also agrees on whether everyone is still fine.
+__device__ __forceinline__ bool softmax_sync(bool ok, int id) {
   uint32_t all;
   asm volatile(
-      "{\n.reg .pred p, q;\nsetp.ne.b32 p, %1, 0;\nbarrier.cta.red.and.pred q, 1, 128, p;\nselp.u32 %0, 1, 0, q;\n}\n"
+      "{\n.reg .pred p, q;\nsetp.ne.b32 p, %1, 0;\nbarrier.cta.red.and.pred q, %2, 128, p;\nselp.u32 %0, 1, 0, q;\n}\n"
       : "=r"(all)
-      : "r"((uint32_t)ok)
+      : "r"((uint32_t)ok), "r"(id)
       : "memory");
   return all != 0;
 }
@@ -178,8 +205,9 @@ __device__ __forceinline__ float reduce_columns(float* v, int lane) {
       v[i] = MAX ? fmaxf(keep, got) : keep + got;
     }
   }
-  if constexpr (NB == 16) {
-    const float got = __shfl_xor_sync(0xffffffffu, v[0], 16);
+#pragma unroll
+  for (int o = NB; o < 32; o <<= 1) {
+    const float got = __shfl_xor_sync(0xffffffffu, v[0], o);
     v[0] = MAX ? fmaxf(v[0], got) : v[0] + got;
   }
   return v[0];
@@ -222,18 +250,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
     mbar_init(&bars->s_full, 1);
-    mbar_init(&bars->p_full, 128);
+    mbar_init(&bars->p_full, 256);
     mbar_init(&bars->o_final, 1);
     for (int i = 0; i < p.ring_pairs; ++i) mbar_init(&bars->pair_full[i], 1), mbar_init(&bars->pair_empty[i], 1);
     for (int i = 0; i < p.ring_rots; ++i) mbar_init(&bars->rot_full[i], 1), mbar_init(&bars->rot_empty[i], 1);
     bars->abort = 0;
     mbar_fence_init();
   }
-  if (warp == 4 && lane == 0) {
+  if (warp == 8 && lane == 0) {
     tma_prefetch_desc(&tmap_q);
     tma_prefetch_desc(&tmap_kv);
   }
-  if (warp == 5) {
+  if (warp == 9) {
     tmem_alloc(&bars->tmem_base, TMEM_COLS);
     tmem_relinquish();
   }
@@ -242,7 +270,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   tc_fence_after_sync();
   const uint32_t tmem = bars->tmem_base;
 
-  if (warp == 4) {
+  if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       mbar_arrive_expect_tx(&bars->q_full, (p.latent_atoms + p.rot_atoms) * Q_ATOM);
@@ -292,7 +320,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           mbar_wait(&bars->pair_full[i % p.ring_pairs], (i / p.ring_pairs) & 1, &never, 714);
       }
     }
-  } else if (warp == 5) {
+  } else if (warp == 9) {
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t IDESC_S = umma_idesc_bf16_f32(DEC_KEYS, NB);
@@ -341,70 +369,73 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       }
     }
   } else {
-    // ------------------------------------------------------------------ softmax: thread = key of the tile
-    const uint32_t t_lane = tmem + ((uint32_t)(warp * 32) << 16);
-    const int key = warp * 32 + lane;
-    float m[NB], l[NB];
+    // ------------------------------------------------------------------ softmax: thread = key of the tile, NC query rows
+    constexpr int NC = NB / 2;
+    const int grp = warp >> 2, w4 = warp & 3, r0 = grp * NC;      // this group's first query row of the block
+    const uint32_t t_s = tmem + ((uint32_t)(w4 * 32) << 16) + r0, t_o = t_s + COL_O;
+    const int key = w4 * 32 + lane;
+    float* red_g = red + grp * 8 * NC;                            // [2][4][NC]
+    float m[NC], l[NC];
 #pragma unroll
-    for (int n = 0; n < NB; ++n) m[n] = -INFINITY, l[n] = 0.f;
+    for (int n = 0; n < NC; ++n) m[n] = -INFINITY, l[n] = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
-      float s[NB];
+      float s[NC];
+      float* red_j = red_g + (j & 1) * 4 * NC;
       ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full, j & 1, abort_flag, 730));
       if (ok) {
         tc_fence_after_sync();
-        tmem_ld_cols<NB>(t_lane, s);
+        tmem_ld_cols<NC>(t_s, s);
         const int k0 = (t0 + j) * DEC_KEYS;
         if (k0 + DEC_KEYS > kv_len - q_len + row0 / p.H + 1) {      // some key of the tile lies behind the first row
 #pragma unroll
-          for (int n = 0; n < NB; ++n)
-            if (k0 + key > kv_len - q_len + (row0 + n) / p.H || k0 + key >= kv_len) s[n] = -INFINITY;
+          for (int n = 0; n < NC; ++n)
+            if (k0 + key > kv_len - q_len + (row0 + r0 + n) / p.H || k0 + key >= kv_len) s[n] = -INFINITY;
         }
-        float v[NB];
+        float v[NC];
 #pragma unroll
-        for (int n = 0; n < NB; ++n) v[n] = s[n];
-        const float top = reduce_columns<NB, true>(v, lane);
-        if (lane < NB) red[((j & 1) * 4 + warp) * NB + lane] = top;
+        for (int n = 0; n < NC; ++n) v[n] = s[n];
+        const float top = reduce_columns<NC, true>(v, lane);
+        if (lane < NC) red_j[w4 * NC + lane] = top;
       }
-      ok = softmax_sync(ok);
+      ok = softmax_sync(ok, 1 + grp);
       if (!ok) break;
-      float mn[NB];
+      float mn[NC];
       bool grow = false;
 #pragma unroll
-      for (int n = 0; n < NB; n += 4) {
-        float4 a = *reinterpret_cast<const float4*>(&red[((j & 1) * 4) * NB + n]);
+      for (int n = 0; n < NC; n += 4) {
+        float4 a = *reinterpret_cast<const float4*>(&red_j[n]);
 #pragma unroll
         for (int w = 1; w < 4; ++w) {
-          const float4 b = *reinterpret_cast<const float4*>(&red[((j & 1) * 4 + w) * NB + n]);
+          const float4 b = *reinterpret_cast<const float4*>(&red_j[w * NC + n]);
           a.x = fmaxf(a.x, b.x), a.y = fmaxf(a.y, b.y), a.z = fmaxf(a.z, b.z), a.w = fmaxf(a.w, b.w);
         }
         mn[n] = fmaxf(m[n], a.x), mn[n + 1] = fmaxf(m[n + 1], a.y), mn[n + 2] = fmaxf(m[n + 2], a.z), mn[n + 3] = fmaxf(m[n + 3], a.w);
       }
 #pragma unroll
-      for (int n = 0; n < NB; ++n) grow |= (mn[n] - m[n]) * p.scale_log2 > 8.f;
-      if (grow) {                    // the same in every thread: move all columns to their current maximum
-        float f[NB];
+      for (int n = 0; n < NC; ++n) grow |= (mn[n] - m[n]) * p.scale_log2 > 8.f;
+      if (grow) {                    // the same in every thread of the group: move its rows to their current maximum
+        float f[NC];
 #pragma unroll
-        for (int n = 0; n < NB; ++n) {
+        for (int n = 0; n < NC; ++n) {
           f[n] = mn[n] == -INFINITY ? 1.f : exp2f((m[n] - mn[n]) * p.scale_log2);
           m[n] = mn[n];
           l[n] *= f[n];
         }
         if (j > 0) {                 // the last PV has completed (s_full of this tile was committed behind it)
           for (int i = 0; i < p.pairs; ++i) {
-            float o[NB];
-            tmem_ld_cols<NB>(t_lane + COL_O + i * NB, o);
+            float o[NC];
+            tmem_ld_cols<NC>(t_o + i * NB, o);
 #pragma unroll
-            for (int n = 0; n < NB; ++n) o[n] *= f[n];
-#pragma unroll
-            for (int c = 0; c < NB; c += 16) tmem_st_cols16(t_lane + COL_O + i * NB + c, o + c);
+            for (int n = 0; n < NC; ++n) o[n] *= f[n];
+            tmem_st_cols<NC>(t_o + i * NB, o);
           }
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      uint8_t* dst = s_p + (key >> 6) * Q_ATOM + (key & 7) * 2;
+      uint8_t* dst = s_p + (key >> 6) * Q_ATOM + r0 * 128 + (key & 7) * 2;
 #pragma unroll
-      for (int n = 0; n < NB; ++n) {
+      for (int n = 0; n < NC; ++n) {
         const float e = exp2f(fmaf(s[n], p.scale_log2, m[n] == -INFINITY ? 0.f : -m[n] * p.scale_log2));
         l[n] += e;
         *reinterpret_cast<bf16*>(dst + n * 128 + ((((key & 63) >> 3) ^ (n & 7)) << 4)) = __float2bfloat16(e);
@@ -414,38 +445,37 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       mbar_arrive(&bars->p_full);
     }
     if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_final, 0, abort_flag, 731));
-    float* lred = red;                               // the last tile used slot (n_tiles - 1) & 1 of the maxima: use the other
-    lred += (n_tiles & 1) * 4 * NB;
+    float* lred = red_g + (n_tiles & 1) * 4 * NC;    // the half that the last tile did not use
     {
-      float v[NB];
+      float v[NC];
 #pragma unroll
-      for (int n = 0; n < NB; ++n) v[n] = l[n];
-      const float sum = reduce_columns<NB, false>(v, lane);
-      if (lane < NB) lred[warp * NB + lane] = sum;
+      for (int n = 0; n < NC; ++n) v[n] = l[n];
+      const float sum = reduce_columns<NC, false>(v, lane);
+      if (lane < NC) lred[w4 * NC + lane] = sum;
     }
-    if (softmax_sync(ok)) {
+    if (softmax_sync(ok, 1 + grp)) {
       tc_fence_after_sync();
-      const size_t base = (size_t)split * p.rows_total + base_row;
+      const size_t base = (size_t)split * p.rows_total + base_row + r0;
 #pragma unroll
-      for (int n = 0; n < NB; ++n)
-        if (threadIdx.x == n && n < nrows) {
+      for (int n = 0; n < NC; ++n)
+        if (key == n && r0 + n < nrows) {
           float* ml = p.part_ml + (base + n) * 2;
           ml[0] = m[n] * p.scale_log2;
-          ml[1] = lred[n] + lred[NB + n] + lred[2 * NB + n] + lred[3 * NB + n];
+          ml[1] = lred[n] + lred[NC + n] + lred[2 * NC + n] + lred[3 * NC + n];
         }
       for (int i = 0; i < p.pairs; ++i) {
-        float o[NB];
-        tmem_ld_cols<NB>(t_lane + COL_O + i * NB, o);
+        float o[NC];
+        tmem_ld_cols<NC>(t_o + i * NB, o);
         const int col = i * 128 + key;
 #pragma unroll
-        for (int n = 0; n < NB; ++n)
-          if (n < nrows && col < p.rk) p.part_o[(base + n) * p.rk + col] = o[n];
+        for (int n = 0; n < NC; ++n)
+          if (r0 + n < nrows && col < p.rk) p.part_o[(base + n) * p.rk + col] = o[n];
       }
     }
   }
   tc_fence_before_sync();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == 9) {
     tc_fence_after_sync();
     tmem_dealloc(tmem, TMEM_COLS);
   }
@@ -471,55 +501,59 @@ struct HeadMmaParams {
 
 constexpr int HM_TOK = 16;   // tokens per CTA: the rows of the MMA
 
-// out[t, h, n] = gate * sum_k a[t, h, k] w[h, n, k]: four warps, NT 8-column MMA tiles each. A lane's eight consecutive k are
+constexpr int HM_WARPS = 8;
+
+// out[t, h, n] = gate * sum_k a[t, h, k] w[h, n, k]: NT 8-column MMA tiles per warp. A lane's eight consecutive k are
 // spread over two MMAs the same way for both operands, so every load is 16 bytes.
 template <int NT, bool MERGE>
-__global__ void __launch_bounds__(128) head_mma_kernel(const HeadMmaParams p) {
+__global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaParams p) {
   extern __shared__ __align__(16) uint8_t hm_smem[];
   const int ld = p.K + 8;
   bf16* sa = reinterpret_cast<bf16*>(hm_smem);                             // [16][K + 8]
   float* wt = reinterpret_cast<float*>(hm_smem + (size_t)HM_TOK * ld * 2); // [16][32]: weight of each split
   const int h = blockIdx.y, t0 = blockIdx.z * HM_TOK, m = min(HM_TOK, p.n - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
-  const int n0 = (blockIdx.x * 4 + warp) * NT * 8;
+  const int n0 = (blockIdx.x * HM_WARPS + warp) * NT * 8;
   pdl_launch_dependents();
   pdl_wait();
   auto token_in = [&](int i) { return p.rows_in ? p.rows_in[t0 + i] : t0 + i; };
   auto token_out = [&](int i) { return p.rows_out ? p.rows_out[t0 + i] : t0 + i; };
   if constexpr (MERGE) {
-    for (int i = threadIdx.x; i < m; i += 128) {
+    for (int i = warp; i < m; i += HM_WARPS) {         // a warp per token: lane = split
       const size_t row = (size_t)token_in(i) * p.H + h;
       const float sk = p.sink[h] * 1.4426950408889634f;
-      float top = sk, den = 0.f;
-      for (int s = 0; s < p.num_splits; ++s) top = fmaxf(top, p.part_ml[((size_t)s * p.rows_total + row) * 2]);
-      for (int s = 0; s < p.num_splits; ++s) {
-        const float* ml = p.part_ml + ((size_t)s * p.rows_total + row) * 2;
-        const float w = ml[1] > 0.f ? exp2f(ml[0] - top) : 0.f;
-        wt[i * 32 + s] = w;
-        den = fmaf(w, ml[1], den);
-      }
-      den = 1.f / (den + exp2f(sk - top));
-      for (int s = 0; s < p.num_splits; ++s) wt[i * 32 + s] *= den;
+      float2 ml = make_float2(-INFINITY, 0.f);
+      if (lane < p.num_splits) ml = *reinterpret_cast<const float2*>(p.part_ml + ((size_t)lane * p.rows_total + row) * 2);
+      const float top = fmaxf(warp_max(ml.x), sk), w = ml.y > 0.f ? exp2f(ml.x - top) : 0.f;
+      const float den = warp_sum(w * ml.y) + exp2f(sk - top);
+      wt[i * 32 + lane] = w / den;
     }
     __syncthreads();
     const int nv = p.K / 4;
-    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += 128) {
+    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += HM_WARPS * 32) {
       const int i = idx / nv, c = (idx % nv) * 4;
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (i < m) {
         const float* o = p.part_o + ((size_t)token_in(i) * p.H + h) * p.K + c;
-        for (int s = 0; s < p.num_splits; ++s) {
-          const float w = wt[i * 32 + s];
-          if (w == 0.f) continue;    // an empty split wrote nothing
-          const float4 x = *reinterpret_cast<const float4*>(o + (size_t)s * p.rows_total * p.K);
-          v.x = fmaf(w, x.x, v.x), v.y = fmaf(w, x.y, v.y), v.z = fmaf(w, x.z, v.z), v.w = fmaf(w, x.w, v.w);
+        const size_t step = (size_t)p.rows_total * p.K;
+        for (int s0 = 0; s0 < p.num_splits; s0 += 4) {
+          float4 x[4];
+          float w[4];
+#pragma unroll
+          for (int s = 0; s < 4; ++s) {                // an empty split wrote nothing and is not read
+            w[s] = s0 + s < p.num_splits ? wt[i * 32 + s0 + s] : 0.f;
+            x[s] = w[s] != 0.f ? *reinterpret_cast<const float4*>(o + (s0 + s) * step) : make_float4(0.f, 0.f, 0.f, 0.f);
+          }
+#pragma unroll
+          for (int s = 0; s < 4; ++s)
+            v.x = fmaf(w[s], x[s].x, v.x), v.y = fmaf(w[s], x[s].y, v.y), v.z = fmaf(w[s], x[s].z, v.z), v.w = fmaf(w[s], x[s].w, v.w);
         }
       }
       *reinterpret_cast<uint2*>(sa + i * ld + c) = make_uint2(attn::pack_bf16(v.x, v.y), attn::pack_bf16(v.z, v.w));
     }
   } else {
     const int nv = p.K / 8;
-    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += 128) {
+    for (int idx = threadIdx.x; idx < HM_TOK * nv; idx += HM_WARPS * 32) {
       const int i = idx / nv, c = (idx % nv) * 8;
       uint4 v = make_uint4(0, 0, 0, 0);
       if (i < m) v = *reinterpret_cast<const uint4*>(p.a + token_in(i) * p.a_tok + (long long)h * p.a_head + c);
@@ -569,8 +603,9 @@ __global__ void __launch_bounds__(128) head_mma_kernel(const HeadMmaParams p) {
 template <int NT, bool MERGE>
 int launch_head_mma(const HeadMmaParams& p, cudaStream_t s) {
   const size_t smem = (size_t)HM_TOK * (p.K + 8) * 2 + (MERGE ? HM_TOK * 32 * 4 : 0);
-  return launch_kernel(head_mma_kernel<NT, MERGE>, dim3((p.N + NT * 32 - 1) / (NT * 32), p.H, (p.n + HM_TOK - 1) / HM_TOK), dim3(128),
-                       smem, s, p);
+  constexpr int COLS = HM_WARPS * NT * 8;
+  return launch_kernel(head_mma_kernel<NT, MERGE>, dim3((p.N + COLS - 1) / COLS, p.H, (p.n + HM_TOK - 1) / HM_TOK),
+                       dim3(HM_WARPS * 32), smem, s, p);
 }
 
 template <int NB>
@@ -604,11 +639,12 @@ int swb_latent_prep(void* buf, int ld, int col_c, const float* w, float eps, con
                     void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
-  if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || (rp % 2) || rank <= 0 || rank > rk || !cache || !slots) return -3;
+  if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || ((dn | rp | rk | ld | col_c) % 8) || rank <= 0 || rank > rk || !cache || !slots)
+    return -3;
   const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot, rp, rank, rk};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return fp32 ? launch_kernel(latent_prep_kernel<float>, dim3((unsigned)T), dim3(256), 0, s, p)
-              : launch_kernel(latent_prep_kernel<bf16>, dim3((unsigned)T), dim3(256), 0, s, p);
+  return fp32 ? launch_kernel(latent_prep_kernel<float>, dim3((unsigned)T), dim3(128), 0, s, p)
+              : launch_kernel(latent_prep_kernel<bf16>, dim3((unsigned)T), dim3(128), 0, s, p);
 }
 
 // out [rows, width] bf16 <- the cached rows of num_seqs sequences (seqs: their indices in block_table, null: 0, 1, ...), those of
@@ -683,7 +719,7 @@ int swb_head_mma(const void* a, long long a_tok, int a_head, const void* w, void
                         out_tok, out_head, reinterpret_cast<const bf16*>(gate), gate_tok, rows_in, rows_out, n, H, N, K, part_o, part_ml, sink,
                         num_splits, rows_total};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return part_o ? launch_head_mma<1, true>(p, s) : launch_head_mma<2, false>(p, s);
+  return part_o ? launch_head_mma<1, true>(p, s) : launch_head_mma<1, false>(p, s);
 }
 
 }  // extern "C"

@@ -418,25 +418,6 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const bf16* __restri
 // out = a N(z) + b N(z^2) + c N(z^3) + e with the powers taken element by element and N(y) = y / sqrt(mean(y^2) + eps) over
 // a row's F values; coef = (a, b, c, e). One CTA per row, statistics in fp32. Rows of at most THREADS * VPT * 8 values stay in
 // registers (VPT > 0), longer ones are read twice.
-template <typename E>
-__device__ __forceinline__ void load_row8(const E* p, float* v) {
-  if constexpr (sizeof(E) == 2) {
-    unpack8(*reinterpret_cast<const uint4*>(p), v);
-  } else {
-    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
-  }
-}
-template <typename E>
-__device__ __forceinline__ void store_row8(E* p, const float* v) {
-  if constexpr (sizeof(E) == 2) {
-    *reinterpret_cast<uint4*>(p) = pack8(v);
-  } else {
-    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-  }
-}
-
 template <typename E, int THREADS, int VPT>
 __global__ void __launch_bounds__(THREADS) poly_norm_kernel(const E* __restrict__ z, int ldz, E* out, int ldo, int F, int Fp,
                                                             const float* __restrict__ coef, float eps) {
@@ -505,11 +486,19 @@ template <typename E>
 int launch_poly_norm(const E* z, int ldz, E* out, int ldo, int T, int F, int Fp, const float* coef, float eps, cudaStream_t s) {
   const int nvec = Fp / 8;
   const dim3 grid((unsigned)T);
-  if (nvec <= 256) return launch_kernel(poly_norm_kernel<E, 256, 1>, grid, dim3(256), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
-  if (nvec <= 512) return launch_kernel(poly_norm_kernel<E, 256, 2>, grid, dim3(256), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
-  if (nvec <= 1024) return launch_kernel(poly_norm_kernel<E, 512, 2>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
-  if (nvec <= 2048) return launch_kernel(poly_norm_kernel<E, 512, 4>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
-  return launch_kernel(poly_norm_kernel<E, 512, 0>, grid, dim3(512), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  auto go = [&](auto kernel, int threads) {
+    return launch_kernel(kernel, grid, dim3(threads), 0, s, z, ldz, out, ldo, F, Fp, coef, eps);
+  };
+  switch ((nvec + 255) / 256) {
+    case 1: return go(poly_norm_kernel<E, 256, 1>, 256);
+    case 2: return go(poly_norm_kernel<E, 256, 2>, 256);
+    case 3: return go(poly_norm_kernel<E, 256, 3>, 256);
+    case 4: return go(poly_norm_kernel<E, 256, 4>, 256);
+    case 5: return go(poly_norm_kernel<E, 256, 5>, 256);
+    case 6: return go(poly_norm_kernel<E, 256, 6>, 256);
+    case 7: case 8: return go(poly_norm_kernel<E, 512, 4>, 512);
+    default: return go(poly_norm_kernel<E, 512, 0>, 512);
+  }
 }
 
 __global__ void __launch_bounds__(256) embedding_kernel(const long long* __restrict__ ids, const bf16* __restrict__ table,

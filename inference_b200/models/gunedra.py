@@ -203,7 +203,7 @@ class GunedraGpu(StackDecoder):
         conv = torch.cat([torch.nn.functional.pad(self._fp32(get(f"{p}{n}.conv", h * d, m.conv)).view(h, d, m.conv),
                                                   (0, 0, 0, padded - d)).reshape(-1, m.conv) for n, (h, d, padded) in parts.items()])
         col_b = 2 * G * dp + H * vp
-        delta = DeltaWeights(H, G, D, dp, E, vp, col_b, conv.contiguous(), self._fp32(get(p + "A_log", H)),
+        delta = DeltaWeights(H, G, D, dp, E, vp, col_b, conv.t().contiguous(), self._fp32(get(p + "A_log", H)),
                              self._fp32(get(p + "dt_bias", H * D).reshape(H, D), dp).reshape(-1), self._fp32(get(p + "norm", E), vp))
         a2 = self._heads(get(p + "a2", H * D, ra), H, [(D, dp)], up8(ra))
         g2 = self._heads(get(p + "g2", H * E, rg), H, [(E, vp)], up8(rg))

@@ -20,7 +20,7 @@ def delta_key_width(dim: int) -> int | None:
 @dataclass
 class DeltaWeights:
     """Sizes and small tensors of one layer. Projection columns: q [kv_heads * dp], k, v [heads * vp], then (from col_b on)
-    one step-size logit per head; conv fp32 [2 kv_heads dp + heads vp, taps] in the same order; a_log fp32 [heads], dt_bias fp32
+    one step-size logit per head; conv fp32 [taps, 2 kv_heads dp + heads vp] in the same order; a_log fp32 [heads], dt_bias fp32
     [heads * dp], norm fp32 [vp]; padding entries are zero."""
     heads: int
     kv_heads: int
@@ -40,7 +40,7 @@ class DeltaWeights:
 
     @property
     def taps(self) -> int:
-        return self.conv.shape[1]
+        return self.conv.shape[0]
 
     def state_shape(self) -> tuple[int, ...]:
         return (self.heads, self.vp, self.dp)

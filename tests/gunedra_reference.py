@@ -157,3 +157,96 @@ def greedy(cfg, weights, prompt, steps):
         toks.append(int(top.indices[0]))
         gaps.append(float(top.values[0] - top.values[1]))
     return toks[len(prompt):], gaps
+
+
+# ---- small random models --------------------------------------------------------------------------------------------
+def latent(heads, dim, rot_dim, vdim, rank, base, scale=None):
+    return ("latent_attention", {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank,
+                                 "scale": (dim + rot_dim) ** -0.5 if scale is None else scale, "rot": {"dims": rot_dim, "base": base}})
+
+
+def delta(heads, kv_heads, dim, vdim, conv):
+    return ("channel_delta", {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv})
+
+
+def config(layers, width, vocab, groups, eps=1e-5, residual_mult=0.5, embed_scale=1.0):
+    return {"architecture": "Gunedra", "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": groups},
+            "residual_mult": residual_mult, "embedding": {"scale": embed_scale},
+            "layers": [{"type": t, "mixer": m, "mlp": None if ff is None else {"kind": "dense", "ff": ff}} for (t, m), ff in layers]}
+
+
+def model_a():
+    """Every layer different; key heads shared by several value heads, a layer without a feed-forward, norm groups of 32."""
+    return config([(latent(3, 40, 24, 56, 96, 500.0), 200), (delta(6, 3, 24, 40, 4), 56), (latent(5, 64, 16, 32, 128, 1e4, 0.2), None),
+                   (delta(4, 4, 48, 24, 3), 72)], 160, 321, 5, eps=1e-3, residual_mult=0.7, embed_scale=1.7)
+
+
+def model_b():
+    """Nothing a multiple of eight, single heads, the shortest convolution with a window."""
+    return config([(delta(2, 1, 10, 12, 2), 30), (latent(1, 18, 6, 14, 20, 100.0), 13), (delta(1, 1, 33, 7, 5), 21)], 90, 77, 3, eps=1e-2,
+                  residual_mult=1.3)
+
+
+def model_c():
+    """Widths beyond the tuned kernels (attention heads above 128, rotated part above 64, rank above 512), no convolution window,
+    one norm group."""
+    return config([(latent(2, 136, 72, 132, 130, 2000.0), 64), (delta(2, 1, 140, 72, 1), None), (latent(3, 32, 8, 24, 600, 900.0), 24)],
+                  256, 150, 1, embed_scale=0.5)
+
+
+def model_d():
+    """For long contexts: many heads on few latents, norm groups of whole 128-column chunks."""
+    return config([(latent(20, 32, 32, 48, 192, 5e5), 300), (delta(4, 2, 64, 64, 4), 128), (latent(4, 128, 64, 128, 256, 1e4), 136)],
+                  384, 200, 3, residual_mult=0.4, embed_scale=2.0)
+
+
+def model_e():
+    """Attention layers only: no recurrent state at all."""
+    return config([(latent(2, 16, 8, 16, 64, 50.0), 40), (latent(4, 24, 16, 16, 40, 300.0), None)], 64, 90, 2)
+
+
+def model_f():
+    """Delta-rule layers only: no pages in use."""
+    return config([(delta(2, 2, 16, 16, 4), 40), (delta(4, 1, 32, 8, 4), None)], 64, 90, 2)
+
+
+MODELS = {"a": model_a, "b": model_b, "c": model_c, "d": model_d, "e": model_e, "f": model_f}
+
+
+def random_weights(cfg, seed=0, peak=2.0):
+    """bf16-representable weights; `peak` sets the spread of the attention scores."""
+    g = torch.Generator().manual_seed(seed)
+    W, V, s = cfg["width"], cfg["vocab"], cfg["embedding"]["scale"]
+
+    def rnd(*shape, std=1.0, mean=0.0):
+        return (torch.randn(shape, generator=g) * std + mean).to(torch.bfloat16)
+
+    def lin(out, inp, std=1.0):
+        return rnd(out, inp, std=std * inp ** -0.5)
+    w = {"embed": rnd(V, W), "final.norm": rnd(W, std=0.3, mean=1.0)}
+    for i, lay in enumerate(cfg["layers"]):
+        L, m, p = f"l{i}.", lay["mixer"], f"l{i}.mix."
+        for n in (1, 2) if lay["mlp"] else (1,):
+            w[f"{L}norm{n}"], w[f"{L}ls{n}"] = rnd(W, std=0.3, mean=1.0), rnd(W, std=0.4, mean=0.8)
+        w[L + "dwa"] = rnd(i + 2, std=0.3)
+        w[L + "dwa"][-1] += 0.7
+        H = m["heads"]
+        if lay["type"] == "latent_attention":
+            D, R, E, rank = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            w[p + "q"] = lin(H * (D + R), W, peak / (m["scale"] * (D + R) ** 0.5 * max(s, 1.0)))
+            w[p + "dkv"], w[p + "dkv.norm"] = lin(rank + R, W), rnd(rank, std=0.3, mean=1.0)
+            w[p + "uk"], w[p + "uv"] = lin(H * D, rank), lin(H * E, rank)
+            w[p + "sink"], w[p + "g"] = rnd(H, std=2.0), lin(H, W, 1.5)
+        else:
+            G, D, E = m["kv_heads"], m["dim"], m["vdim"]
+            for n, c in (("q", G * D), ("k", G * D), ("v", H * E)):
+                w[p + n], w[f"{p}{n}.conv"] = lin(c, W), rnd(c, m["conv"], std=m["conv"] ** -0.5)
+            w[p + "b"], w[p + "A_log"], w[p + "norm"] = lin(H, W, 1.5), rnd(H, std=0.5, mean=-2.0), rnd(E, std=0.3, mean=1.0)
+            ra, rg = max(3, D // 2 + 1), max(2, E // 3)
+            w[p + "a1"], w[p + "a2"], w[p + "dt_bias"] = lin(ra, W), lin(H * D, ra), rnd(H * D, mean=-1.0)
+            w[p + "g1"], w[p + "g2"] = lin(rg, W), lin(H * E, rg, 2.0)
+        w[p + "o"] = lin(W, H * m["vdim"])
+        if lay["mlp"]:
+            ff = lay["mlp"]["ff"]
+            w[L + "mlp.up"], w[L + "mlp.down"], w[L + "mlp.act"] = lin(ff, W), lin(W, ff), rnd(4, std=0.3, mean=0.5)
+    return w
