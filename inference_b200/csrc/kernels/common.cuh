@@ -163,6 +163,21 @@ __device__ __forceinline__ bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
   return ok != 0;
 }
 
+// Never suspends the thread (try_wait may): for a thread that polls several barriers.
+__device__ __forceinline__ bool mbar_test_wait(uint64_t* bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n"
+      ".reg .pred p;\n"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+      "selp.u32 %0, 1, 0, p;\n"
+      "}\n"
+      : "=r"(ok)
+      : "r"(smem_u32(bar)), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+
 // Bounded wait. `abort_flag` is a CTA-shared int: once any role sets it every other role's wait
 // returns false on its next slow-path check, so the whole CTA drains.
 __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, int where) {
@@ -322,6 +337,12 @@ __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __
 __device__ __forceinline__ float relu2_f(float x) {
   const float r = fmaxf(x, 0.f);
   return r * r;
+}
+
+__device__ __forceinline__ void store_row4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_row4(bf16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 
 // Sequence of flat token t: the last one whose first token is not after t (empty sequences are skipped over), or t / uniform.

@@ -2,8 +2,8 @@
 //     S <- g * S          (rows of S are key channels)
 //     u  = beta (v - S^T k),   S <- S + k u^T,   o = S^T q
 // Three launches around the projections:
-//   delta_prep   short causal convolutions with silu, unit q / k, decays, step sizes. A warp takes one head over a run of
-//                tokens and keeps the convolution window in registers;
+//   delta_prep   short causal convolutions with silu, unit q / k, decays, step sizes. A warp takes one head of one token, the
+//                warps of a CTA consecutive tokens, so that all but one of a convolution's rows come from L1;
 //   delta_scan   the recurrence. A column of S (one value channel) never meets the others: sixteen lanes own NC columns, DPL key
 //                channels of each in registers, so that every q, k, g value read from shared memory serves NC columns (reading
 //                them is what bounds the kernel otherwise). Both dots run on the decayed state, o = (g S)^T q + (k . q) u, so one
@@ -37,151 +37,106 @@ struct PrepParams {
   const void* window;        // [slots, taps - 1, 2 G dp + H vp]
   const float *a_log, *dt_bias;
   float *qk, *kq, *g, *v, *beta;       // [T, G, 2, dp] (k, q), [T, G], [T, H, dp], [T, H, vp], [T, H]
-  int tokens_per_cta;
+  int heads_per_cta;
 };
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// for activations and output gates, which do not enter the recurrence as they are
+__device__ __forceinline__ float fast_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
-// Four channels of the convolution at consecutive tokens. TAPS > 0: the last TAPS - 1 inputs stay in registers; 0: any number of
-// taps, every input is loaded again.
+// Four channels of the convolution at token t: silu(sum_j w[taps - 1 - j] x[t - j]). TAPS 0: any number of taps.
 template <typename E, int TAPS>
-struct Conv4 {
+struct Conv {
   const E *buf, *window;     // window: of this sequence's slot, or null (no history)
   const float* w;            // [taps, C]
-  int ld, C, taps, c, start;
-  float4 x[TAPS > 1 ? TAPS - 1 : 1], wt[TAPS > 0 ? TAPS : 1];
+  int ld, C, taps, start, t;
 
-  __device__ __forceinline__ float4 input(int t) const {
-    if (t >= start) return load_row4(buf + (size_t)t * ld + c);
-    if (window) return load_row4(window + (size_t)(taps - 1 + t - start) * C + c);
-    return make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  __device__ __forceinline__ void weights() {
-    if constexpr (TAPS > 0)
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) wt[j] = *reinterpret_cast<const float4*>(w + (size_t)j * C + c);
-  }
-  __device__ __forceinline__ void begin(int t) {       // t: the first token that will be asked for
-    if constexpr (TAPS > 1)
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) x[j] = input(t - (TAPS - 1) + j);
-  }
-  static __device__ __forceinline__ void mac(float4& y, float4 a, float4 b) {
-    y.x = fmaf(a.x, b.x, y.x), y.y = fmaf(a.y, b.y, y.y), y.z = fmaf(a.z, b.z, y.z), y.w = fmaf(a.w, b.w, y.w);
-  }
-  __device__ __forceinline__ float4 next(int t) {      // silu(sum_j w[taps - 1 - j] x[t - j])
+  __device__ __forceinline__ float4 operator()(int c) const {
     float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto input = [&](int r) {
+      if (r >= start) return load_row4(buf + (size_t)r * ld + c);
+      if (window) return load_row4(window + (size_t)(taps - 1 + r - start) * C + c);
+      return make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    auto mac = [&](int j, float4 x) {
+      const float4 b = __ldg(reinterpret_cast<const float4*>(w + (size_t)j * C + c));
+      y.x = fmaf(x.x, b.x, y.x), y.y = fmaf(x.y, b.y, y.y), y.z = fmaf(x.z, b.z, y.z), y.w = fmaf(x.w, b.w, y.w);
+    };
     if constexpr (TAPS > 0) {
-      const float4 now = load_row4(buf + (size_t)t * ld + c);
+      float4 x[TAPS];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) mac(y, wt[j], x[j]);
-      mac(y, wt[TAPS - 1], now);
+      for (int j = 0; j < TAPS; ++j) x[j] = input(t - (TAPS - 1) + j);
 #pragma unroll
-      for (int j = 0; j + 2 < TAPS; ++j) x[j] = x[j + 1];
-      if constexpr (TAPS > 1) x[TAPS - 2] = now;
+      for (int j = 0; j < TAPS; ++j) mac(j, x[j]);
     } else {
-      for (int j = 0; j < taps; ++j) mac(y, *reinterpret_cast<const float4*>(w + (size_t)j * C + c), input(t - (taps - 1) + j));
+      for (int j = 0; j < taps; ++j) mac(j, input(t - (taps - 1) + j));
     }
-    y.x *= sigmoid_f(y.x), y.y *= sigmoid_f(y.y), y.z *= sigmoid_f(y.z), y.w *= sigmoid_f(y.w);
+    y.x *= fast_sigmoid(y.x), y.y *= fast_sigmoid(y.y), y.z *= fast_sigmoid(y.z), y.w *= fast_sigmoid(y.w);
     return y;
   }
 };
 
 __device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+__device__ __forceinline__ float4 scale4(float4 a, float r) { return make_float4(a.x * r, a.y * r, a.z * r, a.w * r); }
 
-// Warp task over a run of tokens: [0, G) unit q and k of a key head; [G, G + H) decays and step sizes of a head; [G + H, G + 2 H)
-// its values. NI: 128-channel pieces of a key head.
+// Tasks of a token: [0, G) unit q and k of a key head; [G, G + H) decays and step size of a head; [G + H, G + 2 H) its values.
+// blockIdx.y takes heads_per_cta of them. NI: 128-channel pieces of a key head.
 template <typename E, int TAPS, int NI>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const PrepParams p) {
   pdl_wait();
   const DeltaShape& s = p.s;
-  const int task = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   const int nq = s.G * s.dp, C = 2 * nq + s.H * s.vp;
   const E* buf = reinterpret_cast<const E*>(p.buf);
-  const int t_lo = blockIdx.x * p.tokens_per_cta, t_hi = min(s.T, t_lo + p.tokens_per_cta);
-  if (task >= s.G && task < s.G + s.H) {
-    const int h = task - s.G;
-    const float rate = -expf(p.a_log[h]);
-    for (int c = lane * 4; c < s.dp; c += 128) {
-      const float4 b = *reinterpret_cast<const float4*>(p.dt_bias + h * s.dp + c);
-#pragma unroll 2
-      for (int t = t_lo; t < t_hi; ++t) {
+  if (t >= s.T) return;
+  const int seq = seq_of_token(s.cu_q, s.num_seqs, s.uniform_q, t);
+  const int start = s.cu_q ? s.cu_q[seq] : seq * s.uniform_q, slot = s.slots[seq];
+  const E* window = s.positions[start] == 0 || slot < 0 ? nullptr
+                                                         : reinterpret_cast<const E*>(p.window) + (size_t)slot * (s.taps - 1) * C;
+  const Conv<E, TAPS> conv{buf, window, p.conv, p.ld, C, s.taps, start, t};
+  const float q_scale = rsqrtf((float)s.dim);
+  const int first = blockIdx.y * p.heads_per_cta, last = min(first + p.heads_per_cta, s.G + 2 * s.H);
+#pragma unroll 1
+  for (int task = first; task < last; ++task) {
+    if (task < s.G) {
+      float4 q[NI], k[NI];
+      float qq = 0.f, kk = 0.f, kq = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int c = lane * 4 + i * 128;
+        q[i] = k[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < s.dp) q[i] = conv(task * s.dp + c), k[i] = conv(nq + task * s.dp + c);
+        qq += dot4(q[i], q[i]), kk += dot4(k[i], k[i]), kq += dot4(k[i], q[i]);
+      }
+      qq = warp_sum(qq), kk = warp_sum(kk), kq = warp_sum(kq);
+      const float rk = rsqrtf(kk + 1e-6f), rq = rsqrtf(qq + 1e-6f) * q_scale;
+      float* out = p.qk + ((size_t)t * s.G + task) * 2 * s.dp;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int c = lane * 4 + i * 128;
+        if (c >= s.dp) continue;
+        *reinterpret_cast<float4*>(out + c) = scale4(k[i], rk);
+        *reinterpret_cast<float4*>(out + s.dp + c) = scale4(q[i], rq);
+      }
+      if (lane == 0) p.kq[(size_t)t * s.G + task] = kq * rk * rq;
+    } else if (task < s.G + s.H) {
+      const int h = task - s.G;
+      const float rate = -expf(p.a_log[h]);
+      for (int c = lane * 4; c < s.dp; c += 128) {
+        const float4 b = *reinterpret_cast<const float4*>(p.dt_bias + h * s.dp + c);
         float4 x = load_row4(reinterpret_cast<const E*>(p.decay) + (size_t)t * p.ld_decay + h * s.dp + c);
         x.x = expf(rate * softplus_f(x.x + b.x)), x.y = expf(rate * softplus_f(x.y + b.y));
         x.z = expf(rate * softplus_f(x.z + b.z)), x.w = expf(rate * softplus_f(x.w + b.w));
         *reinterpret_cast<float4*>(p.g + ((size_t)t * s.H + h) * s.dp + c) = x;
       }
-    }
-    for (int t = t_lo + lane; t < t_hi; t += 32) p.beta[(size_t)t * s.H + h] = sigmoid_f(to_f(buf[(size_t)t * p.ld + p.col_b + h]));
-  } else if (task < s.G + 2 * s.H) {
-    int seq = -1, start = 0, stop = t_lo;
-    const E* window = nullptr;
-    auto enter = [&](int t) {                          // the sequence that token t starts, or lies in
-      seq = seq_of_token(s.cu_q, s.num_seqs, s.uniform_q, t);
-      start = s.cu_q ? s.cu_q[seq] : seq * s.uniform_q;
-      stop = s.cu_q ? s.cu_q[seq + 1] : start + s.uniform_q;
-      const int slot = s.slots[seq];
-      window = s.positions[start] == 0 || slot < 0 ? nullptr : reinterpret_cast<const E*>(p.window) + (size_t)slot * (s.taps - 1) * C;
-    };
-    if (task < s.G) {
-      Conv4<E, TAPS> cq[NI], ck[NI];
-      const float q_scale = rsqrtf((float)s.dim);
-#pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        const int c = min(lane * 4 + i * 128, s.dp - 4);
-        cq[i].buf = ck[i].buf = buf, cq[i].w = ck[i].w = p.conv, cq[i].ld = ck[i].ld = p.ld, cq[i].C = ck[i].C = C;
-        cq[i].taps = ck[i].taps = s.taps, cq[i].c = task * s.dp + c, ck[i].c = nq + task * s.dp + c;
-        cq[i].weights(), ck[i].weights();
-      }
-      for (int t = t_lo; t < t_hi; ++t) {
-        if (t >= stop || t == t_lo) {
-          enter(t);
-#pragma unroll
-          for (int i = 0; i < NI; ++i) {
-            cq[i].window = ck[i].window = window, cq[i].start = ck[i].start = start;
-            cq[i].begin(t), ck[i].begin(t);
-          }
-        }
-        float4 q[NI], k[NI];
-        float qq = 0.f, kk = 0.f, kq = 0.f;
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-          q[i] = cq[i].next(t), k[i] = ck[i].next(t);
-          if (lane * 4 + i * 128 >= s.dp) q[i] = k[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-          qq += dot4(q[i], q[i]), kk += dot4(k[i], k[i]), kq += dot4(k[i], q[i]);
-        }
-        qq = warp_sum(qq), kk = warp_sum(kk), kq = warp_sum(kq);
-        const float rk = rsqrtf(kk + 1e-6f), rq = rsqrtf(qq + 1e-6f) * q_scale;
-        float* out = p.qk + ((size_t)t * s.G + task) * 2 * s.dp;
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-          const int c = lane * 4 + i * 128;
-          if (c >= s.dp) continue;
-          *reinterpret_cast<float4*>(out + c) = make_float4(k[i].x * rk, k[i].y * rk, k[i].z * rk, k[i].w * rk);
-          *reinterpret_cast<float4*>(out + s.dp + c) = make_float4(q[i].x * rq, q[i].y * rq, q[i].z * rq, q[i].w * rq);
-        }
-        if (lane == 0) p.kq[(size_t)t * s.G + task] = kq * rk * rq;
-      }
+      if (lane == 0) p.beta[(size_t)t * s.H + h] = sigmoid_f(to_f(buf[(size_t)t * p.ld + p.col_b + h]));
     } else {
       const int h = task - s.G - s.H;
-      for (int c = lane * 4; c < s.vp; c += 128) {
-        Conv4<E, TAPS> cv;
-        cv.buf = buf, cv.w = p.conv, cv.ld = p.ld, cv.C = C, cv.taps = s.taps, cv.c = 2 * nq + h * s.vp + c;
-        cv.weights();
-        stop = t_lo;
-        for (int t = t_lo; t < t_hi; ++t) {
-          if (t >= stop) {
-            enter(t);
-            cv.window = window, cv.start = start;
-            cv.begin(t);
-          }
-          *reinterpret_cast<float4*>(p.v + ((size_t)t * s.H + h) * s.vp + c) = cv.next(t);
-        }
-      }
+      for (int c = lane * 4; c < s.vp; c += 128)
+        *reinterpret_cast<float4*>(p.v + ((size_t)t * s.H + h) * s.vp + c) = conv(2 * nq + h * s.vp + c);
     }
   }
-  pdl_launch_dependents();
 }
 
 struct ScanParams {
@@ -310,10 +265,11 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
     __syncthreads();
     const float* tok = sm + (b & 1) * TB * TOK;
     const int m = min(TB, n - b * TB);
-    uint64_t k[N2], q[N2], g[N2];
-    if (AHEAD) L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
-    for (int r = 0; r < m; ++r, tok += TOK, orow += (size_t)s.H * s.vp) {
-      if (!AHEAD) L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
+    // one token: operands in (k, q, g), those of the next token are read into (kn, qn, gn) meanwhile
+    auto step = [&](const float* tok, float* o_to, uint64_t* k, uint64_t* q, uint64_t* g, uint64_t* kn, uint64_t* qn, uint64_t* gn,
+                    bool more) {
+      const float kq = tok[3 * DP + COLS], beta = tok[3 * DP + COLS + 1], v = tok[3 * DP + lc + mine];
+      if (AHEAD && more) L::load(tok + TOK, sub, kn), L::load(tok + TOK + DP, sub, qn), L::load(tok + TOK + 2 * DP, sub, gn);
       float a[2 * NC];
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
@@ -326,11 +282,6 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
         }
         a[c] = sum2(ak), a[NC + c] = sum2(aq);
       }
-      const float kq = tok[3 * DP + COLS], beta = tok[3 * DP + COLS + 1], v = tok[3 * DP + lc + mine];
-      uint64_t k_now[N2];
-#pragma unroll
-      for (int i = 0; i < N2; ++i) k_now[i] = k[i];
-      if (AHEAD && r + 1 < m) L::load(tok + TOK, sub, k), L::load(tok + TOK + DP, sub, q), L::load(tok + TOK + 2 * DP, sub, g);
       // fold: each step halves the number of sums a lane still carries, then plain sums over the remaining lane bits
       int o = 8;
 #pragma unroll
@@ -352,9 +303,29 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
         if (c == mine) u_out = u;
         const uint64_t uu = dup2(u);
 #pragma unroll
-        for (int i = 0; i < N2; ++i) S[c][i] = fma2(k_now[i], uu, S[c][i]);
+        for (int i = 0; i < N2; ++i) S[c][i] = fma2(k[i], uu, S[c][i]);
       }
-      if (writes) *orow = fmaf(kq, u_out, a[0]);
+      if (writes) *o_to = fmaf(kq, u_out, a[0]);
+    };
+    const size_t o_step = (size_t)s.H * s.vp;
+    if constexpr (AHEAD) {
+      uint64_t k0[N2], q0[N2], g0[N2], k1[N2], q1[N2], g1[N2];
+      L::load(tok, sub, k0), L::load(tok + DP, sub, q0), L::load(tok + 2 * DP, sub, g0);
+      int r = 0;
+      for (; r + 2 <= m; r += 2, tok += 2 * TOK, orow += 2 * o_step) {
+        step(tok, orow, k0, q0, g0, k1, q1, g1, true);
+        step(tok + TOK, orow + o_step, k1, q1, g1, k0, q0, g0, r + 2 < m);
+      }
+      if (r < m) {
+        step(tok, orow, k0, q0, g0, k1, q1, g1, false);
+        orow += o_step;
+      }
+    } else {
+      for (int r = 0; r < m; ++r, tok += TOK, orow += o_step) {
+        uint64_t k[N2], q[N2], g[N2];
+        L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
+        step(tok, orow, k, q, g, k, q, g, false);
+      }
     }
     __syncthreads();
   }
@@ -377,7 +348,7 @@ struct PostParams {
   const void* buf;           // projections, for the windows
   int ld;
   void* window;
-  int norm_ctas;
+  int norm_ctas, rows_per_warp;
 };
 
 template <typename E>
@@ -404,29 +375,43 @@ __global__ void __launch_bounds__(256) delta_post_kernel(const PostParams p) {
       }
     return;
   }
-  const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (id >= (long long)s.T * s.H) return;
-  const int t = (int)(id / s.H), h = (int)(id % s.H);
-  const float* o = p.o + id * s.vp;
-  float ss = 0.f;
-  for (int c = lane * 8; c < s.vp; c += 256) {       // padding columns are zero
-    float v[8];
-    load_row8(o + c, v);
+  const long long rows = (long long)s.T * s.H, id0 = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * p.rows_per_warp;
+  auto finish = [&](long long id, int c, float4 x, float4 z, float r) {
+    const float4 w = __ldg(reinterpret_cast<const float4*>(p.w + c));
+    store_row4(reinterpret_cast<E*>(p.out) + id * s.vp + c,
+               make_float4(x.x * r * w.x * fast_sigmoid(z.x), x.y * r * w.y * fast_sigmoid(z.y), x.z * r * w.z * fast_sigmoid(z.z),
+                           x.w * r * w.w * fast_sigmoid(z.w)));
+  };
+  auto gate = [&](long long id, int c) {
+    return load_row4(reinterpret_cast<const E*>(p.gate) + (size_t)(id / s.H) * p.ld_gate + (id % s.H) * s.vp + c);
+  };
+  if (s.vp <= 128) {                                 // one piece per lane, the loads of all rows in flight together
+    const int c = lane * 4;
+    constexpr int R = 4;                             // rows_per_warp is 1 or R
+    float4 x[R], z[R];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+    for (int i = 0; i < R; ++i) {
+      x[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < p.rows_per_warp && id0 + i < rows && c < s.vp) x[i] = load_row4(p.o + (id0 + i) * s.vp + c), z[i] = gate(id0 + i, c);
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      if (i >= p.rows_per_warp || id0 + i >= rows) return;
+      const float r = rsqrtf(warp_sum(dot4(x[i], x[i])) / (float)s.vdim + p.eps);    // padding columns are zero
+      if (c < s.vp) finish(id0 + i, c, x[i], z[i], r);
+    }
+    return;
   }
-  const float r = rsqrtf(warp_sum(ss) / (float)s.vdim + p.eps);
-  const E* gate = reinterpret_cast<const E*>(p.gate) + (size_t)t * p.ld_gate + h * s.vp;
-  E* out = reinterpret_cast<E*>(p.out) + id * s.vp;
-  for (int c = lane * 8; c < s.vp; c += 256) {
-    float v[8], w[8], z[8];
-    load_row8(o + c, v);
-    load_row8(p.w + c, w);
-    load_row8(gate + c, z);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] *= r * w[j] * sigmoid_f(z[j]);
-    store_row8(out + c, v);
+  for (long long id = id0; id < min(rows, id0 + p.rows_per_warp); ++id) {
+    const float* o = p.o + id * s.vp;
+    float ss = 0.f;
+    for (int c = lane * 4; c < s.vp; c += 128) {
+      const float4 x = load_row4(o + c);
+      ss += dot4(x, x);
+    }
+    const float r = rsqrtf(warp_sum(ss) / (float)s.vdim + p.eps);
+    for (int c = lane * 4; c < s.vp; c += 128) finish(id, c, load_row4(o + c), gate(id, c), r);
   }
 }
 
@@ -469,7 +454,7 @@ namespace swb {
 namespace {
 template <typename E, int NI>
 int launch_prep(const PrepParams& p, cudaStream_t st) {
-  const dim3 grid((p.s.T + p.tokens_per_cta - 1) / p.tokens_per_cta, (p.s.G + 2 * p.s.H + 7) / 8);
+  const dim3 grid((p.s.T + 7) / 8, (p.s.G + 2 * p.s.H + p.heads_per_cta - 1) / p.heads_per_cta);
   if constexpr (NI > 2) return launch_kernel(delta_prep_kernel<E, 0, NI>, grid, dim3(256), 0, st, p);
   else switch (p.s.taps) {
     case 1: return launch_kernel(delta_prep_kernel<E, 1, NI>, grid, dim3(256), 0, st, p);
@@ -494,7 +479,7 @@ int swb_delta_prep(const int* dims, const int* cu_q, const int* positions, const
                    float* qk, float* kq, float* g, float* v, float* beta, int fp32, void* stream) {
   using namespace swb;
   PrepParams p{make_shape(dims, cu_q, positions, slots), buf, ld, col_b, decay, ld_decay, conv, window, a_log, dt_bias, qk, kq, g, v,
-               beta, dims[0] >= 4096 ? 16 : dims[0] >= 1024 ? 8 : dims[0] >= 256 ? 4 : 1};
+               beta, dims[0] >= 4096 ? 8 : dims[0] >= 1024 ? 4 : 1};
   if (dims[0] <= 0) return 0;
   if (!shape_ok(p.s) || (ld % 4) || (ld_decay % 4)) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
@@ -523,10 +508,10 @@ int swb_delta_scan(const int* dims, const int* cu_q, const int* positions, const
 int swb_delta_post(const int* dims, const int* cu_q, const int* positions, const int* slots, const float* o, const void* gate,
                    int ld_gate, const float* w, float eps, void* out, const void* buf, int ld, void* window, int fp32, void* stream) {
   using namespace swb;
-  PostParams p{make_shape(dims, cu_q, positions, slots), o, gate, ld_gate, w, eps, out, buf, ld, window, 0};
+  PostParams p{make_shape(dims, cu_q, positions, slots), o, gate, ld_gate, w, eps, out, buf, ld, window, 0, dims[0] >= 1024 ? 4 : 1};
   if (dims[0] <= 0) return 0;
   if (!shape_ok(p.s)) return -3;
-  p.norm_ctas = (int)(((long long)p.s.T * p.s.H + 7) / 8);
+  p.norm_ctas = (int)(((long long)p.s.T * p.s.H + 8 * p.rows_per_warp - 1) / (8 * p.rows_per_warp));
   const int C = 2 * p.s.G * p.s.dp + p.s.H * p.s.vp;
   const dim3 grid(p.norm_ctas + (p.s.taps > 1 ? p.s.num_seqs * ((C + 1023) / 1024) : 0));
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

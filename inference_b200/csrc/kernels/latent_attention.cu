@@ -3,10 +3,11 @@
 //   latent_prep     norm of c, rotation of k_rot and of every head's rotated query part, cache write.
 //   latent_decode   attention in the latent space for steps with few tokens per sequence. The queries were taken through the
 //                   key projection, so all heads read the same cached rows, which serve as keys (all columns) and as values
-//                   (the latent columns). Everything is computed transposed on the tensor cores: S^T = K Q^T puts 128 keys on
-//                   the rows of the MMA and the (few) query rows on its columns, O^T = C^T P^T the latent columns on the rows;
+//                   (the latent columns). Everything is computed transposed on the tensor cores: S^T = K Q^T puts 64 keys on
+//                   the rows of the MMA and the (few) query rows on its columns, O^T = C^T P^T 128 latent columns on the rows;
 //                   C^T is the very tile that served as K, read as an MN-major operand. A page row is fetched once per 16 or
-//                   32 query rows. Partial results of KV splits stay un-normalised in fp32.
+//                   32 query rows. Scores and weights are double-buffered, so the softmax of one tile overlaps the MMAs of
+//                   its neighbours and the copies of the next. Partial results of KV splits stay un-normalised in fp32.
 //   head_mma        per-head products with the key and value projections around it; the value side merges the splits, adds
 //                   the sink to the denominator and applies the output gate.
 #include "attention_common.cuh"
@@ -99,9 +100,10 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
 }
 
 // ---- attention in the latent space ---------------------------------------------------------------------------------
-constexpr int DEC_KEYS = 128;                      // keys per tile: the rows of the S^T MMA
-constexpr uint32_t DEC_ATOM = DEC_KEYS * 128;      // 128 rows of one 64-column swizzle atom
-constexpr int DEC_MAX_PAIRS = 16;                  // ring slots of two atoms
+constexpr int DEC_KEYS = 64;                       // keys per tile: the rows of the S^T MMA
+constexpr uint32_t DEC_ATOM = DEC_KEYS * 128;      // 64 rows of one 64-column swizzle atom
+constexpr int DEC_MAX_PAIRS = 16;                  // ring slots of two atoms (16 KB)
+constexpr int DEC_MAX_ROTS = 4;                    // ring slots of the rotated parts
 constexpr int DEC_THREADS = 320;                   // warps 0-3 / 4-7 softmax of half the query rows each, warp 8 TMA, warp 9 MMA
 
 struct LatentDecodeParams {
@@ -117,9 +119,10 @@ struct LatentDecodeParams {
 };
 
 struct DecBarriers {
-  uint64_t q_full, s_full, p_full, o_final;
+  uint64_t q_full, pv_done, o_final;
+  uint64_t s_full[2], p_full[2];                   // tile j uses buffer j & 1
   uint64_t pair_full[DEC_MAX_PAIRS], pair_empty[DEC_MAX_PAIRS];
-  uint64_t rot_full[2], rot_empty[2];
+  uint64_t rot_full[DEC_MAX_ROTS], rot_empty[DEC_MAX_ROTS];
   uint32_t tmem_base;
   int abort;
 };
@@ -217,7 +220,7 @@ template <int NB>
 __global__ void __launch_bounds__(DEC_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_kv,
                      const LatentDecodeParams p) {
-  constexpr uint32_t Q_ATOM = NB * 128, TMEM_COLS = NB == 16 ? 128 : 256, COL_O = NB;
+  constexpr uint32_t Q_ATOM = NB * 128, TMEM_COLS = NB == 16 ? 128 : 256, COL_O = 2 * NB;   // S at [0, NB) and [NB, 2 NB)
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* s_rot = smem + p.ring_pairs * 2 * DEC_ATOM;
@@ -249,9 +252,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   }
   if (threadIdx.x == 0) {
     mbar_init(&bars->q_full, 1);
-    mbar_init(&bars->s_full, 1);
-    mbar_init(&bars->p_full, 256);
+    mbar_init(&bars->pv_done, 1);
     mbar_init(&bars->o_final, 1);
+    for (int i = 0; i < 2; ++i) mbar_init(&bars->s_full[i], 1), mbar_init(&bars->p_full[i], 256);
     for (int i = 0; i < p.ring_pairs; ++i) mbar_init(&bars->pair_full[i], 1), mbar_init(&bars->pair_empty[i], 1);
     for (int i = 0; i < p.ring_rots; ++i) mbar_init(&bars->rot_full[i], 1), mbar_init(&bars->rot_empty[i], 1);
     bars->abort = 0;
@@ -322,45 +325,68 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     }
   } else if (warp == 9) {
     // ------------------------------------------------------------------ MMA issuer
+    // Two streams in one thread: S^T of tile j piece by piece as its copies land (at most one tile ahead of the PV stream,
+    // because S and P have two buffers), O^T of tile j as soon as its weights are written. Whichever is ready goes first.
     if (lane == 0) {
       constexpr uint32_t IDESC_S = umma_idesc_bf16_f32(DEC_KEYS, NB);
       constexpr uint32_t IDESC_O = umma_idesc_bf16_f32(128, NB) | (1u << 15);   // A is MN-major
-      const uint32_t ring = smem_u32(smem), rot = smem_u32(s_rot), q = smem_u32(s_q), pp = smem_u32(s_p);
+      // descriptors of the regions' starts; the address field counts 16-byte units, so an offset is added to it
+      const uint64_t ring_k = umma_desc_kmajor_sw128(smem_u32(smem)), ring_mn = dec_desc_mnmajor(smem_u32(smem)),
+                     rot = umma_desc_kmajor_sw128(smem_u32(s_rot)), q = umma_desc_kmajor_sw128(smem_u32(s_q)),
+                     pp = umma_desc_kmajor_sw128(smem_u32(s_p));
+      constexpr uint32_t ATOM16 = DEC_ATOM / 16, Q16 = Q_ATOM / 16;
       bool ok = mbar_wait(&bars->q_full, 0, abort_flag, 720);
-      int n_pair = 0, n_rot = 0;
-      for (int j = 0; j < n_tiles && ok; ++j) {
-        const int rs = n_rot % p.ring_rots;
-        ok = mbar_wait(&bars->rot_full[rs], (n_rot / p.ring_rots) & 1, abort_flag, 721);
-        if (!ok) break;
-        tc_fence_after_sync();
-        for (int k = 0; k < p.rot_steps; ++k)
-          umma_f16_ss(tmem, umma_desc_kmajor_sw128(rot + (rs * p.rot_atoms + (k >> 2)) * DEC_ATOM + (k & 3) * 32),
-                      umma_desc_kmajor_sw128(q + (p.latent_atoms + (k >> 2)) * Q_ATOM + (k & 3) * 32), IDESC_S, k > 0);
-        umma_commit(&bars->rot_empty[rs]);
-        ++n_rot;
-        for (int i = 0; i < p.pairs && ok; ++i) {
-          const int sl = (n_pair + i) % p.ring_pairs, steps = min(2, p.latent_atoms - 2 * i) * 4;
-          ok = mbar_wait(&bars->pair_full[sl], ((n_pair + i) / p.ring_pairs) & 1, abort_flag, 722);
-          if (!ok) break;
+      int qk = 0, piece = -1, pv = 0;                  // piece -1: the rotated part, else a pair of latent atoms
+      int rot_slot = 0, qk_slot = 0, pv_slot = 0;
+      uint32_t rot_phase = 0, qk_phase = 0;
+      uint64_t idle_since = 0;
+      for (uint32_t spins = 0; ok && pv < n_tiles;) {
+        if (pv < qk && mbar_test_wait(&bars->p_full[pv & 1], (pv >> 1) & 1)) {
           tc_fence_after_sync();
-          for (int k = 0; k < steps; ++k)
-            umma_f16_ss(tmem, umma_desc_kmajor_sw128(ring + (sl * 2 + (k >> 2)) * DEC_ATOM + (k & 3) * 32),
-                        umma_desc_kmajor_sw128(q + (2 * i + (k >> 2)) * Q_ATOM + (k & 3) * 32), IDESC_S, 1);
-        }
-        if (!ok) break;
-        umma_commit(&bars->s_full);
-        ok = mbar_wait(&bars->p_full, j & 1, abort_flag, 723);
-        if (!ok) break;
-        tc_fence_after_sync();
-        for (int i = 0; i < p.pairs; ++i) {
-          const int sl = (n_pair + i) % p.ring_pairs;
+          for (int i = 0; i < p.pairs; ++i) {
 #pragma unroll
-          for (int k = 0; k < DEC_KEYS / 16; ++k)
-            umma_f16_ss(tmem + COL_O + i * NB, dec_desc_mnmajor(ring + sl * 2 * DEC_ATOM + k * 2048),
-                        umma_desc_kmajor_sw128(pp + (k >> 2) * Q_ATOM + (k & 3) * 32), IDESC_O, (j > 0) || (k > 0));
-          umma_commit(&bars->pair_empty[sl]);
+            for (int k = 0; k < DEC_KEYS / 16; ++k)
+              umma_f16_ss(tmem + COL_O + i * NB, ring_mn + pv_slot * 2 * ATOM16 + k * 128, pp + (pv & 1) * Q16 + k * 2, IDESC_O,
+                          (pv > 0) || (k > 0));
+            umma_commit(&bars->pair_empty[pv_slot]);
+            if (++pv_slot == p.ring_pairs) pv_slot = 0;
+          }
+          umma_commit(&bars->pv_done);
+          ++pv, spins = 0;
+        } else if (qk < n_tiles && qk <= pv + 1 &&
+                   (piece < 0 ? mbar_test_wait(&bars->rot_full[rot_slot], rot_phase) : mbar_test_wait(&bars->pair_full[qk_slot], qk_phase))) {
+          tc_fence_after_sync();
+          const uint32_t d = tmem + (qk & 1) * NB;
+          if (piece < 0) {
+            for (int k = 0; k < p.rot_steps; ++k)
+              umma_f16_ss(d, rot + (rot_slot * p.rot_atoms + (k >> 2)) * ATOM16 + (k & 3) * 2,
+                          q + (p.latent_atoms + (k >> 2)) * Q16 + (k & 3) * 2, IDESC_S, k > 0);
+            umma_commit(&bars->rot_empty[rot_slot]);
+            if (++rot_slot == p.ring_rots) rot_slot = 0, rot_phase ^= 1;
+            piece = 0;
+          } else {
+            const int atoms = min(2, p.latent_atoms - 2 * piece);
+            for (int a = 0; a < atoms; ++a)
+#pragma unroll
+              for (int k = 0; k < 4; ++k)
+                umma_f16_ss(d, ring_k + (qk_slot * 2 + a) * ATOM16 + k * 2, q + (2 * piece + a) * Q16 + k * 2, IDESC_S, 1);
+            if (++qk_slot == p.ring_pairs) qk_slot = 0, qk_phase ^= 1;
+            if (++piece == p.pairs) {
+              umma_commit(&bars->s_full[qk & 1]);
+              piece = -1, ++qk;
+            }
+          }
+          spins = 0;
+        } else if ((++spins & 0xFF) == 0) {            // nothing ready: bounded like every wait
+          const uint64_t now = global_timer_ns();
+          if (spins == 0x100) idle_since = now;
+          if (*abort_flag) ok = false;
+          else if (now - idle_since > g_wait_limit_ns) {
+            *abort_flag = 1;
+            report_error(SWB_ERR_WAIT_TIMEOUT, 721, (int)blockIdx.x, pv);
+            ok = false;
+          }
         }
-        n_pair += p.pairs;
       }
       umma_commit(&bars->o_final);   // also on the abort path: it only tracks MMAs already issued
       if (!ok) {                     // TMEM must not be freed under MMAs that are still running
@@ -369,11 +395,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       }
     }
   } else {
-    // ------------------------------------------------------------------ softmax: thread = key of the tile, NC query rows
+    // ------------------------------------------------------------------ softmax: NC query rows per thread. The 64 rows of S^T lie in lanes
+    // 0-15 of every 32: those threads hold a key each, the others only take part in the reductions.
     constexpr int NC = NB / 2;
     const int grp = warp >> 2, w4 = warp & 3, r0 = grp * NC;      // this group's first query row of the block
     const uint32_t t_s = tmem + ((uint32_t)(w4 * 32) << 16) + r0, t_o = t_s + COL_O;
-    const int key = w4 * 32 + lane;
+    const bool has_key = lane < 16;
+    const int key = w4 * 16 + (lane & 15);
     float* red_g = red + grp * 8 * NC;                            // [2][4][NC]
     float m[NC], l[NC];
 #pragma unroll
@@ -382,10 +410,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     for (int j = 0; j < n_tiles; ++j) {
       float s[NC];
       float* red_j = red_g + (j & 1) * 4 * NC;
-      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full, j & 1, abort_flag, 730));
+      ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full[j & 1], (j >> 1) & 1, abort_flag, 730));
       if (ok) {
         tc_fence_after_sync();
-        tmem_ld_cols<NC>(t_s, s);
+        tmem_ld_cols<NC>(t_s + (j & 1) * NB, s);
         const int k0 = (t0 + j) * DEC_KEYS;
         if (k0 + DEC_KEYS > kv_len - q_len + row0 / p.H + 1) {      // some key of the tile lies behind the first row
 #pragma unroll
@@ -394,7 +422,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
         }
         float v[NC];
 #pragma unroll
-        for (int n = 0; n < NC; ++n) v[n] = s[n];
+        for (int n = 0; n < NC; ++n) v[n] = s[n] = has_key ? s[n] : -INFINITY;
         const float top = reduce_columns<NC, true>(v, lane);
         if (lane < NC) red_j[w4 * NC + lane] = top;
       }
@@ -422,7 +450,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           m[n] = mn[n];
           l[n] *= f[n];
         }
-        if (j > 0) {                 // the last PV has completed (s_full of this tile was committed behind it)
+        // O may be touched once the PV of the tile before has completed
+        if (j > 0) ok = __all_sync(0xffffffffu, mbar_wait(&bars->pv_done, (j - 1) & 1, abort_flag, 732));
+        if (j > 0 && ok) {
+          tc_fence_after_sync();
           for (int i = 0; i < p.pairs; ++i) {
             float o[NC];
             tmem_ld_cols<NC>(t_o + i * NB, o);
@@ -433,16 +464,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      uint8_t* dst = s_p + (key >> 6) * Q_ATOM + r0 * 128 + (key & 7) * 2;
+      uint8_t* dst = s_p + (j & 1) * Q_ATOM + r0 * 128 + (key & 7) * 2;
 #pragma unroll
       for (int n = 0; n < NC; ++n) {
         const float e = exp2f(fmaf(s[n], p.scale_log2, m[n] == -INFINITY ? 0.f : -m[n] * p.scale_log2));
         l[n] += e;
-        *reinterpret_cast<bf16*>(dst + n * 128 + ((((key & 63) >> 3) ^ (n & 7)) << 4)) = __float2bfloat16(e);
+        if (has_key) *reinterpret_cast<bf16*>(dst + n * 128 + (((key >> 3) ^ (n & 7)) << 4)) = __float2bfloat16(e);
       }
       fence_proxy_async_smem();
       tc_fence_before_sync();
-      mbar_arrive(&bars->p_full);
+      mbar_arrive(&bars->p_full[j & 1]);
     }
     if (ok) ok = __all_sync(0xffffffffu, mbar_wait(&bars->o_final, 0, abort_flag, 731));
     float* lred = red_g + (n_tiles & 1) * 4 * NC;    // the half that the last tile did not use
@@ -458,7 +489,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       const size_t base = (size_t)split * p.rows_total + base_row + r0;
 #pragma unroll
       for (int n = 0; n < NC; ++n)
-        if (key == n && r0 + n < nrows) {
+        if (w4 * 32 + lane == n && r0 + n < nrows) {
           float* ml = p.part_ml + (base + n) * 2;
           ml[0] = m[n] * p.scale_log2;
           ml[1] = lred[n] + lred[NC + n] + lred[2 * NC + n] + lred[3 * NC + n];
@@ -466,7 +497,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       for (int i = 0; i < p.pairs; ++i) {
         float o[NC];
         tmem_ld_cols<NC>(t_o + i * NB, o);
-        const int col = i * 128 + key;
+        const int col = i * 128 + w4 * 32 + lane;
 #pragma unroll
         for (int n = 0; n < NC; ++n)
           if (r0 + n < nrows && col < p.rk) p.part_o[(base + n) * p.rk + col] = o[n];
@@ -503,9 +534,12 @@ constexpr int HM_TOK = 16;   // tokens per CTA: the rows of the MMA
 
 constexpr int HM_WARPS = 8;
 
-// out[t, h, n] = gate * sum_k a[t, h, k] w[h, n, k]: NT 8-column MMA tiles per warp. A lane's eight consecutive k are
-// spread over two MMAs the same way for both operands, so every load is 16 bytes.
-template <int NT, bool MERGE>
+constexpr int HM_SLABS = 16; // 32-wide K slabs whose weights are fetched ahead (K <= 512)
+
+// out[t, h, n] = gate * sum_k a[t, h, k] w[h, n, k], eight columns per warp. A lane's eight consecutive k are spread over two
+// MMAs the same way for both operands, so every load is 16 bytes. The weights depend on no earlier kernel: they are fetched in
+// front of the dependency wait.
+template <bool MERGE>
 __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaParams p) {
   extern __shared__ __align__(16) uint8_t hm_smem[];
   const int ld = p.K + 8;
@@ -513,7 +547,12 @@ __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaPa
   float* wt = reinterpret_cast<float*>(hm_smem + (size_t)HM_TOK * ld * 2); // [16][32]: weight of each split
   const int h = blockIdx.y, t0 = blockIdx.z * HM_TOK, m = min(HM_TOK, p.n - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
-  const int n0 = (blockIdx.x * HM_WARPS + warp) * NT * 8;
+  const int n0 = (blockIdx.x * HM_WARPS + warp) * 8;
+  const bf16* wr = p.w + ((size_t)h * p.N + min(n0 + g, p.N - 1)) * p.K + t4 * 8;
+  uint4 b[HM_SLABS];
+#pragma unroll
+  for (int s = 0; s < HM_SLABS; ++s)
+    b[s] = s * 32 + t4 * 8 < p.K ? __ldg(reinterpret_cast<const uint4*>(wr + s * 32)) : make_uint4(0, 0, 0, 0);
   pdl_launch_dependents();
   pdl_wait();
   auto token_in = [&](int i) { return p.rows_in ? p.rows_in[t0 + i] : t0 + i; };
@@ -536,16 +575,16 @@ __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaPa
       if (i < m) {
         const float* o = p.part_o + ((size_t)token_in(i) * p.H + h) * p.K + c;
         const size_t step = (size_t)p.rows_total * p.K;
-        for (int s0 = 0; s0 < p.num_splits; s0 += 4) {
-          float4 x[4];
-          float w[4];
+        for (int s0 = 0; s0 < p.num_splits; s0 += 8) {
+          float4 x[8];
+          float w[8];
 #pragma unroll
-          for (int s = 0; s < 4; ++s) {                // an empty split wrote nothing and is not read
+          for (int s = 0; s < 8; ++s) {                // an empty split wrote nothing and is not read
             w[s] = s0 + s < p.num_splits ? wt[i * 32 + s0 + s] : 0.f;
             x[s] = w[s] != 0.f ? *reinterpret_cast<const float4*>(o + (s0 + s) * step) : make_float4(0.f, 0.f, 0.f, 0.f);
           }
 #pragma unroll
-          for (int s = 0; s < 4; ++s)
+          for (int s = 0; s < 8; ++s)
             v.x = fmaf(w[s], x[s].x, v.x), v.y = fmaf(w[s], x[s].y, v.y), v.z = fmaf(w[s], x[s].z, v.z), v.w = fmaf(w[s], x[s].w, v.w);
         }
       }
@@ -562,50 +601,41 @@ __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaPa
   }
   __syncthreads();
   if (n0 >= p.N) return;
-  float acc[NT][4] = {};
-  const bf16* wr[NT];
-#pragma unroll
-  for (int t = 0; t < NT; ++t) wr[t] = p.w + ((size_t)h * p.N + min(n0 + t * 8 + g, p.N - 1)) * p.K + t4 * 8;
-#pragma unroll 4
-  for (int k = 0; k < p.K; k += 32) {
-    const bool in = k + t4 * 8 < p.K;
-    uint4 lo = make_uint4(0, 0, 0, 0), hi = lo, b[NT];
-    if (in) {
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  auto slab = [&](int k, uint4 w) {
+    uint4 lo = make_uint4(0, 0, 0, 0), hi = lo;
+    if (k + t4 * 8 < p.K) {
       lo = *reinterpret_cast<const uint4*>(sa + g * ld + k + t4 * 8);
       hi = *reinterpret_cast<const uint4*>(sa + (g + 8) * ld + k + t4 * 8);
     }
+    const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
+    attn::mma_16816(acc, a0, w.x, w.y);
+    attn::mma_16816(acc, a1, w.z, w.w);
+  };
 #pragma unroll
-    for (int t = 0; t < NT; ++t) b[t] = in ? __ldg(reinterpret_cast<const uint4*>(wr[t] + k)) : make_uint4(0, 0, 0, 0);
+  for (int s = 0; s < HM_SLABS; ++s)
+    if (s * 32 < p.K) slab(s * 32, b[s]);
+  for (int k = HM_SLABS * 32; k < p.K; k += 32)
+    slab(k, k + t4 * 8 < p.K ? __ldg(reinterpret_cast<const uint4*>(wr + k)) : make_uint4(0, 0, 0, 0));
+  const int n = n0 + t4 * 2;
+  if (n >= p.N) return;
 #pragma unroll
-    for (int t = 0; t < NT; ++t) {
-      const uint32_t a0[4] = {lo.x, hi.x, lo.y, hi.y}, a1[4] = {lo.z, hi.z, lo.w, hi.w};
-      attn::mma_16816(acc[t], a0, b[t].x, b[t].y);
-      attn::mma_16816(acc[t], a1, b[t].z, b[t].w);
-    }
-  }
-#pragma unroll
-  for (int t = 0; t < NT; ++t) {
-    const int n = n0 + t * 8 + t4 * 2;
-    if (n >= p.N) continue;
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int i = g + r * 8;
-      if (i >= m) continue;
-      const int tok = token_out(i);
-      float s = 1.f;
-      if (p.gate) s = 1.f / (1.f + expf(-__bfloat162float(p.gate[tok * p.gate_tok + h])));
-      *reinterpret_cast<uint32_t*>(p.out + tok * p.out_tok + (long long)h * p.out_head + n) =
-          attn::pack_bf16(acc[t][2 * r] * s, acc[t][2 * r + 1] * s);
-    }
+  for (int r = 0; r < 2; ++r) {
+    const int i = g + r * 8;
+    if (i >= m) continue;
+    const int tok = token_out(i);
+    float s = 1.f;
+    if (p.gate) s = 1.f / (1.f + expf(-__bfloat162float(p.gate[tok * p.gate_tok + h])));
+    *reinterpret_cast<uint32_t*>(p.out + tok * p.out_tok + (long long)h * p.out_head + n) = attn::pack_bf16(acc[2 * r] * s, acc[2 * r + 1] * s);
   }
 }
 
-template <int NT, bool MERGE>
+template <bool MERGE>
 int launch_head_mma(const HeadMmaParams& p, cudaStream_t s) {
   const size_t smem = (size_t)HM_TOK * (p.K + 8) * 2 + (MERGE ? HM_TOK * 32 * 4 : 0);
-  constexpr int COLS = HM_WARPS * NT * 8;
-  return launch_kernel(head_mma_kernel<NT, MERGE>, dim3((p.N + COLS - 1) / COLS, p.H, (p.n + HM_TOK - 1) / HM_TOK),
-                       dim3(HM_WARPS * 32), smem, s, p);
+  constexpr int COLS = HM_WARPS * 8;
+  return launch_kernel(head_mma_kernel<MERGE>, dim3((p.N + COLS - 1) / COLS, p.H, (p.n + HM_TOK - 1) / HM_TOK), dim3(HM_WARPS * 32), smem,
+                       s, p);
 }
 
 template <int NB>
@@ -613,8 +643,9 @@ int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDec
   constexpr size_t LIMIT = 227 * 1024;
   const size_t fixed = 1024 + (size_t)(p.latent_atoms + p.rot_atoms + 2) * NB * 128 + 8 * NB * 4 + sizeof(DecBarriers);
   const size_t pair = 2 * DEC_ATOM, rot = (size_t)p.rot_atoms * DEC_ATOM;
-  p.ring_rots = fixed + p.pairs * pair + 2 * rot <= LIMIT ? 2 : 1;
-  if (fixed + p.pairs * pair + p.ring_rots * rot > LIMIT) return -3;
+  p.ring_rots = DEC_MAX_ROTS;
+  while (p.ring_rots > 2 && fixed + 3 * p.pairs * pair + p.ring_rots * rot > LIMIT) --p.ring_rots;
+  if (fixed + 2 * p.pairs * pair + p.ring_rots * rot > LIMIT) return -3;   // two tiles are held at a time
   p.ring_pairs = (int)((LIMIT - fixed - p.ring_rots * rot) / pair);
   if (p.ring_pairs > DEC_MAX_PAIRS) p.ring_pairs = DEC_MAX_PAIRS;
   static bool configured[64] = {false};
@@ -719,7 +750,7 @@ int swb_head_mma(const void* a, long long a_tok, int a_head, const void* w, void
                         out_tok, out_head, reinterpret_cast<const bf16*>(gate), gate_tok, rows_in, rows_out, n, H, N, K, part_o, part_ml, sink,
                         num_splits, rows_total};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return part_o ? launch_head_mma<1, true>(p, s) : launch_head_mma<1, false>(p, s);
+  return part_o ? launch_head_mma<true>(p, s) : launch_head_mma<false>(p, s);
 }
 
 }  // extern "C"

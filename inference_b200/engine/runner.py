@@ -178,8 +178,8 @@ class ModelRunner:
     # ---- decode (graph-captured, one token per sequence) ---------------------------------------------
     def _fill_decode_meta(self, seqs: list[PagedSequence], tokens: list[int], pad_to: int = 0) -> int:
         """Writes the step metadata of the live rows; rows len(seqs)..pad_to-1 become copies of row 0 (same
-        token, position, slot and block table), so they recompute row 0 and store identical K / V bytes; they own no
-        recurrent state (slot -1)."""
+        token, position, slot and block table), so they recompute row 0 and store identical K / V bytes. With recurrent
+        layers a copy has no state of its own (state slot -1) and computes something else: it writes no K / V (slot -1)."""
         MB = self.max_batch
         h, table = self._host_np, self._host_table_np
         if self._meta_copy_done is not None:
@@ -212,7 +212,7 @@ class ModelRunner:
             for i in range(len(seqs), pad_to):
                 h[i], h[MB + i], h[2 * MB + i], h[3 * MB + i] = h[0], h[MB], h[2 * MB], h[3 * MB]
                 if self._stateful:
-                    h[4 * MB + i] = -1
+                    h[2 * MB + i] = h[4 * MB + i] = -1
                 table[i, :nb0] = table[0, :nb0]
                 self._row_state[i] = (-1, -1, 0)
         return max_kv

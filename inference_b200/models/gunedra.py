@@ -100,7 +100,7 @@ class GunedraGpu(StackDecoder):
         return out
 
     def decode_splits(self, batch: int, max_kv: int) -> tuple[int, ...]:
-        """KV splits per layer: about one CTA per SM, no split below one 128-key tile."""
+        """KV splits per layer: about one CTA per SM, no split below two 64-key tiles."""
         def splits(m) -> int:
             if not isinstance(m, LatentAttentionSpec):
                 return 1
