@@ -112,9 +112,9 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
     sig("swb_latent_prefill", [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_void_p])
     sig("swb_latent_prep", [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_latent_decode", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                              c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p])
+                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p])
     sig("swb_head_mma", [c_void_p, c_ll, c_int, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                          c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
     sig("swb_delta_prep", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,

@@ -302,6 +302,14 @@ __device__ __forceinline__ void tmem_ld_32x32b_x16(uint32_t taddr, float* v) {
   for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
 
+// One lane of a converged warp (always the same one), for code in which the whole warp runs in step so that descriptors and
+// addresses stay in uniform registers and only the issuing instruction is predicated.
+__device__ __forceinline__ bool elect_one() {
+  uint32_t yes;
+  asm volatile("{\n.reg .pred p;\nelect.sync _|p, 0xffffffff;\nselp.u32 %0, 1, 0, p;\n}\n" : "=r"(yes));
+  return yes != 0;
+}
+
 // UMMA shared-memory matrix descriptor for a K-major tile stored as rows of 128 bytes with the
 // 128-byte swizzle (what a TMA box of 64 bf16 x R rows with SWIZZLE_128B produces): 8-row groups are
 // 1024 bytes apart (stride byte offset), the leading byte offset is unused for swizzled K-major.

@@ -674,6 +674,36 @@ int make_tmap_u32_3d(CUtensorMap* out, const void* ptr, const unsigned long long
   return r == CUDA_SUCCESS ? 0 : -(int)r - 1000;
 }
 
+// Row-major bf16 [rows, cols] (cols a multiple of 64) as (64, rows, cols / 64), box (64, box_rows, cols / 64): one copy brings whole
+// rows and lays them out as 64-column blocks of box_rows rows, 128 bytes each, 128-byte swizzle.
+int make_tmap_bf16_blocks(CUtensorMap* out, const void* ptr, int rows, int cols, int ld, int box_rows) {
+  static std::mutex mu;
+  static std::unordered_map<MapKey, CUtensorMap, MapKeyHash> cache;
+  MapKey key{ptr, rows, cols, ld, box_rows};
+  {
+    std::lock_guard<std::mutex> g(mu);
+    auto it = cache.find(key);
+    if (it != cache.end()) {
+      *out = it->second;
+      return 0;
+    }
+  }
+  auto encode = get_encode_fn();
+  if (!encode) return -1;
+  cuuint64_t dims[3] = {64u, (cuuint64_t)rows, (cuuint64_t)(cols / 64)};
+  cuuint64_t strides[2] = {(cuuint64_t)ld * 2, 128u};
+  cuuint32_t box[3] = {64u, (cuuint32_t)box_rows, (cuuint32_t)(cols / 64)};
+  cuuint32_t estr[3] = {1u, 1u, 1u};
+  CUresult r = encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+                      CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                      CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return -(int)r - 1000;
+  std::lock_guard<std::mutex> g(mu);
+  if (cache.size() > 4096) cache.clear();
+  cache.emplace(key, *out);
+  return 0;
+}
+
 // NHWC bf16 activation [n, h, w, c] (contiguous): dims (c, w, h, n), box (64, box_w, box_h, 1), 128-byte swizzle, zero
 // fill outside (rows of the box land in (y, x) order, 128 bytes each: the K-major A tile the MMA descriptor expects).
 int make_tmap_bf16_nhwc(CUtensorMap* out, const void* ptr, int n, int h, int w, int c, int box_w, int box_h) {

@@ -28,10 +28,10 @@ struct LatentPrepParams {
   const float *cos, *sin;    // [positions, rot / 2]
   const int* positions;
   const long long* slots;    // row of the cache, < 0: none
-  void* cache;               // [rows, rk + rp]
-  void* q_abs;               // optional [rows, H, rk + rp]: receives the rotated query part at column rk
+  void* cache;               // [rows, rk + rc]
+  void* q_abs;               // optional [rows, H, rk + rc]: receives the rotated query part at column rk
   const int* q_row;          // optional [T]: row of q_abs of each token, < 0: none
-  int T, H, dn, rot, rp, rank, rk;
+  int T, H, dn, rot, rp, rc, rank, rk;   // rc: columns of the rotated part in `cache` and `q_abs`, zero beyond rp
 };
 
 // One CTA per token: warp 0 norms the latent, the others rotate in groups of eight dimensions (four pairs).
@@ -39,7 +39,7 @@ template <typename E>
 __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
   pdl_launch_dependents();
   pdl_wait(TL_ROPE_KV);
-  const int t = blockIdx.x, pos = p.positions[t], width = p.rk + p.rp, lane = threadIdx.x & 31;
+  const int t = blockIdx.x, pos = p.positions[t], width = p.rk + p.rc, lane = threadIdx.x & 31;
   E* row = reinterpret_cast<E*>(p.buf) + (size_t)t * p.ld;
   E* c = row + p.col_c;
   const long long slot = p.slots[t];
@@ -64,14 +64,14 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
     }
     return;
   }
-  const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t, per = p.rp / 8;
+  const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t, per = p.rc / 8;
   const float* cs = p.cos + (size_t)pos * (p.rot / 2);
   const float* sn = p.sin + (size_t)pos * (p.rot / 2);
   for (int i = threadIdx.x - 32; i < (p.H + 1) * per; i += 96) {    // the heads' queries, then the shared key part
     const int h = i / per, k = i % per * 8;
     E* x = (h < p.H ? row + h * (p.dn + p.rp) + p.dn : c + p.rk) + k;
-    float v[8];
-    load_row8(x, v);
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (k < p.rp) load_row8(x, v);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       if (k + 2 * j >= p.rot) continue;
@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
       v[2 * j] = u * a - w * b;
       v[2 * j + 1] = w * a + u * b;
     }
-    store_row8(x, v);
+    if (k < p.rp) store_row8(x, v);
     E* to = h < p.H ? (q_row >= 0 ? reinterpret_cast<E*>(p.q_abs) + ((size_t)q_row * p.H + h) * width : nullptr) : dst;
     if (to) store_row8(to + p.rk + k, v);
   }
@@ -101,9 +101,8 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restr
 
 // ---- attention in the latent space ---------------------------------------------------------------------------------
 constexpr int DEC_KEYS = 64;                       // keys per tile: the rows of the S^T MMA
-constexpr uint32_t DEC_ATOM = DEC_KEYS * 128;      // 64 rows of one 64-column swizzle atom
-constexpr int DEC_MAX_PAIRS = 16;                  // ring slots of two atoms (16 KB)
-constexpr int DEC_MAX_ROTS = 4;                    // ring slots of the rotated parts
+constexpr int DEC_STEPS = DEC_KEYS / 16;           // 16-key steps of a tile: the K of an MMA, and what is freed at a time
+constexpr int DEC_MAX_TILES = 8;                   // tiles in flight
 constexpr int DEC_THREADS = 320;                   // warps 0-3 / 4-7 softmax of half the query rows each, warp 8 TMA, warp 9 MMA
 
 struct LatentDecodeParams {
@@ -115,25 +114,25 @@ struct LatentDecodeParams {
   float scale_log2;
   float* part_o;             // [splits, rows_total, rk]
   float* part_ml;            // [splits, rows_total, 2]: running max (log2 units), sum relative to it
-  int rk, latent_atoms, pairs, rot_atoms, rot_steps, ring_pairs, ring_rots;
+  int rk, latent_atoms, pairs, atoms, rot_steps, ring;   // atoms: 64-column blocks of a cached row, rotated part last
 };
 
 struct DecBarriers {
   uint64_t q_full, pv_done, o_final;
   uint64_t s_full[2], p_full[2];                   // tile j uses buffer j & 1
-  uint64_t pair_full[DEC_MAX_PAIRS], pair_empty[DEC_MAX_PAIRS];
-  uint64_t rot_full[DEC_MAX_ROTS], rot_empty[DEC_MAX_ROTS];
+  uint64_t full[DEC_MAX_TILES], empty[DEC_MAX_TILES * DEC_STEPS];
   uint32_t tmem_base;
   int abort;
 };
 
-// A tile [keys][64 columns per atom] as the A operand of O^T += C^T P^T: rows are the MMA's K dimension, the second atom holds
-// columns 64..127 of the 128 MMA rows.
-__device__ __forceinline__ uint64_t dec_desc_mnmajor(uint32_t smem_addr) {
+// A tile in shared memory is 8 groups of 8 keys; a group is `atoms` blocks of 8 rows x 64 columns (1 KB, swizzled). As the A
+// operand of S^T (K-major) 8-row groups are atoms KB apart; as that of O^T (MN-major: keys are the MMA's K dimension) the next 64
+// columns are 1 KB further and the next 8 keys atoms KB.
+__device__ __forceinline__ uint64_t dec_desc(uint32_t smem_addr, uint32_t leading, uint32_t stride) {
   uint64_t d = 0;
   d |= (uint64_t)((smem_addr & 0x3FFFF) >> 4);
-  d |= (uint64_t)(DEC_ATOM >> 4) << 16;
-  d |= (uint64_t)(1024 >> 4) << 32;
+  d |= (uint64_t)(leading >> 4) << 16;
+  d |= (uint64_t)(stride >> 4) << 32;
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;
@@ -223,9 +222,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   constexpr uint32_t Q_ATOM = NB * 128, TMEM_COLS = NB == 16 ? 128 : 256, COL_O = 2 * NB;   // S at [0, NB) and [NB, 2 NB)
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* s_rot = smem + p.ring_pairs * 2 * DEC_ATOM;
-  uint8_t* s_q = s_rot + p.ring_rots * p.rot_atoms * DEC_ATOM;
-  uint8_t* s_p = s_q + (p.latent_atoms + p.rot_atoms) * Q_ATOM;
+  const uint32_t group_bytes = p.atoms * 1024, tile_bytes = 8 * group_bytes;
+  uint8_t* s_q = smem + p.ring * tile_bytes;
+  uint8_t* s_p = s_q + p.atoms * Q_ATOM;
   float* red = reinterpret_cast<float*>(s_p + 2 * Q_ATOM);      // [2][4][NB]
   DecBarriers* bars = reinterpret_cast<DecBarriers*>(red + 8 * NB);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -255,8 +254,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     mbar_init(&bars->pv_done, 1);
     mbar_init(&bars->o_final, 1);
     for (int i = 0; i < 2; ++i) mbar_init(&bars->s_full[i], 1), mbar_init(&bars->p_full[i], 256);
-    for (int i = 0; i < p.ring_pairs; ++i) mbar_init(&bars->pair_full[i], 1), mbar_init(&bars->pair_empty[i], 1);
-    for (int i = 0; i < p.ring_rots; ++i) mbar_init(&bars->rot_full[i], 1), mbar_init(&bars->rot_empty[i], 1);
+    for (int i = 0; i < p.ring; ++i) mbar_init(&bars->full[i], 1);
+    for (int i = 0; i < p.ring * DEC_STEPS; ++i) mbar_init(&bars->empty[i], 1);
     bars->abort = 0;
     mbar_fence_init();
   }
@@ -276,123 +275,107 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
-      mbar_arrive_expect_tx(&bars->q_full, (p.latent_atoms + p.rot_atoms) * Q_ATOM);
-      for (int a = 0; a < p.latent_atoms; ++a) tma_load_2d(s_q + a * Q_ATOM, &tmap_q, &bars->q_full, a * 64, base_row);
-      for (int a = 0; a < p.rot_atoms; ++a)
-        tma_load_2d(s_q + (p.latent_atoms + a) * Q_ATOM, &tmap_q, &bars->q_full, p.rk + a * 64, base_row);
+      mbar_arrive_expect_tx(&bars->q_full, p.atoms * Q_ATOM);
+      tma_load_3d(s_q, &tmap_q, &bars->q_full, 0, base_row, 0);
       const int* pages = p.block_table + (size_t)seq * p.max_blocks;
-      const int per_tile = DEC_KEYS / p.block_size, last_page = (kv_len - 1) / p.block_size;
-      const uint32_t page_bytes = (uint32_t)p.block_size * 128u;
+      const int last_group = (kv_len - 1) / 8;
       bool ok = true;
-      int n_pair = 0, n_rot = 0;                     // slots filled so far
+      int started = 0;                               // tiles with copies under way or landed
       for (int j = 0; j < n_tiles && ok; ++j) {
-        int rows[16];                                // first cache row of each page; pages past the last repeat it (masked)
+        const int slot = j % p.ring;
+        int rows[8];                                 // first cache row of each group; groups past the last repeat it (masked)
 #pragma unroll
-        for (int g = 0; g < 16; ++g) rows[g] = g < per_tile ? pages[min((t0 + j) * per_tile + g, last_page)] * p.block_size : 0;
-        auto load_atom = [&](uint8_t* dst, uint64_t* bar, int x) {
-#pragma unroll
-          for (int g = 0; g < 16; ++g)
-            if (g < per_tile) tma_load_2d(dst + g * page_bytes, &tmap_kv, bar, x, rows[g]);
-        };
-        {
-          const int sl = n_rot % p.ring_rots;
-          ok = mbar_wait(&bars->rot_empty[sl], ((n_rot / p.ring_rots) & 1) ^ 1, abort_flag, 710);
-          if (!ok) break;
-          mbar_arrive_expect_tx(&bars->rot_full[sl], p.rot_atoms * DEC_ATOM);
-          for (int a = 0; a < p.rot_atoms; ++a)
-            load_atom(s_rot + (sl * p.rot_atoms + a) * DEC_ATOM, &bars->rot_full[sl], p.rk + a * 64);
-          ++n_rot;
+        for (int g = 0; g < 8; ++g) {
+          const int key = min((t0 + j) * 8 + g, last_group) * 8;
+          rows[g] = pages[key / p.block_size] * p.block_size + key % p.block_size;
         }
-        for (int i = 0; i < p.pairs; ++i) {
-          const int sl = n_pair % p.ring_pairs, atoms = min(2, p.latent_atoms - 2 * i);
-          ok = mbar_wait(&bars->pair_empty[sl], ((n_pair / p.ring_pairs) & 1) ^ 1, abort_flag, 711);
+#pragma unroll
+        for (int k = 0; k < DEC_STEPS; ++k) {
+          ok = ok && mbar_wait(&bars->empty[slot * DEC_STEPS + k], ((j / p.ring) & 1) ^ 1, abort_flag, 711);
           if (!ok) break;
-          mbar_arrive_expect_tx(&bars->pair_full[sl], atoms * DEC_ATOM);
-          for (int a = 0; a < atoms; ++a)
-            load_atom(smem + (sl * 2 + a) * DEC_ATOM, &bars->pair_full[sl], (2 * i + a) * 64);
-          ++n_pair;
+          if (k == 0) {
+            mbar_arrive_expect_tx(&bars->full[slot], tile_bytes);
+            started = j + 1;
+          }
+          uint8_t* dst = smem + slot * tile_bytes + 2 * k * group_bytes;
+          tma_load_3d(dst, &tmap_kv, &bars->full[slot], 0, rows[2 * k], 0);
+          tma_load_3d(dst + group_bytes, &tmap_kv, &bars->full[slot], 0, rows[2 * k + 1], 0);
         }
       }
       if (!ok) {
-        // drain: every copy this thread started must land before the CTA's shared memory is released
+        // drain: every copy this thread started must land before the CTA's shared memory is released. The last tile may have
+        // been started in part; its barrier then expects more than will come, and this (bounded) wait runs out
         volatile int never = 0;
         mbar_wait(&bars->q_full, 0, &never, 712);
-        for (int i = max(0, n_rot - p.ring_rots); i < n_rot; ++i)
-          mbar_wait(&bars->rot_full[i % p.ring_rots], (i / p.ring_rots) & 1, &never, 713);
-        for (int i = max(0, n_pair - p.ring_pairs); i < n_pair; ++i)
-          mbar_wait(&bars->pair_full[i % p.ring_pairs], (i / p.ring_pairs) & 1, &never, 714);
+        for (int i = max(0, started - p.ring); i < started; ++i) mbar_wait(&bars->full[i % p.ring], (i / p.ring) & 1, &never, 714);
       }
     }
   } else if (warp == 9) {
     // ------------------------------------------------------------------ MMA issuer
-    // Two streams in one thread: S^T of tile j piece by piece as its copies land (at most one tile ahead of the PV stream,
-    // because S and P have two buffers), O^T of tile j as soon as its weights are written. Whichever is ready goes first.
-    if (lane == 0) {
-      constexpr uint32_t IDESC_S = umma_idesc_bf16_f32(DEC_KEYS, NB);
-      constexpr uint32_t IDESC_O = umma_idesc_bf16_f32(128, NB) | (1u << 15);   // A is MN-major
-      // descriptors of the regions' starts; the address field counts 16-byte units, so an offset is added to it
-      const uint64_t ring_k = umma_desc_kmajor_sw128(smem_u32(smem)), ring_mn = dec_desc_mnmajor(smem_u32(smem)),
-                     rot = umma_desc_kmajor_sw128(smem_u32(s_rot)), q = umma_desc_kmajor_sw128(smem_u32(s_q)),
-                     pp = umma_desc_kmajor_sw128(smem_u32(s_p));
-      constexpr uint32_t ATOM16 = DEC_ATOM / 16, Q16 = Q_ATOM / 16;
-      bool ok = mbar_wait(&bars->q_full, 0, abort_flag, 720);
-      int qk = 0, piece = -1, pv = 0;                  // piece -1: the rotated part, else a pair of latent atoms
-      int rot_slot = 0, qk_slot = 0, pv_slot = 0;
-      uint32_t rot_phase = 0, qk_phase = 0;
-      uint64_t idle_since = 0;
-      for (uint32_t spins = 0; ok && pv < n_tiles;) {
-        if (pv < qk && mbar_test_wait(&bars->p_full[pv & 1], (pv >> 1) & 1)) {
-          tc_fence_after_sync();
-          for (int i = 0; i < p.pairs; ++i) {
+    // Two streams: S^T of a tile once its copies have landed (at most one tile ahead of the other stream, because S and P have two
+    // buffers), O^T of a tile once its weights are written. Whichever is ready goes first. The warp runs in step, one lane issues.
+    constexpr uint32_t IDESC_S = umma_idesc_bf16_f32(DEC_KEYS, NB);
+    constexpr uint32_t IDESC_O = umma_idesc_bf16_f32(128, NB) | (1u << 15);     // A is MN-major
+    constexpr uint32_t Q16 = Q_ATOM / 16;                                       // descriptors count 16-byte units
+    const uint32_t tile16 = tile_bytes / 16, step16 = group_bytes / 8;          // one tile; two groups
+    const uint64_t ring_k = dec_desc(smem_u32(smem), 16, group_bytes), ring_mn = dec_desc(smem_u32(smem), 1024, group_bytes),
+                   q = umma_desc_kmajor_sw128(smem_u32(s_q)), pp = umma_desc_kmajor_sw128(smem_u32(s_p));
+    auto ready = [&](uint64_t* bar, uint32_t phase) { return __all_sync(0xffffffffu, mbar_test_wait(bar, phase)) != 0; };
+    bool ok = __all_sync(0xffffffffu, mbar_wait(&bars->q_full, 0, abort_flag, 720));
+    int qk = 0, pv = 0, qk_slot = 0, pv_slot = 0;
+    uint32_t qk_phase = 0, spins = 0;
+    uint64_t idle_since = 0;
+    while (ok && pv < n_tiles) {
+      if (pv < qk && ready(&bars->p_full[pv & 1], (pv >> 1) & 1)) {
+        tc_fence_after_sync();
+        if (elect_one()) {
+          const uint64_t a = ring_mn + pv_slot * tile16, b = pp + (pv & 1) * Q16;
 #pragma unroll
-            for (int k = 0; k < DEC_KEYS / 16; ++k)
-              umma_f16_ss(tmem + COL_O + i * NB, ring_mn + pv_slot * 2 * ATOM16 + k * 128, pp + (pv & 1) * Q16 + k * 2, IDESC_O,
-                          (pv > 0) || (k > 0));
-            umma_commit(&bars->pair_empty[pv_slot]);
-            if (++pv_slot == p.ring_pairs) pv_slot = 0;
+          for (int k = 0; k < DEC_STEPS; ++k) {
+            for (int i = 0; i < p.pairs; ++i)
+              umma_f16_ss(tmem + COL_O + i * NB, a + k * step16 + i * 128, b + k * 2, IDESC_O, (pv > 0) || (k > 0));
+            umma_commit(&bars->empty[pv_slot * DEC_STEPS + k]);
           }
           umma_commit(&bars->pv_done);
-          ++pv, spins = 0;
-        } else if (qk < n_tiles && qk <= pv + 1 &&
-                   (piece < 0 ? mbar_test_wait(&bars->rot_full[rot_slot], rot_phase) : mbar_test_wait(&bars->pair_full[qk_slot], qk_phase))) {
-          tc_fence_after_sync();
+        }
+        __syncwarp();
+        if (++pv_slot == p.ring) pv_slot = 0;
+        ++pv, spins = 0;
+      } else if (qk < n_tiles && qk <= pv + 1 && ready(&bars->full[qk_slot], qk_phase)) {
+        tc_fence_after_sync();
+        if (elect_one()) {
+          const uint64_t a = ring_k + qk_slot * tile16;
           const uint32_t d = tmem + (qk & 1) * NB;
-          if (piece < 0) {
-            for (int k = 0; k < p.rot_steps; ++k)
-              umma_f16_ss(d, rot + (rot_slot * p.rot_atoms + (k >> 2)) * ATOM16 + (k & 3) * 2,
-                          q + (p.latent_atoms + (k >> 2)) * Q16 + (k & 3) * 2, IDESC_S, k > 0);
-            umma_commit(&bars->rot_empty[rot_slot]);
-            if (++rot_slot == p.ring_rots) rot_slot = 0, rot_phase ^= 1;
-            piece = 0;
-          } else {
-            const int atoms = min(2, p.latent_atoms - 2 * piece);
-            for (int a = 0; a < atoms; ++a)
+          for (int i = 0; i < p.latent_atoms; ++i) {
 #pragma unroll
-              for (int k = 0; k < 4; ++k)
-                umma_f16_ss(d, ring_k + (qk_slot * 2 + a) * ATOM16 + k * 2, q + (2 * piece + a) * Q16 + k * 2, IDESC_S, 1);
-            if (++qk_slot == p.ring_pairs) qk_slot = 0, qk_phase ^= 1;
-            if (++piece == p.pairs) {
-              umma_commit(&bars->s_full[qk & 1]);
-              piece = -1, ++qk;
-            }
+            for (int k = 0; k < 4; ++k) umma_f16_ss(d, a + i * 64 + k * 2, q + i * Q16 + k * 2, IDESC_S, (i > 0) || (k > 0));
           }
-          spins = 0;
-        } else if ((++spins & 0xFF) == 0) {            // nothing ready: bounded like every wait
-          const uint64_t now = global_timer_ns();
-          if (spins == 0x100) idle_since = now;
-          if (*abort_flag) ok = false;
-          else if (now - idle_since > g_wait_limit_ns) {
+          for (int k = 0; k < p.rot_steps; ++k)
+            umma_f16_ss(d, a + (p.latent_atoms + (k >> 2)) * 64 + (k & 3) * 2, q + (p.latent_atoms + (k >> 2)) * Q16 + (k & 3) * 2, IDESC_S, 1);
+          umma_commit(&bars->s_full[qk & 1]);
+        }
+        __syncwarp();
+        if (++qk_slot == p.ring) qk_slot = 0, qk_phase ^= 1;
+        ++qk, spins = 0;
+      } else if ((++spins & 0xFF) == 0) {              // nothing ready: bounded like every wait
+        const uint64_t now = global_timer_ns();
+        if (spins == 0x100) idle_since = now;
+        if (__any_sync(0xffffffffu, *abort_flag != 0)) ok = false;
+        else if (__any_sync(0xffffffffu, now - idle_since > g_wait_limit_ns)) {
+          if (lane == 0) {
             *abort_flag = 1;
             report_error(SWB_ERR_WAIT_TIMEOUT, 721, (int)blockIdx.x, pv);
-            ok = false;
           }
+          ok = false;
         }
       }
-      umma_commit(&bars->o_final);   // also on the abort path: it only tracks MMAs already issued
-      if (!ok) {                     // TMEM must not be freed under MMAs that are still running
-        volatile int never = 0;
-        mbar_wait(&bars->o_final, 0, &never, 724);
-      }
+    }
+    __syncwarp();
+    if (elect_one()) umma_commit(&bars->o_final);      // also on the abort path: it only tracks MMAs already issued
+    __syncwarp();
+    if (!ok) {                                         // TMEM must not be freed under MMAs that are still running
+      volatile int never = 0;
+      mbar_wait(&bars->o_final, 0, &never, 724);
     }
   } else {
     // ------------------------------------------------------------------ softmax: NC query rows per thread. The 64 rows of S^T lie in lanes
@@ -641,13 +624,10 @@ int launch_head_mma(const HeadMmaParams& p, cudaStream_t s) {
 template <int NB>
 int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDecodeParams p, int seqs, int max_rows, cudaStream_t s) {
   constexpr size_t LIMIT = 227 * 1024;
-  const size_t fixed = 1024 + (size_t)(p.latent_atoms + p.rot_atoms + 2) * NB * 128 + 8 * NB * 4 + sizeof(DecBarriers);
-  const size_t pair = 2 * DEC_ATOM, rot = (size_t)p.rot_atoms * DEC_ATOM;
-  p.ring_rots = DEC_MAX_ROTS;
-  while (p.ring_rots > 2 && fixed + 3 * p.pairs * pair + p.ring_rots * rot > LIMIT) --p.ring_rots;
-  if (fixed + 2 * p.pairs * pair + p.ring_rots * rot > LIMIT) return -3;   // two tiles are held at a time
-  p.ring_pairs = (int)((LIMIT - fixed - p.ring_rots * rot) / pair);
-  if (p.ring_pairs > DEC_MAX_PAIRS) p.ring_pairs = DEC_MAX_PAIRS;
+  const size_t fixed = 1024 + (size_t)(p.atoms + 2) * NB * 128 + 8 * NB * 4 + sizeof(DecBarriers), tile = (size_t)p.atoms * 8192;
+  if (fixed + 2 * tile > LIMIT) return -3;                                  // two tiles are held at a time
+  p.ring = (int)((LIMIT - fixed) / tile);
+  if (p.ring > DEC_MAX_TILES) p.ring = DEC_MAX_TILES;
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -656,7 +636,7 @@ int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDec
     if (e != cudaSuccess) return -(int)e;
     if (dev >= 0 && dev < 64) configured[dev] = true;
   }
-  const size_t smem = fixed + p.ring_pairs * pair + p.ring_rots * rot;
+  const size_t smem = fixed + p.ring * tile;
   return launch_kernel(latent_decode_kernel<NB>, dim3(p.num_splits, (max_rows + NB - 1) / NB, seqs), dim3(DEC_THREADS), smem, s, tq, tk, p);
 }
 
@@ -666,13 +646,13 @@ int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDec
 extern "C" {
 
 int swb_latent_prep(void* buf, int ld, int col_c, const float* w, float eps, const float* cos, const float* sin, const int* positions,
-                    const long long* slots, void* cache, void* q_abs, const int* q_row, int T, int H, int dn, int rot, int rp, int rank, int rk, int fp32,
+                    const long long* slots, void* cache, void* q_abs, const int* q_row, int T, int H, int dn, int rot, int rp, int rc, int rank, int rk, int fp32,
                     void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
-  if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || ((dn | rp | rk | ld | col_c) % 8) || rank <= 0 || rank > rk || !cache || !slots)
+  if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || ((dn | rp | rc | rk | ld | col_c) % 8) || rc < rp || rank <= 0 || rank > rk || !cache || !slots)
     return -3;
-  const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot, rp, rank, rk};
+  const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot, rp, rc, rank, rk};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return fp32 ? launch_kernel(latent_prep_kernel<float>, dim3((unsigned)T), dim3(128), 0, s, p)
               : launch_kernel(latent_prep_kernel<bf16>, dim3((unsigned)T), dim3(128), 0, s, p);
@@ -705,14 +685,14 @@ int swb_latent_prefill(const void* q, long long q_stride_tok, const void* k, con
                                     reinterpret_cast<cudaStream_t>(stream));
 }
 
-// Attention of q_abs [T * H, rk + rp] over the cached rows [num_blocks * block_size, rk + rp] into split partials (see
-// LatentDecodeParams). max_q: most tokens of a sequence.
+// Attention of q_abs [T * H, rk + rp] over the cached rows [num_blocks * block_size, rk + rc] (q rows likewise) into
+// split partials (see LatentDecodeParams). rc: the rotated part with its padding (zero in q), a multiple of 64; rot of it is used. max_q: most tokens of a sequence.
 int swb_latent_decode(const void* q_abs, const void* cache, int num_blocks, int block_size, const int* block_table, int max_blocks,
                       const int* cu_q, const int* kv_lens, int n_seqs, int uniform_q, int max_q, int T, int H, int rk,
-                      int rp, float scale, int num_splits, float* part_o, float* part_ml, void* stream) {
+                      int rc, int rot, float scale, int num_splits, float* part_o, float* part_ml, void* stream) {
   using namespace swb;
   if (T <= 0 || n_seqs <= 0) return 0;
-  if (rk % 64 || rk < 64 || rk > 512 || rp % 8 || rp < 8 || rp > 128 || block_size < 8 || block_size % 8 || DEC_KEYS % block_size ||
+  if (rk % 64 || rk < 64 || rk > 512 || rc % 64 || rot < 1 || rot > rc || rc > 128 || block_size < 8 || block_size % 8 ||
       !(scale > 0.f) || num_splits < 1 || num_splits > 32 || H < 1 || max_q < 1 || (!cu_q && uniform_q < 1))
     return -3;
   if ((reinterpret_cast<uintptr_t>(q_abs) | reinterpret_cast<uintptr_t>(cache)) & 15) return -3;
@@ -722,13 +702,13 @@ int swb_latent_decode(const void* q_abs, const void* cache, int num_blocks, int 
   p.uniform_q = uniform_q, p.H = H, p.num_splits = num_splits, p.rows_total = T * H;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.part_o = part_o, p.part_ml = part_ml;
-  p.rk = rk, p.latent_atoms = rk / 64, p.pairs = (p.latent_atoms + 1) / 2, p.rot_atoms = (rp + 63) / 64, p.rot_steps = (rp + 15) / 16;
+  p.rk = rk, p.latent_atoms = rk / 64, p.pairs = (p.latent_atoms + 1) / 2, p.atoms = (rk + rc) / 64, p.rot_steps = (rot + 15) / 16;
   const int rows = max_q * H, nb = rows <= 16 ? 16 : 32;
   CUtensorMap tq, tk;
-  int rc = make_tmap_bf16_2d(&tq, q_abs, T * H, rk + rp, rk + rp, nb);
-  if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tk, cache, num_blocks * block_size, rk + rp, rk + rp, block_size);
-  if (rc) return rc;
+  int err = make_tmap_bf16_blocks(&tq, q_abs, T * H, rk + rc, rk + rc, nb);
+  if (err) return err;
+  err = make_tmap_bf16_blocks(&tk, cache, num_blocks * block_size, rk + rc, rk + rc, 8);
+  if (err) return err;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return nb == 16 ? launch_latent_decode<16>(tq, tk, p, n_seqs, rows, s) : launch_latent_decode<32>(tq, tk, p, n_seqs, rows, s);
 }

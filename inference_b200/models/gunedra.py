@@ -77,7 +77,7 @@ class GunedraGpu(StackDecoder):
         for i, lay in enumerate(self.stack.layers):
             if isinstance(lay.mixer, ChannelDeltaSpec) and ops.delta_key_width(lay.mixer.dim) is None:
                 raise Unsupported(f"layer {i}: key width {lay.mixer.dim} of the delta rule is above 512")
-            if isinstance(lay.mixer, LatentAttentionSpec) and self._latent_widths(lay.mixer)[2] + up8(lay.mixer.rot_dim) > 1024:
+            if isinstance(lay.mixer, LatentAttentionSpec) and ops.latent_width(self._latent_widths(lay.mixer)[2], lay.mixer.rot_dim) > 1024:
                 raise Unsupported(f"layer {i}: a cached row of {lay.mixer.kv_rank} + {lay.mixer.rot_dim} is above 1024")
         self.layers: list[_Layer] = []
 
@@ -92,8 +92,7 @@ class GunedraGpu(StackDecoder):
         for lay in self.stack.layers:
             m = lay.mixer
             if isinstance(m, LatentAttentionSpec):
-                _, rp, rk, _ = self._latent_widths(m)
-                out.append(LatentGeometry(rk + rp))
+                out.append(LatentGeometry(ops.latent_width(self._latent_widths(m)[2], m.rot_dim)))
             else:
                 dp, vp = ops.delta_key_width(m.dim), up8(m.vdim)
                 out.append(StateGeometry((m.heads, vp, dp), (m.conv - 1, 2 * m.kv_heads * dp + m.heads * vp)))
@@ -279,12 +278,12 @@ class GunedraGpu(StackDecoder):
         if many is not None:
             if cu_q is None:
                 cu_q = torch.arange(inp.num_seqs + 1, dtype=torch.int32, device=dev) * inp.max_q_len
-            rows = proj[:, w.col_c:w.col_c + w.width]
+            rows = proj[:, w.col_c:w.col_gate]
             if many.cu is not None:
                 rows = ops.latent_gather(cache, table, many.cu, many.keys, many.seqs)
                 self.launches += 1
             expanded = self._linear(rows[:, :w.rk], w.ukv)
-            ops.latent_prefill(proj[:, :w.col_c], expanded, rows[:, w.rk:], w, a.view(T, -1), cu_q=cu_q, max_q_len=many.max_q, gate=gate,
+            ops.latent_prefill(proj[:, :w.col_c], expanded, rows[:, w.rk:w.rk + w.rp], w, a.view(T, -1), cu_q=cu_q, max_q_len=many.max_q, gate=gate,
                                seqs=many.seqs, cu_k=many.cu)
             self.launches += 1
         if few is not None:

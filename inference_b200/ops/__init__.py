@@ -6,7 +6,7 @@ from .llm import (argmax, sample_device, embedding, gated_act_mul, gated_residua
                   spec_verify_greedy)
 from .delta import DeltaWeights, channel_delta, delta_key_width  # noqa: F401
 from .latent import (LatentWeights, SplitPartials, head_product, latent_attention_simple, latent_decode, latent_decode_supported,  # noqa: F401
-                     latent_gather, latent_prefill, latent_prefill_supported, latent_prep)
+                     latent_gather, latent_prefill, latent_prefill_supported, latent_prep, latent_width)
 from .moe import RoutingPlan, gemm_grouped_rows, routed_ffn, table_routing  # noqa: F401
 from .stream import Branch, DepthAverage, NormWeights, stream_embed, stream_norm  # noqa: F401
 from .runtime import KernelError, check_status, device_status  # noqa: F401

@@ -9,10 +9,16 @@ from .._native import kernels
 from .runtime import check, ptr, require_cuda, stream_ptr
 
 
+def latent_width(rk: int, rot: int) -> int:
+    """Columns of a cached row [c | k_rot] with its padding."""
+    return rk + (rot + 63) // 64 * 64
+
+
 @dataclass
 class LatentWeights:
     """Sizes and weights of one layer. Projection columns: q (heads x [dn | rp]), the latent (rk), the shared key part (rp), the
-    gate logits (heads). dn, rp, rk, vp are the padded dim, rot_dim, kv_rank and vdim; padding entries of the weights are zero.
+    gate logits (heads). dn, rp, rk, vp are the padded dim, rot_dim, kv_rank and vdim; in the cache the shared key part takes rc
+    columns (a multiple of 64, zero beyond rp); padding entries of the weights are zero.
     In the activation type: ukv [heads (dn + vp), rk], the rows of all heads' key projections and then of their value projections
     (uv is the latter part as [heads, vp, rk]), and the transposed key projections uk_t [heads, rk, dn]; norm fp32 [rk], sink fp32
     [heads]."""
@@ -45,7 +51,12 @@ class LatentWeights:
 
     @property
     def width(self) -> int:
-        return self.rk + self.rp
+        """Columns of a cached row."""
+        return self.rk + self.rc
+
+    @property
+    def rc(self) -> int:
+        return latent_width(self.rk, self.rot) - self.rk
 
 
 @dataclass
@@ -90,7 +101,7 @@ def head_product(a: torch.Tensor | SplitPartials, w: torch.Tensor, out: torch.Te
 
 def latent_decode_supported(w: LatentWeights, block_size: int) -> bool:
     """Whether the tcgen05 kernel covers the layer (others run on the plain kernel)."""
-    return w.rk <= 512 and w.rp <= 128 and w.scale > 0 and block_size % 8 == 0 and 128 % block_size == 0
+    return w.rk <= 512 and w.rc <= 128 and w.scale > 0 and block_size % 8 == 0
 
 
 def latent_decode(q_abs: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor, w: LatentWeights, *,
@@ -105,7 +116,7 @@ def latent_decode(q_abs: torch.Tensor, cache: torch.Tensor, block_table: torch.T
                          torch.empty((num_splits, T, H, 2), dtype=torch.float32, device=q_abs.device))
     rc = kernels().swb_latent_decode(q_abs.data_ptr(), cache.data_ptr(), cache.shape[0], cache.shape[1], block_table.data_ptr(),
                                      block_table.stride(0), ptr(cu_q), kv_lens.data_ptr(), kv_lens.numel(), max_q_len if cu_q is None else 0, max_q_len,
-                                     T, H, w.rk, w.rp, w.scale, num_splits, part.o.data_ptr(), part.ml.data_ptr(), stream_ptr())
+                                     T, H, w.rk, w.rc, w.rot, w.scale, num_splits, part.o.data_ptr(), part.ml.data_ptr(), stream_ptr())
     check(rc, "swb_latent_decode")
     return part
 
@@ -121,7 +132,7 @@ def latent_prep(proj: torch.Tensor, w: LatentWeights, eps: float, cos: torch.Ten
     assert slots.dtype == torch.int64 and positions.dtype == torch.int32 and cos.shape[-1] == w.rot // 2
     rc = kernels().swb_latent_prep(proj.data_ptr(), proj.stride(0), w.col_c, w.norm.data_ptr(), eps, cos.data_ptr(), sin.data_ptr(),
                                    positions.data_ptr(), slots.data_ptr(), cache.data_ptr(), ptr(q_abs), ptr(q_row), proj.shape[0], w.heads,
-                                   w.dn, w.rot, w.rp, w.rank, w.rk, 1 if proj.dtype == torch.float32 else 0, stream_ptr())
+                                   w.dn, w.rot, w.rp, w.rc, w.rank, w.rk, 1 if proj.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_latent_prep")
 
 
