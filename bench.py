@@ -189,15 +189,19 @@ def main() -> int:
     ap.add_argument("--no-extra", action="store_true", help="skip the TTFT / batch-1 / batch-8 side measurements")
     ap.add_argument("--no-dit", action="store_true", help="skip the DiT 1024x1024 seconds-per-image section")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library-collective (NCCL, unfused) arm")
-    ap.add_argument("--design", default=None, choices=["zobunex"],
+    ap.add_argument("--design", default=None, choices=["zobunex", "gunedra"],
                     help="instead of the headline workload: prefill / decode throughput and kernel rooflines of this design "
-                         "beside the sparse Llama-family decoder at equal size (see benchmarks/bench_zobunex.py)")
+                         "beside the closest Llama-family decoder at equal size (see benchmarks/bench_<design>.py)")
     args = ap.parse_args()
 
     if args.design == "zobunex":
         from benchmarks.bench_zobunex import main as bench_zobunex
 
         return bench_zobunex()
+    if args.design == "gunedra":
+        from benchmarks.bench_gunedra import main as bench_gunedra
+
+        return bench_gunedra()
     if args.impl == "reference":
         print(json.dumps(probe_reference()))
         return 0
