@@ -606,29 +606,35 @@ int swb_attn_paged_prefill_tc(const void* q, long long q_stride_tok, int q_strid
 // (heads contiguous), out [total_tokens, Hq, Dv]. chunk > 0: query i sees key j <= i only if floor(i / chunk) ==
 // floor(j / chunk), positions counted from the sequence's start. sink (nullable fp32 [Hq]): exp(sink[h]) joins the softmax
 // denominator. Widths: multiples of 8 up to 128. mode 0 = prefill (tcgen05 kernel, sequences from cu_q), 1 = decode
-// (TMA-fed kernel, block_size 16, max_q_len * Hq / Hkv <= 16, uniform q_len when cu_q is null). Returns -3 when the
-// problem is outside the two kernels' reach.
+// (TMA-fed kernel, block_size 16, max_q_len * Hq / Hkv <= 16, uniform q_len when cu_q is null). window > 0: query i sees only keys
+// j > i - window. diff (nullable) -> differential attention (DiffAttn): q [total_tokens, Hq, 2, D / 2], key rows of both maps side by
+// side, out [total_tokens, Hq, Dv] already combined; in decode 2 max_q_len * Hq / Hkv <= 16. Returns -3 when the problem is outside
+// the two kernels' reach.
 int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long k_stride_tok, const void* v,
                  long long v_stride_tok, void* out, long long out_stride_tok, const int* block_table, int max_blocks,
                  int block_size, int num_blocks, const int* cu_q, const int* kv_lens, int num_seqs, int max_q_len,
                  int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink, int mode,
-                 int num_splits, void* workspace, size_t workspace_bytes, void* stream) {
+                 int num_splits, void* workspace, size_t workspace_bytes, int window, int diff, float share, float diff_eps,
+                 float post, float cap, const float* q_temp, int v_count, void* stream) {
   using namespace swb;
   if (num_seqs <= 0 || total_tokens <= 0) return 0;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (Hkv <= 0 || Hq % Hkv != 0 || max_q_len <= 0) return -3;
+  if (Hkv <= 0 || Hq % Hkv != 0 || max_q_len <= 0 || window < 0) return -3;
+  if (diff && (D % 16 || v_count < 1 || v_count > Dv || sink || chunk || cap < 0.f)) return -3;
+  const attn::DiffAttn da{diff ? 2 : 0, D / 2, v_count, share, diff_eps, post, cap, q_temp};
   if (mode == 0)
     return attn_ext_tcgen05_launch(q, q_stride_tok, k, k_stride_tok, v, v_stride_tok, out, out_stride_tok, num_seqs,
                                    max_q_len, total_tokens, Hq, Hkv, D, Dv, scale, chunk, sink, cu_q, kv_lens,
-                                   block_table, max_blocks, block_size, num_blocks, st);
+                                   block_table, max_blocks, block_size, num_blocks, st, window, diff ? &da : nullptr);
+  const int per_kv = (diff ? 2 : 1) * (Hq / Hkv);
   if (D < 8 || Dv < 8 || D > HD || Dv > HD || (D % 8) || (Dv % 8) || block_size != 16 || !block_table || !kv_lens ||
-      num_blocks <= 0 || max_q_len * (Hq / Hkv) > 16 || !(scale > 0.f) || chunk < 0 || (q_stride_tok % 8))
+      num_blocks <= 0 || max_q_len * per_kv > 16 || !(scale > 0.f) || chunk < 0 || (q_stride_tok % 8))
     return -3;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -3;
   AttnParams p{};
   p.q = reinterpret_cast<const bf16*>(q);
   p.q_stride_tok = q_stride_tok;
-  p.q_stride_head = D;
+  p.q_stride_head = diff ? D / 2 : D;
   p.out = reinterpret_cast<bf16*>(out);
   p.out_stride_tok = out_stride_tok;
   p.k = reinterpret_cast<const bf16*>(k);
@@ -642,7 +648,9 @@ int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long
   p.num_seqs = num_seqs;
   p.Hq = Hq;
   p.Hkv = Hkv;
-  p.G = Hq / Hkv;
+  p.G = per_kv;
+  p.window = window;
+  p.diff = da;
   p.scale = scale;
   p.causal = 1;
   p.k_dim = D;

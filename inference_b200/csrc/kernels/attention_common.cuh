@@ -9,6 +9,15 @@ constexpr int HD = 128;
 constexpr int KV_TILE = 64;
 constexpr int TILE_BYTES = KV_TILE * HD * 2;  // 16 KB
 
+// Differential attention: every head has two softmax maps over the same values, o = a1 - share a2, normed over the head's n real
+// value columns and scaled by `post`. A key row holds both maps' parts of `dim` columns side by side; the queries of a head are two
+// rows of `dim` columns. Scores are capped (cap > 0: s <- cap tanh(s / cap)) after the factor q_temp[position] (optional).
+struct DiffAttn {
+  int maps, dim, n;      // maps: 2, or 0 for ordinary attention
+  float share, eps, post, cap;
+  const float* q_temp;
+};
+
 struct AttnParams {
   const bf16* q;
   long long q_stride_tok;
@@ -39,6 +48,8 @@ struct AttnParams {
   int k_dim, v_dim;      // head widths of q / k and of v / out (multiples of 8, <= HD)
   int chunk;             // > 0: a query sees only keys of its own chunk, floor(i / chunk) == floor(j / chunk)
   const float* sink;     // optional [Hq]: exp(sink[h]) joins the softmax denominator
+  int window;            // > 0: a query sees only the last `window` keys, its own included
+  DiffAttn diff;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, uint32_t src_bytes) {
@@ -94,10 +105,10 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
                             long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
                             int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
                             const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
-                            int num_blocks, cudaStream_t stream);
+                            int num_blocks, cudaStream_t stream, int window = 0, const attn::DiffAttn* diff = nullptr);
 int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok,
                                const void* k2, long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok,
                                int num_seqs, int max_q_len, int total_tokens, int H, int d1, int d2, int Dv, float scale,
                                const float* sink, const void* gate, long long gate_stride, const int* cu_q, const int* seqs,
-                               const int* cu_k, cudaStream_t stream);
+                               const int* cu_k, cudaStream_t stream, int window = 0);
 }  // namespace swb

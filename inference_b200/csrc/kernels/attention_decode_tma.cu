@@ -53,8 +53,25 @@ __device__ __forceinline__ float softmax_inv(const AttnParams& p, int head, floa
   return L > 0.f ? 1.f / L : 0.f;
 }
 
-// EXT: chunked masking and sinks. FULL: q / k and v are HD wide (their loop bounds are then constants).
-template <bool EXT, bool FULL>
+// Sums of up to eight values per thread over the 128 merging threads (warps 0-3); `red` holds 32 floats.
+__device__ __forceinline__ void sum_over_128(float* v, float* red, int n) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    if (i >= n) break;
+    v[i] = warp_sum(v[i]);
+    if (lane == 0) red[i * 4 + warp] = v[i];
+  }
+  asm volatile("bar.sync 1, 128;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (i < n) v[i] = (red[i * 4] + red[i * 4 + 1]) + (red[i * 4 + 2] + red[i * 4 + 3]);
+}
+
+// EXT: chunked and windowed masking, sinks. FULL: q / k and v are HD wide (their loop bounds are then constants). DIFF: the two maps
+// of a head are neighbouring query rows, each zero outside its own columns of the key row, so that both maps' scores come from one
+// product; the merge subtracts the second map and norms the difference.
+template <bool EXT, bool FULL, bool DIFF>
 __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                               const __grid_constant__ CUtensorMap tmap_v,
                                                               const AttnParams p) {
@@ -68,6 +85,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   uint64_t* bar_empty = bar_full + STAGES;
   volatile int* s_abort = reinterpret_cast<volatile int*>(bar_empty + STAGES);
   float* sMerge = reinterpret_cast<float*>(ring);        // reused after the loop (33 KB)
+  float* sRed = sMerge + STAGES * STAGE_BYTES / 4 - 32;  // DIFF: 32 floats behind it
 
   const int split = blockIdx.x;
   const int kvh = blockIdx.y;
@@ -92,7 +110,8 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   const int nrows = min(16, q_len * p.G);
   const int causal_shift = kv_len - q_len;
   // chunked attention starts at the tile that holds the first key of the first query's chunk
-  const int tile_lo = (EXT && p.chunk > 0) ? max(causal_shift, 0) / p.chunk * p.chunk / KV_TILE : 0;
+  int tile_lo = (EXT && p.chunk > 0) ? max(causal_shift, 0) / p.chunk * p.chunk / KV_TILE : 0;
+  if (EXT && p.window > 0) tile_lo = max(tile_lo, max(causal_shift - p.window + 1, 0) / KV_TILE);
   const int total_tiles = (kv_len + KV_TILE - 1) / KV_TILE;
   const int per = (total_tiles - tile_lo + p.num_splits - 1) / p.num_splits;
   const int t0 = tile_lo + split * per;
@@ -105,10 +124,11 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   for (int idx = threadIdx.x; idx < 256; idx += blockDim.x) {
     const int row = idx >> 4, c = idx & 15;
     uint4 val = make_uint4(0, 0, 0, 0);
-    if (row < nrows && c * 8 < k_dim) {
-      const int qtok = row / p.G, hg = row % p.G;
+    const int qtok = row / p.G, hg = row % p.G;
+    const int c0 = DIFF ? c * 8 - (hg & 1) * p.diff.dim : c * 8;          // column within the head's q row
+    if (row < nrows && c0 >= 0 && c0 < (DIFF ? p.diff.dim : k_dim)) {
       val = *reinterpret_cast<const uint4*>(p.q + (size_t)(q_start + qtok) * p.q_stride_tok +
-                                            (size_t)(kvh * p.G + hg) * p.q_stride_head + c * 8);
+                                            (size_t)(kvh * p.G + hg) * p.q_stride_head + c0);
     }
     *reinterpret_cast<uint4*>(sQp + q_off(row, c)) = val;
   }
@@ -173,6 +193,11 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     }
     int stage = 0;
     uint32_t phase = 0;
+    float row_scale[2] = {p.scale, p.scale};
+    if (DIFF && p.diff.q_temp) {
+#pragma unroll
+      for (int hr = 0; hr < 2; ++hr) row_scale[hr] *= p.diff.q_temp[min((g + hr * 8) / p.G, q_len - 1) + max(causal_shift, 0)];
+    }
     for (int j = 0; j < n_tiles; ++j) {
       if (!mbar_wait(&bar_full[stage], phase, s_abort, 600 + stage)) break;
       const uint32_t sK = smem_u32(ring + stage * STAGE_BYTES);
@@ -195,13 +220,13 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float val = score_transform(s[nt][e], p.scale, p.softcap);
+          const float val = DIFF ? score_transform(s[nt][e], row_scale[e >> 1], p.diff.cap) : score_transform(s[nt][e], p.scale, p.softcap);
           const int col = tok_base + nt * 8 + t4 * 2 + (e & 1);
           const int row = g + ((e >> 1) ? 8 : 0);
           const int qtok = row / p.G;
           const int qpos = qtok + causal_shift;
           const bool ok = (col < kv_len) && (!p.causal || col <= qpos) &&
-                          (!EXT || p.chunk <= 0 || col >= qpos / p.chunk * p.chunk);
+                          (!EXT || ((p.chunk <= 0 || col >= qpos / p.chunk * p.chunk) && (p.window <= 0 || col > qpos - p.window)));
           s[nt][e] = ok ? val : -INFINITY;
         }
       }
@@ -279,6 +304,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     }
   }
   __syncthreads();
+  float keep[8];                           // DIFF: differences of the row pairs
   if (threadIdx.x < 128) {
     const int d = threadIdx.x;
     for (int row = 0; row < nrows; ++row) {
@@ -296,7 +322,9 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       const int qtok = row / p.G, hg = row % p.G;
       if (p.num_splits == 1) {
         const float inv = softmax_inv<EXT>(p, kvh * p.G + hg, M, L);
-        if (d < v_dim)
+        if (DIFF) {
+          sMerge[row * HD + d] = acc * inv;      // warp 0's partial of this row and column, read by this thread alone
+        } else if (d < v_dim)
           p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] =
               __float2bfloat16(acc * inv);
       } else {
@@ -308,6 +336,27 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         }
       }
     }
+  }
+  auto store_pairs = [&](const float* at) {      // at [nrows, HD]: normalised outputs of the two maps of every pair of rows
+    const int d = threadIdx.x, pairs = nrows / 2;
+    float ss[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      keep[i] = i < pairs && d < v_dim ? at[2 * i * HD + d] - p.diff.share * at[(2 * i + 1) * HD + d] : 0.f;
+      ss[i] = keep[i] * keep[i];
+    }
+    sum_over_128(ss, sRed, pairs);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (i >= pairs || d >= v_dim) continue;
+      const int qtok = 2 * i / p.G, hg = 2 * i % p.G;
+      p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)((kvh * p.G + hg) / 2) * v_dim + d] =
+          __float2bfloat16(keep[i] * rsqrtf(ss[i] / (float)p.diff.n + p.diff.eps) * p.diff.post);
+    }
+  };
+  if (DIFF && p.num_splits == 1) {
+    if (threadIdx.x < 128) store_pairs(sMerge);
+    return;
   }
   if (p.num_splits > 1 && p.split_counters) {
     // Merge of the splits inside this launch. Cluster launch (the splits of a (sequence, kv head) form one
@@ -340,7 +389,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     }
     // the partial outputs do not depend on the weights: request them now (up to 4 rows x 8 splits stay in registers)
     float po[4][8];
-    const bool small = nrows <= 4 && S <= 8 && threadIdx.x < 128;
+    const bool small = !DIFF && nrows <= 4 && S <= 8 && threadIdx.x < 128;
     if (small) {
 #pragma unroll
       for (int row = 0; row < 4; ++row)
@@ -365,7 +414,19 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       for (int sp = 0; sp < S; ++sp) sSc[row * 32 + sp] *= inv;
     }
     __syncthreads();
-    if ((int)threadIdx.x < v_dim) {
+    if constexpr (DIFF) {
+      if (threadIdx.x < 128) {
+        float* at = sMerge + 2 * 16 * 32;
+        const int d = threadIdx.x;
+        for (int row = 0; row < nrows; ++row) {
+          float acc = 0.f;
+#pragma unroll 8
+          for (int sp = 0; sp < S; ++sp) acc += sSc[row * 32 + sp] * __ldcg(p.part_o + (base0 + (size_t)sp * 16 + row) * HD + d);
+          at[row * HD + d] = acc;
+        }
+        store_pairs(at);
+      }
+    } else if ((int)threadIdx.x < v_dim) {
       const int d = threadIdx.x;
       if (small) {
 #pragma unroll
@@ -398,11 +459,14 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 
 // Launches the TMA decode kernel; kcache / vcache are one layer's [blocks, Hkv, 16, 128] tensors.
 int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t stream) {
-  const bool ext = p.chunk > 0 || p.sink != nullptr, full = p.k_dim == HD && p.v_dim == HD;
-  const int which = full ? (ext ? 1 : 0) : 2;
-  auto kernel = which == 0 ? attn_decode_tma_kernel<false, true>
-                           : which == 1 ? attn_decode_tma_kernel<true, true> : attn_decode_tma_kernel<true, false>;
-  static bool configured[3][64] = {};
+  const bool ext = p.chunk > 0 || p.sink != nullptr || p.window > 0, full = p.k_dim == HD && p.v_dim == HD;
+  const int which = p.diff.maps ? (full ? 3 : 4) : full ? (ext ? 1 : 0) : 2;
+  auto kernel = which == 0   ? attn_decode_tma_kernel<false, true, false>
+                : which == 1 ? attn_decode_tma_kernel<true, true, false>
+                : which == 2 ? attn_decode_tma_kernel<true, false, false>
+                : which == 3 ? attn_decode_tma_kernel<true, true, true>
+                             : attn_decode_tma_kernel<true, false, true>;
+  static bool configured[5][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[which][dev]) {

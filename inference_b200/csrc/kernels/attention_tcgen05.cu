@@ -80,7 +80,9 @@ struct FaParams {
   // Extended problems (the EXT instantiations only):
   int chunk;           // > 0: query i sees key j <= i only if floor(i / chunk) == floor(j / chunk), positions of the sequence
   const float* sink;   // optional [Hq]: exp(sink[h]) joins the softmax denominator (no key, no value, not scaled)
+  int window;          // > 0: query i sees only keys j > i - window
   int v_dim;           // width of the v heads and of the output heads (<= VD; the tile is zero filled beyond it)
+  attn::DiffAttn diff; // DIFF only
   // Latent attention (LAT): q and k in two parts, k's second part shared by the heads; keys and values are rows
   // [cu_k[z], cu_k[z + 1]) of one flat axis (null: those of the queries), the queries the last positions of them.
   const int* seqs;     // optional: sequence of blockIdx.z (cu_q is indexed by it, cu_k by blockIdx.z)
@@ -154,6 +156,11 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&h);
@@ -172,9 +179,12 @@ struct Barriers {
 
 // 168 registers per thread is the cap for ten warps: two of the four scheduler partitions hold three warps, and a
 // partition's file is 16 K registers (a build with 200 registers per thread does not launch).
-// EXT adds chunked masking, attention sinks and head widths below the tile widths (q . k and P V then run over zero
+// EXT adds chunked and windowed masking, attention sinks and head widths below the tile widths (q . k and P V then run over zero
 // columns that the tensor maps fill in). LAT adds what latent attention needs: two-part q / k, key ranges, output gates.
-template <int QK, int VD, bool EXT, bool LAT>
+// DIFF is differential attention: the two tiles of a CTA are the two softmax maps of the same 128 query rows. Each map's keys are
+// one 64-column atom of the K tile (columns of the other map that fall into it meet zero columns of q), the V tile serves both, and
+// the second map's result is handed to the first one's threads through shared memory for the difference and its norm.
+template <int QK, int VD, bool EXT, bool LAT, bool DIFF>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_q2,
@@ -187,7 +197,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   Barriers* bars = reinterpret_cast<Barriers*>(smem + SMEM_BAR);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int q_base = blockIdx.x * (p.tiles * BM);
+  constexpr int TILE_STEP = DIFF ? 0 : BM;                  // query rows between the two tiles of a CTA
+  const int cta_rows = DIFF ? BM : p.tiles * BM;
+  const int q_base = blockIdx.x * cta_rows;
   const int head = blockIdx.y;
   // packed variable-length batch: this CTA's sequence covers tokens [tok0, tok0 + q_len) of one flat token axis
   const int seq = (LAT && p.seqs) ? p.seqs[blockIdx.z] : blockIdx.z;
@@ -200,9 +212,14 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   const int batch = p.cu_q ? 0 : blockIdx.z;
   if (q_base >= q_len || kv_len <= 0) return;   // uniform for the whole CTA, before any barrier or TMEM allocation
   const int kv_head = head / (p.Hq / p.Hkv);
-  const int kv_end = p.causal ? min(kv_len, q_base + p.tiles * BM + coff) : kv_len;
-  // first key tile that any row of this CTA sees (rows are ascending, so the first row's chunk starts lowest)
-  const int j0 = (EXT && p.chunk > 0) ? (q_base + coff) / p.chunk * p.chunk / BN : 0;
+  const int kv_end = p.causal ? min(kv_len, q_base + cta_rows + coff) : kv_len;
+  // first key that a row sees, and first key tile that any row of this CTA sees (rows are ascending, so the first row's is lowest)
+  auto first_key_of = [&](int pos) {
+    int first = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+    if (p.window > 0) first = max(first, pos - p.window + 1);
+    return first;
+  };
+  const int j0 = EXT ? first_key_of(q_base + coff) / BN : 0;
   const int n_tiles = (kv_end + BN - 1) / BN - j0;
   volatile int* abort_flag = &bars->abort;
 
@@ -245,9 +262,13 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   if (warp == 8) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
-      mbar_arrive_expect_tx(&bars->q_full, p.tiles * TILE_BYTES);
+      mbar_arrive_expect_tx(&bars->q_full, DIFF ? 2 * ATOM_BYTES : p.tiles * TILE_BYTES);
       for (int q = 0; q < p.tiles; ++q)
-        for (int a = 0; a < ATOMS; ++a) {
+        for (int a = 0; a < (DIFF ? 1 : ATOMS); ++a) {
+          if constexpr (DIFF) {
+            tma_load_4d(smem + SMEM_Q + q * TILE_BYTES, &tmap_q, &bars->q_full, 0, 2 * head + q, tok0 + q_base, batch);
+            continue;
+          }
           const bool second = LAT && a >= p.first_atoms;
           tma_load_4d(smem + SMEM_Q + q * TILE_BYTES + a * ATOM_BYTES, second ? &tmap_q2 : &tmap_q, &bars->q_full,
                       (second ? a - p.first_atoms : a) * 64, head, tok0 + q_base + q * BM, batch);
@@ -261,19 +282,20 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const uint32_t page_bytes = paged ? (uint32_t)p.block_size * 128u : 0u;
       auto load_tile = [&](uint32_t dst_off, const CUtensorMap* map, uint64_t* bar, int jrel, int atoms, bool is_k) {
         const int j = jrel + j0;
+        const int atom_cols = DIFF && is_k ? p.diff.dim : 64;        // DIFF: each map's keys start an atom
         if (!paged) {
           for (int a = 0; a < atoms; ++a) {
             if (LAT && is_k && a >= p.first_atoms)
               tma_load_4d(smem + dst_off + a * ATOM_BYTES, &tmap_k2, bar, (a - p.first_atoms) * 64, 0, key0_row + j * BN, batch);
             else
-              tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * 64, kv_head, key0_row + j * BN, batch);
+              tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * atom_cols, kv_head, key0_row + j * BN, batch);
           }
           return;
         }
         for (int g = 0; g < per_tile; ++g) {
           const int page = pages[min(j * per_tile + g, last_page)];
           for (int a = 0; a < atoms; ++a)
-            tma_load_4d(smem + dst_off + a * ATOM_BYTES + g * page_bytes, map, bar, a * 64, 0, kv_head, page);
+            tma_load_4d(smem + dst_off + a * ATOM_BYTES + g * page_bytes, map, bar, a * atom_cols, 0, kv_head, page);
         }
       };
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -308,6 +330,13 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const uint32_t q_addr = smem_u32(smem + SMEM_Q), k_addr = smem_u32(smem + SMEM_K),
                      v_addr = smem_u32(smem + SMEM_V);
       auto issue_qk = [&](int q, int s) {
+        if constexpr (DIFF) {
+          for (int k = 0; k < (p.diff.dim + 15) / 16; ++k)
+            umma_f16_ss(tmem + col_s[q], umma_desc_kmajor_sw128(q_addr + q * TILE_BYTES + k * 32),
+                        umma_desc_kmajor_sw128(k_addr + s * TILE_BYTES + q * ATOM_BYTES + k * 32), IDESC_QK, k > 0);
+          umma_commit(&bars->s_full[q]);
+          return;
+        }
 #pragma unroll
         for (int k = 0; k < QK / 16; ++k) {
           const uint32_t off = (k >> 2) * ATOM_BYTES + (k & 3) * 32;
@@ -358,7 +387,14 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t t_s = tmem + lane_base + (q ? COL_S1 : COL_S0);
     const uint32_t t_o = tmem + lane_base + (q ? COL_O1 : COL_O0);
-    const int row = q_base + q * BM + (warp & 3) * 32 + lane;
+    const int row = q_base + q * TILE_STEP + (warp & 3) * 32 + lane;
+    const float cap = DIFF ? p.diff.cap : 0.f;
+    float to_cap = 0.f;             // 2 log2(e) scale / cap: the capped score is cap (1 - 2 / (2^(to_cap s) + 1))
+    float scale_log2 = p.scale_log2;
+    if constexpr (DIFF) {
+      if (p.diff.q_temp && row < q_len) scale_log2 *= p.diff.q_temp[row + coff];
+      if (cap > 0.f) to_cap = 2.f * scale_log2 / cap, scale_log2 = 1.4426950408889634f;
+    }
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < my_tiles; ++j) {
@@ -369,18 +405,23 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) tmem_ld_x32(t_s + c * 32, s + c * 32);
       tmem_ld_wait();
+      if (DIFF && cap > 0.f) {
+#pragma unroll
+        for (int i = 0; i < BN; ++i)
+          s[i] = __float_as_uint(fmaf(-2.f * cap, rcp_approx(ex2(__uint_as_float(s[i]) * to_cap) + 1.f), cap));
+      }
       // keys past the sequence (zero fill, or the next sequence of a packed batch) and, when causal, keys after the
       // query position never contribute
       const int key0 = (j + j0) * BN;
-      if (key0 + BN > kv_len || (p.causal && key0 + BN > q_base + q * BM + coff)) {
+      if (key0 + BN > kv_len || (p.causal && key0 + BN > q_base + q * TILE_STEP + coff)) {
         const int last_key = p.causal ? min(kv_len - 1, row + coff) : kv_len - 1;
 #pragma unroll
         for (int i = 0; i < BN; ++i)
           if (key0 + i > last_key) s[i] = __float_as_uint(-INFINITY);
       }
-      if constexpr (EXT) {   // keys of earlier chunks; only tiles below the last row's chunk start can hold any
-        if (p.chunk > 0 && key0 < (q_base + q * BM + BM - 1 + coff) / p.chunk * p.chunk) {
-          const int first_key = (row + coff) / p.chunk * p.chunk;
+      if constexpr (EXT) {   // keys in front of the chunk or window; only tiles below the last row's first key can hold any
+        if (key0 < first_key_of(q_base + q * TILE_STEP + BM - 1 + coff)) {
+          const int first_key = first_key_of(row + coff);
 #pragma unroll
           for (int i = 0; i < BN; ++i)
             if (key0 + i < first_key) s[i] = __float_as_uint(-INFINITY);
@@ -395,9 +436,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         mx3 = fmaxf(mx3, __uint_as_float(s[i + 3]));
       }
       const float m_new = fmaxf(fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)), m_used);
-      const bool grow = (m_new - m_used) * p.scale_log2 > RESCALE_THRESHOLD;   // true on the first tile (m_used = -inf)
+      const bool grow = (m_new - m_used) * scale_log2 > RESCALE_THRESHOLD;   // true on the first tile (m_used = -inf)
       if (__any_sync(0xffffffffu, grow)) {
-        const float f = grow ? ex2((m_used - m_new) * p.scale_log2) : 1.f;      // -inf -> 0 on the first tile
+        const float f = grow ? ex2((m_used - m_new) * scale_log2) : 1.f;      // -inf -> 0 on the first tile
         if (grow) {
           l *= f;
           m_used = m_new;
@@ -415,15 +456,15 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
       }
       // a row whose chunk starts beyond this tile has seen no key yet: its exponentials are all zero
-      const float neg_m = (EXT && m_used == -INFINITY) ? 0.f : -m_used * p.scale_log2;
+      const float neg_m = (EXT && m_used == -INFINITY) ? 0.f : -m_used * scale_log2;
       float l0 = 0.f, l1 = 0.f;
       // (Measured alternatives for this loop, all slower on B200: every 4th / 2nd exponential as a cubic on the FMA pipe
       // -8 % / -17 %; pairs of exponentials as one bf16x2 special-function operation -6 %; three-input max with
       // two-lane fp32 multiply-add and add -30 %, from register-pair moves and spills. The loop is issue-bound.)
 #pragma unroll
       for (int i = 0; i < BN; i += 2) {   // packed P overwrites the row in place (index i/2 <= i)
-        const float e0 = ex2(fmaf(__uint_as_float(s[i]), p.scale_log2, neg_m));
-        const float e1 = ex2(fmaf(__uint_as_float(s[i + 1]), p.scale_log2, neg_m));
+        const float e0 = ex2(fmaf(__uint_as_float(s[i]), scale_log2, neg_m));
+        const float e1 = ex2(fmaf(__uint_as_float(s[i + 1]), scale_log2, neg_m));
         l0 += e0;
         l1 += e1;
         s[i >> 1] = pack_bf16x2(e0, e1);
@@ -436,12 +477,13 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       mbar_arrive(&bars->p_full[q]);
     }
     if (ok && my_tiles > 0) ok = mbar_wait(&bars->o_final, 0, abort_flag, 32 + q);
+    if constexpr (DIFF) ok = __all_sync(0xffffffffu, ok);      // the barrier below is taken warp by warp
     if (ok && my_tiles > 0) {
       tc_fence_after_sync();
       float inv = l > 0.f ? 1.f / l : 0.f;
       if constexpr (EXT) {
         if (p.sink) {   // join the sink in a frame whose largest exponent is zero
-          const float sk = p.sink[head] * 1.4426950408889634f, mm = m_used * p.scale_log2;
+          const float sk = p.sink[head] * 1.4426950408889634f, mm = m_used * scale_log2;
           const float top = fmaxf(sk, mm), e = ex2(mm - top);
           inv = e / (l * e + ex2(sk - top));
         }
@@ -456,8 +498,44 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       // VD / 8 lanes x 16 bytes: contiguous runs for local stores and for stores that cross NVLink alike.
       // 16-byte chunk c of row r sits at c ^ (r & 7).
       uint8_t* slab = smem + SMEM_Q + warp * (32 * ROW_BYTES);
+      if constexpr (DIFF) {
+        // fp32 hand-over in the (idle) K region, row r of VD numbers, 16-byte chunk c at c ^ (r & 31 within the row's chunks)
+        float4* hand = reinterpret_cast<float4*>(smem + SMEM_K) + (size_t)((warp & 3) * 32 + lane) * (VD / 4);
+        const float f = q ? inv * p.diff.share : inv;
+        float ss = 0.f;
+        if (q == 0) asm volatile("bar.sync 1, 256;" ::: "memory");
 #pragma unroll
-      for (int c = 0; c < VD / 32; ++c) {
+        for (int c = 0; c < VD / 32; ++c) {
+          uint32_t o[32];
+          tmem_ld_x32(t_o + c * 32, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int v = 0; v < 8; ++v) {
+            float4* at = hand + ((c * 8 + v) ^ (lane & (VD / 4 - 1)));
+            float4 x = make_float4(__uint_as_float(o[v * 4]) * f, __uint_as_float(o[v * 4 + 1]) * f, __uint_as_float(o[v * 4 + 2]) * f,
+                                   __uint_as_float(o[v * 4 + 3]) * f);
+            if (q == 0) {
+              const float4 y = *at;
+              x.x -= y.x, x.y -= y.y, x.z -= y.z, x.w -= y.w;
+              ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);      // columns past v_dim are zero in both maps
+            }
+            *at = x;
+          }
+        }
+        if (q == 0) {
+          const float r = rsqrtf(ss / (float)p.diff.n + p.diff.eps) * p.diff.post;
+#pragma unroll
+          for (int c = 0; c < VD / 8; ++c) {
+            const float4 x = hand[(2 * c) ^ (lane & (VD / 4 - 1))], y = hand[(2 * c + 1) ^ (lane & (VD / 4 - 1))];
+            uint4 u;
+            u.x = pack_bf16x2(x.x * r, x.y * r), u.y = pack_bf16x2(x.z * r, x.w * r);
+            u.z = pack_bf16x2(y.x * r, y.y * r), u.w = pack_bf16x2(y.z * r, y.w * r);
+            *reinterpret_cast<uint4*>(slab + lane * ROW_BYTES + ((c ^ (lane & 7)) << 4)) = u;
+          }
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < (DIFF ? 0 : VD / 32); ++c) {
         uint32_t o[32];
         tmem_ld_x32(t_o + c * 32, o);
         tmem_ld_wait();
@@ -472,9 +550,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
       }
       __syncwarp();
-      const int row0 = q_base + q * BM + (warp & 3) * 32;
+      const int row0 = q_base + q * TILE_STEP + (warp & 3) * 32;
 #pragma unroll 4
-      for (int it = 0; it < CHUNKS; ++it) {            // CHUNKS lanes write one row: 32 / CHUNKS rows per pass
+      for (int it = 0; it < (DIFF && q ? 0 : CHUNKS); ++it) {            // CHUNKS lanes write one row: 32 / CHUNKS rows per pass
         const int r = (32 / CHUNKS) * it + lane / CHUNKS, ch = lane % CHUNKS;
         const int grow = row0 + r;
         if (grow < q_len) {
@@ -492,6 +570,9 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
           *reinterpret_cast<uint4*>(dst + ch * 8) = val;
         }
       }
+    }
+    if constexpr (DIFF) {          // the hand-over barrier takes all 256 threads, whatever became of the waits
+      if (q == 1 || !ok) asm volatile("bar.sync 1, 256;" ::: "memory");
     }
   }
   tc_fence_before_sync();
@@ -586,10 +667,10 @@ struct FaMaps {
   CUtensorMap q, k, v, q2, k2;     // q2 / k2: second parts of latent attention
 };
 
-template <int QK, int VD, bool EXT, bool LAT>
+template <int QK, int VD, bool EXT, bool LAT, bool DIFF = false>
 int launch_fa(dim3 grid, cudaStream_t stream, const FaMaps& m, const FaParams& p) {
   static bool configured[64] = {false};
-  auto kernel = attn_dense_tcgen05_kernel<QK, VD, EXT, LAT>;
+  auto kernel = attn_dense_tcgen05_kernel<QK, VD, EXT, LAT, DIFF>;
   constexpr size_t SMEM = FaCfg<QK, VD>::SMEM_BYTES;
   int dev = 0;
   cudaGetDevice(&dev);
@@ -601,11 +682,15 @@ int launch_fa(dim3 grid, cudaStream_t stream, const FaMaps& m, const FaParams& p
   return launch_kernel(kernel, grid, dim3(THREADS), SMEM, stream, m.q, m.k, m.v, m.q2, m.k2, p);
 }
 
-enum class FaKind { DENSE, EXT, LATENT };
+enum class FaKind { DENSE, EXT, LATENT, DIFF };
 
 // qk: tile width of q and k
 int launch_tiles(int qk, FaKind kind, int q_len, int Hq, int batch, cudaStream_t stream, const FaMaps& m, FaParams& p) {
   // one-tile CTAs when that shortens the schedule: a one-tile CTA takes ~0.85 of a two-tile CTA's time (measured)
+  if (kind == FaKind::DIFF) {
+    p.tiles = 2;
+    return launch_fa<128, 128, true, false, true>(dim3((q_len + BM - 1) / BM, Hq, batch), stream, m, p);
+  }
   const int sms = 148;
   const long c2 = (long)((q_len + 2 * BM - 1) / (2 * BM)) * Hq * batch, c1 = (long)((q_len + BM - 1) / BM) * Hq * batch;
   const double t2 = (double)((c2 + sms - 1) / sms), t1 = 0.85 * (double)((c1 + sms - 1) / sms);
@@ -688,8 +773,9 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
                             long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
                             int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
                             const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
-                            int num_blocks, cudaStream_t stream) {
+                            int num_blocks, cudaStream_t stream, int window, const attn::DiffAttn* diff) {
   const bool paged = block_table != nullptr;
+  if (window < 0 || (diff && (sink || chunk || D % 16))) return -3;
   if (D < 8 || Dv < 8 || D > 128 || Dv > 128 || (D % 8) || (Dv % 8) || !cu_q || Hq % Hkv || !(scale > 0.f) || chunk < 0) return -3;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
        reinterpret_cast<uintptr_t>(out)) & 15)
@@ -699,7 +785,8 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
             : ((k_stride_tok | v_stride_tok) % 8 != 0))
     return -3;
   FaMaps m{};
-  int rc = make_tmap_heads(&m.q, q, D, Hq, total_tokens, 1, D, q_stride_tok, q_stride_tok * total_tokens);
+  int rc = diff ? make_tmap_heads(&m.q, q, D / 2, 2 * Hq, total_tokens, 1, D / 2, q_stride_tok, q_stride_tok * total_tokens)
+                : make_tmap_heads(&m.q, q, D, Hq, total_tokens, 1, D, q_stride_tok, q_stride_tok * total_tokens);
   if (rc) return rc;
   rc = make_tmap_heads(&m.k, k, D, Hkv, total_tokens, paged ? num_blocks : 1, D, k_stride_tok, k_stride_tok * total_tokens,
                        paged ? block_size : 0);
@@ -721,7 +808,12 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
   p.block_size = block_size;
   p.chunk = chunk;
   p.sink = sink;
+  p.window = window;
   p.v_dim = Dv;
+  if (diff) {
+    p.diff = *diff;
+    return launch_tiles(128, FaKind::DIFF, max_q_len, Hq, num_seqs, stream, m, p);
+  }
   return launch_tiles(D > 64 || Dv > 64 ? 128 : 64, FaKind::EXT, max_q_len, Hq, num_seqs, stream, m, p);
 }
 
@@ -733,7 +825,8 @@ int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void
                                const void* k2, long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok,
                                int num_seqs, int max_q_len, int total_tokens, int H, int d1, int d2, int Dv, float scale,
                                const float* sink, const void* gate, long long gate_stride, const int* cu_q, const int* seqs,
-                               const int* cu_k, cudaStream_t stream) {
+                               const int* cu_k, cudaStream_t stream, int window) {
+  if (window < 0) return -3;
   if (d1 < 8 || d2 < 8 || Dv < 8 || d1 > 128 || d2 > 64 || Dv > 128 || ((d1 | d2 | Dv) % 8) || !cu_q || !(scale > 0.f)) return -3;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
        reinterpret_cast<uintptr_t>(k2) | reinterpret_cast<uintptr_t>(out)) & 15)
@@ -755,6 +848,7 @@ int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void
   p.causal = 1;
   p.cu_q = cu_q;
   p.sink = sink;
+  p.window = window;
   p.v_dim = Dv;
   p.seqs = seqs;
   p.cu_k = cu_k;

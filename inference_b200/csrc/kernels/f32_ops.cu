@@ -12,10 +12,11 @@ namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16;
 
-// out[r, n] = act(sum_k a[src ? src[r] : r, k] w[e, n, k]); 64 x 64 tile, 4 x 4 per thread. Grouped: blockIdx.z = expert.
+// out[r, n] = act(sum_k a[src ? src[r] : r, k] w[e, n, k] + bias[n]); 64 x 64 tile, 4 x 4 per thread. Grouped: blockIdx.z = expert.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ a, int lda, const int* __restrict__ src,
                                                        const int* __restrict__ offsets, const float* __restrict__ w, int ldw,
-                                                       float* out, int ldo, int T, int N, int K, int act) {
+                                                       float* out, int ldo, int T, int N, int K, int act,
+                                                       const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float sa[TK][TM + 4], sw[TK][TN + 4];
@@ -58,6 +59,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float v = acc[i][j];
+      if (bias) v += bias[n];
       if (act == SWB_ACT_RELU2) v = relu2_f(v);
       else if (act == SWB_ACT_SILU) v = silu_f(v);
       else if (act == SWB_ACT_GELU_TANH) v = gelu_tanh_f(v);
@@ -69,52 +71,68 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 constexpr int AW = 4;          // warps per CTA: keys are dealt out to them
 constexpr int MAX_PER_LANE = 32;   // head widths up to 1024
 
+// What a query sees and how its scores are formed, beyond scale and causality.
+struct SimpleAttnParams {
+  long long q_stride_tok, out_stride_tok;
+  const int* block_table;
+  int max_blocks, block_size;
+  const int *cu_q, *kv_lens;
+  int num_seqs, uniform_q, Hq, Hkv, D, Dv;
+  int k_row, v_row;          // elements between the key / value rows of consecutive tokens of a page
+  float scale;
+  int chunk;                 // > 0: only keys of the query's own run of `chunk` positions
+  int window;                // > 0: only the last `window` keys, the query's own included
+  float softcap;             // > 0: score <- softcap tanh(score / softcap)
+  const float* q_temp;       // optional, by position: factor of the scores in front of the cap
+  const float* sink;
+  int maps;                  // query heads h, h + 1, ... take turns on `maps` key parts of D columns each within a key row
+};
+
 // One CTA per (query token, head). Each warp runs an online softmax over its share of the visible keys; lanes split the
 // head dimension. The sink joins the denominator when the four partial results are merged.
 template <typename E, int PL>
-__global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restrict__ q, long long q_stride_tok,
-                                                              const E* __restrict__ kc, const E* __restrict__ vc, E* out,
-                                                              long long out_stride_tok, const int* __restrict__ block_table,
-                                                              int max_blocks, int block_size, const int* __restrict__ cu_q,
-                                                              const int* __restrict__ kv_lens, int num_seqs, int uniform_q,
-                                                              int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
-                                                              const float* __restrict__ sink) {
+__global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restrict__ q, const E* __restrict__ kc, const E* __restrict__ vc,
+                                                              E* out, const SimpleAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, head = blockIdx.y, kvh = head / (Hq / Hkv);
+  const int t = blockIdx.x, head = blockIdx.y, kvh = head / (p.Hq / p.Hkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int seq = seq_of_token(cu_q, num_seqs, uniform_q, t);
-  const int q0 = cu_q ? cu_q[seq] : seq * uniform_q, q_len = cu_q ? cu_q[seq + 1] - q0 : uniform_q;
-  const int pos = kv_lens[seq] - q_len + (t - q0);
-  const int first = chunk > 0 ? pos / chunk * chunk : 0;
-  const int* table = block_table + (size_t)seq * max_blocks;
-  const E* qr = q + (size_t)t * q_stride_tok + (size_t)head * D;
+  const int seq = seq_of_token(p.cu_q, p.num_seqs, p.uniform_q, t);
+  const int q0 = p.cu_q ? p.cu_q[seq] : seq * p.uniform_q, q_len = p.cu_q ? p.cu_q[seq + 1] - q0 : p.uniform_q;
+  const int pos = p.kv_lens[seq] - q_len + (t - q0);
+  int first = p.chunk > 0 ? pos / p.chunk * p.chunk : 0;
+  if (p.window > 0) first = max(first, pos - p.window + 1);
+  const int* table = p.block_table + (size_t)seq * p.max_blocks;
+  const E* qr = q + (size_t)t * p.q_stride_tok + (size_t)head * p.D;
+  const float scale = p.scale * (p.q_temp ? p.q_temp[pos] : 1.f);
+  const int k_off = p.maps > 1 ? head % p.maps * p.D : 0;
   float qv[PL], o[PL];
 #pragma unroll
   for (int i = 0; i < PL; ++i) {
     const int d = lane + i * 32;
-    qv[i] = d < D ? to_f(qr[d]) : 0.f;
+    qv[i] = d < p.D ? to_f(qr[d]) : 0.f;
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
   for (int j = first + warp; j <= pos; j += AW) {
-    const size_t row = ((size_t)table[j / block_size] * Hkv + kvh) * block_size + j % block_size;
-    const E* kr = kc + row * D;
-    const E* vr = vc + row * v_row;
+    const size_t row = ((size_t)table[j / p.block_size] * p.Hkv + kvh) * p.block_size + j % p.block_size;
+    const E* kr = kc + row * p.k_row + k_off;
+    const E* vr = vc + row * p.v_row;
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < PL; ++i) {
       const int d = lane + i * 32;
-      if (d < D) s = fmaf(qv[i], to_f(kr[d]), s);
+      if (d < p.D) s = fmaf(qv[i], to_f(kr[d]), s);
     }
     s = warp_sum(s) * scale;
+    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     const float mn = fmaxf(m, s), f = expf(m - mn), e = expf(s - mn);
     l = l * f + e;
     m = mn;
 #pragma unroll
     for (int i = 0; i < PL; ++i) {
       const int d = lane + i * 32;
-      if (d < Dv) o[i] = fmaf(e, to_f(vr[d]), o[i] * f);
+      if (d < p.Dv) o[i] = fmaf(e, to_f(vr[d]), o[i] * f);
     }
   }
   __shared__ float so[AW][32 * PL], sm[AW], sl[AW];
@@ -122,14 +140,14 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
   for (int i = 0; i < PL; ++i) so[warp][lane + i * 32] = o[i];
   if (lane == 0) sm[warp] = m, sl[warp] = l;
   __syncthreads();
-  float top = sink ? sink[head] : -INFINITY;
+  float top = p.sink ? p.sink[head] : -INFINITY;
   for (int w = 0; w < AW; ++w) top = fmaxf(top, sm[w]);
-  float den = sink ? expf(sink[head] - top) : 0.f;
+  float den = p.sink ? expf(p.sink[head] - top) : 0.f;
   for (int w = 0; w < AW; ++w) den += sl[w] * expf(sm[w] - top);
-  for (int d = threadIdx.x; d < Dv; d += AW * 32) {
+  for (int d = threadIdx.x; d < p.Dv; d += AW * 32) {
     float v = 0.f;
     for (int w = 0; w < AW; ++w) v = fmaf(so[w][d], expf(sm[w] - top), v);
-    from_f(out[(size_t)t * out_stride_tok + (size_t)head * Dv + d], v / den);
+    from_f(out[(size_t)t * p.out_stride_tok + (size_t)head * p.Dv + d], v / den);
   }
 }
 
@@ -171,16 +189,13 @@ __global__ void __launch_bounds__(64) head_product_kernel(const E* __restrict__ 
 }
 
 template <typename E>
-int launch_attn_simple(const E* q, long long q_stride_tok, const E* k, const E* v, E* out, long long out_stride_tok,
-                       const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
-                       int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
-                       const float* sink, cudaStream_t s) {
-  const dim3 grid((unsigned)total_tokens, Hq), block(AW * 32);
+int launch_attn_simple(const void* q, const void* k, const void* v, void* out, const SimpleAttnParams& p, int total_tokens, cudaStream_t s) {
+  const dim3 grid((unsigned)total_tokens, p.Hq), block(AW * 32);
   auto go = [&](auto kernel) {
-    return launch_kernel(kernel, grid, block, 0, s, q, q_stride_tok, k, v, out, out_stride_tok, block_table, max_blocks, block_size,
-                         cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv, v_row, scale, chunk, sink);
+    return launch_kernel(kernel, grid, block, 0, s, reinterpret_cast<const E*>(q), reinterpret_cast<const E*>(k), reinterpret_cast<const E*>(v),
+                         reinterpret_cast<E*>(out), p);
   };
-  const int widest = max(D, Dv);
+  const int widest = max(p.D, p.Dv);
   if (widest <= 128) return go(attn_simple_kernel<E, 4>);
   if (widest <= 320) return go(attn_simple_kernel<E, 10>);
   if (widest <= 640) return go(attn_simple_kernel<E, 20>);
@@ -195,37 +210,32 @@ extern "C" {
 // fp32 GEMM without reduced-precision modes. Dense: offsets null, groups 1. Grouped: w [groups, N, ldw], rows of group g
 // are [offsets[g], offsets[g + 1]), at most T rows in all; src (nullable) names the row of `a` for each row.
 int swb_gemm_f32(const float* a, int lda, const int* src, const int* offsets, int groups, const float* w, int ldw, float* out,
-                 int ldo, int T, int N, int K, int act, void* stream) {
+                 int ldo, int T, int N, int K, int act, const float* bias, void* stream) {
   using namespace swb;
   if (T <= 0 || N <= 0 || K <= 0) return 0;
-  if (groups < 1 || (groups > 1 && !offsets) || gemm_act_pairs(act)) return -3;
+  if (groups < 1 || (bias && offsets) || (groups > 1 && !offsets) || gemm_act_pairs(act)) return -3;
   return launch_kernel(gemm_f32_kernel, dim3((N + TN - 1) / TN, (T + TM - 1) / TM, groups), dim3(256), 0,
-                       reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act);
+                       reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act, bias);
 }
 
 // Paged attention for any head widths up to 1024 in fp32 arithmetic; elements fp32 or bf16 (fp32 flag). Arguments as in
-// swb_attn_ext; causal, sequences from cu_q or uniform lengths of uniform_q tokens. v_row: elements between the value rows of
-// consecutive tokens of a page (0: Dv), so that values may be the leading columns of wider rows.
+// swb_attn_ext and SimpleAttnParams; causal, sequences from cu_q or uniform lengths of uniform_q tokens. v_row: elements between the
+// value rows of consecutive tokens of a page (0: Dv), so that values may be the leading columns of wider rows. Key rows are maps * D
+// wide (D up to 1024 each).
 int swb_attn_simple(const void* q, long long q_stride_tok, const void* k, const void* v, void* out, long long out_stride_tok,
                     const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
                     int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
-                    const float* sink, int fp32, void* stream) {
+                    const float* sink, int window, float softcap, const float* q_temp, int maps, int fp32, void* stream) {
   using namespace swb;
   if (total_tokens <= 0 || num_seqs <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || D < 1 || Dv < 1 || D > 32 * MAX_PER_LANE || Dv > 32 * MAX_PER_LANE || block_size <= 0 ||
-      !block_table || !kv_lens || chunk < 0 || (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)) ||
-      (v_row && v_row < Dv))
+      !block_table || !kv_lens || chunk < 0 || window < 0 || softcap < 0.f || maps < 1 || (Hq / Hkv) % maps ||
+      (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)) || (v_row && v_row < Dv))
     return -3;
+  const SimpleAttnParams p{q_stride_tok, out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv,
+                           maps * D, v_row ? v_row : Dv, scale, chunk, window, softcap, q_temp, sink, maps};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (!v_row) v_row = Dv;
-  if (fp32)
-    return launch_attn_simple(reinterpret_cast<const float*>(q), q_stride_tok, reinterpret_cast<const float*>(k),
-                              reinterpret_cast<const float*>(v), reinterpret_cast<float*>(out), out_stride_tok, block_table,
-                              max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, total_tokens, Hq, Hkv, D, Dv, v_row, scale,
-                              chunk, sink, s);
-  return launch_attn_simple(reinterpret_cast<const bf16*>(q), q_stride_tok, reinterpret_cast<const bf16*>(k),
-                            reinterpret_cast<const bf16*>(v), reinterpret_cast<bf16*>(out), out_stride_tok, block_table, max_blocks,
-                            block_size, cu_q, kv_lens, num_seqs, uniform_q, total_tokens, Hq, Hkv, D, Dv, v_row, scale, chunk, sink, s);
+  return fp32 ? launch_attn_simple<float>(q, k, v, out, p, total_tokens, s) : launch_attn_simple<bf16>(q, k, v, out, p, total_tokens, s);
 }
 
 // Per-head products of any sizes and strides (elements): out[t, h, n] = sigmoid(gate[t, h]) sum_k a[t, h, k] w[h, n, k].

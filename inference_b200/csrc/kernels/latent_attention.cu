@@ -1,6 +1,7 @@
 // Latent attention: a token's keys and values of all heads are projections of one cached row [c | k_rot], c the normed latent
 // (rank numbers) and k_rot the rotated key part shared by the heads.
-//   latent_prep     norm of c, rotation of k_rot and of every head's rotated query part, cache write.
+//   latent_prep     norm of c (and of a low-rank query latent beside it), rotation of k_rot and of every head's rotated query part,
+//                   cache write. Queries that come out of a low-rank latent only exist later: a second launch rotates them.
 //   latent_decode   attention in the latent space for steps with few tokens per sequence. The queries were taken through the
 //                   key projection, so all heads read the same cached rows, which serve as keys (all columns) and as values
 //                   (the latent columns). Everything is computed transposed on the tensor cores: S^T = K Q^T puts 64 keys on
@@ -21,9 +22,13 @@ SWB_REGISTER_STATUS_UNIT(latent_attention);
 namespace {
 
 struct LatentPrepParams {
-  void* buf;                 // projections [T, ld]: q (H heads of dn + rp) at 0, c (rk) at col_c, k_rot (rp) behind it
+  void* q;                   // queries [T, ldq]: H heads of dn + rp (H 0: none in this launch)
+  int ldq;
+  void* buf;                 // optional projections [T, ld]: c (rk) at col_c, k_rot (rp) behind it, a query latent (qk) at 0
   int ld, col_c;
   const float* w;            // [rk]
+  const float* wq;           // optional [qk]: norm of the query latent, q_rank real columns
+  int q_rank, qk;
   float eps;
   const float *cos, *sin;    // [positions, rot / 2]
   const int* positions;
@@ -34,42 +39,56 @@ struct LatentPrepParams {
   int T, H, dn, rot, rp, rc, rank, rk;   // rc: columns of the rotated part in `cache` and `q_abs`, zero beyond rp
 };
 
-// One CTA per token: warp 0 norms the latent, the others rotate in groups of eight dimensions (four pairs).
+// v <- v / sqrt(mean(v^2) + eps) * w over a row of `n` padded columns (`real` of them in the mean), by one warp; also to dst.
+template <typename E>
+__device__ __forceinline__ void norm_latent(E* v, const float* w, int n, int real, float eps, E* dst, int lane) {
+  float ss = 0.f;
+  for (int i = lane * 8; i < n; i += 256) {            // padding columns are zero
+    float x[8];
+    load_row8(v + i, x);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(x[j], x[j], ss);
+  }
+  const float r = rsqrtf(warp_sum(ss) / (float)real + eps);
+  for (int i = lane * 8; i < n; i += 256) {
+    float x[8], y[8];
+    load_row8(v + i, x);
+    load_row8(w + i, y);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] *= r * y[j];
+    store_row8(v + i, x);
+    if (dst) store_row8(dst + i, x);
+  }
+}
+
+// One CTA per token: warp 0 norms the latent and warp 1 the query latent, the others rotate in groups of eight dimensions (four pairs).
 template <typename E>
 __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
   pdl_launch_dependents();
   pdl_wait(TL_ROPE_KV);
-  const int t = blockIdx.x, pos = p.positions[t], width = p.rk + p.rc, lane = threadIdx.x & 31;
+  const int t = blockIdx.x, pos = p.positions[t], width = p.rk + p.rc, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   E* row = reinterpret_cast<E*>(p.buf) + (size_t)t * p.ld;
   E* c = row + p.col_c;
-  const long long slot = p.slots[t];
+  const long long slot = p.buf ? p.slots[t] : -1;
   E* dst = slot >= 0 ? reinterpret_cast<E*>(p.cache) + (size_t)slot * width : nullptr;
-  if (threadIdx.x < 32) {
-    float ss = 0.f;
-    for (int i = lane * 8; i < p.rk; i += 256) {       // padding columns are zero
-      float v[8];
-      load_row8(c + i, v);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+  int busy = 0;                                        // warps that norm
+  if (p.buf) {
+    if (warp == 0) norm_latent(c, p.w, p.rk, p.rank, p.eps, dst, lane);
+    busy = 1;
+    if (p.wq) {
+      if (warp == 1) norm_latent(row, p.wq, p.qk, p.q_rank, p.eps, (E*)nullptr, lane);
+      busy = 2;
     }
-    const float r = rsqrtf(warp_sum(ss) / (float)p.rank + p.eps);
-    for (int i = lane * 8; i < p.rk; i += 256) {
-      float v[8], w[8];
-      load_row8(c + i, v);
-      load_row8(p.w + i, w);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] *= r * w[j];
-      store_row8(c + i, v);
-      if (dst) store_row8(dst + i, v);
-    }
-    return;
   }
+  if (warp < busy) return;
   const int q_row = !p.q_abs ? -1 : p.q_row ? p.q_row[t] : t, per = p.rc / 8;
   const float* cs = p.cos + (size_t)pos * (p.rot / 2);
   const float* sn = p.sin + (size_t)pos * (p.rot / 2);
-  for (int i = threadIdx.x - 32; i < (p.H + 1) * per; i += 96) {    // the heads' queries, then the shared key part
+  E* q = reinterpret_cast<E*>(p.q) + (size_t)t * p.ldq;
+  const int heads = p.H + (p.buf ? 1 : 0);
+  for (int i = threadIdx.x - busy * 32; i < heads * per; i += 128 - busy * 32) {    // the heads' queries, then the shared key part
     const int h = i / per, k = i % per * 8;
-    E* x = (h < p.H ? row + h * (p.dn + p.rp) + p.dn : c + p.rk) + k;
+    E* x = (h < p.H ? q + h * (p.dn + p.rp) + p.dn : c + p.rk) + k;
     float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
     if (k < p.rp) load_row8(x, v);
 #pragma unroll
@@ -85,15 +104,15 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
   }
 }
 
-// Cached rows of several sequences side by side: out row cu_k[s] + i is row i of sequence s (16-byte pieces).
+// Cached rows of several sequences side by side: out row cu_k[s] + i is row first[s] + i of sequence s (16-byte pieces).
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table,
                                                             int max_blocks, int block_size, const int* __restrict__ seqs,
-                                                            const int* __restrict__ cu_k, int num_seqs, int rows, int pieces, uint4* out) {
+                                                            const int* __restrict__ first, const int* __restrict__ cu_k, int num_seqs, int rows, int pieces, uint4* out) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < (long long)rows * pieces; i += (long long)gridDim.x * 256) {
     const int r = (int)(i / pieces), c = (int)(i % pieces);
-    const int z = seq_of_token(cu_k, num_seqs, 1, r), k = r - cu_k[z], s = seqs ? seqs[z] : z;
+    const int z = seq_of_token(cu_k, num_seqs, 1, r), k = r - cu_k[z] + (first ? first[z] : 0), s = seqs ? seqs[z] : z;
     const int page = block_table[(size_t)s * max_blocks + k / block_size];
     out[i] = cache[((size_t)page * block_size + k % block_size) * pieces + c];
   }
@@ -111,6 +130,7 @@ struct LatentDecodeParams {
   const int* cu_q;           // [num_seqs + 1] or null (uniform_q tokens each)
   const int* kv_lens;
   int uniform_q, H, num_splits, rows_total;
+  int window;                // > 0: a query sees only the last `window` keys, its own included
   float scale_log2;
   float* part_o;             // [splits, rows_total, rk]
   float* part_ml;            // [splits, rows_total, 2]: running max (log2 units), sum relative to it
@@ -240,8 +260,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   const int kv_len = p.kv_lens[seq], base_row = q_start * p.H + row0;
   // keys that the last row of this block sees
   const int kv_end = min(kv_len, kv_len - q_len + (row0 + nrows - 1) / p.H + 1);
-  const int tiles = (kv_end + DEC_KEYS - 1) / DEC_KEYS, per = (tiles + p.num_splits - 1) / p.num_splits;
-  const int t0 = split * per, n_tiles = min(tiles, t0 + per) - t0;
+  // first tile that the first row sees
+  const int tile_lo = p.window > 0 ? max(kv_len - q_len + row0 / p.H - p.window + 1, 0) / DEC_KEYS : 0;
+  const int tiles = (kv_end + DEC_KEYS - 1) / DEC_KEYS, per = (tiles - tile_lo + p.num_splits - 1) / p.num_splits;
+  const int t0 = tile_lo + split * per, n_tiles = min(tiles, t0 + per) - t0;
   if (n_tiles <= 0) {
     for (int i = threadIdx.x; i < nrows; i += DEC_THREADS) {
       float* ml = p.part_ml + ((size_t)split * p.rows_total + base_row + i) * 2;
@@ -403,6 +425,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           for (int n = 0; n < NC; ++n)
             if (k0 + key > kv_len - q_len + (row0 + r0 + n) / p.H || k0 + key >= kv_len) s[n] = -INFINITY;
         }
+        if (p.window > 0 && k0 <= kv_len - q_len + (row0 + nrows - 1) / p.H - p.window) {      // some key is out of the last row's window
+#pragma unroll
+          for (int n = 0; n < NC; ++n)
+            if (k0 + key <= kv_len - q_len + (row0 + r0 + n) / p.H - p.window) s[n] = -INFINITY;
+        }
         float v[NC];
 #pragma unroll
         for (int n = 0; n < NC; ++n) v[n] = s[n] = has_key ? s[n] : -INFINITY;
@@ -511,6 +538,11 @@ struct HeadMmaParams {
   // MERGE: a is the merged split partials
   const float *part_o, *part_ml, *sink;
   int num_splits, rows_total;
+  // optional (not MERGE): columns [rot_in, rot_in + rot_pad) of a's head rows are rotated (the first `rot`, neighbouring pairs) and
+  // stored at column rot_out of out's head rows, zero up to rot_cols
+  const float *cos, *sin;
+  const int* positions;
+  int rot_in, rot_out, rot, rot_pad, rot_cols;
 };
 
 constexpr int HM_TOK = 16;   // tokens per CTA: the rows of the MMA
@@ -543,11 +575,11 @@ __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaPa
   if constexpr (MERGE) {
     for (int i = warp; i < m; i += HM_WARPS) {         // a warp per token: lane = split
       const size_t row = (size_t)token_in(i) * p.H + h;
-      const float sk = p.sink[h] * 1.4426950408889634f;
+      const float sk = p.sink ? p.sink[h] * 1.4426950408889634f : -INFINITY;
       float2 ml = make_float2(-INFINITY, 0.f);
       if (lane < p.num_splits) ml = *reinterpret_cast<const float2*>(p.part_ml + ((size_t)lane * p.rows_total + row) * 2);
       const float top = fmaxf(warp_max(ml.x), sk), w = ml.y > 0.f ? exp2f(ml.x - top) : 0.f;
-      const float den = warp_sum(w * ml.y) + exp2f(sk - top);
+      const float den = warp_sum(w * ml.y) + (p.sink ? exp2f(sk - top) : 0.f);
       wt[i * 32 + lane] = w / den;
     }
     __syncthreads();
@@ -580,6 +612,25 @@ __global__ void __launch_bounds__(HM_WARPS * 32) head_mma_kernel(const HeadMmaPa
       uint4 v = make_uint4(0, 0, 0, 0);
       if (i < m) v = *reinterpret_cast<const uint4*>(p.a + token_in(i) * p.a_tok + (long long)h * p.a_head + c);
       *reinterpret_cast<uint4*>(sa + i * ld + c) = v;
+    }
+  }
+  if (!MERGE && p.cos && blockIdx.x == 0) {
+    const int per = p.rot_cols / 8;
+    for (int idx = threadIdx.x; idx < m * per; idx += HM_WARPS * 32) {
+      const int i = idx / per, k = idx % per * 8, ti = token_in(i);
+      const bf16* x = p.a + ti * p.a_tok + (long long)h * p.a_head + p.rot_in + k;
+      const float* cs = p.cos + (size_t)p.positions[ti] * (p.rot / 2);
+      const float* sn = p.sin + (size_t)p.positions[ti] * (p.rot / 2);
+      float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (k < p.rot_pad) load_row8(x, v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (k + 2 * j >= p.rot) continue;
+        const float c = cs[k / 2 + j], s = sn[k / 2 + j], u = v[2 * j], w = v[2 * j + 1];
+        v[2 * j] = u * c - w * s;
+        v[2 * j + 1] = w * c + u * s;
+      }
+      store_row8(p.out + token_out(i) * p.out_tok + (long long)h * p.out_head + p.rot_out + k, v);
     }
   }
   __syncthreads();
@@ -645,30 +696,34 @@ int launch_latent_decode(const CUtensorMap& tq, const CUtensorMap& tk, LatentDec
 
 extern "C" {
 
-int swb_latent_prep(void* buf, int ld, int col_c, const float* w, float eps, const float* cos, const float* sin, const int* positions,
-                    const long long* slots, void* cache, void* q_abs, const int* q_row, int T, int H, int dn, int rot, int rp, int rc, int rank, int rk, int fp32,
-                    void* stream) {
+// See LatentPrepParams. buf null: only the queries of q are rotated; H 0: only the latents.
+int swb_latent_prep(void* q, int ldq, void* buf, int ld, int col_c, const float* w, const float* wq, int q_rank, int qk, float eps,
+                    const float* cos, const float* sin, const int* positions, const long long* slots, void* cache, void* q_abs,
+                    const int* q_row, int T, int H, int dn, int rot, int rp, int rc, int rank, int rk, int fp32, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
-  if (H <= 0 || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || ((dn | rp | rc | rk | ld | col_c) % 8) || rc < rp || rank <= 0 || rank > rk || !cache || !slots)
+  if (H < 0 || (H > 0 && !q) || (!buf && H == 0) || dn <= 0 || rot <= 0 || (rot % 2) || rot > rp || ((dn | rp | rc | rk | ldq) % 8) || rc < rp)
     return -3;
-  const LatentPrepParams p{buf, ld, col_c, w, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot, rp, rc, rank, rk};
+  if (buf && (((ld | col_c) % 8) || !w || rank <= 0 || rank > rk || !cache || !slots)) return -3;
+  if (wq && (!buf || (qk % 8) || q_rank <= 0 || q_rank > qk || qk > col_c)) return -3;
+  const LatentPrepParams p{q, ldq, buf, ld, col_c, w, wq, q_rank, qk, eps, cos, sin, positions, slots, cache, q_abs, q_row, T, H, dn, rot,
+                           rp, rc, rank, rk};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return fp32 ? launch_kernel(latent_prep_kernel<float>, dim3((unsigned)T), dim3(128), 0, s, p)
               : launch_kernel(latent_prep_kernel<bf16>, dim3((unsigned)T), dim3(128), 0, s, p);
 }
 
 // out [rows, width] bf16 <- the cached rows of num_seqs sequences (seqs: their indices in block_table, null: 0, 1, ...), those of
-// sequence s at [cu_k[s], cu_k[s + 1]). width % 8 == 0.
-int swb_latent_gather(const void* cache, const int* block_table, int max_blocks, int block_size, const int* seqs, const int* cu_k,
-                      int num_seqs, int rows, int width, void* out, void* stream) {
+// sequence s from its row first[s] (null: 0) on at [cu_k[s], cu_k[s + 1]). width % 8 == 0.
+int swb_latent_gather(const void* cache, const int* block_table, int max_blocks, int block_size, const int* seqs, const int* first,
+                      const int* cu_k, int num_seqs, int rows, int width, void* out, void* stream) {
   using namespace swb;
   if (rows <= 0) return 0;
   if (width % 8 || num_seqs <= 0 || block_size <= 0 || ((reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(out)) & 15)) return -3;
   const long long n = (long long)rows * (width / 8);
   const unsigned grid = (unsigned)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
   return launch_kernel(latent_gather_kernel, dim3(grid), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream),
-                       reinterpret_cast<const uint4*>(cache), block_table, max_blocks, block_size, seqs, cu_k, num_seqs, rows, width / 8,
+                       reinterpret_cast<const uint4*>(cache), block_table, max_blocks, block_size, seqs, first, cu_k, num_seqs, rows, width / 8,
                        reinterpret_cast<uint4*>(out));
 }
 
@@ -676,30 +731,30 @@ int swb_latent_gather(const void* cache, const int* block_table, int max_blocks,
 int swb_latent_prefill(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok, const void* k2,
                        long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
                        int total_tokens, int H, int d1, int d2, int Dv, float scale, const float* sink, const void* gate,
-                       long long gate_stride, const int* cu_q, const int* seqs, const int* cu_k, void* stream) {
+                       long long gate_stride, const int* cu_q, const int* seqs, const int* cu_k, int window, void* stream) {
   using namespace swb;
   if (num_seqs <= 0 || total_tokens <= 0) return 0;
   if (max_q_len <= 0 || key_rows <= 0) return -3;
   return attn_latent_tcgen05_launch(q, q_stride_tok, k, v, kv_stride_tok, k2, k2_stride_tok, key_rows, out, out_stride_tok, num_seqs,
                                     max_q_len, total_tokens, H, d1, d2, Dv, scale, sink, gate, gate_stride, cu_q, seqs, cu_k,
-                                    reinterpret_cast<cudaStream_t>(stream));
+                                    reinterpret_cast<cudaStream_t>(stream), window);
 }
 
 // Attention of q_abs [T * H, rk + rp] over the cached rows [num_blocks * block_size, rk + rc] (q rows likewise) into
 // split partials (see LatentDecodeParams). rc: the rotated part with its padding (zero in q), a multiple of 64; rot of it is used. max_q: most tokens of a sequence.
 int swb_latent_decode(const void* q_abs, const void* cache, int num_blocks, int block_size, const int* block_table, int max_blocks,
                       const int* cu_q, const int* kv_lens, int n_seqs, int uniform_q, int max_q, int T, int H, int rk,
-                      int rc, int rot, float scale, int num_splits, float* part_o, float* part_ml, void* stream) {
+                      int rc, int rot, float scale, int num_splits, int window, float* part_o, float* part_ml, void* stream) {
   using namespace swb;
   if (T <= 0 || n_seqs <= 0) return 0;
   if (rk % 64 || rk < 64 || rk > 512 || rc % 64 || rot < 1 || rot > rc || rc > 128 || block_size < 8 || block_size % 8 ||
-      !(scale > 0.f) || num_splits < 1 || num_splits > 32 || H < 1 || max_q < 1 || (!cu_q && uniform_q < 1))
+      !(scale > 0.f) || num_splits < 1 || num_splits > 32 || H < 1 || max_q < 1 || window < 0 || (!cu_q && uniform_q < 1))
     return -3;
   if ((reinterpret_cast<uintptr_t>(q_abs) | reinterpret_cast<uintptr_t>(cache)) & 15) return -3;
   LatentDecodeParams p{};
   p.block_table = block_table, p.max_blocks = max_blocks, p.block_size = block_size;
   p.cu_q = cu_q, p.kv_lens = kv_lens;
-  p.uniform_q = uniform_q, p.H = H, p.num_splits = num_splits, p.rows_total = T * H;
+  p.uniform_q = uniform_q, p.H = H, p.num_splits = num_splits, p.rows_total = T * H, p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.part_o = part_o, p.part_ml = part_ml;
   p.rk = rk, p.latent_atoms = rk / 64, p.pairs = (p.latent_atoms + 1) / 2, p.atoms = (rk + rc) / 64, p.rot_steps = (rot + 15) / 16;
@@ -714,21 +769,25 @@ int swb_latent_decode(const void* q_abs, const void* cache, int num_blocks, int 
 }
 
 // out[t, h, n] = sigmoid(gate[t, h]) sum_k a[t, h, k] w[h, n, k] in bf16 for n tokens: row i is token rows_in[i] of a and
-// rows_out[i] of out and gate (null: i). With
-// part_o, a[t, h] are the merged split partials of swb_latent_decode with sinks (K = rk) and `a` is unused. K, N and all strides
+// rows_out[i] of out and gate (null: i). With cos, the rotated query parts travel along (see HeadMmaParams). With
+// part_o, a[t, h] are the merged split partials of swb_latent_decode (K = rk), with optional sinks, and `a` is unused. K, N and all strides
 // are multiples of 8.
 int swb_head_mma(const void* a, long long a_tok, int a_head, const void* w, void* out, long long out_tok, int out_head, const void* gate,
                  long long gate_tok, const int* rows_in, const int* rows_out, int n, int H, int N, int K, const float* part_o, const float* part_ml,
-                 const float* sink, int num_splits, int rows_total, void* stream) {
+                 const float* sink, int num_splits, int rows_total, const float* cos, const float* sin, const int* positions, int rot_in,
+                 int rot_out, int rot, int rot_pad, int rot_cols, void* stream) {
   using namespace swb;
   if (n <= 0 || H <= 0) return 0;
-  if (N < 8 || N % 8 || K < 8 || K % 8 || K > 1024 || (out_tok % 8) || (out_head % 8) || (part_o && (!part_ml || !sink || num_splits > 32)) ||
+  if (cos && (part_o || !sin || !positions || rot < 2 || (rot % 2) || rot > rot_pad || rot_pad > rot_cols || ((rot_in | rot_out | rot_pad | rot_cols) % 8) ||
+              (reinterpret_cast<uintptr_t>(out) & 15)))
+    return -3;
+  if (N < 8 || N % 8 || K < 8 || K % 8 || K > 1024 || (out_tok % 8) || (out_head % 8) || (part_o && (!part_ml || num_splits > 32)) ||
       (!part_o && (!a || (a_tok % 8) || (a_head % 8) || (reinterpret_cast<uintptr_t>(a) & 15))) ||
       (reinterpret_cast<uintptr_t>(w) & 15) || (reinterpret_cast<uintptr_t>(out) & 3))
     return -3;
   const HeadMmaParams p{reinterpret_cast<const bf16*>(a), a_tok, a_head, reinterpret_cast<const bf16*>(w), reinterpret_cast<bf16*>(out),
                         out_tok, out_head, reinterpret_cast<const bf16*>(gate), gate_tok, rows_in, rows_out, n, H, N, K, part_o, part_ml, sink,
-                        num_splits, rows_total};
+                        num_splits, rows_total, cos, sin, positions, rot_in, rot_out, rot, rot_pad, rot_cols};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return part_o ? launch_head_mma<true>(p, s) : launch_head_mma<false>(p, s);
 }

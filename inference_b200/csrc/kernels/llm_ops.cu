@@ -382,10 +382,128 @@ __global__ void __launch_bounds__(256) rope_kv_write_d128_kernel(
   }
 }
 
+// Norms over whole query / key projections (all heads of a token at once), rotation, cache write: one CTA per token.
+struct RowRopeParams {
+  void* buf;                  // [T, ld]: q (H heads of D) at 0, k (G heads of D) behind it, v (G heads of Dv) at v_col
+  int ld, v_col, H, G, D, Dv, rot;
+  const float *wq, *wk;       // norm weights [H * D], [G * D]; null: no norm
+  int nq, nk;                 // numbers that enter the mean of q and k (padding columns are zero)
+  float eps;
+  const float *cos, *sin;     // [positions, rot / 2]; pairs are neighbouring dimensions
+  const int* positions;
+  const long long* slots;     // row of the caches, < 0: none
+  void *kcache, *vcache;      // [block, G, block_size, D | Dv]
+  int block_size;
+  int v_from_k;               // values are the keys as projected (Dv == D)
+  int store_v;                // v_from_k: also store them at v_col
+};
+
+template <typename E>
+__global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p) {
+  pdl_launch_dependents();
+  pdl_wait(TL_ROPE_KV);
+  __shared__ float red[2][8];
+  const int t = blockIdx.x, nq8 = p.H * p.D / 8, nk8 = p.G * p.D / 8, nv8 = p.G * p.Dv / 8;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  E* q = reinterpret_cast<E*>(p.buf) + (size_t)t * p.ld;
+  E* k = q + nq8 * 8;
+  E* v = q + p.v_col;
+  float rq = 1.f, rk = 1.f;
+  if (p.wk) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < nq8 + nk8; i += blockDim.x) {
+      float x[8], ss = 0.f;
+      load_row8(q + i * 8, x);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(x[j], x[j], ss);
+      if (i < nq8) sq += ss;
+      else sk += ss;
+    }
+    sq = warp_sum(sq), sk = warp_sum(sk);
+    if (lane == 0) red[0][warp] = sq, red[1][warp] = sk;
+    __syncthreads();
+    sq = sk = 0.f;
+    for (int w = 0; w < warps; ++w) sq += red[0][w], sk += red[1][w];
+    rq = rsqrtf(sq / (float)p.nq + p.eps), rk = rsqrtf(sk / (float)p.nk + p.eps);
+  }
+  const long long slot = p.slots[t];
+  E *kc = nullptr, *vc = nullptr;
+  const size_t page = slot >= 0 ? (size_t)(slot / p.block_size) * p.G * p.block_size + slot % p.block_size : 0;
+  if (slot >= 0) kc = reinterpret_cast<E*>(p.kcache), vc = reinterpret_cast<E*>(p.vcache);
+  const int half = p.rot / 2;
+  const float* cs = p.cos + (size_t)p.positions[t] * half;
+  const float* sn = p.sin + (size_t)p.positions[t] * half;
+  const int first = p.wk || p.rot > 0 ? 0 : nq8;            // nothing to do for the queries
+  for (int i = first + threadIdx.x; i < nq8 + nk8; i += blockDim.x) {
+    const bool is_q = i < nq8;
+    const int j8 = is_q ? i : i - nq8, h = j8 * 8 / p.D, d = j8 * 8 - h * p.D;
+    E* at = is_q ? q + j8 * 8 : k + j8 * 8;
+    float x[8];
+    load_row8(at, x);
+    if (!is_q && p.v_from_k) {
+      if (vc) store_row8(vc + (page + (size_t)h * p.block_size) * p.Dv + d, x);
+      if (p.store_v) store_row8(v + j8 * 8, x);
+    }
+    if (p.wk) {
+      float w[8];
+      load_row8((is_q ? p.wq : p.wk) + j8 * 8, w);
+      const float r = is_q ? rq : rk;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] *= r * w[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (d + 2 * j >= p.rot) continue;
+      const float c = cs[d / 2 + j], s = sn[d / 2 + j], a = x[2 * j], b = x[2 * j + 1];
+      x[2 * j] = a * c - b * s;
+      x[2 * j + 1] = b * c + a * s;
+    }
+    if (p.wk || p.rot > 0) store_row8(at, x);
+    if (!is_q && kc) store_row8(kc + (page + (size_t)h * p.block_size) * p.D + d, x);
+  }
+  if (!p.v_from_k && vc) {
+    for (int i = threadIdx.x; i < nv8; i += blockDim.x) {
+      const int h = i * 8 / p.Dv, d = i * 8 - h * p.Dv;
+      float x[8];
+      load_row8(v + i * 8, x);
+      store_row8(vc + (page + (size_t)h * p.block_size) * p.Dv + d, x);
+    }
+  }
+}
+
+// Differential attention: o = a1 - lambda a2 for the two maps of a head, divided by its root mean square, times `post`. One warp per
+// (token, head); in [T, H, 2, Dv] strided by token, out [T, H * Dv] likewise. N: real columns of the Dv.
+template <typename E>
+__global__ void __launch_bounds__(256) diff_combine_kernel(const E* __restrict__ in, long long in_tok, E* out, long long out_tok, int T, int H,
+                                                           int Dv, int N, float lambda, float eps, float post) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long gw = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (gw >= (long long)T * H) return;
+  const int t = (int)(gw / H), h = (int)(gw % H);
+  const E* a = in + t * in_tok + (long long)h * 2 * Dv;
+  E* o = out + t * out_tok + (long long)h * Dv;
+  float ss = 0.f;
+  for (int d = lane; d < Dv; d += 32) {
+    const float x = to_f(a[d]) - lambda * to_f(a[Dv + d]);
+    ss = fmaf(x, x, ss);
+  }
+  const float r = rsqrtf(warp_sum(ss) / (float)N + eps) * post;
+  for (int d = lane; d < Dv; d += 32) from_f(o[d], (to_f(a[d]) - lambda * to_f(a[Dv + d])) * r);
+}
+
+__device__ __forceinline__ float gated_act(float g, bool gelu, bool exact) {
+  if (gelu) return gelu_tanh_f(g);
+  return exact ? g / (1.f + expf(-g)) : silu_f(g);
+}
+
 // out[t, f] = act(gu[t, f]) * gu[t, F + f]; act 1 = SiLU (SwiGLU), 2 = tanh-GELU (GeGLU). act 3 / 4: the same two
-// activations on a pair-interleaved projection output, out[t, f] = act(gu[t, 2f]) * gu[t, 2f + 1].
-__global__ void __launch_bounds__(256) gated_act_mul_kernel(const bf16* __restrict__ gu, int ld_gu, bf16* out,
-                                                           int ldo, int T, int F, int act) {
+// activations on a pair-interleaved projection output, out[t, f] = act(gu[t, 2f]) * gu[t, 2f + 1]. row_gate (fp32 logits, one per
+// row, `gate_ld` apart): the row is scaled by its sigmoid.
+template <typename E>
+__global__ void __launch_bounds__(256) gated_act_mul_kernel(const E* __restrict__ gu, int ld_gu, E* out, int ldo, int T, int F, int act,
+                                                           const float* __restrict__ row_gate, int gate_ld) {
   pdl_launch_dependents();
   pdl_wait(TL_GATED_ACT);
   const int nvec = F / 8;
@@ -396,8 +514,8 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const bf16* __restri
   float g[8], u[8], o[8];
   if (act >= 3) {
     float lo[8], hi[8];
-    unpack8(*reinterpret_cast<const uint4*>(gu + (size_t)t * ld_gu + v * 16), lo);
-    unpack8(*reinterpret_cast<const uint4*>(gu + (size_t)t * ld_gu + v * 16 + 8), hi);
+    load_row8(gu + (size_t)t * ld_gu + v * 16, lo);
+    load_row8(gu + (size_t)t * ld_gu + v * 16 + 8, hi);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       g[j] = lo[2 * j];
@@ -406,13 +524,18 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const bf16* __restri
       u[4 + j] = hi[2 * j + 1];
     }
   } else {
-    unpack8(*reinterpret_cast<const uint4*>(gu + (size_t)t * ld_gu + v * 8), g);
-    unpack8(*reinterpret_cast<const uint4*>(gu + (size_t)t * ld_gu + F + v * 8), u);
+    load_row8(gu + (size_t)t * ld_gu + v * 8, g);
+    load_row8(gu + (size_t)t * ld_gu + F + v * 8, u);
   }
   const bool gelu = act == 2 || act == 4;
 #pragma unroll
-  for (int j = 0; j < 8; ++j) o[j] = (gelu ? gelu_tanh_f(g[j]) : silu_f(g[j])) * u[j];
-  *reinterpret_cast<uint4*>(out + (size_t)t * ldo + v * 8) = pack8(o);
+  for (int j = 0; j < 8; ++j) o[j] = gated_act(g[j], gelu, sizeof(E) == 4) * u[j];
+  if (row_gate) {
+    const float s = 1.f / (1.f + expf(-row_gate[(size_t)t * gate_ld]));
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] *= s;
+  }
+  store_row8(out + (size_t)t * ldo + v * 8, o);
 }
 
 // out = a N(z) + b N(z^2) + c N(z^3) + e with the powers taken element by element and N(y) = y / sqrt(mean(y^2) + eps) over
@@ -676,13 +799,54 @@ int swb_poly_norm(const void* z, int ldz, void* out, int ldo, int T, int F, int 
   if (fp32) return launch_poly_norm(reinterpret_cast<const float*>(z), ldz, reinterpret_cast<float*>(out), ldo, T, F, Fp, coef, eps, s);
   return launch_poly_norm(reinterpret_cast<const bf16*>(z), ldz, reinterpret_cast<bf16*>(out), ldo, T, F, Fp, coef, eps, s);
 }
-int swb_gated_act_mul(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, void* stream) {
+// row_gate: see gated_act_mul_kernel; fp32 selects the element type of gate_up and out.
+int swb_gated_act_mul_ex(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, const float* row_gate, int gate_ld,
+                         int fp32, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
   if (F % 8 != 0 || ld_gu % 8 != 0 || ldo % 8 != 0) return -3;
   const long long n = (long long)T * (F / 8);
-  launch_rc = launch_kernel(gated_act_mul_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), reinterpret_cast<const bf16*>(gate_up), ld_gu, reinterpret_cast<bf16*>(out), ldo, T, F, act);
-  return last_err();
+  const dim3 grid((unsigned)((n + 255) / 256)), block(256);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (fp32)
+    return launch_kernel(gated_act_mul_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(gate_up), ld_gu,
+                         reinterpret_cast<float*>(out), ldo, T, F, act, row_gate, gate_ld);
+  return launch_kernel(gated_act_mul_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(gate_up), ld_gu,
+                       reinterpret_cast<bf16*>(out), ldo, T, F, act, row_gate, gate_ld);
+}
+int swb_gated_act_mul(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, void* stream) {
+  return swb_gated_act_mul_ex(gate_up, ld_gu, out, ldo, T, F, act, nullptr, 0, 0, stream);
+}
+
+// See RowRopeParams. D, Dv, ld and v_col multiples of 8, buffers 16-byte aligned (32 in fp32).
+int swb_row_rope_kv_write(void* buf, int ld, int v_col, int H, int G, int D, int Dv, int rot, const float* wq, const float* wk, int nq, int nk,
+                          float eps, const float* cos, const float* sin, const int* positions, const long long* slots, void* kcache,
+                          void* vcache, int block_size, int v_from_k, int store_v, int T, int fp32, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (H < 0 || G < 1 || D < 8 || Dv < 8 || ((D | Dv | ld | v_col) % 8) || rot < 0 || rot > D || (rot % 2) || block_size < 1 || !kcache || !vcache ||
+      !slots || (wk && (nk < 1 || (H > 0 && (!wq || nq < 1)))) || (v_from_k && Dv != D))
+    return -3;
+  const RowRopeParams p{buf, ld, v_col, H, G, D, Dv, rot, wq, wk, nq > 0 ? nq : 1, nk > 0 ? nk : 1, eps, cos, sin, positions, slots, kcache,
+                        vcache, block_size, v_from_k, store_v};
+  const int work = (H + G) * D / 8;
+  const dim3 grid((unsigned)T), block(work <= 64 ? 64 : work <= 128 ? 128 : 256);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  return fp32 ? launch_kernel(row_rope_kv_kernel<float>, grid, block, 0, s, p) : launch_kernel(row_rope_kv_kernel<bf16>, grid, block, 0, s, p);
+}
+
+int swb_diff_combine(const void* in, long long in_tok, void* out, long long out_tok, int T, int H, int Dv, int N, float lambda, float eps,
+                     float post, int fp32, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (H < 1 || Dv < 1 || N < 1 || N > Dv) return -3;
+  const dim3 grid((unsigned)(((long long)T * H + 7) / 8)), block(256);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (fp32)
+    return launch_kernel(diff_combine_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(in), in_tok,
+                         reinterpret_cast<float*>(out), out_tok, T, H, Dv, N, lambda, eps, post);
+  return launch_kernel(diff_combine_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(in), in_tok,
+                       reinterpret_cast<bf16*>(out), out_tok, T, H, Dv, N, lambda, eps, post);
 }
 
 int swb_embedding(const long long* ids, const void* table, void* out, int T, int H, int vocab_start, int vocab_end,

@@ -1,4 +1,8 @@
-// Mixture-of-experts feed-forward for routings that are known before the layer runs, and the small-batch grouped GEMM.
+// Mixture-of-experts feed-forward: routing plans, from a table or from router logits, and the small-batch grouped GEMM.
+//
+// moe_route_kernel / moe_layout_kernel: softmax over a token's router logits (fp32), the `top` largest, and their places in an
+// expert-sorted buffer of the same two layouts as below. Small steps do it in one launch (the last CTA to finish lays the pairs
+// out); large ones lay out in a second, which also copies the rows to their places. The counters clean up after themselves.
 //
 // moe_table_plan_kernel: a router without arithmetic. A table [vocab, top] names each token id's experts, so the token ids
 // of a step fix the routing of every layer before the first one starts: one launch plans all layers (one CTA each).
@@ -111,6 +115,159 @@ __global__ void __launch_bounds__(1024) moe_table_plan_kernel(const long long* _
   }
 }
 
+struct RouteParams {
+  const float* logits;       // [T, ld]
+  int ld, T, E, top, pad;
+  int* expert;               // [T * top]
+  int* rank;                 // [T * top] place of the pair among those of its expert
+  float* weights;            // [T * top] softmax scores
+  int* counters;             // [E + 2] pairs per expert, two tickets; zero between launches
+  int* dest;                 // [T * top]
+  int* src;                  // optional [rows_cap]
+  int* offsets;              // [E + 1]
+  int* active;               // optional [min(E, T * top)]
+  int* tile_group;           // optional [rows_cap / 128]
+  int rows_cap;
+  const uint4* rows_in;      // optional: row t goes to row dest[t, k] of rows_out, 16-byte pieces
+  uint4* rows_out;
+  long long ld_in, ld_out;
+  int pieces;
+};
+
+// First row of every expert's (padded) segment from the counts, by the whole block; start [E + 1] in shared memory.
+__device__ __forceinline__ void segment_starts(const RouteParams& p, int* start) {
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    int carry = 0;
+    for (int e0 = 0; e0 < p.E; e0 += 32) {
+      const int e = e0 + lane;
+      const int n = e < p.E ? (__ldcg(p.counters + e) + p.pad - 1) / p.pad * p.pad : 0;
+      int s = n;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += y;
+      }
+      if (e < p.E) start[e] = carry + s - n;
+      carry += __shfl_sync(0xffffffffu, s, 31);
+    }
+    if (lane == 0) start[p.E] = carry;
+  }
+  __syncthreads();
+}
+
+// What one block writes about the segments as a whole.
+__device__ __forceinline__ void describe_segments(const RouteParams& p, const int* start) {
+  for (int e = threadIdx.x; e <= p.E; e += blockDim.x) p.offsets[e] = start[e];
+  if (p.tile_group) {
+    for (int i = threadIdx.x; i < p.rows_cap / 128; i += blockDim.x) {
+      int lo = 0, hi = p.E;
+      while (lo < hi) {
+        const int mid = (lo + hi) >> 1;
+        if (start[mid + 1] <= i * 128) lo = mid + 1;
+        else hi = mid;
+      }
+      p.tile_group[i] = lo < p.E ? lo : -1;
+    }
+  }
+  if (p.active) {
+    __shared__ int n_active;
+    if (threadIdx.x == 0) n_active = 0;
+    __syncthreads();
+    for (int e = threadIdx.x; e < p.E; e += blockDim.x)
+      if (__ldcg(p.counters + e) > 0) p.active[atomicAdd(&n_active, 1)] = e;
+    __syncthreads();
+    for (int i = n_active + threadIdx.x; i < min(p.E, p.T * p.top); i += blockDim.x) p.active[i] = -1;
+  }
+}
+
+__device__ __forceinline__ void place_pair(const RouteParams& p, const int* start, int pair) {
+  const int row = start[__ldcg(p.expert + pair)] + __ldcg(p.rank + pair);
+  p.dest[pair] = row;
+  if (p.src) p.src[row] = pair / p.top;
+}
+
+// One warp per token. Ties go to the lower expert number. WHOLE: the last block to finish also lays the pairs out.
+template <bool WHOLE>
+__global__ void __launch_bounds__(256) moe_route_kernel(const RouteParams p) {
+  pdl_wait();
+  extern __shared__ int route_start[];
+  const int lane = threadIdx.x & 31, t = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (t < p.T) {
+    const float* z = p.logits + (size_t)t * p.ld;
+    float top = -INFINITY, sum = 0.f;
+    for (int e = lane; e < p.E; e += 32) top = fmaxf(top, z[e]);
+    top = warp_max(top);
+    for (int e = lane; e < p.E; e += 32) sum += expf(z[e] - top);
+    sum = warp_sum(sum);
+    float last = INFINITY, mine = 0.f;      // lane k mod 32 keeps choice k until 32 of them (or all) are filed together
+    int last_e = -1, mine_e = 0;
+    for (int k = 0; k < p.top; ++k) {
+      float best = -INFINITY;
+      int best_e = p.E;
+      for (int e = lane; e < p.E; e += 32) {
+        const float v = z[e];
+        const bool after = v < last || (v == last && e > last_e);     // not taken yet: what follows the last one in order
+        if (after && (v > best || best_e == p.E)) best = v, best_e = e;
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, best, o);
+        const int e = __shfl_xor_sync(0xffffffffu, best_e, o);
+        if (e < p.E && (best_e == p.E || v > best || (v == best && e < best_e))) best = v, best_e = e;
+      }
+      last = best, last_e = best_e;
+      if (lane == (k & 31)) mine = best, mine_e = min(best_e, p.E - 1);     // logits that are not numbers: any expert
+      if ((k & 31) == 31 || k == p.top - 1) {
+        const int pair = t * p.top + (k & ~31) + lane;
+        if (lane <= (k & 31)) {
+          p.expert[pair] = mine_e;
+          p.weights[pair] = expf(mine - top) / sum;
+          p.rank[pair] = atomicAdd(p.counters + mine_e, 1);
+        }
+      }
+    }
+  }
+  if constexpr (WHOLE) {
+    __shared__ int is_last;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) is_last = atomicAdd(p.counters + p.E, 1) == (int)gridDim.x - 1;
+    __syncthreads();
+    if (!is_last) return;
+    __threadfence();
+    segment_starts(p, route_start);
+    describe_segments(p, route_start);
+    for (int pair = threadIdx.x; pair < p.T * p.top; pair += blockDim.x) place_pair(p, route_start, pair);
+    __syncthreads();
+    for (int e = threadIdx.x; e < p.E + 1; e += blockDim.x) p.counters[e] = 0;
+  }
+}
+
+// Lays out the pairs of a large step, a warp per pair, and copies each token's row to its places.
+__global__ void __launch_bounds__(256) moe_layout_kernel(const RouteParams p) {
+  pdl_wait();
+  extern __shared__ int layout_start[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, pairs = p.T * p.top;
+  segment_starts(p, layout_start);
+  if (blockIdx.x == 0) describe_segments(p, layout_start);
+  for (int pair = blockIdx.x * 8 + warp; pair < pairs; pair += gridDim.x * 8) {
+    if (lane == 0) place_pair(p, layout_start, pair);
+    if (p.rows_out) {
+      const int row = layout_start[p.expert[pair]] + p.rank[pair];
+      const uint4* from = p.rows_in + (size_t)(pair / p.top) * p.ld_in;
+      uint4* to = p.rows_out + (size_t)row * p.ld_out;
+      for (int i = lane; i < p.pieces; i += 32) to[i] = __ldg(from + i);
+    }
+  }
+  __syncthreads();
+  __shared__ int is_last;
+  if (threadIdx.x == 0) is_last = atomicAdd(p.counters + p.E + 1, 1) == (int)gridDim.x - 1;     // every block has read the counts
+  __syncthreads();
+  if (!is_last) return;
+  for (int e = threadIdx.x; e < p.E + 2; e += blockDim.x) p.counters[e] = 0;
+}
+
 constexpr int GR_WARPS = 8;
 
 __device__ __forceinline__ void mma16816(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -133,7 +290,8 @@ struct GroupedRowsParams {
   const int* active;     // experts with rows; < 0 = none
   const bf16* w;         // [E, N, K]
   bf16* out;
-  int ldo, N, K, act;
+  int ldo, N, K, act;    // act may be a gated pair: rows of w in (gate, up) pairs, out [*, N / 2]
+  int plan_ahead;        // the plan was complete before the kernel in front of this one started
 };
 
 // One pass over the CTA's 16 * MT weight rows for up to 8 * NT token rows [r0, r0 + n).
@@ -183,6 +341,19 @@ __device__ __forceinline__ void grouped_pass(const GroupedRowsParams& p, const b
 #pragma unroll
       for (int e = 0; e < 4; ++e) mine[(t * 8 + t4 * 2 + (e & 1)) * FW + m * 16 + g + (e >> 1) * 8] = acc[m][t][e];
   __syncthreads();
+  if (gemm_act_pairs(p.act)) {
+    for (int i = threadIdx.x; i < n * 8 * MT; i += GR_WARPS * 32) {
+      const int tok = i / (8 * MT), f = i % (8 * MT) * 2;
+      if (f0 + f < p.N) {
+        float a = 0.f, b = 0.f;
+#pragma unroll
+        for (int w = 0; w < GR_WARPS; ++w) a += red[w * (8 * NT * FW) + tok * FW + f], b += red[w * (8 * NT * FW) + tok * FW + f + 1];
+        p.out[(size_t)(r0 + tok) * p.ldo + (f0 + f) / 2] = __float2bfloat16((p.act == SWB_ACT_GEGLU_PAIRS ? gelu_tanh_f(a) : silu_f(a)) * b);
+      }
+    }
+    __syncthreads();
+    return;
+  }
   for (int i = threadIdx.x; i < n * 16 * MT; i += GR_WARPS * 32) {
     const int tok = i / (16 * MT), f = i % (16 * MT);
     if (f0 + f < p.N) {
@@ -202,12 +373,13 @@ template <int MT>
 __global__ void __launch_bounds__(GR_WARPS * 32) grouped_rows_kernel(const GroupedRowsParams p) {
   pdl_launch_dependents();
   __shared__ float red[GR_WARPS * 32 * (16 * MT + 1)];
+  if (!p.plan_ahead) pdl_wait();
   const int e = p.active[blockIdx.y];
   const int f0 = blockIdx.x * (16 * MT);
   const bf16* wrow = p.w + (size_t)max(e, 0) * p.N * p.K;
   int lo = 0, hi = 0;
   if (e >= 0) lo = p.offsets[e], hi = p.offsets[e + 1];
-  pdl_wait();
+  if (p.plan_ahead) pdl_wait();
   if (e < 0) return;
   for (int r = lo; r < hi; r += 32) {
     const int n = min(32, hi - r);
@@ -240,17 +412,43 @@ int swb_moe_table_plan(const long long* ids, int T, const int* tables, int layer
                        tile_group, rows_cap);
 }
 
+// Routing plan of one layer from router logits [T, ld] (fp32): the `top` experts of the largest softmax scores over all E, weights
+// [T, top] = their scores as they are. dest, src, offsets, active, tile_group, pad and rows_cap as in swb_moe_table_plan.
+// expert and rank: int32 scratch [T * top]; counters: int32 [E + 2], zero at the first launch, launches that share it ordered on
+// one stream. rows_in (nullable): bf16 / fp32 rows of `pieces` 16-byte pieces, ld_in pieces apart, copied to rows dest[t, k] of rows_out.
+int swb_moe_route(const float* logits, int ld, int T, int E, int top, int pad, int* expert, int* rank, float* weights, int* counters,
+                  int* dest, int* src, int* offsets, int* active, int* tile_group, int rows_cap, const void* rows_in, long long ld_in,
+                  void* rows_out, long long ld_out, int pieces, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (top <= 0 || E <= 0 || E > 4096 || top > E || ld < E || (pad != 1 && pad != 128) || (tile_group && (pad != 128 || rows_cap % 128)) ||
+      (long long)T * top + (long long)E * (pad - 1) > (long long)rows_cap || !expert || !rank || !weights || !counters || !dest || !offsets ||
+      (rows_in && (!rows_out || pieces <= 0)))
+    return -3;
+  const RouteParams p{logits, ld, T, E, top, pad, expert, rank, weights, counters, dest, src, offsets, active, tile_group, rows_cap,
+                      reinterpret_cast<const uint4*>(rows_in), reinterpret_cast<uint4*>(rows_out), ld_in, ld_out, pieces};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((unsigned)((T + 7) / 8));
+  const size_t smem = (size_t)(E + 1) * sizeof(int);
+  if (T <= 128 && !rows_in) return launch_kernel(moe_route_kernel<true>, grid, dim3(256), smem, s, p);
+  const int rc = launch_kernel(moe_route_kernel<false>, grid, dim3(256), 0, s, p);
+  if (rc) return rc;
+  const long long blocks = ((long long)T * top + 7) / 8;
+  return launch_kernel(moe_layout_kernel, dim3((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), smem, s, p);
+}
+
 // out[r, :] = act(x[src ? src[r] : r, :] W[e]^T) for every row r of expert e's segment [offsets[e], offsets[e + 1]).
-// W [E, N, K] bf16, K % 8 == 0, ldx % 8 == 0, x and W 16-byte aligned; n_active = length of `active`.
+// W [E, N, K] bf16, K % 8 == 0, ldx % 8 == 0, x and W 16-byte aligned; n_active = length of `active`. plan_ahead: see
+// GroupedRowsParams.
 int swb_gemm_grouped_rows(const void* x, int ldx, const int* src, const int* offsets, const int* active, int n_active,
-                          const void* w, void* out, int ldo, int N, int K, int act, void* stream) {
+                          const void* w, void* out, int ldo, int N, int K, int act, int plan_ahead, void* stream) {
   using namespace swb;
   if (n_active <= 0 || N <= 0 || K <= 0) return 0;
-  if ((K % 8) || (ldx % 8) || !offsets || !active || gemm_act_pairs(act) ||
+  if ((K % 8) || (ldx % 8) || !offsets || !active || (gemm_act_pairs(act) && (N & 1)) ||
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15))
     return -3;
   GroupedRowsParams p{reinterpret_cast<const bf16*>(x), ldx, src, offsets, active, reinterpret_cast<const bf16*>(w),
-                      reinterpret_cast<bf16*>(out), ldo, N, K, act};
+                      reinterpret_cast<bf16*>(out), ldo, N, K, act, plan_ahead};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   // 32 weight rows per CTA halve the token re-reads; 16 when that is needed to give every SM two CTAs
   if ((long long)((N + 31) / 32) * n_active >= 2 * 148)

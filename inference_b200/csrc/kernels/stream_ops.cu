@@ -8,8 +8,9 @@
 // mean, never a difference of large sums). The output is stored once per token, or to every row of an expert-sorted buffer that the token's
 // routing names, so the gather in front of a grouped GEMM costs no launch of its own.
 // The EXT instantiations add what some designs need on top: RMS norms over equal groups of columns, a stream that is read
-// from another buffer than it is written to, and the depth average, in which the joined stream is filed as one more result
-// and x becomes a weighted sum of all results so far.
+// from another buffer than it is written to, the depth average, in which the joined stream is filed as one more result
+// and x becomes a weighted sum of all results so far, and a second part of the branch: weighted expert output rows beside a
+// dense row (parallel sublayers join the stream together).
 // Rows are padded to a multiple of 8 columns; padding columns of the stream, the weights and the outputs are zero and do
 // not enter the statistics.
 #include "common.cuh"
@@ -45,6 +46,11 @@ struct StreamNormParams {
   long long hist_stride;
   int n_hist;
   const float* mix;          // [n_hist + 1]: x <- sum_j mix[j] hist[j] + mix[n_hist] x; the joined x becomes hist[n_hist]
+  const void* extra;         // optional bf16 / fp32 [*, ld_extra]: rows extra_rows[t, k] times extra_weights[t, k] join the branch
+  int ld_extra, extra_fp32;
+  const int* extra_rows;     // [T, extra_top]
+  const float* extra_weights;
+  int extra_top;
 };
 
 __device__ __forceinline__ float4 load4(const void* base, size_t off, int fp32) {
@@ -235,6 +241,24 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const StreamNormPa
       for (int i = 0; i < VPT; ++i)
         v[i].x *= p.branch_weight, v[i].y *= p.branch_weight, v[i].z *= p.branch_weight, v[i].w *= p.branch_weight;
     }
+    if constexpr (EXT) {
+      if (p.extra) {
+#pragma unroll 4
+        for (int k = 0; k < p.extra_top; ++k) {
+          const size_t er = (size_t)p.extra_rows[row * p.extra_top + k] * p.ld_extra;
+          const float w = p.extra_weights[row * p.extra_top + k];
+#pragma unroll
+          for (int i = 0; i < VPT; ++i) {
+            const int c = threadIdx.x + i * THREADS;
+            if (c < nvec) {
+              const float4 y = load4(p.extra, er + c * 4, p.extra_fp32);
+              v[i].x = fmaf(w, y.x, v[i].x), v[i].y = fmaf(w, y.y, v[i].y);
+              v[i].z = fmaf(w, y.z, v[i].z), v[i].w = fmaf(w, y.w, v[i].w);
+            }
+          }
+        }
+      }
+    }
     if (p.w1) {
       if (EXT && p.groups > 1) group_norm_row<THREADS, VPT>(v, p.w1, p.H, nvec, p.groups, p.eps, part);
       else norm_row<THREADS, VPT>(v, p.w1, p.b1, p.H, nvec, p.eps, p.center, red);
@@ -314,9 +338,55 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const long long* __re
   if (out_b) store4(out_b, (size_t)t * ld_b + c, out_fp32, v);
 }
 
+// Token pair embedding: x[t] = table[id] + pairs[row], row = (previous id * mul_prev + id * mul_cur) mod buckets, or `buckets` at
+// the first position of a sequence. Every token files its id in the paged token cache; a sequence's first token of a step finds
+// its predecessor there, the others in `ids`.
+struct PairEmbedParams {
+  const long long* ids;
+  const void *table, *pairs;       // [vocab, Hp], [buckets + 1, Hp], both fp32 or bf16
+  int fp32, vocab;
+  long long mul_prev, mul_cur, buckets;
+  const int* positions;
+  const long long* slots;          // row of the token cache, < 0: none
+  int* tokens;                     // [blocks * block_size]
+  const int* block_table;
+  int max_blocks, block_size;
+  const int* cu_q;                 // [num_seqs + 1] or null (uniform_q tokens each)
+  int num_seqs, uniform_q;
+  float* x;
+  int T, Hp;
+};
+
+__global__ void __launch_bounds__(128) stream_embed_pairs_kernel(const PairEmbedParams p) {
+  pdl_launch_dependents();
+  pdl_wait(TL_EMBED);
+  const int t = blockIdx.x, pos = p.positions[t];
+  const long long id = p.ids[t];
+  long long row = p.buckets;
+  if (pos > 0) {
+    const int seq = seq_of_token(p.cu_q, p.num_seqs, p.uniform_q, t), q0 = p.cu_q ? p.cu_q[seq] : seq * p.uniform_q;
+    long long prev;
+    if (t > q0) {
+      prev = p.ids[t - 1];
+    } else {
+      const int page = p.block_table[(size_t)seq * p.max_blocks + (pos - 1) / p.block_size];
+      prev = p.tokens[(size_t)page * p.block_size + (pos - 1) % p.block_size];
+    }
+    row = (prev * p.mul_prev + id * p.mul_cur) % p.buckets;
+    if (row < 0) row += p.buckets;
+  }
+  if (threadIdx.x == 0 && p.slots[t] >= 0) p.tokens[p.slots[t]] = (int)id;
+  const bool known = id >= 0 && id < p.vocab;
+  for (int c = threadIdx.x * 4; c < p.Hp; c += 512) {
+    const float4 a = known ? load4(p.table, (size_t)id * p.Hp + c, p.fp32) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 b = load4(p.pairs, (size_t)row * p.Hp + c, p.fp32);
+    *reinterpret_cast<float4*>(p.x + (size_t)t * p.Hp + c) = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+  }
+}
+
 template <int THREADS, int VPT>
 int launch_sn(const StreamNormParams& p, int T, cudaStream_t s) {
-  if (p.groups <= 1 && !p.x_in && !p.hist)
+  if (p.groups <= 1 && !p.x_in && !p.hist && !p.extra)
     return launch_kernel(stream_norm_kernel<THREADS, VPT, false>, dim3((unsigned)T), dim3(THREADS), 0, s, p);
   size_t smem = 0;
   if (p.groups > 1) smem = (p.H / p.groups) % 128 == 0 ? THREADS / 32 * VPT * sizeof(float) : (size_t)(p.Hp + p.groups) * sizeof(float);
@@ -339,9 +409,11 @@ int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch,
                     const int* branch_rows, int branch_top, float branch_weight, const float* w1, const float* b1,
                     const float* w2, const float* b2, void* out, int ldo, int out_fp32, const int* out_rows, int out_top,
                     int T, int H, int Hp, float eps, float out_scale, int center, int groups, const void* x_in, void* hist,
-                    long long hist_stride, int n_hist, const float* mix, void* stream) {
+                    long long hist_stride, int n_hist, const float* mix, const void* extra, int ld_extra, int extra_fp32,
+                    const int* extra_rows, const float* extra_weights, int extra_top, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
+  if (extra && (!branch || (ld_extra % 4) || !extra_rows || !extra_weights || extra_top <= 0)) return -3;
   if (groups < 1 || H % groups || (groups > 1 && (center || b1 || b2)) || (hist && (!mix || !branch || n_hist < 0 || (hist_stride % 4))) ||
       (rows && (x_in || hist)))
     return -3;
@@ -374,6 +446,8 @@ int swb_stream_norm(void* x, int ldx, const long long* rows, const void* branch,
   p.hist_stride = hist_stride;
   p.n_hist = n_hist;
   p.mix = mix;
+  p.extra = extra, p.ld_extra = ld_extra, p.extra_fp32 = extra_fp32;
+  p.extra_rows = extra_rows, p.extra_weights = extra_weights, p.extra_top = extra_top;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int nvec = Hp / 4;
   if (nvec <= 128) return launch_sn<128, 1>(p, T, s);
@@ -395,6 +469,20 @@ int swb_stream_embed(const long long* ids, const void* table, int table_fp32, in
   return launch_kernel(stream_embed_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0,
                        reinterpret_cast<cudaStream_t>(stream), ids, table, table_fp32, vocab,
                        reinterpret_cast<float*>(x), ldx, out_a, ld_a, out_b, ld_b, out_fp32, scale, T, Hp);
+}
+
+// See PairEmbedParams; x [T, Hp] fp32, rows 16-byte aligned, Hp a multiple of 8.
+int swb_stream_embed_pairs(const long long* ids, const void* table, const void* pairs, int fp32, int vocab, long long mul_prev,
+                           long long mul_cur, long long buckets, const int* positions, const long long* slots, int* tokens,
+                           const int* block_table, int max_blocks, int block_size, const int* cu_q, int num_seqs, int uniform_q,
+                           float* x, int T, int Hp, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if ((Hp % 8) || buckets < 1 || num_seqs < 1 || block_size < 1 || !tokens || !block_table || !slots || (!cu_q && (long long)num_seqs * uniform_q != T))
+    return -3;
+  const PairEmbedParams p{ids, table, pairs, fp32, vocab, mul_prev, mul_cur, buckets, positions, slots, tokens, block_table, max_blocks,
+                          block_size, cu_q, num_seqs, uniform_q, x, T, Hp};
+  return launch_kernel(stream_embed_pairs_kernel, dim3((unsigned)T), dim3(128), 0, reinterpret_cast<cudaStream_t>(stream), p);
 }
 
 }  // extern "C"

@@ -60,6 +60,15 @@ class LatentGeometry:
 
 
 @dataclass(frozen=True)
+class TokenGeometry:
+    """Pages of token ids, for models whose input at a position depends on the ids in front of it. Paged like keys, so that rollbacks,
+    forks and shared prefixes need nothing else."""
+
+    def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
+        return [(block_size,)]
+
+
+@dataclass(frozen=True)
 class StateGeometry:
     """Recurrent layer: per sequence a fp32 state and a window of recent inputs in the activation type; no pages."""
     state: tuple[int, ...]
@@ -71,12 +80,12 @@ class StateGeometry:
 
 class LayeredKvPool:
     """Paged pool of a model whose layers differ in what they keep, or run more than once: every run owns its page tensors
-    [blocks, ...] (K and V, or latent rows). Block ids are shared by all runs (one allocator), so sequences, forks and
+    [blocks, ...] (K and V, latent rows, or token ids). Block ids are shared by all runs (one allocator), so sequences, forks and
     rollbacks work as on the uniform pool. Recurrent layers own tensors [state_slots, ...] instead; a sequence holds one slot
     for all of them from its first token to its release. A slot needs no clearing: the kernels take the state of a sequence
     as zero at position 0."""
 
-    def __init__(self, geometry: list[KvGeometry | LatentGeometry | StateGeometry], num_blocks: int, block_size: int = 16,
+    def __init__(self, geometry: list[KvGeometry | LatentGeometry | TokenGeometry | StateGeometry], num_blocks: int, block_size: int = 16,
                  device: torch.device | str = "cuda", dtype: torch.dtype = torch.bfloat16, state_slots: int = 0):
         self.geometry, self.num_layers = list(geometry), len(geometry)
         self.num_blocks, self.block_size = num_blocks, block_size
@@ -88,7 +97,8 @@ class LayeredKvPool:
             if isinstance(g, StateGeometry):
                 return (torch.zeros((state_slots, *g.state), dtype=torch.float32, device=device),
                         torch.zeros((state_slots, *g.window), dtype=dtype, device=device))
-            return tuple(torch.zeros((num_blocks, *s), dtype=dtype, device=device) for s in g.page_shapes(block_size))
+            kind = torch.int32 if isinstance(g, TokenGeometry) else dtype
+            return tuple(torch.zeros((num_blocks, *s), dtype=kind, device=device) for s in g.page_shapes(block_size))
         self.data = [tensors(g) for g in geometry]
         self.allocator = BlockAllocator(num_blocks)
         self.slots = BlockAllocator(state_slots) if self.has_state else None
@@ -111,7 +121,7 @@ class LayeredKvPool:
 
     @staticmethod
     def block_bytes(geometry, block_size: int = 16, elem: int = 2) -> int:
-        return sum(math.prod(s) for g in geometry for s in g.page_shapes(block_size)) * elem
+        return sum(math.prod(s) * (4 if isinstance(g, TokenGeometry) else elem) for g in geometry for s in g.page_shapes(block_size))
 
 
 class PagedSequence:

@@ -5,6 +5,7 @@ parsing and defaults), :540-596 (RoPE construction, GQA groups, attention scale)
 """
 from __future__ import annotations
 
+import dataclasses
 import enum
 import json
 import math
@@ -27,6 +28,7 @@ class Architecture(enum.Enum):
     QWEN35 = "qwen3_5"       # hybrid Gated-DeltaNet / gated full attention
     QWEN3_VL = "qwen3_vl"    # VLM-wrapped Qwen3 decoder with interleaved M-RoPE
     ZOBUNEX = "zobunex"      # listed layers with a loop, chunked sink attention, sandwich layer norms, token-routed experts
+    ROTALORN = "rotalorn"    # listed layers with parallel sublayers: windowed, latent and differential attention, dense / routed experts
     GUNEDRA = "gunedra"      # listed layers: latent attention and channel-wise delta rule, output norms, depth averages
 
     @staticmethod
@@ -79,7 +81,7 @@ class Architecture(enum.Enum):
         return self in (Architecture.GEMMA2, Architecture.GLM4)
 
 
-LISTED = (Architecture.ZOBUNEX, Architecture.GUNEDRA)     # designs whose config lists the layers one by one
+LISTED = (Architecture.ZOBUNEX, Architecture.GUNEDRA, Architecture.ROTALORN)     # designs whose config lists the layers one by one
 
 
 @dataclass(frozen=True)
@@ -137,8 +139,9 @@ class RopeSpec:
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    """One attention mixer: `rot_dims` leading dimensions of q and k are rotated, `chunk` > 0 limits a query to the keys of
-    its own run of `chunk` positions, `scale` multiplies the scores."""
+    """One attention mixer: `rot_dims` leading dimensions of q and k are rotated (frequencies rescaled by `rot_scaling`), `chunk` > 0
+    limits a query to the keys of its own run of `chunk` positions, `window` > 0 to the last `window` keys (its own included), `scale`
+    multiplies the scores."""
     heads: int
     kv_heads: int
     dim: int
@@ -147,6 +150,8 @@ class AttentionSpec:
     chunk: int
     rot_dims: int
     rot_base: float
+    rot_scaling: RopeScaling | None = None
+    window: int = 0
 
     @property
     def groups(self) -> int:
@@ -156,7 +161,8 @@ class AttentionSpec:
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Latent attention: keys and values of every head are projections of one cached vector of `kv_rank` numbers per token;
-    `rot_dim` further query / key dimensions are rotated, their key part is shared by the heads."""
+    `rot_dim` further query / key dimensions are rotated, their key part is shared by the heads. q_rank > 0: queries come out of a normed
+    latent of that size. `window` as in AttentionSpec."""
     heads: int
     dim: int
     rot_dim: int
@@ -164,6 +170,9 @@ class LatentAttentionSpec:
     kv_rank: int
     scale: float
     rot_base: float
+    q_rank: int = 0
+    window: int = 0
+    rot_scaling: RopeScaling | None = None
 
     @property
     def kv_heads(self) -> int:
@@ -172,6 +181,26 @@ class LatentAttentionSpec:
     @property
     def groups(self) -> int:
         return self.heads
+
+
+@dataclass(frozen=True)
+class DifferentialSpec:
+    """Differential attention: two softmax maps per head with q / k of `dim` each over the same values, the second one's result subtracted
+    with a learned share (offset `diff`). No rotation; queries grow with the position p by 1 + temp_coef ln(floor((p + 1) / temp_every) +
+    1), scores s become softcap tanh(s / softcap)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float
+    diff: float
+    temp_coef: float
+    temp_every: float
+
+    @property
+    def groups(self) -> int:
+        return 2 * (self.heads // self.kv_heads)     # query rows that meet one row of keys
 
 
 @dataclass(frozen=True)
@@ -194,6 +223,7 @@ class ExpertsSpec:
     experts: int
     top: int
     ff: int
+    shared: int = 0      # feed-forward width of an expert that every token uses
 
 
 @dataclass(frozen=True)
@@ -203,8 +233,17 @@ class DenseSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | LatentAttentionSpec | ChannelDeltaSpec
+    mixer: AttentionSpec | LatentAttentionSpec | DifferentialSpec | ChannelDeltaSpec
     mlp: ExpertsSpec | DenseSpec | None
+
+
+@dataclass(frozen=True)
+class BigramSpec:
+    """Every token adds the row (previous id * mul_prev + id * mul_cur) mod buckets of a table to its embedding, a sequence's first
+    token the row `buckets`."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
@@ -232,6 +271,46 @@ def _real(d: Any, key: str, where: str) -> float:
     if isinstance(v, bool) or not isinstance(v, (int, float)):
         raise ConfigError(f"config.json: `{where}{key}` must be a number, not {v!r}")
     return float(v)
+
+
+def _rot_scaling(rot: Any, at: str) -> RopeScaling | None:
+    s = rot.get("scaling")
+    if s is None:
+        return None
+    at += "rot.scaling."
+    out = RopeScaling(_real(s, "factor", at), _real(s, "low", at), _real(s, "high", at), _real(s, "original", at))
+    if out.factor <= 0 or out.low_freq_factor <= 0 or out.high_freq_factor <= out.low_freq_factor:
+        raise ConfigError(f"config.json: `{at}` needs factor > 0 and high > low > 0")
+    return out
+
+
+def _window(m: Any, at: str) -> int:
+    return _count(m["mask"], "size", at + "mask.") if m.get("mask") else 0
+
+
+def _windowed_spec(m: Any, at: str) -> AttentionSpec:
+    """Grouped heads whose values are the projected keys, within a window."""
+    rot = m.get("rot") or {"dims": 0, "base": 1.0}
+    spec = AttentionSpec(_count(m, "heads", at), _count(m, "kv_heads", at), _count(m, "dim", at), _count(m, "vdim", at), _real(m, "scale", at), 0,
+                         _count(rot, "dims", at + "rot.", 0), _real(rot, "base", at + "rot."), _rot_scaling(rot, at), _window(m, at))
+    if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim or spec.vdim != spec.dim:
+        raise ConfigError(f"config.json: `{at}` heads / kv_heads / dim / vdim / rot.dims do not fit together")
+    return spec
+
+
+def _low_rank_latent_spec(m: Any, at: str) -> LatentAttentionSpec:
+    s = _latent_spec(m, at)
+    return dataclasses.replace(s, q_rank=_count(m, "q_rank", at), window=_window(m, at), rot_scaling=_rot_scaling(m["rot"], at))
+
+
+def _differential_spec(m: Any, at: str) -> DifferentialSpec:
+    temp = m.get("q_temp") or {"coef": 0.0, "every": 1}
+    spec = DifferentialSpec(_count(m, "heads", at), _count(m, "kv_heads", at), _count(m, "dim", at), _count(m, "vdim", at), _real(m, "scale", at),
+                            _real(m, "softcap", at) if m.get("softcap") is not None else 0.0, _real(m, "diff", at),
+                            _real(temp, "coef", at + "q_temp."), _real(temp, "every", at + "q_temp."))
+    if spec.heads % spec.kv_heads or spec.softcap < 0 or spec.temp_every <= 0:
+        raise ConfigError(f"config.json: `{at}` heads / kv_heads / softcap / q_temp.every do not fit together")
+    return spec
 
 
 def _attention_spec(m: Any, at: str) -> AttentionSpec:
@@ -267,6 +346,13 @@ def _experts_spec(f: Any, at: str) -> ExpertsSpec:
                        _count(_need(f, "expert", at), "ff", at + "expert."))
 
 
+def _shared_experts_spec(f: Any, at: str) -> ExpertsSpec:
+    s = dataclasses.replace(_experts_spec(f, at), shared=_count(_need(f, "shared", at), "ff", at + "shared."))
+    if s.top > s.experts:
+        raise ConfigError(f"config.json: `{at}router.top` is above the number of experts")
+    return s
+
+
 def _dense_spec(f: Any, at: str) -> DenseSpec:
     return DenseSpec(_count(f, "ff", at))
 
@@ -275,6 +361,8 @@ def _dense_spec(f: Any, at: str) -> DenseSpec:
 _LAYER_PARTS = {
     Architecture.ZOBUNEX: ({"attention": _attention_spec}, {"moe": _experts_spec}),
     Architecture.GUNEDRA: ({"latent_attention": _latent_spec, "channel_delta": _channel_delta_spec}, {"dense": _dense_spec}),
+    Architecture.ROTALORN: ({"attention": _windowed_spec, "latent_attention": _low_rank_latent_spec, "attention_2": _differential_spec},
+                            {"dense": _dense_spec, "moe": _shared_experts_spec}),
 }
 
 
@@ -286,6 +374,7 @@ class StackConfig:
     logit_scale: float
     embed_scale: float = 1.0       # the embedding rows enter the stream times this
     residual_mult: float = 1.0     # every sublayer's result joins the stream times this
+    bigram: BigramSpec | None = None
     norm_groups: int = 1           # the stream norms take the root mean square of this many equal parts separately
 
     def runs(self) -> list[tuple[int, bool]]:
@@ -320,7 +409,11 @@ class StackConfig:
             if width % groups:
                 raise ConfigError("config.json: `norm.groups` does not divide `width`")
             return StackConfig(tuple(layers), None, 1.0, _real(_need(top, "embedding", ""), "scale", "embedding."),
-                               _real(top, "residual_mult", ""), groups)
+                               _real(top, "residual_mult", ""), norm_groups=groups)
+        if arch is Architecture.ROTALORN:
+            b, at = _need(_need(top, "embedding", ""), "bigram", "embedding."), "embedding.bigram."
+            return StackConfig(tuple(layers), None, 1.0, bigram=BigramSpec(_count(b, "buckets", at), _count(b, "mul_prev", at, 0),
+                                                                           _count(b, "mul_cur", at, 0)))
         loop, lp = None, top.get("loop")
         if lp:
             loop = LoopSpec(_count(lp, "start", "loop.", 0), _count(lp, "stop", "loop.", 0), _count(lp, "times", "loop."))
@@ -548,6 +641,24 @@ def _plain_inv_freq(dim: int, theta: float) -> list[float]:
     return [1.0 / theta ** ((2 * i) / dim) for i in range(dim // 2)]
 
 
+def rescale_frequencies(freqs: list[float], rs: RopeScaling) -> list[float]:
+    """Llama-3 frequency bands: wavelengths above original / low are stretched by `factor`, those below original / high stay, and between
+    the two the frequencies are mixed."""
+    low_wl = rs.original_context / rs.low_freq_factor
+    high_wl = rs.original_context / rs.high_freq_factor
+    out = []
+    for inv in freqs:
+        wl = 2.0 * math.pi / inv
+        if wl > low_wl:
+            out.append(inv / rs.factor)
+        elif wl < high_wl:
+            out.append(inv)
+        else:
+            smooth = (rs.original_context / wl - rs.low_freq_factor) / (rs.high_freq_factor - rs.low_freq_factor)
+            out.append((1.0 - smooth) * inv / rs.factor + smooth * inv)
+    return out
+
+
 def build_rope(cfg: ModelConfig) -> RopeSpec:
     """Inverse-frequency table for the configured RoPE variant (standard, partial / interleaved, Llama-3
     frequency-band scaling, YaRN). Parity: candle-llm/src/primitives/rope.rs:35-170, config.rs:540-575."""
@@ -575,16 +686,5 @@ def build_rope(cfg: ModelConfig) -> RopeSpec:
     rs = cfg.rope_scaling
     if rs is None:
         return RopeSpec(tuple(base), cfg.head_dim, False)
-    low_wl = rs.original_context / rs.low_freq_factor
-    high_wl = rs.original_context / rs.high_freq_factor
-    out = []
-    for inv in base:
-        wl = 2.0 * math.pi / inv
-        if wl > low_wl:
-            out.append(inv / rs.factor)
-        elif wl < high_wl:
-            out.append(inv)
-        else:
-            smooth = (rs.original_context / wl - rs.low_freq_factor) / (rs.high_freq_factor - rs.low_freq_factor)
-            out.append((1.0 - smooth) * inv / rs.factor + smooth * inv)
+    out = rescale_frequencies(base, rs)
     return RopeSpec(tuple(out), cfg.head_dim, False)

@@ -27,26 +27,9 @@ from ..engine.kv_pool import LatentGeometry, StateGeometry
 from ..ops import Branch, DeltaWeights, DepthAverage, LatentWeights, NormWeights
 from ..parallel.comm import Communicator
 from .config import ChannelDeltaSpec, LatentAttentionSpec, LayerSpec, ModelConfig
+from .latent_mixer import LatentDecoder, Ragged
 from .llama import StepInputs
-from .stack import StackDecoder, up8
-
-
-def _up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
-
-
-@dataclass
-class _Ragged:
-    """Sequences of a step that take one attention path. `rows` int32: their tokens, or None when they are all of the step."""
-    n: int
-    tokens: int
-    max_q: int
-    max_kv: int
-    seqs: torch.Tensor | None = None
-    rows: torch.Tensor | None = None
-    cu: torch.Tensor | None = None       # token offsets among `rows` (few) or key-row offsets (many); None when not needed
-    keys: int = 0
-    q_row: torch.Tensor | None = None    # int32 [T]: index in `rows` of each token, -1: not one of them
+from .stack import up8
 
 
 @dataclass
@@ -67,7 +50,7 @@ class _Layer:
     ff: int = 0
 
 
-class GunedraGpu(StackDecoder):
+class GunedraGpu(LatentDecoder):
     name = "Gunedra"
 
     def __init__(self, cfg: ModelConfig, comm: Communicator | None = None, device: torch.device | None = None,
@@ -77,16 +60,11 @@ class GunedraGpu(StackDecoder):
         for i, lay in enumerate(self.stack.layers):
             if isinstance(lay.mixer, ChannelDeltaSpec) and ops.delta_key_width(lay.mixer.dim) is None:
                 raise Unsupported(f"layer {i}: key width {lay.mixer.dim} of the delta rule is above 512")
-            if isinstance(lay.mixer, LatentAttentionSpec) and ops.latent_width(self._latent_widths(lay.mixer)[2], lay.mixer.rot_dim) > 1024:
-                raise Unsupported(f"layer {i}: a cached row of {lay.mixer.kv_rank} + {lay.mixer.rot_dim} is above 1024")
+            if isinstance(lay.mixer, LatentAttentionSpec):
+                self._check_latent(i, lay.mixer)
         self.layers: list[_Layer] = []
 
     # ---- cache geometry and scheduling hooks ------------------------------------------------------------------------
-    @staticmethod
-    def _latent_widths(m: LatentAttentionSpec) -> tuple[int, int, int, int]:
-        """Padded dim, rot_dim, kv_rank, vdim."""
-        return _up(m.dim, 16), up8(m.rot_dim), _up(m.kv_rank, 64), _up(m.vdim, 16)
-
     def kv_geometry(self) -> list:
         out = []
         for lay in self.stack.layers:
@@ -99,16 +77,8 @@ class GunedraGpu(StackDecoder):
         return out
 
     def decode_splits(self, batch: int, max_kv: int) -> tuple[int, ...]:
-        """KV splits per layer: about one CTA per SM, no split below two 64-key tiles."""
-        def splits(m) -> int:
-            if not isinstance(m, LatentAttentionSpec):
-                return 1
-            blocks = batch * ((m.heads + 31) // 32)
-            want, s = min(148 // blocks, (max_kv + 127) // 128, 32), 1
-            while s * 2 <= want:
-                s *= 2
-            return s
-        return tuple(splits(lay.mixer) for lay in self.stack.layers)
+        return tuple(self._latent_splits(lay.mixer, batch, max_kv) if isinstance(lay.mixer, LatentAttentionSpec) else 1
+                     for lay in self.stack.layers)
 
     def rotations(self) -> set[tuple[int, float]]:
         return {(lay.mixer.rot_dim, lay.mixer.rot_base) for lay in self.stack.layers if isinstance(lay.mixer, LatentAttentionSpec)}
@@ -160,34 +130,10 @@ class GunedraGpu(StackDecoder):
             self.layers.append(lay)
         return self
 
-    def _heads(self, t: torch.Tensor, n: int, parts: list[tuple[int, int]], cols: int | None = None) -> torch.Tensor:
-        """Rows laid out head by head in parts of the given (size, padded size) -> the same with every part padded; columns
-        padded to `cols` (default: the stream's padded width)."""
-        t = t.to(self.device, self.dtype).reshape(n, sum(a for a, _ in parts), -1)
-        out = torch.zeros((n, sum(b for _, b in parts), cols or self.hp), dtype=self.dtype, device=self.device)
-        src = dst = 0
-        for a, b in parts:
-            out[:, dst:dst + a, :t.shape[2]] = t[:, src:src + a]
-            src, dst = src + a, dst + b
-        return out.reshape(-1, out.shape[2])
-
-    def _out(self, o: torch.Tensor, heads: int, d: int, dp: int) -> torch.Tensor:
-        out = torch.zeros((self.hp, heads, dp), dtype=self.dtype, device=self.device)
-        out[:self.width, :, :d] = o.to(self.device, self.dtype).reshape(self.width, heads, d)
-        return out.reshape(self.hp, heads * dp)
-
     def _latent_layer(self, spec: LayerSpec, p: str, get, norm1: NormWeights, dwa: torch.Tensor) -> _Layer:
-        m, W = spec.mixer, self.width
-        H, R, dn, rp, rk, vp = m.heads, m.kv_rank, *self._latent_widths(m)
-        w_in = torch.cat([self._heads(get(p + "q", H * (m.dim + m.rot_dim), W), H, [(m.dim, dn), (m.rot_dim, rp)]),
-                          self._heads(get(p + "dkv", R + m.rot_dim, W), 1, [(R, rk), (m.rot_dim, rp)]),
-                          self._heads(get(p + "g", H, W), 1, [(H, up8(H))])])
-        uk = self._heads(get(p + "uk", H * m.dim, R), H, [(m.dim, dn)], rk).view(H, dn, rk)
-        uv = self._heads(get(p + "uv", H * m.vdim, R), H, [(m.vdim, vp)], rk).view(H, vp, rk)
-        latent = LatentWeights(H, m.dim, dn, m.rot_dim, rp, R, rk, m.vdim, vp, m.scale, self._fp32(get(p + "dkv.norm", R), rk),
-                               self._fp32(get(p + "sink", H)), torch.cat([uk.view(H * dn, rk), uv.view(H * vp, rk)]),
-                               uk.transpose(1, 2).contiguous())
-        return _Layer(norm1, dwa, w_in, self._out(get(p + "o", W, H * m.vdim), H, m.vdim, vp), latent=latent,
+        m = spec.mixer
+        w_in, latent = self._latent_weights(m, p, get, sink=self._fp32(get(p + "sink", m.heads)))
+        return _Layer(norm1, dwa, w_in, self._out(get(p + "o", self.width, m.heads * m.vdim), m.heads, m.vdim, latent.vp), latent=latent,
                       rope=(m.rot_dim, m.rot_base))
 
     def _delta_layer(self, spec: LayerSpec, p: str, get, norm1: NormWeights, dwa: torch.Tensor) -> _Layer:
@@ -217,87 +163,11 @@ class GunedraGpu(StackDecoder):
         return sum(t.nbytes for t in ts)
 
     # ---- forward --------------------------------------------------------------------------------------------------------
-    few_tokens = 16      # measured on B200: up to so many tokens of a sequence attend in the latent space
-
-    def _split_step(self, inp: StepInputs) -> tuple[_Ragged | None, _Ragged | None]:
-        """(few, many): sequences with few new tokens attend in the latent space, where all heads share the cached rows; for the
-        others expanding the latents into keys and values of every head costs less than it saves. A decode step, and 32-bit
-        mode, is all few."""
-        T, S = inp.input_ids.numel(), inp.num_seqs
-        spans = inp.spans
-        if spans is None:
-            return _Ragged(S, T, inp.max_q_len, 0, cu=inp.cu_q), None
-        limit = self.few_tokens if self.dtype == torch.bfloat16 else max(q for q, _ in spans)
-        few, many = [i for i in range(S) if spans[i][0] <= limit], [i for i in range(S) if spans[i][0] > limit]
-        dev_i32 = lambda v: torch.tensor(v, dtype=torch.int32).to(self.device, non_blocking=True)   # noqa: E731
-        starts = [0]
-        for q, _ in spans:
-            starts.append(starts[-1] + q)
-
-        def ragged(ids: list[int], is_many: bool) -> _Ragged | None:
-            if not ids:
-                return None
-            r = _Ragged(len(ids), sum(spans[i][0] for i in ids), max(spans[i][0] for i in ids), max(spans[i][1] for i in ids))
-            if len(ids) < S:
-                r.seqs = dev_i32(ids)
-            if is_many:
-                if len(ids) < S or any(q != n for q, n in spans):       # earlier context: keys come from the cache
-                    ends = [0]
-                    for i in ids:
-                        ends.append(ends[-1] + spans[i][1])
-                    r.cu, r.keys = dev_i32(ends), ends[-1]
-            elif len(ids) < S:
-                rows = [t for i in ids for t in range(starts[i], starts[i + 1])]
-                q_row, ends = [-1] * T, [0]
-                for k, t in enumerate(rows):
-                    q_row[t] = k
-                for i in ids:
-                    ends.append(ends[-1] + spans[i][0])
-                r.rows, r.q_row, r.cu = dev_i32(rows), dev_i32(q_row), dev_i32(ends)
-            else:
-                r.cu = inp.cu_q
-            return r
-        return ragged(few, False), ragged(many, True)
-
-    def _latent(self, lay: _Layer, h: torch.Tensor, inp: StepInputs, kv, splits: int, few: _Ragged | None,
-                many: _Ragged | None) -> torch.Tensor:
-        w, T, cache, dev = lay.latent, h.shape[0], kv[0], self.device
-        proj = self._linear(h, lay.w_in)
-        cos, sin = self._rope[lay.rope]
-        table, lens, fast = inp.block_table, inp.kv_lens, self.dtype == torch.bfloat16
-        cu_q = inp.cu_q
-        if many is not None and not ops.latent_prefill_supported(w):
-            # heads wider than the prefill kernel: everything attends in the latent space
-            few, many = _Ragged(inp.num_seqs, T, inp.max_q_len, max(n for _, n in inp.spans), cu=cu_q), None
-        q_abs = torch.empty((few.tokens, w.heads, w.width), dtype=self.dtype, device=dev) if few is not None else None
-        ops.latent_prep(proj, w, self.cfg.rms_norm_eps, cos, sin, inp.positions, inp.slot_mapping, cache, q_abs,
-                        few.q_row if few is not None else None)
-        gate = proj[:, w.col_gate:w.col_gate + w.heads]
-        a = torch.empty((T, w.heads, w.vp), dtype=self.dtype, device=dev)
-        self.launches += 1
-        if many is not None:
-            if cu_q is None:
-                cu_q = torch.arange(inp.num_seqs + 1, dtype=torch.int32, device=dev) * inp.max_q_len
-            rows = proj[:, w.col_c:w.col_gate]
-            if many.cu is not None:
-                rows = ops.latent_gather(cache, table, many.cu, many.keys, many.seqs)
-                self.launches += 1
-            expanded = self._linear(rows[:, :w.rk], w.ukv)
-            ops.latent_prefill(proj[:, :w.col_c], expanded, rows[:, w.rk:w.rk + w.rp], w, a.view(T, -1), cu_q=cu_q, max_q_len=many.max_q, gate=gate,
-                               seqs=many.seqs, cu_k=many.cu)
-            self.launches += 1
-        if few is not None:
-            q = proj[:, :w.col_c].view(T, w.heads, w.dn + w.rp)[..., :w.dn]
-            ops.head_product(q, w.uk_t, q_abs[..., :w.rk], rows_in=few.rows, rows_out=None)
-            if few.seqs is not None:
-                table, lens = table[few.seqs], lens[few.seqs]
-            ragged = dict(cu_q=few.cu, max_q_len=few.max_q)
-            if fast and ops.latent_decode_supported(w, cache.shape[1]):
-                lat = ops.latent_decode(q_abs, cache, table, lens, w, num_splits=splits, **ragged)
-            else:
-                lat = ops.latent_attention_simple(q_abs, cache, table, lens, w, **ragged)
-            ops.head_product(lat, w.uv, a, gate=gate, sink=w.sink, rows_out=few.rows)
-            self.launches += 3
+    def _latent(self, lay: _Layer, h: torch.Tensor, inp: StepInputs, kv, splits: int, few: Ragged | None,
+                many: Ragged | None) -> torch.Tensor:
+        w, T = lay.latent, h.shape[0]
+        a = torch.empty((T, w.heads, w.vp), dtype=self.dtype, device=self.device)
+        self._latent_attend(w, lay.rope, self._linear(h, lay.w_in), inp, kv[0], splits, few, many, a)
         return self._linear(a.view(T, -1), lay.o)
 
     def _delta(self, lay: _Layer, h: torch.Tensor, inp: StepInputs, kv) -> torch.Tensor:

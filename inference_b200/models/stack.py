@@ -7,7 +7,7 @@ from .. import ops
 from ..contracts.errors import LoadError, Unsupported
 from ..engine.kv_pool import LayeredKvPool
 from ..parallel.comm import Communicator, single
-from .config import ModelConfig
+from .config import ModelConfig, rescale_frequencies
 
 
 def up8(n: int) -> int:
@@ -34,7 +34,7 @@ class StackDecoder:
         self.width, self.hp = cfg.hidden_size, up8(cfg.hidden_size)
         self.layers: list = []
         self.embed = self.final = None
-        self._rope: dict[tuple[int, float], tuple[torch.Tensor, torch.Tensor]] = {}
+        self._rope: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
         self.max_positions = 0
         self.launches = 0
 
@@ -50,16 +50,19 @@ class StackDecoder:
 
     # ---- rotary tables --------------------------------------------------------------------------------------------
     def rotations(self) -> set[tuple[int, float]]:
-        """(rotated dimensions, base) of every layer that rotates."""
+        """(rotated dimensions, base) or (rotated dimensions, base, rescaling) of every layer that rotates."""
         raise NotImplementedError
 
     def ensure_rope(self, max_positions: int) -> None:
         if max_positions <= self.max_positions:
             return
-        for dims, base in self.rotations():
-            i = torch.arange(dims // 2, dtype=torch.float64)
-            ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * (base ** (-2.0 * i / max(dims, 1)))[None, :]
-            self._rope[(dims, base)] = (ang.cos().float().to(self.device).contiguous(),
+        for key in self.rotations():
+            dims, base = key[:2]
+            freq = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+            if len(key) > 2 and key[2] is not None:
+                freq = rescale_frequencies(freq, key[2])
+            ang = torch.arange(max_positions, dtype=torch.float64)[:, None] * torch.tensor(freq, dtype=torch.float64)[None, :]
+            self._rope[key] = (ang.cos().float().to(self.device).contiguous(),
                                         ang.sin().float().to(self.device).contiguous())
         self.max_positions = max_positions
 
@@ -82,13 +85,29 @@ class StackDecoder:
         t = t.to(self.device, torch.float32)
         return torch.nn.functional.pad(t, (0, (pad_to or t.shape[-1]) - t.shape[-1])).contiguous()
 
+    def _heads(self, t: torch.Tensor, n: int, parts: list[tuple[int, int]], cols: int | None = None) -> torch.Tensor:
+        """Rows laid out head by head in parts of the given (size, padded size) -> the same with every part padded; columns
+        padded to `cols` (default: the stream's padded width)."""
+        t = t.to(self.device, self.dtype).reshape(n, sum(a for a, _ in parts), -1)
+        out = torch.zeros((n, sum(b for _, b in parts), cols or self.hp), dtype=self.dtype, device=self.device)
+        src = dst = 0
+        for a, b in parts:
+            out[:, dst:dst + a, :t.shape[2]] = t[:, src:src + a]
+            src, dst = src + a, dst + b
+        return out.reshape(-1, out.shape[2])
+
+    def _out(self, o: torch.Tensor, heads: int, d: int, dp: int) -> torch.Tensor:
+        out = torch.zeros((self.hp, heads, dp), dtype=self.dtype, device=self.device)
+        out[:self.width, :, :d] = o.to(self.device, self.dtype).reshape(self.width, heads, d)
+        return out.reshape(self.hp, heads * dp)
+
     # ---- forward ----------------------------------------------------------------------------------------------------
     def _linear(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
-                out: torch.Tensor | None = None) -> torch.Tensor:
+                out: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
         self.launches += 1
         if self.dtype == torch.float32:
-            return ops.gemm_f32(a, w, out=out)
-        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16)
+            return ops.gemm_f32(a, w, out=out, bias=bias)
+        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16, bias=bias)
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         if hidden.shape[0] == 0:

@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 
 import torch
 
@@ -131,31 +132,52 @@ def varlen_causal_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, c
     return out
 
 
+@dataclass
+class Differential:
+    """Differential attention: two softmax maps per head over the same values, o = N(a1 - share a2) post, N the RMS norm over the head's
+    first `width` value columns. softcap > 0: scores s become softcap tanh(s / softcap). q_temp fp32 [positions]: factor of a query's
+    scores in front of the cap."""
+    share: float
+    post: float
+    eps: float
+    width: int
+    softcap: float = 0.0
+    q_temp: torch.Tensor | None = None
+
+
 def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor,
                     kv_lens: torch.Tensor, *, cu_q: torch.Tensor | None, max_q_len: int, scale: float, chunk: int = 0,
-                    sink: torch.Tensor | None = None, decode: bool = False, num_splits: int = 1,
-                    fresh_kv: tuple[torch.Tensor, torch.Tensor] | None = None, kernel: str = "auto") -> torch.Tensor:
-    """Causal paged attention with head widths of its own for q / k (D) and v (Dv), optional chunked masking and sinks.
+                    sink: torch.Tensor | None = None, decode: bool = False, num_splits: int = 1, window: int = 0,
+                    fresh_kv: tuple[torch.Tensor, torch.Tensor] | None = None, diff: Differential | None = None,
+                    out: torch.Tensor | None = None, kernel: str = "auto") -> torch.Tensor:
+    """Causal paged attention with head widths of its own for q / k (D) and v (Dv), optional chunked or windowed masking and sinks.
 
     q [T, Hq, D] (heads contiguous), caches [blocks, Hkv, block_size, D] and [blocks, Hkv, block_size, Dv], block_table /
     kv_lens / cu_q as in paged_attention -> [T, Hq * Dv]. chunk > 0: position i sees j <= i only when both lie in the same
-    run of `chunk` positions, counted from the start of the sequence. sink fp32 [Hq]: exp(sink) joins each head's softmax
-    denominator. fresh_kv = (k [T, Hkv, D], v [T, Hkv, Dv]) strided views: every sequence starts in this step, so a prefill
-    reads its keys there instead of the pages.
+    run of `chunk` positions, counted from the start of the sequence. window > 0: position i sees only 0 <= i - j < window. sink
+    fp32 [Hq]: exp(sink) joins each head's softmax denominator. diff: q [T, Hq, 2, D / 2], the two maps' keys side by side in each
+    key row, the result combined. fresh_kv = (k [T, Hkv, D], v [T, Hkv, Dv]) strided views: every sequence starts in this step, so a
+    prefill reads its keys there instead of the pages.
     bf16 widths that are multiples of 8 up to 128 run on the tcgen05 kernel (prefill) or the TMA-fed decode kernel; other
     widths, fp32 and non-positive scales on the plain fp32-arithmetic kernel (kernel="simple" forces it)."""
-    require_cuda(q, kcache, vcache, block_table, kv_lens, sink)
-    T, Hq, D = q.shape
-    nblk, Hkv, bs, Dk = kcache.shape
+    require_cuda(q, kcache, vcache, block_table, kv_lens, sink, out)
+    maps = 1 if diff is None else 2
+    T, Hq = q.shape[:2]
+    nblk, Hkv, bs, D = kcache.shape
     Dv = vcache.shape[3]
-    assert Dk == D and vcache.shape[:3] == kcache.shape[:3] and kcache.is_contiguous() and vcache.is_contiguous()
-    assert q.stride(2) == 1 and q.stride(1) == D and q.dtype == kcache.dtype == vcache.dtype
+    assert vcache.shape[:3] == kcache.shape[:3] and kcache.is_contiguous() and vcache.is_contiguous()
+    assert q.shape[2:] == ((D,) if diff is None else (2, D // 2)) and q.stride(-1) == 1 and q.stride(1) == D
+    assert q.dtype == kcache.dtype == vcache.dtype and (diff is None or (D % 2 == 0 and q.stride(2) == D // 2))
     assert block_table.dtype == torch.int32 and kv_lens.dtype == torch.int32 and block_table.stride(1) == 1
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == Hq and sink.is_contiguous())
+    temp = diff.q_temp if diff is not None else None
+    assert temp is None or (temp.is_cuda and temp.dtype == torch.float32 and temp.is_contiguous())
     num_seqs = kv_lens.numel()
-    out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
-    if q.dtype == torch.bfloat16 and kernel == "auto" and scale > 0 and max(D, Dv) <= 128 and D % 8 == 0 and Dv % 8 == 0:
-        decode = decode and max_q_len * (Hq // Hkv) <= 16 and bs == 16
+    if out is None:
+        out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
+    assert out.shape == (T, Hq * Dv) and out.stride(1) == 1 and out.dtype == q.dtype
+    if q.dtype == torch.bfloat16 and kernel == "auto" and scale > 0 and max(D, Dv) <= 128 and D % (8 * maps) == 0 and Dv % 8 == 0:
+        decode = decode and max_q_len * maps * (Hq // Hkv) <= 16 and bs == 16
         ws_ptr, ws_bytes, k, v, ks, vs, table = None, 0, kcache, vcache, 0, 0, block_table
         if decode and num_splits > 1:
             ws = decode_workspace(q.device, kernels().swb_attn_decode_workspace_bytes(num_seqs, Hkv, num_splits))
@@ -167,16 +189,24 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                 k, v = fresh_kv
                 assert k.stride(2) == 1 and v.stride(2) == 1 and k.stride(1) == D and v.stride(1) == Dv
                 ks, vs, table = k.stride(0), v.stride(0), None
+        d = diff or Differential(0.0, 1.0, 0.0, Dv)
         rc = kernels().swb_attn_ext(q.data_ptr(), q.stride(0), k.data_ptr(), ks, v.data_ptr(), vs, out.data_ptr(),
                                     out.stride(0), ptr(table), block_table.stride(0), bs, nblk, ptr(cu_q),
                                     kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq, Hkv, D, Dv, scale, chunk, ptr(sink),
-                                    1 if decode else 0, num_splits, ws_ptr, ws_bytes, stream_ptr())
+                                    1 if decode else 0, num_splits, ws_ptr, ws_bytes, window, 0 if diff is None else 1, d.share, d.eps, d.post,
+                                    d.softcap, ptr(temp), d.width, stream_ptr())
         if rc != -3:
             check(rc, "swb_attn_ext")
             return out
-    rc = kernels().swb_attn_simple(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), out.data_ptr(),
-                                   out.stride(0), block_table.data_ptr(), block_table.stride(0), bs, ptr(cu_q),
-                                   kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq, Hkv, D, Dv, 0, scale, chunk, ptr(sink),
+    res = out if diff is None else torch.empty((T, Hq, 2, Dv), dtype=q.dtype, device=q.device)
+    rc = kernels().swb_attn_simple(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), res.data_ptr(),
+                                   res.stride(0), block_table.data_ptr(), block_table.stride(0), bs, ptr(cu_q),
+                                   kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq * maps, Hkv, D // maps, Dv, 0, scale, chunk, ptr(sink),
+                                   window, diff.softcap if diff is not None else 0.0, ptr(temp), maps,
                                    1 if q.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_attn_simple")
+    if diff is not None:
+        from .llm import diff_combine
+
+        diff_combine(res, out, diff.share, diff.eps, diff.post, diff.width)
     return out

@@ -119,7 +119,7 @@ def gated_fused(T: int, N: int, K: int) -> bool:
     return bool(kernels().swb_gemm_gated_supported(T, N, K))
 
 
-def linear_gated(x: torch.Tensor, w_pairs: torch.Tensor, act: str = "silu") -> torch.Tensor:
+def linear_gated(x: torch.Tensor, w_pairs: torch.Tensor, act: str = "silu", out: torch.Tensor | None = None) -> torch.Tensor:
     """act(x W_gate^T) * (x W_up^T) for a gate-up weight whose rows are interleaved (gate_0, up_0, gate_1, ...).
 
     Decode-sized token counts apply the gated activation in the GEMM's epilogue (the reference runs the projection,
@@ -132,9 +132,11 @@ def linear_gated(x: torch.Tensor, w_pairs: torch.Tensor, act: str = "silu") -> t
     N = w_pairs.shape[0]
     gelu = act in ("gelu", "gelu_tanh")
     if kernels().swb_gemm_gated_supported(T, N, K):
-        y = gemm_bf16(x2, w_pairs, act="geglu_pairs" if gelu else "swiglu_pairs")
+        y = gemm_bf16(x2, w_pairs, act="geglu_pairs" if gelu else "swiglu_pairs", out=out)
     else:
-        y = gated_act_mul(gemm_bf16(x2, w_pairs), act, paired=True)
+        y = gated_act_mul(gemm_bf16(x2, w_pairs), act, paired=True, out=out)
+    if out is not None:
+        return out
     return y.reshape(*x.shape[:-1], N // 2)
 
 
@@ -145,20 +147,21 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *
     return y.reshape(*lead, w.shape[0])
 
 
-def gemm_f32(a: torch.Tensor, w: torch.Tensor, *, act: str | None = None, out: torch.Tensor | None = None,
+def gemm_f32(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = None, act: str | None = None, out: torch.Tensor | None = None,
              offsets: torch.Tensor | None = None, src: torch.Tensor | None = None, rows: int | None = None) -> torch.Tensor:
-    """True 32-bit product (no TF32): out[T, N] = act(a[T, K] @ w[N, K]^T). Grouped: w [G, N, K], offsets int32 [G + 1] on
+    """True 32-bit product (no TF32): out[T, N] = act(a[T, K] @ w[N, K]^T + bias). Grouped: w [G, N, K], offsets int32 [G + 1] on
     the device, rows [offsets[g], offsets[g + 1]) use w[g] and read a[src[r]] (r itself without src); `rows` bounds them."""
     require_cuda(a, w)
     assert a.dtype == torch.float32 and w.dtype == torch.float32 and a.stride(1) == 1 and w.is_contiguous()
     G = w.shape[0] if offsets is not None else 1
     N, K = w.shape[-2:]
     T = rows if rows is not None else a.shape[0]
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous())
     assert a.shape[1] == K and (w.dim() == 3) == (offsets is not None)
     if out is None:
         out = torch.empty((T, N), dtype=torch.float32, device=a.device)
     assert out.shape == (T, N) and out.dtype == torch.float32 and out.stride(1) == 1
     rc = kernels().swb_gemm_f32(a.data_ptr(), a.stride(0), ptr(src), ptr(offsets), G, w.data_ptr(), K, out.data_ptr(),
-                                out.stride(0), T, N, K, ACT[act], stream_ptr())
+                                out.stride(0), T, N, K, ACT[act], ptr(bias), stream_ptr())
     check(rc, "swb_gemm_f32")
     return out

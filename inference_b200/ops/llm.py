@@ -90,19 +90,59 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: torc
 
 
 def gated_act_mul(gate_up: torch.Tensor, act: str = "silu", out: torch.Tensor | None = None,
-                  paired: bool = False) -> torch.Tensor:
+                  paired: bool = False, row_gate: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f] (SwiGLU / GeGLU, candle-llm models/llama.rs:1386-1391).
-    paired: the projection's rows are interleaved (gate_0, up_0, gate_1, ...), out[t, f] = act(gu[t, 2f]) * gu[t, 2f+1]."""
-    require_cuda(gate_up)
+    paired: the projection's rows are interleaved (gate_0, up_0, gate_1, ...), out[t, f] = act(gu[t, 2f]) * gu[t, 2f+1].
+    row_gate fp32 [T] logits (strided): row t is scaled by their sigmoid. bf16 or fp32."""
+    require_cuda(gate_up, row_gate)
     g2 = gate_up.reshape(-1, gate_up.shape[-1])
     T, F2 = g2.shape
     F = F2 // 2
     if out is None:
         out = torch.empty((T, F), dtype=gate_up.dtype, device=gate_up.device)
-    rc = kernels().swb_gated_act_mul(g2.data_ptr(), g2.stride(0), out.data_ptr(), out.stride(0), T, F,
-                                     (2 if act in ("gelu", "gelu_tanh") else 1) + (2 if paired else 0), stream_ptr())
+    assert g2.stride(1) == 1 and out.stride(1) == 1 and out.shape == (T, F) and out.dtype == g2.dtype
+    assert row_gate is None or (row_gate.dtype == torch.float32 and row_gate.shape == (T,))
+    rc = kernels().swb_gated_act_mul_ex(g2.data_ptr(), g2.stride(0), out.data_ptr(), out.stride(0), T, F,
+                                        (2 if act in ("gelu", "gelu_tanh") else 1) + (2 if paired else 0), ptr(row_gate),
+                                        row_gate.stride(0) if row_gate is not None else 0, 1 if g2.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_gated_act_mul")
-    return out.reshape(*gate_up.shape[:-1], F)
+    return out.reshape(*gate_up.shape[:-1], F) if gate_up.dim() != 2 else out
+
+
+def row_rope_kv_write(buf: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, n_heads: int,
+                      n_kv_heads: int, head_dim: int, *, v_col: int = 0, rope: tuple[torch.Tensor, torch.Tensor] | None = None,
+                      q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, norm_counts: tuple[int, int] = (0, 0),
+                      eps: float = 0.0, v_from_k: bool = False, store_v: bool = False) -> None:
+    """In place on buf [T, >= (Hq + Hkv) * D]: RMS norms over the whole q and the whole k of a token (fp32 weights q_norm [Hq * D] and
+    k_norm [Hkv * D]; norm_counts: how many numbers enter each mean, the rest being zero padding), then rotation of the leading dimensions
+    of every head in neighbouring pairs (rope = cos and sin tables fp32 [positions, rot / 2]). k and v go to the paged caches [blocks, Hkv,
+    block_size, D | Dv] at `slots` (int64, -1 = skip). Values are the columns from v_col on, or with v_from_k the keys as projected, which
+    store_v also copies there. Without norm and rotation the queries are left alone. bf16 or fp32 throughout."""
+    require_cuda(buf, positions, slots, kcache, vcache, q_norm, k_norm)
+    T, Dv = buf.shape[0], vcache.shape[-1]
+    assert buf.stride(1) == 1 and kcache.dtype == vcache.dtype == buf.dtype and kcache.is_contiguous() and vcache.is_contiguous()
+    assert kcache.shape[-1] == head_dim and kcache.shape[1] == n_kv_heads and positions.dtype == torch.int32 and slots.dtype == torch.int64
+    for w, n in ((q_norm, n_heads), (k_norm, n_kv_heads)):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == n * head_dim and w.is_contiguous())
+    cos, sin = rope if rope is not None else (None, None)
+    rc = kernels().swb_row_rope_kv_write(buf.data_ptr(), buf.stride(0), v_col, n_heads, n_kv_heads, head_dim, Dv,
+                                         0 if cos is None else 2 * cos.shape[-1], ptr(q_norm), ptr(k_norm), norm_counts[0], norm_counts[1], eps,
+                                         ptr(cos), ptr(sin), positions.data_ptr(), slots.data_ptr(), kcache.data_ptr(), vcache.data_ptr(),
+                                         kcache.shape[2], 1 if v_from_k else 0, 1 if store_v else 0, T, 1 if buf.dtype == torch.float32 else 0,
+                                         stream_ptr())
+    check(rc, "swb_row_rope_kv_write")
+
+
+def diff_combine(maps: torch.Tensor, out: torch.Tensor, share: float, eps: float, post: float, width: int | None = None) -> torch.Tensor:
+    """Differential attention: out[t, h] = post * N(maps[t, h, 0] - share * maps[t, h, 1]) with N(y) = y / sqrt(mean(y^2) + eps) over the first
+    `width` columns. maps [T, H, 2, Dv] (contiguous per token), out [T, H * Dv] strided; bf16 or fp32."""
+    require_cuda(maps, out)
+    T, H, _, Dv = maps.shape
+    assert maps.is_contiguous() and out.shape == (T, H * Dv) and out.stride(1) == 1 and out.dtype == maps.dtype
+    rc = kernels().swb_diff_combine(maps.data_ptr(), maps.stride(0), out.data_ptr(), out.stride(0), T, H, Dv, width or Dv, share, eps, post,
+                                    1 if maps.dtype == torch.float32 else 0, stream_ptr())
+    check(rc, "swb_diff_combine")
+    return out
 
 
 def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, width: int | None = None, out: torch.Tensor | None = None) -> torch.Tensor:

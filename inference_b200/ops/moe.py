@@ -1,4 +1,4 @@
-"""Mixture-of-experts pieces whose routing is known before the layer runs (csrc/kernels/moe_routed.cu)."""
+"""Mixture-of-experts pieces: routing plans from a table or from router logits, grouped products (csrc/kernels/moe_routed.cu)."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -23,6 +23,8 @@ class RoutingPlan:
     offsets: torch.Tensor | None = None
     active: torch.Tensor | None = None
     tile_group: torch.Tensor | None = None
+    weights: torch.Tensor | None = None      # fp32 [T, top] (logits routing)
+    ahead: bool = False                      # planned at the start of the step (table routing)
 
     @property
     def padded(self) -> bool:
@@ -50,7 +52,44 @@ def table_routing(ids: torch.Tensor, tables: torch.Tensor, num_experts: int, *, 
                                       stream_ptr())
     check(rc, "swb_moe_table_plan")
     return [RoutingPlan(dest[i], rows, src[i] if src is not None else None, offsets[i],
-                        active[i] if active is not None else None, tiles[i] if tiles is not None else None) for i in range(L)]
+                        active[i] if active is not None else None, tiles[i] if tiles is not None else None, ahead=True) for i in range(L)]
+
+
+_COUNTERS: dict[int, torch.Tensor] = {}
+
+
+def _counters(device: torch.device) -> torch.Tensor:
+    """Per-device counters of the routing kernels, zero between launches."""
+    idx = device.index if device.index is not None else torch.cuda.current_device()
+    if idx not in _COUNTERS:
+        _COUNTERS[idx] = torch.zeros(4096 + 2, dtype=torch.int32, device=device)
+    return _COUNTERS[idx]
+
+
+def logits_routing(logits: torch.Tensor, num_experts: int, top: int, *, rows: torch.Tensor | None = None) -> tuple[RoutingPlan, torch.Tensor | None]:
+    """Softmax router: the `top` experts of the largest scores per token, weighted by these scores as they are. logits fp32 [T, >=
+    num_experts]. Without `rows` a dense plan; with rows [T, H] a padded plan and the rows copied to their places in the expert-sorted
+    buffer."""
+    require_cuda(logits, rows)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= num_experts >= top
+    T, E, dev, padded = logits.shape[0], num_experts, logits.device, rows is not None
+    pairs = T * top
+    cap = (pairs + E * (TILE - 1) + TILE - 1) // TILE * TILE if padded else pairs
+
+    def ints(*shape):
+        return torch.empty(shape, dtype=torch.int32, device=dev)
+    dest, offsets, scratch = ints(T, top), ints(E + 1), ints(2, pairs)
+    weights = torch.empty((T, top), dtype=torch.float32, device=dev)
+    src, active, tiles = (None, None, ints(cap // TILE)) if padded else (ints(cap), ints(min(E, pairs)), None)
+    buf = torch.empty((cap, rows.shape[1]), dtype=rows.dtype, device=dev) if padded else None
+    per = 16 // rows.element_size() if padded else 1
+    assert not padded or (rows.stride(1) == 1 and rows.stride(0) % per == 0 and rows.shape[1] % per == 0)
+    rc = kernels().swb_moe_route(logits.data_ptr(), logits.stride(0), T, E, top, TILE if padded else 1, scratch[0].data_ptr(),
+                                 scratch[1].data_ptr(), weights.data_ptr(), _counters(dev).data_ptr(), dest.data_ptr(), ptr(src),
+                                 offsets.data_ptr(), ptr(active), ptr(tiles), cap, ptr(rows), rows.stride(0) // per if padded else 0, ptr(buf),
+                                 rows.shape[1] // per if padded else 0, rows.shape[1] // per if padded else 0, stream_ptr())
+    check(rc, "swb_moe_route")
+    return RoutingPlan(dest, cap, src, offsets, active, tiles, weights), buf
 
 
 def gemm_grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: RoutingPlan, *, gather: bool, act: str | None = None) -> torch.Tensor:
@@ -59,10 +98,10 @@ def gemm_grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: RoutingPlan, *, ga
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and x.stride(1) == 1
     E, N, K = w.shape
     assert x.shape[1] == K and not plan.padded
-    out = torch.empty((plan.rows, N), dtype=torch.bfloat16, device=x.device)
+    out = torch.empty((plan.rows, N // 2 if act in ("swiglu_pairs", "geglu_pairs") else N), dtype=torch.bfloat16, device=x.device)
     rc = kernels().swb_gemm_grouped_rows(x.data_ptr(), x.stride(0), plan.src.data_ptr() if gather else None,
                                          plan.offsets.data_ptr(), plan.active.data_ptr(), plan.active.numel(), w.data_ptr(),
-                                         out.data_ptr(), out.stride(0), N, K, ACT[act], stream_ptr())
+                                         out.data_ptr(), out.stride(0), N, K, ACT[act], 1 if plan.ahead else 0, stream_ptr())
     check(rc, "swb_gemm_grouped_rows")
     return out
 
@@ -76,3 +115,17 @@ def routed_ffn(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, plan: Rout
     if plan.padded:
         return gemm_bf16_grouped(gemm_bf16_grouped(h, up, plan.tile_group, act=act), down, plan.tile_group)
     return gemm_grouped_rows(gemm_grouped_rows(h, up, plan, gather=True, act=act), down, plan, gather=False)
+
+
+def routed_gated_ffn(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, plan: RoutingPlan, act: str) -> torch.Tensor:
+    """Expert outputs [plan.rows, H] in the plan's row order: down_e(act(gate_e x) * (up_e x)). gate_up [E, 2 F, H] with its rows in
+    (gate, up) pairs, down [E, H, F]; h as in routed_ffn."""
+    from .llm import gated_act_mul
+
+    if h.dtype == torch.float32:
+        u = gated_act_mul(gemm_f32(h, gate_up, offsets=plan.offsets, src=plan.src, rows=plan.rows), act, paired=True)
+        return gemm_f32(u, down, offsets=plan.offsets, rows=plan.rows)
+    if plan.padded:
+        return gemm_bf16_grouped(gated_act_mul(gemm_bf16_grouped(h, gate_up, plan.tile_group), act, paired=True), down, plan.tile_group)
+    pairs = "geglu_pairs" if act in ("gelu", "gelu_tanh") else "swiglu_pairs"
+    return gemm_grouped_rows(gemm_grouped_rows(h, gate_up, plan, gather=True, act=pairs), down, plan, gather=False)

@@ -17,14 +17,23 @@ class NormWeights:
 
 
 @dataclass
+class RoutedRows:
+    """Expert outputs: token t gets the sum over k of weights[t, k] y[rows[t, k]]; rows int32, weights fp32, both [T, top]."""
+    y: torch.Tensor
+    rows: torch.Tensor
+    weights: torch.Tensor
+
+
+@dataclass
 class Branch:
     """A sublayer output that has not joined the stream yet: rows [*, Hp] in bf16 / fp32, normed on the way in. With
-    `rows` (int32 [T, top]) the branch of token t is the sum of y[rows[t, k]] over k times `weight`."""
+    `rows` (int32 [T, top]) the branch of token t is the sum of y[rows[t, k]] over k times `weight`. `extra` is added to it."""
     y: torch.Tensor
     norm: NormWeights | None
     rows: torch.Tensor | None = None
     top: int = 1
     weight: float = 1.0
+    extra: RoutedRows | None = None
 
 
 @dataclass
@@ -49,7 +58,11 @@ def stream_norm(x: torch.Tensor, width: int, eps: float, *, branch: Branch | Non
     T = rows.numel() if rows is not None else x.shape[0]
     assert x.dtype == torch.float32 and x.stride(1) == 1
     b, w1, w2 = branch, (branch.norm if branch is not None else None), norm
-    for t in (b.y if b is not None else None, out):
+    ex = b.extra if b is not None else None
+    if ex is not None:
+        assert ex.rows.dtype == torch.int32 and ex.weights.dtype == torch.float32 and ex.rows.is_contiguous() and ex.weights.is_contiguous()
+        assert ex.rows.shape == ex.weights.shape and ex.rows.shape[0] == T
+    for t in (b.y if b is not None else None, out, ex.y if ex is not None else None):
         assert t is None or (t.stride(1) == 1 and t.shape[1] == Hp and t.dtype in (torch.bfloat16, torch.float32))
     for n in (w1, w2):
         assert n is None or (n.w.dtype == torch.float32 and n.w.numel() == Hp and n.w.is_contiguous())
@@ -66,7 +79,9 @@ def stream_norm(x: torch.Tensor, width: int, eps: float, *, branch: Branch | Non
         ptr(out), out.stride(0) if out is not None else 0, 1 if out is not None and out.dtype == torch.float32 else 0,
         ptr(out_rows), out_top, T, width, Hp, eps, out_scale, 1 if center else 0, groups, ptr(x_in),
         ptr(av.results) if av is not None else None, av.results.stride(0) if av is not None else 0, av.filled if av is not None else 0,
-        ptr(av.weights) if av is not None else None, stream_ptr())
+        ptr(av.weights) if av is not None else None, ptr(ex.y) if ex is not None else None, ex.y.stride(0) if ex is not None else 0,
+        1 if ex is not None and ex.y.dtype == torch.float32 else 0, ptr(ex.rows) if ex is not None else None,
+        ptr(ex.weights) if ex is not None else None, ex.rows.shape[1] if ex is not None else 0, stream_ptr())
     check(rc, "swb_stream_norm")
     return out
 
@@ -90,4 +105,25 @@ def stream_embed(ids: torch.Tensor, table: torch.Tensor, *, copies: list[torch.T
                                     1 if c[0] is not None and c[0].dtype == torch.float32 else 0, scale, T, Hp,
                                     stream_ptr())
     check(rc, "swb_stream_embed")
+    return x
+
+
+def stream_embed_pairs(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, mul_prev: int, mul_cur: int, *, positions: torch.Tensor,
+                       slots: torch.Tensor, tokens: torch.Tensor, block_table: torch.Tensor, cu_q: torch.Tensor | None, num_seqs: int,
+                       max_q_len: int) -> torch.Tensor:
+    """fp32 rows table[id] + pairs[(previous id * mul_prev + id * mul_cur) mod buckets]; a sequence's first token takes the last row
+    of `pairs` [buckets + 1, Hp]. tokens int32 [blocks, block_size]: paged cache of the ids, in which every token files its own and
+    the first token of a sequence in this step finds its predecessor."""
+    require_cuda(ids, table, pairs, positions, slots, tokens, block_table, cu_q)
+    assert ids.dtype == torch.int64 and table.is_contiguous() and pairs.is_contiguous() and table.dtype == pairs.dtype
+    assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and tokens.dtype == torch.int32 and tokens.is_contiguous()
+    assert block_table.dtype == torch.int32 and block_table.stride(1) == 1 and pairs.shape[1] == table.shape[1]
+    flat = ids.reshape(-1)
+    T, Hp = flat.numel(), table.shape[1]
+    x = torch.empty((T, Hp), dtype=torch.float32, device=table.device)
+    rc = kernels().swb_stream_embed_pairs(flat.data_ptr(), table.data_ptr(), pairs.data_ptr(), 1 if table.dtype == torch.float32 else 0,
+                                          table.shape[0], mul_prev, mul_cur, pairs.shape[0] - 1, positions.data_ptr(), slots.data_ptr(),
+                                          tokens.data_ptr(), block_table.data_ptr(), block_table.stride(0), tokens.shape[1], ptr(cu_q),
+                                          num_seqs, max_q_len, x.data_ptr(), T, Hp, stream_ptr())
+    check(rc, "swb_stream_embed_pairs")
     return x
