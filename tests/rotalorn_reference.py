@@ -148,6 +148,12 @@ def route(h, router, top):
     return e, w
 
 
+def margin(h, router, top):
+    """How far the last chosen expert's logit is above the first one left out (infinite when all are chosen)."""
+    z = (h @ router.T).sort(-1, descending=True).values
+    return z[:, top - 1] - z[:, top] if top < z.shape[1] else torch.full((len(h),), math.inf, dtype=F)
+
+
 def mixture(h, W, p, f):
     """Routed experts plus the gated shared one."""
     e, w = route(h, W[p + "router"], f["router"]["top"])
@@ -161,8 +167,8 @@ def mixture(h, W, p, f):
 MIXERS = {"attention": attention, "latent_attention": latent_attention, "attention_2": differential_attention}
 
 
-def run(cfg, weights, tokens):
-    """Whole sequence at once: (logits [T, vocab], residual stream after every layer)."""
+def run(cfg, weights, tokens, margins=None):
+    """Whole sequence at once: (logits [T, vocab], residual stream after every layer). `margins` collects the routers' margins."""
     W = {k: t.to(F) for k, t in weights.items()}
     eps, trail = cfg["norm"]["eps"], []
     norm = lambda x, n: layer_norm(x, W[n], W[n + ".b"], eps)   # noqa: E731
@@ -170,6 +176,8 @@ def run(cfg, weights, tokens):
     for i, lay in enumerate(cfg["layers"]):
         L, f = f"l{i}.", lay["mlp"]
         h = norm(x, L + "norm1")
+        if margins is not None and f is not None and f["kind"] == "moe":
+            margins.append(margin(h, W[L + "mlp.router"], f["router"]["top"]))
         y = MIXERS[lay["type"]](h, W, L + "mix.", lay["mixer"], eps)
         if f is not None:
             y = y + (gated(h, W, L + "mlp.", gelu) if f["kind"] == "dense" else mixture(h, W, L + "mlp.", f))
