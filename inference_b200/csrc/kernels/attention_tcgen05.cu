@@ -166,6 +166,11 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
+// tanh(x) / x on |x| <= 1 as a polynomial in x^2: a least-squares fit reweighted towards equal ripples; |error of tanh| < 2.4e-7.
+constexpr float TANH_0 = 0.99999685f, TANH_1 = -0.33324004f, TANH_2 = 0.13253525f, TANH_3 = -0.05097286f, TANH_4 = 0.01611418f,
+                TANH_5 = -0.00283947f;
+constexpr float MAX_FIXED_CAP = 64.f;      // sums of exp(cap) over 2^20 keys stay finite in fp32
+
 struct Barriers {
   uint64_t q_full;
   uint64_t k_full[MAX_STAGES], k_empty[MAX_STAGES];
@@ -183,8 +188,9 @@ struct Barriers {
 // columns that the tensor maps fill in). LAT adds what latent attention needs: two-part q / k, key ranges, output gates.
 // DIFF is differential attention: the two tiles of a CTA are the two softmax maps of the same 128 query rows. Each map's keys are
 // one 64-column atom of the K tile (columns of the other map that fall into it meet zero columns of q), the V tile serves both, and
-// the second map's result is handed to the first one's threads through shared memory for the difference and its norm.
-template <int QK, int VD, bool EXT, bool LAT, bool DIFF>
+// the second map's result is handed to the first one's threads through shared memory for the difference and its norm. DIFF 2 is for
+// caps up to MAX_FIXED_CAP: the scores are bounded, so the exponentials are taken as they are, without a running maximum.
+template <int QK, int VD, bool EXT, bool LAT, int DIFF>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                           const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_q2,
@@ -265,7 +271,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       mbar_arrive_expect_tx(&bars->q_full, DIFF ? 2 * ATOM_BYTES : p.tiles * TILE_BYTES);
       for (int q = 0; q < p.tiles; ++q)
         for (int a = 0; a < (DIFF ? 1 : ATOMS); ++a) {
-          if constexpr (DIFF) {
+          if constexpr (DIFF != 0) {
             tma_load_4d(smem + SMEM_Q + q * TILE_BYTES, &tmap_q, &bars->q_full, 0, 2 * head + q, tok0 + q_base, batch);
             continue;
           }
@@ -330,7 +336,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       const uint32_t q_addr = smem_u32(smem + SMEM_Q), k_addr = smem_u32(smem + SMEM_K),
                      v_addr = smem_u32(smem + SMEM_V);
       auto issue_qk = [&](int q, int s) {
-        if constexpr (DIFF) {
+        if constexpr (DIFF != 0) {
           for (int k = 0; k < (p.diff.dim + 15) / 16; ++k)
             umma_f16_ss(tmem + col_s[q], umma_desc_kmajor_sw128(q_addr + q * TILE_BYTES + k * 32),
                         umma_desc_kmajor_sw128(k_addr + s * TILE_BYTES + q * ATOM_BYTES + k * 32), IDESC_QK, k > 0);
@@ -391,7 +397,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
     const float cap = DIFF ? p.diff.cap : 0.f;
     float to_cap = 0.f;             // 2 log2(e) scale / cap: the capped score is cap (1 - 2 / (2^(to_cap s) + 1))
     float scale_log2 = p.scale_log2;
-    if constexpr (DIFF) {
+    if constexpr (DIFF != 0) {
       if (p.diff.q_temp && row < q_len) scale_log2 *= p.diff.q_temp[row + coff];
       if (cap > 0.f) to_cap = 2.f * scale_log2 / cap, scale_log2 = 1.4426950408889634f;
     }
@@ -405,6 +411,57 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) tmem_ld_x32(t_s + c * 32, s + c * 32);
       tmem_ld_wait();
+      if constexpr (DIFF == 2) {
+        const int key0 = (j + j0) * BN, last = q_base + BM - 1 + coff;
+        const float to_x = 0.34657359f * to_cap, k = 1.4426950408889634f * cap;       // x = score / cap; exponents in log2 units
+        float far0 = 0.f, far1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < BN; i += 2) {
+          const float x0 = __uint_as_float(s[i]) * to_x, x1 = __uint_as_float(s[i + 1]) * to_x;
+          far0 = fmaxf(far0, fabsf(x0)), far1 = fmaxf(far1, fabsf(x1));
+          s[i] = __float_as_uint(x0), s[i + 1] = __float_as_uint(x1);
+        }
+        const bool edge = key0 + BN > min(kv_len, q_base + 1 + coff) || key0 < first_key_of(last);     // some pair is masked
+        float l0 = 0.f, l1 = 0.f;
+        if (!edge && __all_sync(0xffffffffu, fmaxf(far0, far1) <= 1.f)) {
+          auto weight = [&](uint32_t u) {
+            const float x = __uint_as_float(u), t = x * x;
+            float r = fmaf(t, k * TANH_5, k * TANH_4);
+            r = fmaf(t, r, k * TANH_3);
+            r = fmaf(t, r, k * TANH_2);
+            r = fmaf(t, r, k * TANH_1);
+            r = fmaf(t, r, k * TANH_0);
+            return ex2(x * r);
+          };
+#pragma unroll
+          for (int i = 0; i < BN; i += 2) {
+            const float e0 = weight(s[i]), e1 = weight(s[i + 1]);
+            l0 += e0;
+            l1 += e1;
+            s[i >> 1] = pack_bf16x2(e0, e1);
+          }
+        } else {
+          const int last_rel = min(kv_len - 1, row + coff) - key0, first_rel = first_key_of(row + coff) - key0;
+          auto weight = [&](uint32_t u, int i) {
+            const float y = ex2(__uint_as_float(u) * 2.8853900818f) + 1.f;
+            return i > last_rel || i < first_rel ? 0.f : ex2(fmaf(-2.f * k, rcp_approx(y), k));
+          };
+#pragma unroll
+          for (int i = 0; i < BN; i += 2) {
+            const float e0 = weight(s[i], i), e1 = weight(s[i + 1], i + 1);
+            l0 += e0;
+            l1 += e1;
+            s[i >> 1] = pack_bf16x2(e0, e1);
+          }
+        }
+        l += l0 + l1;
+        tmem_st_x32(t_s, s);
+        tmem_st_x32(t_s + 32, s + 32);
+        tmem_st_wait();
+        tc_fence_before_sync();
+        mbar_arrive(&bars->p_full[q]);
+        continue;
+      }
       if (DIFF && cap > 0.f) {
 #pragma unroll
         for (int i = 0; i < BN; ++i)
@@ -477,7 +534,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       mbar_arrive(&bars->p_full[q]);
     }
     if (ok && my_tiles > 0) ok = mbar_wait(&bars->o_final, 0, abort_flag, 32 + q);
-    if constexpr (DIFF) ok = __all_sync(0xffffffffu, ok);      // the barrier below is taken warp by warp
+    if constexpr (DIFF != 0) ok = __all_sync(0xffffffffu, ok);      // the barrier below is taken warp by warp
     if (ok && my_tiles > 0) {
       tc_fence_after_sync();
       float inv = l > 0.f ? 1.f / l : 0.f;
@@ -498,7 +555,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       // VD / 8 lanes x 16 bytes: contiguous runs for local stores and for stores that cross NVLink alike.
       // 16-byte chunk c of row r sits at c ^ (r & 7).
       uint8_t* slab = smem + SMEM_Q + warp * (32 * ROW_BYTES);
-      if constexpr (DIFF) {
+      if constexpr (DIFF != 0) {
         // fp32 hand-over in the (idle) K region, row r of VD numbers, 16-byte chunk c at c ^ (r & 31 within the row's chunks)
         float4* hand = reinterpret_cast<float4*>(smem + SMEM_K) + (size_t)((warp & 3) * 32 + lane) * (VD / 4);
         const float f = q ? inv * p.diff.share : inv;
@@ -571,7 +628,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         }
       }
     }
-    if constexpr (DIFF) {          // the hand-over barrier takes all 256 threads, whatever became of the waits
+    if constexpr (DIFF != 0) {          // the hand-over barrier takes all 256 threads, whatever became of the waits
       if (q == 1 || !ok) asm volatile("bar.sync 1, 256;" ::: "memory");
     }
   }
@@ -667,7 +724,7 @@ struct FaMaps {
   CUtensorMap q, k, v, q2, k2;     // q2 / k2: second parts of latent attention
 };
 
-template <int QK, int VD, bool EXT, bool LAT, bool DIFF = false>
+template <int QK, int VD, bool EXT, bool LAT, int DIFF = 0>
 int launch_fa(dim3 grid, cudaStream_t stream, const FaMaps& m, const FaParams& p) {
   static bool configured[64] = {false};
   auto kernel = attn_dense_tcgen05_kernel<QK, VD, EXT, LAT, DIFF>;
@@ -689,7 +746,9 @@ int launch_tiles(int qk, FaKind kind, int q_len, int Hq, int batch, cudaStream_t
   // one-tile CTAs when that shortens the schedule: a one-tile CTA takes ~0.85 of a two-tile CTA's time (measured)
   if (kind == FaKind::DIFF) {
     p.tiles = 2;
-    return launch_fa<128, 128, true, false, true>(dim3((q_len + BM - 1) / BM, Hq, batch), stream, m, p);
+    const dim3 rows((q_len + BM - 1) / BM, Hq, batch);
+    return p.diff.cap > 0.f && p.diff.cap <= MAX_FIXED_CAP ? launch_fa<128, 128, true, false, 2>(rows, stream, m, p)
+                                                           : launch_fa<128, 128, true, false, 1>(rows, stream, m, p);
   }
   const int sms = 148;
   const long c2 = (long)((q_len + 2 * BM - 1) / (2 * BM)) * Hq * batch, c1 = (long)((q_len + BM - 1) / BM) * Hq * batch;
