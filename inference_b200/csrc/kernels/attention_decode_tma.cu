@@ -53,6 +53,13 @@ __device__ __forceinline__ float softmax_inv(const AttnParams& p, int head, floa
   return L > 0.f ? 1.f / L : 0.f;
 }
 
+// cap tanh(s scale / cap) in log2 units, tanh y = 1 - 2 / (e^(2 y) + 1); the absolute error is that of fp32 numbers of the size of cap
+__device__ __forceinline__ float capped_score(float s, float scale, float to_cap, float cap) {
+  if (cap <= 0.f) return s * (scale * 1.4426950408889634f);
+  const float k = 1.4426950408889634f * cap;
+  return fmaf(-2.f * k, __fdividef(1.f, exp2f(s * to_cap) + 1.f), k);
+}
+
 // Sums of up to eight values per thread over the 128 merging threads (warps 0-3); `red` holds 32 floats.
 __device__ __forceinline__ void sum_over_128(float* v, float* red, int n) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -198,6 +205,8 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 #pragma unroll
       for (int hr = 0; hr < 2; ++hr) row_scale[hr] *= p.diff.q_temp[min((g + hr * 8) / p.G, q_len - 1) + max(causal_shift, 0)];
     }
+    float row_cap[2] = {0.f, 0.f};         // 2 log2(e) scale / cap
+    if (DIFF && p.diff.cap > 0.f) row_cap[0] = 2.8853900818f * row_scale[0] / p.diff.cap, row_cap[1] = 2.8853900818f * row_scale[1] / p.diff.cap;
     for (int j = 0; j < n_tiles; ++j) {
       if (!mbar_wait(&bar_full[stage], phase, s_abort, 600 + stage)) break;
       const uint32_t sK = smem_u32(ring + stage * STAGE_BYTES);
@@ -220,7 +229,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
       for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float val = DIFF ? score_transform(s[nt][e], row_scale[e >> 1], p.diff.cap) : score_transform(s[nt][e], p.scale, p.softcap);
+          const float val = DIFF ? capped_score(s[nt][e], row_scale[e >> 1], row_cap[e >> 1], p.diff.cap) : score_transform(s[nt][e], p.scale, p.softcap);
           const int col = tok_base + nt * 8 + t4 * 2 + (e & 1);
           const int row = g + ((e >> 1) ? 8 : 0);
           const int qtok = row / p.G;
