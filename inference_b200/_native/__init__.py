@@ -81,6 +81,8 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
     sig("swb_gemm_workspace_min", [], c_size_t)
     sig("swb_gemm_bf16", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                           c_int, c_int, c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p])
+    sig("swb_gemm_bf16_act", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                              c_int, c_int, c_float, c_float, c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p])
     sig("swb_rmsnorm_prefetch", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                                  c_float, c_void_p, c_ll, c_void_p])
     sig("swb_rmsnorm", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float,
@@ -103,15 +105,21 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
                              c_float, c_int, c_int, c_void_p])
     sig("swb_moe_table_plan", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                c_void_p, c_void_p, c_int, c_void_p])
-    sig("swb_moe_route", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+    sig("swb_moe_route", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_void_p, c_int, c_void_p, c_ll, c_void_p, c_ll, c_int, c_void_p])
     sig("swb_gemm_grouped_rows", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                                  c_int, c_int, c_int, c_void_p])
+                                  c_int, c_int, c_float, c_int, c_void_p])
     sig("swb_gemm_f32", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                         c_int, c_void_p, c_void_p])
+                         c_int, c_float, c_float, c_void_p, c_void_p])
+    sig("swb_hyper_step", [c_void_p, c_void_p, c_ll, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p,
+                           c_void_p, c_void_p])
+    sig("swb_short_conv", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                           c_int, c_void_p])
+    sig("swb_head_mix", [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_attn_simple", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float,
-                            c_void_p, c_int, c_int, c_void_p])
+                            c_void_p, c_int, c_int, c_void_p, c_ll, c_int, c_void_p])
     sig("swb_head_product_simple", [c_void_p, c_ll, c_int, c_void_p, c_ll, c_int, c_int, c_void_p, c_ll, c_int, c_void_p, c_ll, c_int,
                                     c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_latent_gather", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p])
@@ -128,16 +136,18 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     sig("swb_delta_scan", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                            c_void_p, c_void_p])
-    sig("swb_delta_post", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p,
+    sig("swb_delta_post", [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p,
                            c_int, c_void_p, c_int, c_void_p])
     sig("swb_poly_norm", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p])
     sig("swb_attn_ext", [c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_ll, c_void_p, c_int, c_int, c_int,
                          c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
-                         c_int, c_int, c_void_p, c_size_t, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p, c_int, c_void_p])
+                         c_int, c_int, c_void_p, c_size_t, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p, c_int, c_int, c_void_p,
+                         c_ll, c_void_p])
     sig("swb_row_rope_kv_write", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float,
-                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                  c_void_p])
     sig("swb_diff_combine", [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p])
-    sig("swb_gated_act_mul_ex", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+    sig("swb_gated_act_mul_ex", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p])
     sig("swb_gated_act_mul", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_embedding", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
     sig("swb_gated_residual", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p])

@@ -17,10 +17,13 @@ extern "C" {
 // [13] partials delivered, [14] first group's sum of squares sent). Pass null to switch it off.
 void swb_gemm_set_trace(void* device_buffer) { swb::g_trace = reinterpret_cast<unsigned long long*>(device_buffer); }
 
-int swb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* D, int ldd, int T, int N, int K,
-                  const void* bias, const void* residual, int ld_res, int act, int out_fp32, void* workspace,
-                  size_t workspace_bytes, int force_mode, int force_block_n, int force_ctas, void* stream) {
+// act_a, act_b: parameters of activations that have any (see GemmAct).
+int swb_gemm_bf16_act(const void* A, int lda, const void* W, int ldw, void* D, int ldd, int T, int N, int K,
+                      const void* bias, const void* residual, int ld_res, int act, float act_a, float act_b, int out_fp32,
+                      void* workspace, size_t workspace_bytes, int force_mode, int force_block_n, int force_ctas, void* stream) {
   swb::GemmArgs a;
+  a.act_a = act_a;
+  a.act_b = act_b;
   a.A = A;
   a.lda = lda;
   a.W = W;
@@ -41,6 +44,13 @@ int swb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* D, int l
   a.force_block_n = force_block_n;
   a.force_ctas = force_ctas;
   return swb::gemm_bf16_launch(a, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int swb_gemm_bf16(const void* A, int lda, const void* W, int ldw, void* D, int ldd, int T, int N, int K,
+                  const void* bias, const void* residual, int ld_res, int act, int out_fp32, void* workspace,
+                  size_t workspace_bytes, int force_mode, int force_block_n, int force_ctas, void* stream) {
+  return swb_gemm_bf16_act(A, lda, W, ldw, D, ldd, T, N, K, bias, residual, ld_res, act, 0.f, 0.f, out_fp32, workspace,
+                           workspace_bytes, force_mode, force_block_n, force_ctas, stream);
 }
 
 // 3x3 convolution, stride 1, zero padding 1, over an NHWC bf16 activation x [n, h, w, c] as an implicit GEMM on the

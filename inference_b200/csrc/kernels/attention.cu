@@ -608,24 +608,28 @@ int swb_attn_paged_prefill_tc(const void* q, long long q_stride_tok, int q_strid
 // denominator. Widths: multiples of 8 up to 128. mode 0 = prefill (tcgen05 kernel, sequences from cu_q), 1 = decode
 // (TMA-fed kernel, block_size 16, max_q_len * Hq / Hkv <= 16, uniform q_len when cu_q is null). window > 0: query i sees only keys
 // j > i - window. diff (nullable) -> differential attention (DiffAttn): q [total_tokens, Hq, 2, D / 2], key rows of both maps side by
-// side, out [total_tokens, Hq, Dv] already combined; in decode 2 max_q_len * Hq / Hkv <= 16. Returns -3 when the problem is outside
-// the two kernels' reach.
+// side, out [total_tokens, Hq, Dv] already combined; in decode 2 max_q_len * Hq / Hkv <= 16. v_heads > 0: vcache [num_blocks, v_heads,
+// block_size, Dv], every query head is applied to all value heads, out [total_tokens, Hq, v_heads, Dv]. gate (nullable): logits in the
+// layout of the output, rows gate_stride apart; the output is scaled by their sigmoid. Returns -3 when the problem is outside the two
+// kernels' reach.
 int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long k_stride_tok, const void* v,
                  long long v_stride_tok, void* out, long long out_stride_tok, const int* block_table, int max_blocks,
                  int block_size, int num_blocks, const int* cu_q, const int* kv_lens, int num_seqs, int max_q_len,
                  int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink, int mode,
                  int num_splits, void* workspace, size_t workspace_bytes, int window, int diff, float share, float diff_eps,
-                 float post, float cap, const float* q_temp, int v_count, void* stream) {
+                 float post, float cap, const float* q_temp, int v_count, int v_heads, const void* gate, long long gate_stride,
+                 void* stream) {
   using namespace swb;
   if (num_seqs <= 0 || total_tokens <= 0) return 0;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (Hkv <= 0 || Hq % Hkv != 0 || max_q_len <= 0 || window < 0) return -3;
-  if (diff && (D % 16 || v_count < 1 || v_count > Dv || sink || chunk || cap < 0.f)) return -3;
+  if (v_heads < 0 || (gate && gate_stride % 8) || (reinterpret_cast<uintptr_t>(gate) & 15)) return -3;
+  if (diff && (v_heads || gate || D % 16 || v_count < 1 || v_count > Dv || sink || chunk || cap < 0.f)) return -3;
   const attn::DiffAttn da{diff ? 2 : 0, D / 2, v_count, share, diff_eps, post, cap, q_temp};
   if (mode == 0)
     return attn_ext_tcgen05_launch(q, q_stride_tok, k, k_stride_tok, v, v_stride_tok, out, out_stride_tok, num_seqs,
                                    max_q_len, total_tokens, Hq, Hkv, D, Dv, scale, chunk, sink, cu_q, kv_lens,
-                                   block_table, max_blocks, block_size, num_blocks, st, window, diff ? &da : nullptr);
+                                   block_table, max_blocks, block_size, num_blocks, st, window, diff ? &da : nullptr, v_heads, gate, gate_stride);
   const int per_kv = (diff ? 2 : 1) * (Hq / Hkv);
   if (D < 8 || Dv < 8 || D > HD || Dv > HD || (D % 8) || (Dv % 8) || block_size != 16 || !block_table || !kv_lens ||
       num_blocks <= 0 || max_q_len * per_kv > 16 || !(scale > 0.f) || chunk < 0 || (q_stride_tok % 8))
@@ -651,6 +655,9 @@ int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long
   p.G = per_kv;
   p.window = window;
   p.diff = da;
+  p.v_heads = v_heads;
+  p.gate = reinterpret_cast<const bf16*>(gate);
+  p.gate_stride = gate_stride;
   p.scale = scale;
   p.causal = 1;
   p.k_dim = D;
@@ -661,9 +668,10 @@ int swb_attn_ext(const void* q, long long q_stride_tok, const void* k, long long
   if (num_splits > 32) num_splits = 32;
   p.num_splits = num_splits;
   if (num_splits > 1) {
-    if (!workspace || workspace_bytes < swb_attn_decode_workspace_bytes(num_seqs, Hkv, num_splits)) return -5;
-    p.part_o = reinterpret_cast<float*>(reinterpret_cast<char*>(workspace) + attn_counter_bytes(num_seqs, Hkv));
-    p.part_ml = p.part_o + (size_t)num_seqs * Hkv * num_splits * 16 * HD;
+    const int problems = Hkv * (v_heads > 0 ? v_heads : 1);      // per sequence
+    if (!workspace || workspace_bytes < swb_attn_decode_workspace_bytes(num_seqs, problems, num_splits)) return -5;
+    p.part_o = reinterpret_cast<float*>(reinterpret_cast<char*>(workspace) + attn_counter_bytes(num_seqs, problems));
+    p.part_ml = p.part_o + (size_t)num_seqs * problems * num_splits * 16 * HD;
     p.split_counters = reinterpret_cast<int*>(workspace);
   }
   return attn_decode_tma_launch(p, num_blocks, st);

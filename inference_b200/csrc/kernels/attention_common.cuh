@@ -50,6 +50,9 @@ struct AttnParams {
   const float* sink;     // optional [Hq]: exp(sink[h]) joins the softmax denominator
   int window;            // > 0: a query sees only the last `window` keys, its own included
   DiffAttn diff;
+  int v_heads;           // > 0: every query head is applied to all `v_heads` value heads, out [token, Hq, v_heads, v_dim]
+  const bf16* gate;      // optional logits in the layout of a token's output, rows gate_stride apart: out is scaled by their sigmoid
+  long long gate_stride;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, uint32_t src_bytes) {
@@ -105,7 +108,8 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
                             long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
                             int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
                             const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
-                            int num_blocks, cudaStream_t stream, int window = 0, const attn::DiffAttn* diff = nullptr);
+                            int num_blocks, cudaStream_t stream, int window = 0, const attn::DiffAttn* diff = nullptr, int v_heads = 0,
+                            const void* gate = nullptr, long long gate_stride = 0);
 int attn_latent_tcgen05_launch(const void* q, long long q_stride_tok, const void* k, const void* v, long long kv_stride_tok,
                                const void* k2, long long k2_stride_tok, int key_rows, void* out, long long out_stride_tok,
                                int num_seqs, int max_q_len, int total_tokens, int H, int d1, int d2, int Dv, float scale,

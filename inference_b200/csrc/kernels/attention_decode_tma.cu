@@ -75,7 +75,7 @@ __device__ __forceinline__ void sum_over_128(float* v, float* red, int n) {
     if (i < n) v[i] = (red[i * 4] + red[i * 4 + 1]) + (red[i * 4 + 2] + red[i * 4 + 3]);
 }
 
-// EXT: chunked and windowed masking, sinks. FULL: q / k and v are HD wide (their loop bounds are then constants). DIFF: the two maps
+// EXT: chunked and windowed masking, sinks, output gates, values of every head (blockIdx.y then runs over key head, value head). FULL: q / k and v are HD wide (their loop bounds are then constants). DIFF: the two maps
 // of a head are neighbouring query rows, each zero outside its own columns of the key row, so that both maps' scores come from one
 // product; the merge subtracts the second map and norms the difference.
 template <bool EXT, bool FULL, bool DIFF>
@@ -95,9 +95,12 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   float* sRed = sMerge + STAGES * STAGE_BYTES / 4 - 32;  // DIFF: 32 floats behind it
 
   const int split = blockIdx.x;
-  const int kvh = blockIdx.y;
+  const int v_heads = EXT && p.v_heads > 0 ? p.v_heads : 1;
+  const int kvh = EXT ? blockIdx.y / v_heads : blockIdx.y;
+  const int vh = EXT && p.v_heads > 0 ? blockIdx.y % v_heads : kvh, v_rows = EXT && p.v_heads > 0 ? v_heads : p.Hkv;
   const int seq = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t part0 = ((size_t)seq * gridDim.y + blockIdx.y) * p.num_splits * 16;     // first row of this problem's partials
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) {
@@ -167,11 +170,11 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
           const int tstart = tok0 + b * 16;
           // blocks wholly past the context reuse the first block: finite data, masked in the softmax
           const int blk = tstart < kv_len ? __ldg(&table[tstart >> 4]) : first_block;
-          const int row0 = (blk * p.Hkv + kvh) * 16;
+          const int row0 = (blk * p.Hkv + kvh) * 16, vrow0 = (blk * v_rows + vh) * 16;
           tma_load_2d(sK + (b * 2 + 0) * 2048, &tmap_k, &bar_full[stage], 0, row0);
           if (k_halves > 1) tma_load_2d(sK + (b * 2 + 1) * 2048, &tmap_k, &bar_full[stage], 64, row0);
-          tma_load_2d(sV + (b * 2 + 0) * 2048, &tmap_v, &bar_full[stage], 0, row0);
-          if (v_halves > 1) tma_load_2d(sV + (b * 2 + 1) * 2048, &tmap_v, &bar_full[stage], 64, row0);
+          tma_load_2d(sV + (b * 2 + 0) * 2048, &tmap_v, &bar_full[stage], 0, vrow0);
+          if (v_halves > 1) tma_load_2d(sV + (b * 2 + 1) * 2048, &tmap_v, &bar_full[stage], 64, vrow0);
         }
         outstanding |= 1u << stage;
         issue_phase = (issue_phase & ~(1u << stage)) | (phase << stage);
@@ -314,6 +317,15 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
   }
   __syncthreads();
   float keep[8];                           // DIFF: differences of the row pairs
+  auto put = [&](int row, int d, float x) {      // output column d of query row `row`
+    const int head = kvh * p.G + row % p.G;
+    const size_t tok = q_start + row / p.G, col = (size_t)(EXT && p.v_heads > 0 ? head * v_heads + vh : head) * v_dim + d;
+    if (EXT && !DIFF && p.gate) {
+      const float z = __bfloat162float(p.gate[tok * p.gate_stride + col]);
+      x *= __fdividef(1.f, 1.f + __expf(-z));
+    }
+    p.out[tok * p.out_stride_tok + col] = __float2bfloat16(x);
+  };
   if (threadIdx.x < 128) {
     const int d = threadIdx.x;
     for (int row = 0; row < nrows; ++row) {
@@ -328,16 +340,13 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         L += sc * sMerge[4 * 16 * HD + 4 * 16 + w * 16 + row];
         acc += sc * sMerge[w * 16 * HD + row * HD + d];
       }
-      const int qtok = row / p.G, hg = row % p.G;
       if (p.num_splits == 1) {
-        const float inv = softmax_inv<EXT>(p, kvh * p.G + hg, M, L);
+        const float inv = softmax_inv<EXT>(p, kvh * p.G + row % p.G, M, L);
         if (DIFF) {
           sMerge[row * HD + d] = acc * inv;      // warp 0's partial of this row and column, read by this thread alone
-        } else if (d < v_dim)
-          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] =
-              __float2bfloat16(acc * inv);
+        } else if (d < v_dim) put(row, d, acc * inv);
       } else {
-        const size_t base = (((size_t)seq * p.Hkv + kvh) * p.num_splits + split) * 16 + row;
+        const size_t base = part0 + (size_t)split * 16 + row;
         p.part_o[base * HD + d] = acc;
         if (d == 0) {
           p.part_ml[base * 2] = M;
@@ -371,7 +380,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     // Merge of the splits inside this launch. Cluster launch (the splits of a (sequence, kv head) form one
     // thread-block cluster): a cluster barrier orders the partials, the first CTA merges. Otherwise the last split
     // to arrive (ticket counter in the workspace, reset by the merger) merges.
-    int* ctr = p.split_counters + (size_t)seq * p.Hkv + kvh;
+    int* ctr = p.split_counters + (size_t)seq * gridDim.y + blockIdx.y;
     if (p.cluster_merge) {
       asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
       asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -388,7 +397,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     const int S = p.num_splits;            // <= 32
     float* sSc = sMerge;                   // [16][32] weights of the splits, then normalised
     float* sL = sMerge + 16 * 32;          // [16][32]
-    const size_t base0 = ((size_t)seq * p.Hkv + kvh) * S * 16;
+    const size_t base0 = part0;
     __syncthreads();                       // (cluster path: the cross-warp merge area is free)
     for (int i = threadIdx.x; i < nrows * S; i += blockDim.x) {
       const int row = i / S, sp = i % S;
@@ -445,8 +454,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 #pragma unroll
             for (int sp = 0; sp < 8; ++sp)
               if (sp < S) acc += sSc[row * 32 + sp] * po[row][sp];
-            const int qtok = row / p.G, hg = row % p.G;
-            p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] = __float2bfloat16(acc);
+            put(row, d, acc);
           }
         }
       } else {
@@ -455,8 +463,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 #pragma unroll 8
           for (int sp = 0; sp < S; ++sp)
             acc += sSc[row * 32 + sp] * __ldcg(p.part_o + (base0 + (size_t)sp * 16 + row) * HD + d);
-          const int qtok = row / p.G, hg = row % p.G;
-          p.out[(size_t)(q_start + qtok) * p.out_stride_tok + (size_t)(kvh * p.G + hg) * v_dim + d] = __float2bfloat16(acc);
+          put(row, d, acc);
         }
       }
     }
@@ -468,7 +475,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 
 // Launches the TMA decode kernel; kcache / vcache are one layer's [blocks, Hkv, 16, 128] tensors.
 int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t stream) {
-  const bool ext = p.chunk > 0 || p.sink != nullptr || p.window > 0, full = p.k_dim == HD && p.v_dim == HD;
+  const bool ext = p.chunk > 0 || p.sink != nullptr || p.window > 0 || p.v_heads > 0 || p.gate, full = p.k_dim == HD && p.v_dim == HD;
   const int which = p.diff.maps ? (full ? 3 : 4) : full ? (ext ? 1 : 0) : 2;
   auto kernel = which == 0   ? attn_decode_tma_kernel<false, true, false>
                 : which == 1 ? attn_decode_tma_kernel<true, true, false>
@@ -487,9 +494,9 @@ int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t str
   const int rows = num_blocks * p.Hkv * 16;
   int rc = make_tmap_bf16_2d(&tk, p.k, rows, p.k_dim, p.k_dim, 16);
   if (rc) return rc;
-  rc = make_tmap_bf16_2d(&tv, p.v, rows, p.v_dim, p.v_dim, 16);
+  rc = make_tmap_bf16_2d(&tv, p.v, p.v_heads > 0 ? num_blocks * p.v_heads * 16 : rows, p.v_dim, p.v_dim, 16);
   if (rc) return rc;
-  dim3 grid(p.num_splits, p.Hkv, p.num_seqs);
+  dim3 grid(p.num_splits, p.Hkv * (p.v_heads > 0 ? p.v_heads : 1), p.num_seqs);
   if (p.num_splits > 1 && p.num_splits <= 8 && p.split_counters) {
     // the splits of one (sequence, kv head) as a thread-block cluster: merged after a cluster barrier
     AttnParams pc = p;

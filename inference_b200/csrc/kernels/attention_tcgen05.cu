@@ -83,6 +83,9 @@ struct FaParams {
   int window;          // > 0: query i sees only keys j > i - window
   int v_dim;           // width of the v heads and of the output heads (<= VD; the tile is zero filled beyond it)
   attn::DiffAttn diff; // DIFF only
+  int v_heads;         // > 0: blockIdx.y runs over (query head, value head); every query head is applied to all value heads
+  const bf16* out_gate;         // optional logits in the layout of a token's output: out is scaled by their sigmoid
+  long long out_gate_stride;
   // Latent attention (LAT): q and k in two parts, k's second part shared by the heads; keys and values are rows
   // [cu_k[z], cu_k[z + 1]) of one flat axis (null: those of the queries), the queries the last positions of them.
   const int* seqs;     // optional: sequence of blockIdx.z (cu_q is indexed by it, cu_k by blockIdx.z)
@@ -184,7 +187,7 @@ struct Barriers {
 
 // 168 registers per thread is the cap for ten warps: two of the four scheduler partitions hold three warps, and a
 // partition's file is 16 K registers (a build with 200 registers per thread does not launch).
-// EXT adds chunked and windowed masking, attention sinks and head widths below the tile widths (q . k and P V then run over zero
+// EXT adds chunked and windowed masking, attention sinks, output gates, values of every head for every query head, and head widths below the tile widths (q . k and P V then run over zero
 // columns that the tensor maps fill in). LAT adds what latent attention needs: two-part q / k, key ranges, output gates.
 // DIFF is differential attention: the two tiles of a CTA are the two softmax maps of the same 128 query rows. Each map's keys are
 // one 64-column atom of the K tile (columns of the other map that fall into it meet zero columns of q), the V tile serves both, and
@@ -206,7 +209,8 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   constexpr int TILE_STEP = DIFF ? 0 : BM;                  // query rows between the two tiles of a CTA
   const int cta_rows = DIFF ? BM : p.tiles * BM;
   const int q_base = blockIdx.x * cta_rows;
-  const int head = blockIdx.y;
+  constexpr bool WIDE = EXT && !LAT && DIFF == 0;             // v_heads and out_gate are looked at
+  const int head = WIDE && p.v_heads > 0 ? blockIdx.y / p.v_heads : blockIdx.y;
   // packed variable-length batch: this CTA's sequence covers tokens [tok0, tok0 + q_len) of one flat token axis
   const int seq = (LAT && p.seqs) ? p.seqs[blockIdx.z] : blockIdx.z;
   const int tok0 = p.cu_q ? p.cu_q[seq] : 0;
@@ -217,7 +221,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
   const int coff = paged || ranged ? max(kv_len - q_len, 0) : 0;   // position of query 0 among the sequence's keys
   const int batch = p.cu_q ? 0 : blockIdx.z;
   if (q_base >= q_len || kv_len <= 0) return;   // uniform for the whole CTA, before any barrier or TMEM allocation
-  const int kv_head = head / (p.Hq / p.Hkv);
+  const int kv_head = head / (p.Hq / p.Hkv), v_head = WIDE && p.v_heads > 0 ? blockIdx.y % p.v_heads : kv_head;
   const int kv_end = p.causal ? min(kv_len, q_base + cta_rows + coff) : kv_len;
   // first key that a row sees, and first key tile that any row of this CTA sees (rows are ascending, so the first row's is lowest)
   auto first_key_of = [&](int pos) {
@@ -294,14 +298,14 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             if (LAT && is_k && a >= p.first_atoms)
               tma_load_4d(smem + dst_off + a * ATOM_BYTES, &tmap_k2, bar, (a - p.first_atoms) * 64, 0, key0_row + j * BN, batch);
             else
-              tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * atom_cols, kv_head, key0_row + j * BN, batch);
+              tma_load_4d(smem + dst_off + a * ATOM_BYTES, map, bar, a * atom_cols, is_k ? kv_head : v_head, key0_row + j * BN, batch);
           }
           return;
         }
         for (int g = 0; g < per_tile; ++g) {
           const int page = pages[min(j * per_tile + g, last_page)];
           for (int a = 0; a < atoms; ++a)
-            tma_load_4d(smem + dst_off + a * ATOM_BYTES + g * page_bytes, map, bar, a * atom_cols, 0, kv_head, page);
+            tma_load_4d(smem + dst_off + a * ATOM_BYTES + g * page_bytes, map, bar, a * atom_cols, 0, is_k ? kv_head : v_head, page);
         }
       };
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -613,10 +617,20 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
         const int r = (32 / CHUNKS) * it + lane / CHUNKS, ch = lane % CHUNKS;
         const int grow = row0 + r;
         if (grow < q_len) {
-          const uint4 val = *reinterpret_cast<const uint4*>(slab + r * ROW_BYTES + ((ch ^ (r & 7)) << 4));
+          uint4 val = *reinterpret_cast<const uint4*>(slab + r * ROW_BYTES + ((ch ^ (r & 7)) << 4));
           if (EXT && ch * 8 >= p.v_dim) continue;
-          bf16* dst = p.out + ((long long)batch * p.q_len + tok0 + grow) * p.out_stride_tok +
-                      (long long)head * (EXT ? p.v_dim : VD);
+          const long long col = (long long)(WIDE ? blockIdx.y : head) * (EXT ? p.v_dim : VD);
+          if constexpr (WIDE) {
+            if (p.out_gate) {
+              float x[8], z[8];
+              load_row8(reinterpret_cast<const bf16*>(&val), x);
+              load_row8(p.out_gate + (tok0 + grow) * p.out_gate_stride + col + ch * 8, z);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) x[i] *= rcp_approx(1.f + ex2(-1.4426950408889634f * z[i]));
+              store_row8(reinterpret_cast<bf16*>(&val), x);
+            }
+          }
+          bf16* dst = p.out + ((long long)batch * p.q_len + tok0 + grow) * p.out_stride_tok + col;
           if (p.scatter.enabled) {
             const OutScatter& sc = p.scatter;
             const int g2 = grow - sc.split;
@@ -757,8 +771,10 @@ int launch_tiles(int qk, FaKind kind, int q_len, int Hq, int batch, cudaStream_t
   const dim3 grid((q_len + p.tiles * BM - 1) / (p.tiles * BM), Hq, batch);
   if (kind == FaKind::LATENT)
     return qk == 192 ? launch_fa<192, 128, true, true>(grid, stream, m, p) : launch_fa<128, 128, true, true>(grid, stream, m, p);
-  if (kind == FaKind::EXT)
+  if (kind == FaKind::EXT) {
+    if (qk == 64 && p.v_dim > 64) return launch_fa<64, 128, true, false>(grid, stream, m, p);
     return qk == 64 ? launch_fa<64, 64, true, false>(grid, stream, m, p) : launch_fa<128, 128, true, false>(grid, stream, m, p);
+  }
   return qk == 64 ? launch_fa<64, 64, false, false>(grid, stream, m, p) : launch_fa<128, 128, false, false>(grid, stream, m, p);
 }
 
@@ -832,7 +848,8 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
                             long long v_stride_tok, void* out, long long out_stride_tok, int num_seqs, int max_q_len,
                             int total_tokens, int Hq, int Hkv, int D, int Dv, float scale, int chunk, const float* sink,
                             const int* cu_q, const int* kv_lens, const int* block_table, int max_blocks, int block_size,
-                            int num_blocks, cudaStream_t stream, int window, const attn::DiffAttn* diff) {
+                            int num_blocks, cudaStream_t stream, int window, const attn::DiffAttn* diff, int v_heads, const void* gate,
+                            long long gate_stride) {
   const bool paged = block_table != nullptr;
   if (window < 0 || (diff && (sink || chunk || D % 16))) return -3;
   if (D < 8 || Dv < 8 || D > 128 || Dv > 128 || (D % 8) || (Dv % 8) || !cu_q || Hq % Hkv || !(scale > 0.f) || chunk < 0) return -3;
@@ -850,7 +867,7 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
   rc = make_tmap_heads(&m.k, k, D, Hkv, total_tokens, paged ? num_blocks : 1, D, k_stride_tok, k_stride_tok * total_tokens,
                        paged ? block_size : 0);
   if (rc) return rc;
-  rc = make_tmap_heads(&m.v, v, Dv, Hkv, total_tokens, paged ? num_blocks : 1, Dv, v_stride_tok, v_stride_tok * total_tokens,
+  rc = make_tmap_heads(&m.v, v, Dv, v_heads > 0 ? v_heads : Hkv, total_tokens, paged ? num_blocks : 1, Dv, v_stride_tok, v_stride_tok * total_tokens,
                        paged ? block_size : 0);
   if (rc) return rc;
   FaParams p{};
@@ -869,11 +886,14 @@ int attn_ext_tcgen05_launch(const void* q, long long q_stride_tok, const void* k
   p.sink = sink;
   p.window = window;
   p.v_dim = Dv;
+  p.v_heads = v_heads;
+  p.out_gate = reinterpret_cast<const bf16*>(gate);
+  p.out_gate_stride = gate_stride;
   if (diff) {
     p.diff = *diff;
     return launch_tiles(128, FaKind::DIFF, max_q_len, Hq, num_seqs, stream, m, p);
   }
-  return launch_tiles(D > 64 || Dv > 64 ? 128 : 64, FaKind::EXT, max_q_len, Hq, num_seqs, stream, m, p);
+  return launch_tiles(D > 64 ? 128 : 64, FaKind::EXT, max_q_len, Hq * (v_heads > 0 ? v_heads : 1), num_seqs, stream, m, p);
 }
 
 // Latent attention on expanded keys and values, causal: q [total_tokens] rows of H heads of [d1 | d2] (stride q_stride_tok), k

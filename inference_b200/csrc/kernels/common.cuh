@@ -347,6 +347,24 @@ __device__ __forceinline__ float relu2_f(float x) {
   return r * r;
 }
 
+// xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below. The second form takes the series of e^z - 1 - z near zero and the fast
+// exponential elsewhere (for outputs that are rounded to bf16).
+__device__ __forceinline__ float xielu_exact_f(float z, float a, float b) {
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+  const float low = z > -0.03f ? z * z * fmaf(z, 1.f / 6.f, 0.5f) : __expf(z) - 1.f - z;
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, low, 0.5f * z);
+}
+// Gated unit whose parts are clamped: g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
+template <bool EXACT>
+__device__ __forceinline__ float clamped_gate_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  const float s = EXACT ? g / (1.f + expf(-1.702f * g)) : __fdividef(g, 1.f + __expf(-1.702f * g));
+  return s * (u + 1.f);
+}
+
 __device__ __forceinline__ void store_row4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ void store_row4(bf16* p, float4 v) {
   const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);

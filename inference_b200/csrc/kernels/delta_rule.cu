@@ -1,4 +1,4 @@
-// Gated delta rule with a decay per head and key channel, over a flat ragged batch of sequences:
+// Gated delta rule with a decay per head and key channel, or one per head, over a flat ragged batch of sequences:
 //     S <- g * S          (rows of S are key channels)
 //     u  = beta (v - S^T k),   S <- S + k u^T,   o = S^T q
 // Three launches around the projections:
@@ -10,6 +10,7 @@
 //                cross-lane reduction per token is on the critical path; it folds the 2 NC sums into different lanes on the way.
 //                Arithmetic is fp32 in token order: results do not depend on how a prompt was cut.
 //   delta_post   RMS norm over a head's value channels, weight and gate; moves the convolution windows on.
+// With one decay per head the dots run on the state as it is, a factor g behind them, and the decay joins the update.
 // States and windows live in slots; a sequence's state is zero at position 0, a slot below 0 is neither read nor written.
 #include "common.cuh"
 
@@ -25,13 +26,14 @@ struct DeltaShape {
   const int* positions;      // [T]
   const int* slots;          // [num_seqs]
   int H, G, dim, dp, vdim, vp, taps;   // dp / vp: padded widths
+  int head_decay;            // 1: one decay per head
 };
 
 struct PrepParams {
   DeltaShape s;
   const void* buf;           // projections [T, ld]: q (G dp) at 0, k, v (H vp), then beta logits at col_b
   int ld, col_b;
-  const void* decay;         // [T, ld_decay]: decay logits, H dp
+  const void* decay;         // [T, ld_decay]: decay logits, H dp (H with one per head, as are dt_bias and g)
   int ld_decay;
   const float* conv;         // [taps, 2 G dp + H vp]
   const void* window;        // [slots, taps - 1, 2 G dp + H vp]
@@ -123,7 +125,11 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const PrepParams p) {
     } else if (task < s.G + s.H) {
       const int h = task - s.G;
       const float rate = -expf(p.a_log[h]);
-      for (int c = lane * 4; c < s.dp; c += 128) {
+      if (s.head_decay) {
+        if (lane == 0)
+          p.g[(size_t)t * s.H + h] =
+              expf(rate * softplus_f(to_f(reinterpret_cast<const E*>(p.decay)[(size_t)t * p.ld_decay + h]) + p.dt_bias[h]));
+      } else for (int c = lane * 4; c < s.dp; c += 128) {
         const float4 b = *reinterpret_cast<const float4*>(p.dt_bias + h * s.dp + c);
         float4 x = load_row4(reinterpret_cast<const E*>(p.decay) + (size_t)t * p.ld_decay + h * s.dp + c);
         x.x = expf(rate * softplus_f(x.x + b.x)), x.y = expf(rate * softplus_f(x.y + b.y));
@@ -200,10 +206,11 @@ struct Lane {
   }
 };
 
-// TB tokens per staged block; layout of one token in shared memory: k [dp], q [dp], g [dp], v [COLS], (kq, beta, -, -)
-template <int DPL, int NC, int TB>
+// TB tokens per staged block; layout of one token in shared memory: k [dp], q [dp], g [dp], v [COLS], (kq, beta, -, -). HEAD: one decay
+// per head, no g [dp] but (kq, beta, g, -).
+template <int DPL, int NC, int TB, bool HEAD>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanParams p) {
-  constexpr int DP = DPL * SCAN_LANES, COLS = SCAN_WARPS * 2 * NC, TOK = 3 * DP + COLS + 4, N2 = DPL / 2;
+  constexpr int DP = DPL * SCAN_LANES, COLS = SCAN_WARPS * 2 * NC, VO = HEAD ? 2 * DP : 3 * DP, TAIL = VO + COLS, TOK = TAIL + 4, N2 = DPL / 2;
   constexpr bool AHEAD = DPL <= 16;                  // operands of the next token are read while this one is computed
   using L = Lane<DPL>;
   extern __shared__ __align__(16) float sm[];        // 2 blocks of TB tokens
@@ -237,15 +244,16 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
       float* d = dst0 + r * TOK + c;
       cp_async16(d, qk);
       cp_async16(d + DP, qk + DP);
-      cp_async16(d + 2 * DP, p.g + (t * s.H + h) * DP + c);
+      if constexpr (!HEAD) cp_async16(d + 2 * DP, p.g + (t * s.H + h) * DP + c);
     }
     for (int i = tid; i < m * (COLS / 4); i += SCAN_WARPS * 32) {
       const int r = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
-      if (c < ncols) cp_async16(dst0 + r * TOK + 3 * DP + c, p.v + ((size_t)(start + t0 + r) * s.H + h) * s.vp + c0 + c);
+      if (c < ncols) cp_async16(dst0 + r * TOK + VO + c, p.v + ((size_t)(start + t0 + r) * s.H + h) * s.vp + c0 + c);
     }
     for (int r = tid; r < m; r += SCAN_WARPS * 32) {
-      cp_async4(dst0 + r * TOK + 3 * DP + COLS, p.kq + (size_t)(start + t0 + r) * s.G + kvh);
-      cp_async4(dst0 + r * TOK + 3 * DP + COLS + 1, p.beta + (size_t)(start + t0 + r) * s.H + h);
+      cp_async4(dst0 + r * TOK + TAIL, p.kq + (size_t)(start + t0 + r) * s.G + kvh);
+      cp_async4(dst0 + r * TOK + TAIL + 1, p.beta + (size_t)(start + t0 + r) * s.H + h);
+      if constexpr (HEAD) cp_async4(dst0 + r * TOK + TAIL + 2, p.g + (size_t)(start + t0 + r) * s.H + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -268,15 +276,19 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
     // one token: operands in (k, q, g), those of the next token are read into (kn, qn, gn) meanwhile
     auto step = [&](const float* tok, float* o_to, uint64_t* k, uint64_t* q, uint64_t* g, uint64_t* kn, uint64_t* qn, uint64_t* gn,
                     bool more) {
-      const float kq = tok[3 * DP + COLS], beta = tok[3 * DP + COLS + 1], v = tok[3 * DP + lc + mine];
-      if (AHEAD && more) L::load(tok + TOK, sub, kn), L::load(tok + TOK + DP, sub, qn), L::load(tok + TOK + 2 * DP, sub, gn);
+      const float kq = tok[TAIL], beta = tok[TAIL + 1], v = tok[VO + lc + mine], gh = HEAD ? tok[TAIL + 2] : 1.f;
+      const uint64_t gg = dup2(gh);
+      if (AHEAD && more) {
+        L::load(tok + TOK, sub, kn), L::load(tok + TOK + DP, sub, qn);
+        if constexpr (!HEAD) L::load(tok + TOK + 2 * DP, sub, gn);
+      }
       float a[2 * NC];
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
         uint64_t ak = 0ull, aq = 0ull;
 #pragma unroll
         for (int i = 0; i < N2; ++i) {
-          S[c][i] = mul2(S[c][i], g[i]);
+          if constexpr (!HEAD) S[c][i] = mul2(S[c][i], g[i]);
           ak = i ? fma2(S[c][i], k[i], ak) : mul2(S[c][i], k[i]);
           aq = i ? fma2(S[c][i], q[i], aq) : mul2(S[c][i], q[i]);
         }
@@ -295,6 +307,7 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
       }
 #pragma unroll
       for (; o > 0; o >>= 1) a[0] += __shfl_xor_sync(0xffffffffu, a[0], o);
+      if constexpr (HEAD) a[0] *= gh;
       const float u_mine = beta * (v - a[0]);        // meaningful in the lanes that hold a dot with k
       float u_out = 0.f;
 #pragma unroll
@@ -303,14 +316,15 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
         if (c == mine) u_out = u;
         const uint64_t uu = dup2(u);
 #pragma unroll
-        for (int i = 0; i < N2; ++i) S[c][i] = fma2(k[i], uu, S[c][i]);
+        for (int i = 0; i < N2; ++i) S[c][i] = fma2(k[i], uu, HEAD ? mul2(S[c][i], gg) : S[c][i]);
       }
       if (writes) *o_to = fmaf(kq, u_out, a[0]);
     };
     const size_t o_step = (size_t)s.H * s.vp;
     if constexpr (AHEAD) {
       uint64_t k0[N2], q0[N2], g0[N2], k1[N2], q1[N2], g1[N2];
-      L::load(tok, sub, k0), L::load(tok + DP, sub, q0), L::load(tok + 2 * DP, sub, g0);
+      L::load(tok, sub, k0), L::load(tok + DP, sub, q0);
+      if constexpr (!HEAD) L::load(tok + 2 * DP, sub, g0);
       int r = 0;
       for (; r + 2 <= m; r += 2, tok += 2 * TOK, orow += 2 * o_step) {
         step(tok, orow, k0, q0, g0, k1, q1, g1, true);
@@ -323,7 +337,8 @@ __global__ void __launch_bounds__(SCAN_WARPS * 32) delta_scan_kernel(const ScanP
     } else {
       for (int r = 0; r < m; ++r, tok += TOK, orow += o_step) {
         uint64_t k[N2], q[N2], g[N2];
-        L::load(tok, sub, k), L::load(tok + DP, sub, q), L::load(tok + 2 * DP, sub, g);
+        L::load(tok, sub, k), L::load(tok + DP, sub, q);
+        if constexpr (!HEAD) L::load(tok + 2 * DP, sub, g);
         step(tok, orow, k, q, g, k, q, g, false);
       }
     }
@@ -344,6 +359,7 @@ struct PostParams {
   int ld_gate;
   const float* w;            // [vp]
   float eps;
+  int gate_silu;             // the gate is silu of its logits (else their sigmoid)
   void* out;                 // [T, H vp]
   const void* buf;           // projections, for the windows
   int ld;
@@ -379,6 +395,7 @@ __global__ void __launch_bounds__(256) delta_post_kernel(const PostParams p) {
   const long long rows = (long long)s.T * s.H, id0 = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * p.rows_per_warp;
   auto finish = [&](long long id, int c, float4 x, float4 z, float r) {
     const float4 w = __ldg(reinterpret_cast<const float4*>(p.w + c));
+    if (p.gate_silu) x = make_float4(x.x * z.x, x.y * z.y, x.z * z.z, x.w * z.w);
     store_row4(reinterpret_cast<E*>(p.out) + id * s.vp + c,
                make_float4(x.x * r * w.x * fast_sigmoid(z.x), x.y * r * w.y * fast_sigmoid(z.y), x.z * r * w.z * fast_sigmoid(z.z),
                            x.w * r * w.w * fast_sigmoid(z.w)));
@@ -415,22 +432,26 @@ __global__ void __launch_bounds__(256) delta_post_kernel(const PostParams p) {
   }
 }
 
-template <int DPL, int NC, int TB>
+template <int DPL, int NC, int TB, bool HEAD>
 int launch_scan(const ScanParams& p, cudaStream_t st) {
   constexpr int DP = DPL * SCAN_LANES, COLS = SCAN_WARPS * 2 * NC;
-  constexpr size_t smem = 2 * TB * (3 * DP + COLS + 4) * sizeof(float);
+  constexpr size_t smem = 2 * TB * ((HEAD ? 2 : 3) * DP + COLS + 4) * sizeof(float);
   if (smem > 48 * 1024) {
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64 || !configured[dev]) {
-      const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DPL, NC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DPL, NC, TB, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return -(int)e;
       if (dev >= 0 && dev < 64) configured[dev] = true;
     }
   }
-  return launch_kernel(delta_scan_kernel<DPL, NC, TB>, dim3((p.s.vp + COLS - 1) / COLS, p.s.H, p.s.num_seqs), dim3(SCAN_WARPS * 32),
+  return launch_kernel(delta_scan_kernel<DPL, NC, TB, HEAD>, dim3((p.s.vp + COLS - 1) / COLS, p.s.H, p.s.num_seqs), dim3(SCAN_WARPS * 32),
                        smem, st, p);
+}
+template <int DPL, int NC, int TB>
+int launch_scan(const ScanParams& p, cudaStream_t st) {
+  return p.s.head_decay ? launch_scan<DPL, NC, TB, true>(p, st) : launch_scan<DPL, NC, TB, false>(p, st);
 }
 
 bool shape_ok(const DeltaShape& s) {
@@ -440,8 +461,8 @@ bool shape_ok(const DeltaShape& s) {
 }
 
 DeltaShape make_shape(const int* dims, const int* cu_q, const int* positions, const int* slots) {
-  // dims: T, num_seqs, uniform_q, H, G, dim, dp, vdim, vp, taps
-  return DeltaShape{dims[0], dims[1], dims[2], cu_q, positions, slots, dims[3], dims[4], dims[5], dims[6], dims[7], dims[8], dims[9]};
+  // dims: T, num_seqs, uniform_q, H, G, dim, dp, vdim, vp, taps, head_decay
+  return DeltaShape{dims[0], dims[1], dims[2], cu_q, positions, slots, dims[3], dims[4], dims[5], dims[6], dims[7], dims[8], dims[9], dims[10]};
 }
 
 }  // namespace
@@ -472,7 +493,7 @@ int launch_prep(const PrepParams& p, cudaStream_t st) {
 }  // namespace swb
 extern "C" {
 
-// dims: host int[10] = T, num_seqs, uniform_q (cu_q null), H, G, dim, dp, vdim, vp, taps. fp32 selects the element type of
+// dims: host int[11] = T, num_seqs, uniform_q (cu_q null), H, G, dim, dp, vdim, vp, taps, head_decay. fp32 selects the element type of
 // the projections, windows and decay logits.
 int swb_delta_prep(const int* dims, const int* cu_q, const int* positions, const int* slots, const void* buf, int ld, int col_b,
                    const void* decay, int ld_decay, const float* conv, const void* window, const float* a_log, const float* dt_bias,
@@ -481,7 +502,7 @@ int swb_delta_prep(const int* dims, const int* cu_q, const int* positions, const
   PrepParams p{make_shape(dims, cu_q, positions, slots), buf, ld, col_b, decay, ld_decay, conv, window, a_log, dt_bias, qk, kq, g, v,
                beta, dims[0] >= 4096 ? 8 : dims[0] >= 1024 ? 4 : 1};
   if (dims[0] <= 0) return 0;
-  if (!shape_ok(p.s) || (ld % 4) || (ld_decay % 4)) return -3;
+  if (!shape_ok(p.s) || (ld % 4) || (!p.s.head_decay && ld_decay % 4)) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return fp32 ? launch_prep<float>(p, st) : launch_prep<bf16>(p, st);
 }
@@ -506,9 +527,11 @@ int swb_delta_scan(const int* dims, const int* cu_q, const int* positions, const
 }
 
 int swb_delta_post(const int* dims, const int* cu_q, const int* positions, const int* slots, const float* o, const void* gate,
-                   int ld_gate, const float* w, float eps, void* out, const void* buf, int ld, void* window, int fp32, void* stream) {
+                   int ld_gate, const float* w, float eps, int gate_silu, void* out, const void* buf, int ld, void* window, int fp32,
+                   void* stream) {
   using namespace swb;
-  PostParams p{make_shape(dims, cu_q, positions, slots), o, gate, ld_gate, w, eps, out, buf, ld, window, 0, dims[0] >= 1024 ? 4 : 1};
+  PostParams p{make_shape(dims, cu_q, positions, slots), o, gate, ld_gate, w, eps, gate_silu, out, buf, ld, window, 0,
+               dims[0] >= 1024 ? 4 : 1};
   if (dims[0] <= 0) return 0;
   if (!shape_ok(p.s)) return -3;
   p.norm_ctas = (int)(((long long)p.s.T * p.s.H + 8 * p.rows_per_warp - 1) / (8 * p.rows_per_warp));

@@ -15,7 +15,7 @@ constexpr int TM = 64, TN = 64, TK = 16;
 // out[r, n] = act(sum_k a[src ? src[r] : r, k] w[e, n, k] + bias[n]); 64 x 64 tile, 4 x 4 per thread. Grouped: blockIdx.z = expert.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ a, int lda, const int* __restrict__ src,
                                                        const int* __restrict__ offsets, const float* __restrict__ w, int ldw,
-                                                       float* out, int ldo, int T, int N, int K, int act,
+                                                       float* out, int ldo, int T, int N, int K, int act, float act_a, float act_b,
                                                        const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
@@ -63,6 +63,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
       if (act == SWB_ACT_RELU2) v = relu2_f(v);
       else if (act == SWB_ACT_SILU) v = silu_f(v);
       else if (act == SWB_ACT_GELU_TANH) v = gelu_tanh_f(v);
+      else if (act == SWB_ACT_XIELU) v = xielu_exact_f(v, act_a, act_b);
       out[(size_t)r * ldo + n] = v;
     }
   }
@@ -86,16 +87,20 @@ struct SimpleAttnParams {
   const float* q_temp;       // optional, by position: factor of the scores in front of the cap
   const float* sink;
   int maps;                  // query heads h, h + 1, ... take turns on `maps` key parts of D columns each within a key row
+  int v_heads;               // > 0: every query head is applied to all value heads; out [token, Hq, v_heads, Dv]
+  const void* gate;          // optional logits in the layout of a token's output, rows gate_stride apart: out is scaled by their sigmoid
+  long long gate_stride;
 };
 
-// One CTA per (query token, head). Each warp runs an online softmax over its share of the visible keys; lanes split the
+// One CTA per (query token, head) or, with v_heads, (query token, head, value head). Each warp runs an online softmax over its share of the visible keys; lanes split the
 // head dimension. The sink joins the denominator when the four partial results are merged.
 template <typename E, int PL>
 __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restrict__ q, const E* __restrict__ kc, const E* __restrict__ vc,
                                                               E* out, const SimpleAttnParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, head = blockIdx.y, kvh = head / (p.Hq / p.Hkv);
+  const int t = blockIdx.x, nv = p.v_heads > 0 ? p.v_heads : 1, head = blockIdx.y / nv, kvh = head / (p.Hq / p.Hkv);
+  const int v_rows = p.v_heads > 0 ? nv : p.Hkv, vh = p.v_heads > 0 ? blockIdx.y % nv : kvh;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = seq_of_token(p.cu_q, p.num_seqs, p.uniform_q, t);
   const int q0 = p.cu_q ? p.cu_q[seq] : seq * p.uniform_q, q_len = p.cu_q ? p.cu_q[seq + 1] - q0 : p.uniform_q;
@@ -115,9 +120,9 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
   }
   float m = -INFINITY, l = 0.f;
   for (int j = first + warp; j <= pos; j += AW) {
-    const size_t row = ((size_t)table[j / p.block_size] * p.Hkv + kvh) * p.block_size + j % p.block_size;
-    const E* kr = kc + row * p.k_row + k_off;
-    const E* vr = vc + row * p.v_row;
+    const size_t page = table[j / p.block_size], at = j % p.block_size;
+    const E* kr = kc + ((page * p.Hkv + kvh) * p.block_size + at) * p.k_row + k_off;
+    const E* vr = vc + ((page * v_rows + vh) * p.block_size + at) * p.v_row;
     float s = 0.f;
 #pragma unroll
     for (int i = 0; i < PL; ++i) {
@@ -147,7 +152,10 @@ __global__ void __launch_bounds__(AW * 32) attn_simple_kernel(const E* __restric
   for (int d = threadIdx.x; d < p.Dv; d += AW * 32) {
     float v = 0.f;
     for (int w = 0; w < AW; ++w) v = fmaf(so[w][d], expf(sm[w] - top), v);
-    from_f(out[(size_t)t * p.out_stride_tok + (size_t)head * p.Dv + d], v / den);
+    const size_t col = (size_t)blockIdx.y * p.Dv + d;
+    v /= den;
+    if (p.gate) v /= 1.f + expf(-to_f(reinterpret_cast<const E*>(p.gate)[t * p.gate_stride + col]));
+    from_f(out[(size_t)t * p.out_stride_tok + col], v);
   }
 }
 
@@ -190,7 +198,7 @@ __global__ void __launch_bounds__(64) head_product_kernel(const E* __restrict__ 
 
 template <typename E>
 int launch_attn_simple(const void* q, const void* k, const void* v, void* out, const SimpleAttnParams& p, int total_tokens, cudaStream_t s) {
-  const dim3 grid((unsigned)total_tokens, p.Hq), block(AW * 32);
+  const dim3 grid((unsigned)total_tokens, p.Hq * (p.v_heads > 0 ? p.v_heads : 1)), block(AW * 32);
   auto go = [&](auto kernel) {
     return launch_kernel(kernel, grid, block, 0, s, reinterpret_cast<const E*>(q), reinterpret_cast<const E*>(k), reinterpret_cast<const E*>(v),
                          reinterpret_cast<E*>(out), p);
@@ -210,12 +218,12 @@ extern "C" {
 // fp32 GEMM without reduced-precision modes. Dense: offsets null, groups 1. Grouped: w [groups, N, ldw], rows of group g
 // are [offsets[g], offsets[g + 1]), at most T rows in all; src (nullable) names the row of `a` for each row.
 int swb_gemm_f32(const float* a, int lda, const int* src, const int* offsets, int groups, const float* w, int ldw, float* out,
-                 int ldo, int T, int N, int K, int act, const float* bias, void* stream) {
+                 int ldo, int T, int N, int K, int act, float act_a, float act_b, const float* bias, void* stream) {
   using namespace swb;
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if (groups < 1 || (bias && offsets) || (groups > 1 && !offsets) || gemm_act_pairs(act)) return -3;
   return launch_kernel(gemm_f32_kernel, dim3((N + TN - 1) / TN, (T + TM - 1) / TM, groups), dim3(256), 0,
-                       reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act, bias);
+                       reinterpret_cast<cudaStream_t>(stream), a, lda, src, offsets, w, ldw, out, ldo, T, N, K, act, act_a, act_b, bias);
 }
 
 // Paged attention for any head widths up to 1024 in fp32 arithmetic; elements fp32 or bf16 (fp32 flag). Arguments as in
@@ -225,15 +233,16 @@ int swb_gemm_f32(const float* a, int lda, const int* src, const int* offsets, in
 int swb_attn_simple(const void* q, long long q_stride_tok, const void* k, const void* v, void* out, long long out_stride_tok,
                     const int* block_table, int max_blocks, int block_size, const int* cu_q, const int* kv_lens, int num_seqs,
                     int uniform_q, int total_tokens, int Hq, int Hkv, int D, int Dv, int v_row, float scale, int chunk,
-                    const float* sink, int window, float softcap, const float* q_temp, int maps, int fp32, void* stream) {
+                    const float* sink, int window, float softcap, const float* q_temp, int maps, int v_heads, const void* gate,
+                    long long gate_stride, int fp32, void* stream) {
   using namespace swb;
   if (total_tokens <= 0 || num_seqs <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv || D < 1 || Dv < 1 || D > 32 * MAX_PER_LANE || Dv > 32 * MAX_PER_LANE || block_size <= 0 ||
-      !block_table || !kv_lens || chunk < 0 || window < 0 || softcap < 0.f || maps < 1 || (Hq / Hkv) % maps ||
+      !block_table || !kv_lens || chunk < 0 || window < 0 || softcap < 0.f || maps < 1 || v_heads < 0 || (maps > 1 && v_heads) || (Hq / Hkv) % maps ||
       (!cu_q && (uniform_q <= 0 || num_seqs * uniform_q != total_tokens)) || (v_row && v_row < Dv))
     return -3;
   const SimpleAttnParams p{q_stride_tok, out_stride_tok, block_table, max_blocks, block_size, cu_q, kv_lens, num_seqs, uniform_q, Hq, Hkv, D, Dv,
-                           maps * D, v_row ? v_row : Dv, scale, chunk, window, softcap, q_temp, sink, maps};
+                           maps * D, v_row ? v_row : Dv, scale, chunk, window, softcap, q_temp, sink, maps, v_heads, gate, gate_stride};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return fp32 ? launch_attn_simple<float>(q, k, v, out, p, total_tokens, s) : launch_attn_simple<bf16>(q, k, v, out, p, total_tokens, s);
 }

@@ -148,11 +148,17 @@ __device__ __forceinline__ unsigned long long ssq_fixed(float ss) {
   return __float2ull_rn(fminf(ss, 5.0e11f) * 16777216.f);
 }
 
-__device__ __forceinline__ float act_apply(float x, int act) {
+__device__ __forceinline__ float act_apply(float x, const GemmParams& p) {
+  const int act = p.act;
   if (act == SWB_ACT_SILU) return silu_f(x);
   if (act == SWB_ACT_GELU_TANH) return gelu_tanh_f(x);
   if (act == SWB_ACT_RELU2) return relu2_f(x);
+  if (act == SWB_ACT_XIELU) return xielu_f(x, p.act_a, p.act_b);
   return x;
+}
+__device__ __forceinline__ float gated_pair(float gate, float up, const GemmParams& p) {
+  if (p.act == SWB_ACT_CLAMPED_PAIRS) return clamped_gate_f<false>(gate, up, p.act_a);
+  return (p.act == SWB_ACT_SWIGLU_PAIRS ? silu_f(gate) : gelu_tanh_f(gate)) * up;
 }
 
 // PEER instantiates the cross-rank epilogue (its batched peer loads need more registers than the plain store path).
@@ -564,16 +570,15 @@ gemm_decode_cluster_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
           }
           if (gemm_act_pairs(p.act)) {
             // rows come in (gate, up) pairs: four gated outputs, one 8-byte store
-            const int a1 = p.act == SWB_ACT_SWIGLU_PAIRS ? SWB_ACT_SILU : SWB_ACT_GELU_TANH;
             uint2 o;
             __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
-            oh[0] = __floats2bfloat162_rn(act_apply(acc[0], a1) * acc[1], act_apply(acc[2], a1) * acc[3]);
-            oh[1] = __floats2bfloat162_rn(act_apply(acc[4], a1) * acc[5], act_apply(acc[6], a1) * acc[7]);
+            oh[0] = __floats2bfloat162_rn(gated_pair(acc[0], acc[1], p), gated_pair(acc[2], acc[3], p));
+            oh[1] = __floats2bfloat162_rn(gated_pair(acc[4], acc[5], p), gated_pair(acc[6], acc[7], p));
             *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(p.out) + (size_t)tok * p.ldd + (feat >> 1)) = o;
           } else {
             if (p.act != SWB_ACT_NONE) {
 #pragma unroll
-              for (int j = 0; j < 8; ++j) acc[j] = act_apply(acc[j], p.act);
+              for (int j = 0; j < 8; ++j) acc[j] = act_apply(acc[j], p);
             }
             if (p.residual) {
               const uint4 r = res_vec ? resv[PREFETCH_RES ? it : 0]
@@ -606,15 +611,14 @@ gemm_decode_cluster_kernel(const __grid_constant__ CUtensorMap tmap_w, const __g
             }
           }
         } else if (gemm_act_pairs(p.act)) {
-          const int a1 = p.act == SWB_ACT_SWIGLU_PAIRS ? SWB_ACT_SILU : SWB_ACT_GELU_TANH;
           for (int j = 0; j + 1 < nvalid; j += 2) {
             const float gte = acc[j] + (p.bias ? __bfloat162float(p.bias[feat + j]) : 0.f);
             const float up = acc[j + 1] + (p.bias ? __bfloat162float(p.bias[feat + j + 1]) : 0.f);
-            reinterpret_cast<bf16*>(p.out)[(size_t)tok * p.ldd + ((feat + j) >> 1)] = __float2bfloat16(act_apply(gte, a1) * up);
+            reinterpret_cast<bf16*>(p.out)[(size_t)tok * p.ldd + ((feat + j) >> 1)] = __float2bfloat16(gated_pair(gte, up, p));
           }
         } else {
           for (int j = 0; j < nvalid; ++j) {
-            float x = act_apply(acc[j] + (p.bias ? __bfloat162float(p.bias[feat + j]) : 0.f), p.act);
+            float x = act_apply(acc[j] + (p.bias ? __bfloat162float(p.bias[feat + j]) : 0.f), p);
             if (p.residual) x += __bfloat162float(p.residual[(size_t)tok * p.ld_res + feat + j]);
             if (p.out_fp32)
               reinterpret_cast<float*>(p.out)[off + j] = x;
@@ -730,6 +734,7 @@ int gemm_decode_cluster_launch(const GemmArgs& a, int force_cluster, cudaStream_
   p.residual = reinterpret_cast<const __nv_bfloat16*>(a.residual);
   p.ld_res = a.ld_res;
   p.act = a.act;
+  p.act_a = a.act_a, p.act_b = a.act_b;
   p.ssq_out = reinterpret_cast<unsigned long long*>(a.ssq_out);
   p.ssq_in = reinterpret_cast<const unsigned long long*>(a.ssq_in);
   p.ssq_zero = reinterpret_cast<unsigned long long*>(a.ssq_zero);

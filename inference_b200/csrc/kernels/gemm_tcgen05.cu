@@ -102,10 +102,12 @@ struct SegIter {
   }
 };
 
-__device__ __forceinline__ float apply_act(float x, int act) {
+__device__ __forceinline__ float apply_act(float x, const GemmParams& p) {
+  const int act = p.act;
   if (act == SWB_ACT_SILU) return silu_f(x);
   if (act == SWB_ACT_GELU_TANH) return gelu_tanh_f(x);
   if (act == SWB_ACT_RELU2) return relu2_f(x);
+  if (act == SWB_ACT_XIELU) return xielu_f(x, p.act_a, p.act_b);
   return x;
 }
 
@@ -132,7 +134,7 @@ __device__ __forceinline__ void epilogue_store16(const GemmParams& p, float* v, 
       }
       if (p.act != SWB_ACT_NONE) {
 #pragma unroll
-        for (int j = 0; j < 16; ++j) v[j] = apply_act(v[j], p.act);
+        for (int j = 0; j < 16; ++j) v[j] = apply_act(v[j], p);
       }
       if (p.residual) {
         const uint4* rp = reinterpret_cast<const uint4*>(p.residual + (size_t)row * p.ld_res + col0);
@@ -178,7 +180,7 @@ __device__ __forceinline__ void epilogue_store16(const GemmParams& p, float* v, 
       for (int j = 0; j < nvalid; ++j) {
         float x = v[j];
         if (p.bias) x += __bfloat162float(p.bias[col0 + j]);
-        x = apply_act(x, p.act);
+        x = apply_act(x, p);
         if (p.residual) x += __bfloat162float(p.residual[(size_t)row * p.ld_res + col0 + j]);
         if (p.out_fp32)
           reinterpret_cast<float*>(p.out)[off + j] = x;
@@ -191,7 +193,7 @@ __device__ __forceinline__ void epilogue_store16(const GemmParams& p, float* v, 
 #pragma unroll 4
     for (int j = 0; j < nvalid; ++j) {
       const int tok = col0 + j;
-      float x = apply_act(v[j] + b, p.act);
+      float x = apply_act(v[j] + b, p);
       if (p.residual) x += __bfloat162float(p.residual[(size_t)tok * p.ld_res + row]);
       const size_t off = (size_t)tok * p.ldd + row;
       if (p.out_fp32)
@@ -245,7 +247,7 @@ __device__ __forceinline__ void epilogue_scatter_staged(const GemmParams& p, uin
       }
       if (p.act != SWB_ACT_NONE) {
 #pragma unroll
-        for (int j = 0; j < 16; ++j) v[j] = apply_act(v[j], p.act);
+        for (int j = 0; j < 16; ++j) v[j] = apply_act(v[j], p);
       }
       if (p.residual && row0 + lane < p.M && col0 < p.N) {
         const uint4* rp = reinterpret_cast<const uint4*>(p.residual + (size_t)(row0 + lane) * p.ld_res + col0);
@@ -831,6 +833,7 @@ int gemm_bf16_launch(const GemmArgs& a, cudaStream_t stream) {
   p.residual = reinterpret_cast<const bf16*>(a.residual);
   p.ld_res = a.ld_res;
   p.act = a.act;
+  p.act_a = a.act_a, p.act_b = a.act_b;
   p.status = nullptr;
   if (a.scatter) {
     p.scatter = *a.scatter;

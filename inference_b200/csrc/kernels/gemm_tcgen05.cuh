@@ -10,10 +10,12 @@ namespace swb {
 
 // 3 / 4: gated pairs. Output features come in (gate, up) row pairs of the weight: out[t, f] = silu|gelu(acc[2f]) * acc[2f+1],
 // so the output is half as wide as the weight has rows (SwiGLU / GeGLU fused into the gate-up projection).
-// 5: square of relu (ungated).
+// 5: square of relu (ungated). 6: xIELU (ungated) with act_a, act_b. 7: gated pairs with both parts clamped at act_a.
 enum GemmAct : int { SWB_ACT_NONE = 0, SWB_ACT_SILU = 1, SWB_ACT_GELU_TANH = 2, SWB_ACT_SWIGLU_PAIRS = 3,
-                     SWB_ACT_GEGLU_PAIRS = 4, SWB_ACT_RELU2 = 5 };
-__host__ __device__ inline bool gemm_act_pairs(int act) { return act == SWB_ACT_SWIGLU_PAIRS || act == SWB_ACT_GEGLU_PAIRS; }
+                     SWB_ACT_GEGLU_PAIRS = 4, SWB_ACT_RELU2 = 5, SWB_ACT_XIELU = 6, SWB_ACT_CLAMPED_PAIRS = 7 };
+__host__ __device__ inline bool gemm_act_pairs(int act) {
+  return act == SWB_ACT_SWIGLU_PAIRS || act == SWB_ACT_GEGLU_PAIRS || act == SWB_ACT_CLAMPED_PAIRS;
+}
 
 // The first SWB_GEMM_COUNTER_BYTES of a GEMM workspace hold per-tile arrival counters (zero between
 // launches: the caller zeroes them once, the kernel restores zero); fp32 split-K partials follow.
@@ -77,6 +79,7 @@ struct GemmParams {
   const __nv_bfloat16* residual;
   int ld_res;
   int act;
+  float act_a, act_b;   // parameters of the activation, where it has any
   float* workspace;
   int* counters;
   int* status;
@@ -135,6 +138,7 @@ struct GemmArgs {
   float norm_eps = 0.f;
   const GemmPeerReduce* peer = nullptr;  // see GemmPeerReduce (decode cluster kernel only)
   int conv_n = 0, conv_h = 0, conv_w = 0, conv_c = 0;   // see GemmParams: A = NHWC activation, T = n h w, K = 9 c
+  float act_a = 0.f, act_b = 0.f;
 };
 
 int gemm_bf16_launch(const GemmArgs& a, cudaStream_t stream);

@@ -382,7 +382,8 @@ __global__ void __launch_bounds__(256) rope_kv_write_d128_kernel(
   }
 }
 
-// Norms over whole query / key projections (all heads of a token at once), rotation, cache write: one CTA per token.
+// Norms over whole query / key projections (all heads of a token at once) or over every head by itself, rotation, cache write: one CTA
+// per token.
 struct RowRopeParams {
   void* buf;                  // [T, ld]: q (H heads of D) at 0, k (G heads of D) behind it, v (G heads of Dv) at v_col
   int ld, v_col, H, G, D, Dv, rot;
@@ -396,6 +397,8 @@ struct RowRopeParams {
   int block_size;
   int v_from_k;               // values are the keys as projected (Dv == D)
   int store_v;                // v_from_k: also store them at v_col
+  int GV;                     // value heads
+  int unit;                   // > 0: q and k heads are divided by their own root mean square over `unit` columns, no weight
 };
 
 template <typename E>
@@ -403,7 +406,8 @@ __global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p)
   pdl_launch_dependents();
   pdl_wait(TL_ROPE_KV);
   __shared__ float red[2][8];
-  const int t = blockIdx.x, nq8 = p.H * p.D / 8, nk8 = p.G * p.D / 8, nv8 = p.G * p.Dv / 8;
+  extern __shared__ float part[];            // unit: sums of squares of the pieces of eight columns
+  const int t = blockIdx.x, nq8 = p.H * p.D / 8, nk8 = p.G * p.D / 8, nv8 = p.GV * p.Dv / 8;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   E* q = reinterpret_cast<E*>(p.buf) + (size_t)t * p.ld;
   E* k = q + nq8 * 8;
@@ -426,14 +430,25 @@ __global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p)
     for (int w = 0; w < warps; ++w) sq += red[0][w], sk += red[1][w];
     rq = rsqrtf(sq / (float)p.nq + p.eps), rk = rsqrtf(sk / (float)p.nk + p.eps);
   }
+  if (p.unit > 0) {           // a rotation leaves the sum of squares as it is
+    for (int i = threadIdx.x; i < nq8 + nk8; i += blockDim.x) {
+      float x[8], ss = 0.f;
+      load_row8(q + i * 8, x);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(x[j], x[j], ss);
+      part[i] = ss;
+    }
+    __syncthreads();
+  }
   const long long slot = p.slots[t];
   E *kc = nullptr, *vc = nullptr;
   const size_t page = slot >= 0 ? (size_t)(slot / p.block_size) * p.G * p.block_size + slot % p.block_size : 0;
+  const size_t vpage = slot >= 0 ? (size_t)(slot / p.block_size) * p.GV * p.block_size + slot % p.block_size : 0;
   if (slot >= 0) kc = reinterpret_cast<E*>(p.kcache), vc = reinterpret_cast<E*>(p.vcache);
   const int half = p.rot / 2;
   const float* cs = p.cos + (size_t)p.positions[t] * half;
   const float* sn = p.sin + (size_t)p.positions[t] * half;
-  const int first = p.wk || p.rot > 0 ? 0 : nq8;            // nothing to do for the queries
+  const int first = p.wk || p.unit > 0 || p.rot > 0 ? 0 : nq8;            // nothing to do for the queries
   for (int i = first + threadIdx.x; i < nq8 + nk8; i += blockDim.x) {
     const bool is_q = i < nq8;
     const int j8 = is_q ? i : i - nq8, h = j8 * 8 / p.D, d = j8 * 8 - h * p.D;
@@ -451,6 +466,14 @@ __global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p)
 #pragma unroll
       for (int j = 0; j < 8; ++j) x[j] *= r * w[j];
     }
+    if (p.unit > 0) {
+      const float* ps = part + i - d / 8;                   // the pieces of this head
+      float ss = 0.f;
+      for (int m = 0; m < p.D / 8; ++m) ss += ps[m];
+      const float r = rsqrtf(ss / (float)p.unit + p.eps);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] *= r;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       if (d + 2 * j >= p.rot) continue;
@@ -458,7 +481,7 @@ __global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p)
       x[2 * j] = a * c - b * s;
       x[2 * j + 1] = b * c + a * s;
     }
-    if (p.wk || p.rot > 0) store_row8(at, x);
+    if (p.wk || p.unit > 0 || p.rot > 0) store_row8(at, x);
     if (!is_q && kc) store_row8(kc + (page + (size_t)h * p.block_size) * p.D + d, x);
   }
   if (!p.v_from_k && vc) {
@@ -466,7 +489,7 @@ __global__ void __launch_bounds__(256) row_rope_kv_kernel(const RowRopeParams p)
       const int h = i * 8 / p.Dv, d = i * 8 - h * p.Dv;
       float x[8];
       load_row8(v + i * 8, x);
-      store_row8(vc + (page + (size_t)h * p.block_size) * p.Dv + d, x);
+      store_row8(vc + (vpage + (size_t)h * p.block_size) * p.Dv + d, x);
     }
   }
 }
@@ -493,16 +516,78 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(const E* __restrict__
   for (int d = lane; d < Dv; d += 32) from_f(o[d], (to_f(a[d]) - lambda * to_f(a[Dv + d])) * r);
 }
 
+// Heads that exchange their attention weights: with a[t, g, c] the weights of query head g applied to the values of key/value head c,
+//     out[t, h] = sigmoid(gate[t, h]) sum_g talk[h, g] a[t, g, c(h)],   c(h) = h / (H / G)
+// because the weighted sum over the heads' weights passes through the (linear) application to the values. A thread owns two columns of
+// one c for TT tokens and up to HM of its query heads.
+constexpr int HM = 8;
+struct HeadMixParams {
+  const void* a;              // [T, H, G, Dv] (a token's part contiguous), a_tok apart
+  long long a_tok;
+  const float* talk;          // [H (g), G (c), HP]: talk[c * H / G + i, g] at i, HP = H / G rounded up to HM, zeros behind
+  const void* gate;           // optional logits [T, >= H], gate_tok apart
+  long long gate_tok;
+  void* out;                  // [T, H * Dv], out_tok apart
+  long long out_tok;
+  int T, H, G, Dv;
+};
+
+template <typename E, int TT>
+__global__ void __launch_bounds__(128) head_mix_kernel(const HeadMixParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int col = (blockIdx.x * 128 + threadIdx.x) * 2, width = p.G * p.Dv, t0 = blockIdx.y * TT;
+  if (col >= width) return;
+  const int c = col / p.Dv, per = p.H / p.G, hp = (per + HM - 1) / HM * HM, h0 = blockIdx.z * HM;
+  const E* a = reinterpret_cast<const E*>(p.a) + col;
+  const float* talk = p.talk + (size_t)c * hp + h0;
+  float acc[HM][TT][2] = {};
+#pragma unroll 4
+  for (int g = 0; g < p.H; ++g) {
+    const float4 w0 = __ldg(reinterpret_cast<const float4*>(talk + (size_t)g * p.G * hp)), w1 = __ldg(reinterpret_cast<const float4*>(talk + (size_t)g * p.G * hp) + 1);
+    const float w[HM] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+    for (int i = 0; i < TT; ++i) {
+      if (t0 + i >= p.T) break;
+      const E* at = a + (t0 + i) * p.a_tok + (size_t)g * width;
+      float x, y;
+      if constexpr (sizeof(E) == 2) {
+        const uint32_t u = *reinterpret_cast<const uint32_t*>(at);
+        x = __uint_as_float(u << 16), y = __uint_as_float(u & 0xffff0000u);
+      } else {
+        const float2 u = *reinterpret_cast<const float2*>(at);
+        x = u.x, y = u.y;
+      }
+#pragma unroll
+      for (int h = 0; h < HM; ++h) acc[h][i][0] = fmaf(w[h], x, acc[h][i][0]), acc[h][i][1] = fmaf(w[h], y, acc[h][i][1]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < TT; ++i) {
+    const int t = t0 + i;
+    if (t >= p.T) break;
+#pragma unroll
+    for (int h = 0; h < HM; ++h) {
+      if (h0 + h >= per) break;
+      const int head = c * per + h0 + h;
+      const float s = p.gate ? 1.f / (1.f + expf(-to_f(reinterpret_cast<const E*>(p.gate)[t * p.gate_tok + head]))) : 1.f;
+      E* o = reinterpret_cast<E*>(p.out) + t * p.out_tok + (size_t)head * p.Dv + col % p.Dv;
+      from_f(o[0], acc[h][i][0] * s), from_f(o[1], acc[h][i][1] * s);
+    }
+  }
+}
+
 __device__ __forceinline__ float gated_act(float g, bool gelu, bool exact) {
   if (gelu) return gelu_tanh_f(g);
   return exact ? g / (1.f + expf(-g)) : silu_f(g);
 }
 
 // out[t, f] = act(gu[t, f]) * gu[t, F + f]; act 1 = SiLU (SwiGLU), 2 = tanh-GELU (GeGLU). act 3 / 4: the same two
-// activations on a pair-interleaved projection output, out[t, f] = act(gu[t, 2f]) * gu[t, 2f + 1]. row_gate (fp32 logits, one per
+// activations on a pair-interleaved projection output, out[t, f] = act(gu[t, 2f]) * gu[t, 2f + 1]. act 5 / 6: the gated unit with both
+// parts clamped at `limit`, side by side / interleaved. row_gate (fp32 logits, one per
 // row, `gate_ld` apart): the row is scaled by its sigmoid.
 template <typename E>
-__global__ void __launch_bounds__(256) gated_act_mul_kernel(const E* __restrict__ gu, int ld_gu, E* out, int ldo, int T, int F, int act,
+__global__ void __launch_bounds__(256) gated_act_mul_kernel(const E* __restrict__ gu, int ld_gu, E* out, int ldo, int T, int F, int act, float limit,
                                                            const float* __restrict__ row_gate, int gate_ld) {
   pdl_launch_dependents();
   pdl_wait(TL_GATED_ACT);
@@ -512,7 +597,7 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const E* __restrict_
   const int t = (int)(idx / nvec);
   const int v = (int)(idx % nvec);
   float g[8], u[8], o[8];
-  if (act >= 3) {
+  if (act == 3 || act == 4 || act == 6) {
     float lo[8], hi[8];
     load_row8(gu + (size_t)t * ld_gu + v * 16, lo);
     load_row8(gu + (size_t)t * ld_gu + v * 16 + 8, hi);
@@ -529,7 +614,8 @@ __global__ void __launch_bounds__(256) gated_act_mul_kernel(const E* __restrict_
   }
   const bool gelu = act == 2 || act == 4;
 #pragma unroll
-  for (int j = 0; j < 8; ++j) o[j] = gated_act(g[j], gelu, sizeof(E) == 4) * u[j];
+  for (int j = 0; j < 8; ++j)
+    o[j] = act >= 5 ? clamped_gate_f<sizeof(E) == 4>(g[j], u[j], limit) : gated_act(g[j], gelu, sizeof(E) == 4) * u[j];
   if (row_gate) {
     const float s = 1.f / (1.f + expf(-row_gate[(size_t)t * gate_ld]));
 #pragma unroll
@@ -800,7 +886,7 @@ int swb_poly_norm(const void* z, int ldz, void* out, int ldo, int T, int F, int 
   return launch_poly_norm(reinterpret_cast<const bf16*>(z), ldz, reinterpret_cast<bf16*>(out), ldo, T, F, Fp, coef, eps, s);
 }
 // row_gate: see gated_act_mul_kernel; fp32 selects the element type of gate_up and out.
-int swb_gated_act_mul_ex(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, const float* row_gate, int gate_ld,
+int swb_gated_act_mul_ex(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, float limit, const float* row_gate, int gate_ld,
                          int fp32, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
@@ -810,29 +896,49 @@ int swb_gated_act_mul_ex(const void* gate_up, int ld_gu, void* out, int ldo, int
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (fp32)
     return launch_kernel(gated_act_mul_kernel<float>, grid, block, 0, s, reinterpret_cast<const float*>(gate_up), ld_gu,
-                         reinterpret_cast<float*>(out), ldo, T, F, act, row_gate, gate_ld);
+                         reinterpret_cast<float*>(out), ldo, T, F, act, limit, row_gate, gate_ld);
   return launch_kernel(gated_act_mul_kernel<bf16>, grid, block, 0, s, reinterpret_cast<const bf16*>(gate_up), ld_gu,
-                       reinterpret_cast<bf16*>(out), ldo, T, F, act, row_gate, gate_ld);
+                       reinterpret_cast<bf16*>(out), ldo, T, F, act, limit, row_gate, gate_ld);
 }
 int swb_gated_act_mul(const void* gate_up, int ld_gu, void* out, int ldo, int T, int F, int act, void* stream) {
-  return swb_gated_act_mul_ex(gate_up, ld_gu, out, ldo, T, F, act, nullptr, 0, 0, stream);
+  return swb_gated_act_mul_ex(gate_up, ld_gu, out, ldo, T, F, act, 0.f, nullptr, 0, 0, stream);
 }
 
-// See RowRopeParams. D, Dv, ld and v_col multiples of 8, buffers 16-byte aligned (32 in fp32).
+// See RowRopeParams. D, Dv, ld and v_col multiples of 8, buffers 16-byte aligned (32 in fp32). GV 0: as many value heads as key heads.
 int swb_row_rope_kv_write(void* buf, int ld, int v_col, int H, int G, int D, int Dv, int rot, const float* wq, const float* wk, int nq, int nk,
                           float eps, const float* cos, const float* sin, const int* positions, const long long* slots, void* kcache,
-                          void* vcache, int block_size, int v_from_k, int store_v, int T, int fp32, void* stream) {
+                          void* vcache, int block_size, int v_from_k, int store_v, int GV, int unit, int T, int fp32, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
+  if (GV <= 0) GV = G;
+  if (unit < 0 || unit > D || (unit && wk) || (v_from_k && GV != G)) return -3;
   if (H < 0 || G < 1 || D < 8 || Dv < 8 || ((D | Dv | ld | v_col) % 8) || rot < 0 || rot > D || (rot % 2) || block_size < 1 || !kcache || !vcache ||
       !slots || (wk && (nk < 1 || (H > 0 && (!wq || nq < 1)))) || (v_from_k && Dv != D))
     return -3;
   const RowRopeParams p{buf, ld, v_col, H, G, D, Dv, rot, wq, wk, nq > 0 ? nq : 1, nk > 0 ? nk : 1, eps, cos, sin, positions, slots, kcache,
-                        vcache, block_size, v_from_k, store_v};
+                        vcache, block_size, v_from_k, store_v, GV, unit};
   const int work = (H + G) * D / 8;
   const dim3 grid((unsigned)T), block(work <= 64 ? 64 : work <= 128 ? 128 : 256);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return fp32 ? launch_kernel(row_rope_kv_kernel<float>, grid, block, 0, s, p) : launch_kernel(row_rope_kv_kernel<bf16>, grid, block, 0, s, p);
+  const size_t smem = unit ? (size_t)work * sizeof(float) : 0;
+  if (smem > 48 * 1024) return -3;
+  return fp32 ? launch_kernel(row_rope_kv_kernel<float>, grid, block, smem, s, p) : launch_kernel(row_rope_kv_kernel<bf16>, grid, block, smem, s, p);
+}
+
+// See HeadMixParams. Dv and the strides even, rows 8-byte aligned; talk 16-byte aligned.
+int swb_head_mix(const void* a, long long a_tok, const float* talk, const void* gate, long long gate_tok, void* out, long long out_tok, int T,
+                 int H, int G, int Dv, int fp32, void* stream) {
+  using namespace swb;
+  if (T <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || Dv < 2 || ((Dv | a_tok | out_tok) % 2) || !talk) return -3;
+  const HeadMixParams p{a, a_tok, talk, gate, gate_tok, out, out_tok, T, H, G, Dv};
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const unsigned x = (G * Dv / 2 + 127) / 128, z = (H / G + HM - 1) / HM;
+  if (T < 512)
+    return fp32 ? launch_kernel(head_mix_kernel<float, 1>, dim3(x, T, z), dim3(128), 0, s, p)
+                : launch_kernel(head_mix_kernel<bf16, 1>, dim3(x, T, z), dim3(128), 0, s, p);
+  return fp32 ? launch_kernel(head_mix_kernel<float, 4>, dim3(x, (T + 3) / 4, z), dim3(128), 0, s, p)
+              : launch_kernel(head_mix_kernel<bf16, 4>, dim3(x, (T + 3) / 4, z), dim3(128), 0, s, p);
 }
 
 int swb_diff_combine(const void* in, long long in_tok, void* out, long long out_tok, int T, int H, int Dv, int N, float lambda, float eps,

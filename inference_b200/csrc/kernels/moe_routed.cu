@@ -1,6 +1,6 @@
 // Mixture-of-experts feed-forward: routing plans, from a table or from router logits, and the small-batch grouped GEMM.
 //
-// moe_route_kernel / moe_layout_kernel: softmax over a token's router logits (fp32), the `top` largest, and their places in an
+// moe_route_kernel / moe_layout_kernel: softmax over a token's router logits (fp32), the `top` largest (as they are, or divided by their sum), and their places in an
 // expert-sorted buffer of the same two layouts as below. Small steps do it in one launch (the last CTA to finish lays the pairs
 // out); large ones lay out in a second, which also copies the rows to their places. The counters clean up after themselves.
 //
@@ -121,6 +121,7 @@ struct RouteParams {
   int* expert;               // [T * top]
   int* rank;                 // [T * top] place of the pair among those of its expert
   float* weights;            // [T * top] softmax scores
+  int renorm;                // 1: divided by the sum of the chosen ones
   int* counters;             // [E + 2] pairs per expert, two tickets; zero between launches
   int* dest;                 // [T * top]
   int* src;                  // optional [rows_cap]
@@ -202,6 +203,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const RouteParams p) {
     sum = warp_sum(sum);
     float last = INFINITY, mine = 0.f;      // lane k mod 32 keeps choice k until 32 of them (or all) are filed together
     int last_e = -1, mine_e = 0;
+    float chosen = 0.f;                     // sum of the chosen scores, times `sum`
     for (int k = 0; k < p.top; ++k) {
       float best = -INFINITY;
       int best_e = p.E;
@@ -217,6 +219,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const RouteParams p) {
         if (e < p.E && (best_e == p.E || v > best || (v == best && e < best_e))) best = v, best_e = e;
       }
       last = best, last_e = best_e;
+      chosen += expf(best - top);
       if (lane == (k & 31)) mine = best, mine_e = min(best_e, p.E - 1);     // logits that are not numbers: any expert
       if ((k & 31) == 31 || k == p.top - 1) {
         const int pair = t * p.top + (k & ~31) + lane;
@@ -226,6 +229,11 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const RouteParams p) {
           p.rank[pair] = atomicAdd(p.counters + mine_e, 1);
         }
       }
+    }
+    if (p.renorm) {
+      __syncwarp();
+      const float share = chosen / sum + 1e-20f;
+      for (int k = lane; k < p.top; k += 32) p.weights[t * p.top + k] /= share;      // written by this lane above
     }
   }
   if constexpr (WHOLE) {
@@ -291,6 +299,7 @@ struct GroupedRowsParams {
   const bf16* w;         // [E, N, K]
   bf16* out;
   int ldo, N, K, act;    // act may be a gated pair: rows of w in (gate, up) pairs, out [*, N / 2]
+  float act_a;           // its parameter
   int plan_ahead;        // the plan was complete before the kernel in front of this one started
 };
 
@@ -348,7 +357,9 @@ __device__ __forceinline__ void grouped_pass(const GroupedRowsParams& p, const b
         float a = 0.f, b = 0.f;
 #pragma unroll
         for (int w = 0; w < GR_WARPS; ++w) a += red[w * (8 * NT * FW) + tok * FW + f], b += red[w * (8 * NT * FW) + tok * FW + f + 1];
-        p.out[(size_t)(r0 + tok) * p.ldo + (f0 + f) / 2] = __float2bfloat16((p.act == SWB_ACT_GEGLU_PAIRS ? gelu_tanh_f(a) : silu_f(a)) * b);
+        const float y = p.act == SWB_ACT_CLAMPED_PAIRS ? clamped_gate_f<false>(a, b, p.act_a)
+                                                       : (p.act == SWB_ACT_GEGLU_PAIRS ? gelu_tanh_f(a) : silu_f(a)) * b;
+        p.out[(size_t)(r0 + tok) * p.ldo + (f0 + f) / 2] = __float2bfloat16(y);
       }
     }
     __syncthreads();
@@ -413,10 +424,10 @@ int swb_moe_table_plan(const long long* ids, int T, const int* tables, int layer
 }
 
 // Routing plan of one layer from router logits [T, ld] (fp32): the `top` experts of the largest softmax scores over all E, weights
-// [T, top] = their scores as they are. dest, src, offsets, active, tile_group, pad and rows_cap as in swb_moe_table_plan.
+// [T, top] = their scores, as they are or (renorm) divided by their sum + 1e-20. dest, src, offsets, active, tile_group, pad and rows_cap as in swb_moe_table_plan.
 // expert and rank: int32 scratch [T * top]; counters: int32 [E + 2], zero at the first launch, launches that share it ordered on
 // one stream. rows_in (nullable): bf16 / fp32 rows of `pieces` 16-byte pieces, ld_in pieces apart, copied to rows dest[t, k] of rows_out.
-int swb_moe_route(const float* logits, int ld, int T, int E, int top, int pad, int* expert, int* rank, float* weights, int* counters,
+int swb_moe_route(const float* logits, int ld, int T, int E, int top, int renorm, int pad, int* expert, int* rank, float* weights, int* counters,
                   int* dest, int* src, int* offsets, int* active, int* tile_group, int rows_cap, const void* rows_in, long long ld_in,
                   void* rows_out, long long ld_out, int pieces, void* stream) {
   using namespace swb;
@@ -425,7 +436,7 @@ int swb_moe_route(const float* logits, int ld, int T, int E, int top, int pad, i
       (long long)T * top + (long long)E * (pad - 1) > (long long)rows_cap || !expert || !rank || !weights || !counters || !dest || !offsets ||
       (rows_in && (!rows_out || pieces <= 0)))
     return -3;
-  const RouteParams p{logits, ld, T, E, top, pad, expert, rank, weights, counters, dest, src, offsets, active, tile_group, rows_cap,
+  const RouteParams p{logits, ld, T, E, top, pad, expert, rank, weights, renorm, counters, dest, src, offsets, active, tile_group, rows_cap,
                       reinterpret_cast<const uint4*>(rows_in), reinterpret_cast<uint4*>(rows_out), ld_in, ld_out, pieces};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid((unsigned)((T + 7) / 8));
@@ -441,14 +452,14 @@ int swb_moe_route(const float* logits, int ld, int T, int E, int top, int pad, i
 // W [E, N, K] bf16, K % 8 == 0, ldx % 8 == 0, x and W 16-byte aligned; n_active = length of `active`. plan_ahead: see
 // GroupedRowsParams.
 int swb_gemm_grouped_rows(const void* x, int ldx, const int* src, const int* offsets, const int* active, int n_active,
-                          const void* w, void* out, int ldo, int N, int K, int act, int plan_ahead, void* stream) {
+                          const void* w, void* out, int ldo, int N, int K, int act, float act_a, int plan_ahead, void* stream) {
   using namespace swb;
   if (n_active <= 0 || N <= 0 || K <= 0) return 0;
   if ((K % 8) || (ldx % 8) || !offsets || !active || (gemm_act_pairs(act) && (N & 1)) ||
       ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15))
     return -3;
   GroupedRowsParams p{reinterpret_cast<const bf16*>(x), ldx, src, offsets, active, reinterpret_cast<const bf16*>(w),
-                      reinterpret_cast<bf16*>(out), ldo, N, K, act, plan_ahead};
+                      reinterpret_cast<bf16*>(out), ldo, N, K, act, act_a, plan_ahead};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   // 32 weight rows per CTA halve the token re-reads; 16 when that is needed to give every SM two CTAs
   if ((long long)((N + 31) / 32) * n_active >= 2 * 148)

@@ -41,13 +41,14 @@ class PagedKvPool:
 
 @dataclass(frozen=True)
 class KvGeometry:
-    """K / V pages of one cache-owning layer run."""
+    """K / V pages of one cache-owning layer run. v_heads: value heads, where they are not cached like the keys (0: like the keys)."""
     kv_heads: int
     k_dim: int
     v_dim: int
+    v_heads: int = 0
 
     def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
-        return [(self.kv_heads, block_size, self.k_dim), (self.kv_heads, block_size, self.v_dim)]
+        return [(self.kv_heads, block_size, self.k_dim), (self.v_heads or self.kv_heads, block_size, self.v_dim)]
 
 
 @dataclass(frozen=True)
@@ -78,18 +79,30 @@ class StateGeometry:
         return []
 
 
+@dataclass(frozen=True)
+class WindowGeometry:
+    """Short convolution over time: per sequence a window of recent inputs in the activation type; no pages."""
+    window: tuple[int, ...]
+
+    def page_shapes(self, block_size: int) -> list[tuple[int, ...]]:
+        return []
+
+
+PER_SEQUENCE = (StateGeometry, WindowGeometry)      # what a state slot holds
+
+
 class LayeredKvPool:
     """Paged pool of a model whose layers differ in what they keep, or run more than once: every run owns its page tensors
-    [blocks, ...] (K and V, latent rows, or token ids). Block ids are shared by all runs (one allocator), so sequences, forks and
-    rollbacks work as on the uniform pool. Recurrent layers own tensors [state_slots, ...] instead; a sequence holds one slot
+    [blocks, ...] (K and V, latent rows, or token ids), or several such entries. Block ids are shared by all runs (one allocator), so sequences, forks and
+    rollbacks work as on the uniform pool. Recurrent layers and short convolutions own tensors [state_slots, ...] instead; a sequence holds one slot
     for all of them from its first token to its release. A slot needs no clearing: the kernels take the state of a sequence
     as zero at position 0."""
 
-    def __init__(self, geometry: list[KvGeometry | LatentGeometry | TokenGeometry | StateGeometry], num_blocks: int, block_size: int = 16,
+    def __init__(self, geometry: list[KvGeometry | LatentGeometry | TokenGeometry | StateGeometry | WindowGeometry], num_blocks: int, block_size: int = 16,
                  device: torch.device | str = "cuda", dtype: torch.dtype = torch.bfloat16, state_slots: int = 0):
         self.geometry, self.num_layers = list(geometry), len(geometry)
         self.num_blocks, self.block_size = num_blocks, block_size
-        self.has_state = any(isinstance(g, StateGeometry) for g in geometry)
+        self.has_state = any(isinstance(g, PER_SEQUENCE) for g in geometry)
         if self.has_state and state_slots < 1:
             raise ValueError("a pool with recurrent layers needs state slots")
 
@@ -97,6 +110,8 @@ class LayeredKvPool:
             if isinstance(g, StateGeometry):
                 return (torch.zeros((state_slots, *g.state), dtype=torch.float32, device=device),
                         torch.zeros((state_slots, *g.window), dtype=dtype, device=device))
+            if isinstance(g, WindowGeometry):
+                return (torch.zeros((state_slots, *g.window), dtype=dtype, device=device),)
             kind = torch.int32 if isinstance(g, TokenGeometry) else dtype
             return tuple(torch.zeros((num_blocks, *s), dtype=kind, device=device) for s in g.page_shapes(block_size))
         self.data = [tensors(g) for g in geometry]
@@ -109,13 +124,13 @@ class LayeredKvPool:
 
     def copy_block(self, src: int, dst: int) -> None:
         for g, kv in zip(self.geometry, self.data):
-            if not isinstance(g, StateGeometry):
+            if not isinstance(g, PER_SEQUENCE):
                 for t in kv:
                     t[dst].copy_(t[src])
 
     def copy_state(self, src: int, dst: int) -> None:
         for g, kv in zip(self.geometry, self.data):
-            if isinstance(g, StateGeometry):
+            if isinstance(g, PER_SEQUENCE):
                 for t in kv:
                     t[dst].copy_(t[src])
 

@@ -29,6 +29,7 @@ class Architecture(enum.Enum):
     QWEN3_VL = "qwen3_vl"    # VLM-wrapped Qwen3 decoder with interleaved M-RoPE
     ZOBUNEX = "zobunex"      # listed layers with a loop, chunked sink attention, sandwich layer norms, token-routed experts
     ROTALORN = "rotalorn"    # listed layers with parallel sublayers: windowed, latent and differential attention, dense / routed experts
+    NAFELIX = "nafelix"      # listed layers with a loop over several streams: talking heads beside a delta rule, gated attention
     GUNEDRA = "gunedra"      # listed layers: latent attention and channel-wise delta rule, output norms, depth averages
 
     @staticmethod
@@ -81,7 +82,7 @@ class Architecture(enum.Enum):
         return self in (Architecture.GEMMA2, Architecture.GLM4)
 
 
-LISTED = (Architecture.ZOBUNEX, Architecture.GUNEDRA, Architecture.ROTALORN)     # designs whose config lists the layers one by one
+LISTED = (Architecture.ZOBUNEX, Architecture.GUNEDRA, Architecture.ROTALORN, Architecture.NAFELIX)     # designs whose config lists the layers one by one
 
 
 @dataclass(frozen=True)
@@ -219,11 +220,44 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class HeadDeltaSpec(ChannelDeltaSpec):
+    """The same with one decay per head."""
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers side by side on one input: attention whose heads exchange their weights, and a delta rule."""
+    left: AttentionSpec
+    right: HeadDeltaSpec
+
+    @property
+    def heads(self) -> int:
+        return max(self.left.heads, self.right.heads)
+
+    @property
+    def kv_heads(self) -> int:
+        return self.left.kv_heads
+
+    @property
+    def dim(self) -> int:
+        return max(self.left.dim, self.right.dim)
+
+    @property
+    def vdim(self) -> int:
+        return max(self.left.vdim, self.right.vdim)
+
+    @property
+    def groups(self) -> int:
+        return self.left.groups
+
+
+@dataclass(frozen=True)
 class ExpertsSpec:
     experts: int
     top: int
     ff: int
     shared: int = 0      # feed-forward width of an expert that every token uses
+    limit: float = 0.0   # > 0: both parts of the gated unit are clamped there
 
 
 @dataclass(frozen=True)
@@ -233,7 +267,7 @@ class DenseSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | LatentAttentionSpec | DifferentialSpec | ChannelDeltaSpec
+    mixer: AttentionSpec | LatentAttentionSpec | DifferentialSpec | ChannelDeltaSpec | ParallelSpec
     mlp: ExpertsSpec | DenseSpec | None
 
 
@@ -288,13 +322,21 @@ def _window(m: Any, at: str) -> int:
     return _count(m["mask"], "size", at + "mask.") if m.get("mask") else 0
 
 
-def _windowed_spec(m: Any, at: str) -> AttentionSpec:
-    """Grouped heads whose values are the projected keys, within a window."""
+def _grouped_spec(m: Any, at: str) -> AttentionSpec:
+    """Grouped heads within a window."""
     rot = m.get("rot") or {"dims": 0, "base": 1.0}
     spec = AttentionSpec(_count(m, "heads", at), _count(m, "kv_heads", at), _count(m, "dim", at), _count(m, "vdim", at), _real(m, "scale", at), 0,
                          _count(rot, "dims", at + "rot.", 0), _real(rot, "base", at + "rot."), _rot_scaling(rot, at), _window(m, at))
-    if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim or spec.vdim != spec.dim:
-        raise ConfigError(f"config.json: `{at}` heads / kv_heads / dim / vdim / rot.dims do not fit together")
+    if spec.heads % spec.kv_heads or spec.rot_dims % 2 or spec.rot_dims > spec.dim:
+        raise ConfigError(f"config.json: `{at}` heads / kv_heads / rot.dims do not fit together")
+    return spec
+
+
+def _windowed_spec(m: Any, at: str) -> AttentionSpec:
+    """The same with the projected keys as values."""
+    spec = _grouped_spec(m, at)
+    if spec.vdim != spec.dim:
+        raise ConfigError(f"config.json: `{at}` dim / vdim do not fit together")
     return spec
 
 
@@ -340,6 +382,21 @@ def _channel_delta_spec(m: Any, at: str) -> ChannelDeltaSpec:
     return spec
 
 
+def _head_delta_spec(m: Any, at: str) -> HeadDeltaSpec:
+    return HeadDeltaSpec(**dataclasses.asdict(_channel_delta_spec(m, at)))
+
+
+def _parallel_spec(m: Any, at: str) -> ParallelSpec:
+    return ParallelSpec(_grouped_spec(_need(m, "left", at), at + "left."), _head_delta_spec(_need(m, "right", at), at + "right."))
+
+
+def _clamped_experts_spec(f: Any, at: str) -> ExpertsSpec:
+    s = dataclasses.replace(_experts_spec(f, at), limit=_real(f["expert"], "limit", at + "expert."))
+    if s.top > s.experts or s.limit <= 0:
+        raise ConfigError(f"config.json: `{at}` needs router.top <= router.experts and expert.limit > 0")
+    return s
+
+
 def _experts_spec(f: Any, at: str) -> ExpertsSpec:
     r = _need(f, "router", at)
     return ExpertsSpec(_count(r, "experts", at + "router."), _count(r, "top", at + "router."),
@@ -363,6 +420,7 @@ _LAYER_PARTS = {
     Architecture.GUNEDRA: ({"latent_attention": _latent_spec, "channel_delta": _channel_delta_spec}, {"dense": _dense_spec}),
     Architecture.ROTALORN: ({"attention": _windowed_spec, "latent_attention": _low_rank_latent_spec, "attention_2": _differential_spec},
                             {"dense": _dense_spec, "moe": _shared_experts_spec}),
+    Architecture.NAFELIX: ({"parallel": _parallel_spec, "attention": _grouped_spec}, {"dense": _dense_spec, "moe": _clamped_experts_spec}),
 }
 
 
@@ -376,6 +434,9 @@ class StackConfig:
     residual_mult: float = 1.0     # every sublayer's result joins the stream times this
     bigram: BigramSpec | None = None
     norm_groups: int = 1           # the stream norms take the root mean square of this many equal parts separately
+    streams: int = 1               # residual streams side by side
+    canon_taps: int = 0            # taps of a convolution over time on every sublayer's input (0: none)
+    tied: bool = True              # the embedding table gives the logits
 
     def runs(self) -> list[tuple[int, bool]]:
         """(layer, first layer of a loop pass) in execution order; every run owns a cache."""
@@ -421,6 +482,9 @@ class StackConfig:
                 raise ConfigError("config.json: `loop` does not lie within the layers")
             if loop.start == loop.stop:
                 loop = None
+        if arch is Architecture.NAFELIX:
+            return StackConfig(tuple(layers), loop, 1.0, streams=_count(top, "streams", ""), tied=False,
+                               canon_taps=_count(_need(top, "canon", ""), "taps", "canon."))
         return StackConfig(tuple(layers), loop, _real(top, "logit_scale", "") if top.get("logit_scale") is not None else 1.0)
 
 
@@ -561,7 +625,7 @@ class ModelConfig:
             hidden_size=int(top["width"]), intermediate_size=max(ffs, default=0), num_layers=len(stack.layers),
             num_heads=max(m.heads for m in mix), num_kv_heads=max(m.kv_heads for m in mix),
             head_dim=max(max(m.dim, m.vdim) for m in mix), vocab_size=int(top["vocab"]), rms_norm_eps=float(norm["eps"]),
-            tie_word_embeddings=True, architecture=arch, max_position_embeddings=int(mpe) if isinstance(mpe, int) else 0,
+            tie_word_embeddings=stack.tied, architecture=arch, max_position_embeddings=int(mpe) if isinstance(mpe, int) else 0,
             stack=stack, raw=dict(top))
 
     @staticmethod

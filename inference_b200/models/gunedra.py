@@ -23,7 +23,7 @@ import torch
 
 from .. import ops
 from ..contracts.errors import Unsupported
-from ..engine.kv_pool import LatentGeometry, StateGeometry
+from ..engine.kv_pool import LatentGeometry
 from ..ops import Branch, DeltaWeights, DepthAverage, LatentWeights, NormWeights
 from ..parallel.comm import Communicator
 from .config import ChannelDeltaSpec, LatentAttentionSpec, LayerSpec, ModelConfig
@@ -72,8 +72,7 @@ class GunedraGpu(LatentDecoder):
             if isinstance(m, LatentAttentionSpec):
                 out.append(LatentGeometry(ops.latent_width(self._latent_widths(m)[2], m.rot_dim)))
             else:
-                dp, vp = ops.delta_key_width(m.dim), up8(m.vdim)
-                out.append(StateGeometry((m.heads, vp, dp), (m.conv - 1, 2 * m.kv_heads * dp + m.heads * vp)))
+                out.append(self._delta_geometry(m))
         return out
 
     def decode_splits(self, batch: int, max_kv: int) -> tuple[int, ...]:
@@ -139,16 +138,14 @@ class GunedraGpu(LatentDecoder):
     def _delta_layer(self, spec: LayerSpec, p: str, get, norm1: NormWeights, dwa: torch.Tensor) -> _Layer:
         m, W = spec.mixer, self.width
         H, G, D, E, dp, vp = m.heads, m.kv_heads, m.dim, m.vdim, ops.delta_key_width(m.dim), up8(m.vdim)
-        hb, parts = up8(H), {"q": (G, D, dp), "k": (G, D, dp), "v": (H, E, vp)}
+        hb = up8(H)
         low = {"a1": get(p + "a1", None, W), "g1": get(p + "g1", None, W)}
         ra, rg = low["a1"].shape[0], low["g1"].shape[0]
-        rows = [self._heads(get(p + n, h * d, W), h, [(d, padded)]) for n, (h, d, padded) in parts.items()]
+        rows, conv = self._delta_inputs(m, p, get)
         rows += [self._heads(get(p + "b", H, W), 1, [(H, hb)]), self._heads(low["a1"], 1, [(ra, up8(ra))]),
                  self._heads(low["g1"], 1, [(rg, up8(rg))])]
-        conv = torch.cat([torch.nn.functional.pad(self._fp32(get(f"{p}{n}.conv", h * d, m.conv)).view(h, d, m.conv),
-                                                  (0, 0, 0, padded - d)).reshape(-1, m.conv) for n, (h, d, padded) in parts.items()])
         col_b = 2 * G * dp + H * vp
-        delta = DeltaWeights(H, G, D, dp, E, vp, col_b, conv.t().contiguous(), self._fp32(get(p + "A_log", H)),
+        delta = DeltaWeights(H, G, D, dp, E, vp, col_b, conv, self._fp32(get(p + "A_log", H)),
                              self._fp32(get(p + "dt_bias", H * D).reshape(H, D), dp).reshape(-1), self._fp32(get(p + "norm", E), vp))
         a2 = self._heads(get(p + "a2", H * D, ra), H, [(D, dp)], up8(ra))
         g2 = self._heads(get(p + "g2", H * E, rg), H, [(E, vp)], up8(rg))

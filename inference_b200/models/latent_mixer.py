@@ -11,17 +11,11 @@ from ..contracts.errors import Unsupported
 from ..ops import LatentWeights, QueryRotation
 from .config import LatentAttentionSpec
 from .llama import StepInputs
-from .stack import StackDecoder, up8
+from .stack import StackDecoder, half_pairs, up8
 
 
 def _up(n: int, m: int) -> int:
     return (n + m - 1) // m * m
-
-
-def half_pairs(dim: int, rot: int) -> list[int]:
-    """Order of a head's dimensions that makes the partners (i, i + rot / 2) of a rotation neighbours; the kernels rotate neighbours, and
-    a head's scores do not depend on the order of its dimensions."""
-    return [j for i in range(rot // 2) for j in (i, i + rot // 2)] + list(range(rot, dim))
 
 
 @dataclass

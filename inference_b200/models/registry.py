@@ -32,6 +32,10 @@ def gpu_model(cfg: ModelConfig, comm=None, device: torch.device | None = None, d
         from .rotalorn import RotalornGpu
 
         return RotalornGpu(cfg, comm=comm, device=device, dtype=dtype)
+    if cfg.architecture is Architecture.NAFELIX:
+        from .nafelix import NafelixGpu
+
+        return NafelixGpu(cfg, comm=comm, device=device, dtype=dtype)
     if dtype != torch.bfloat16:
         raise Unsupported(f"{cfg.architecture.value}: the sm_100a decoder computes in bfloat16")
     from .llama import LlamaGpu

@@ -29,9 +29,9 @@ from ..engine.kv_pool import KvGeometry, LatentGeometry, TokenGeometry
 from ..ops import Branch, Differential, LatentWeights, NormWeights, RoutedRows
 from ..parallel.comm import Communicator
 from .config import AttentionSpec, DenseSpec, DifferentialSpec, ExpertsSpec, LatentAttentionSpec, ModelConfig
-from .latent_mixer import LatentDecoder, Ragged, half_pairs
+from .latent_mixer import LatentDecoder, Ragged
 from .llama import StepInputs, splits_for
-from .stack import up8
+from .stack import half_pairs, up8
 
 
 @dataclass
@@ -175,13 +175,6 @@ class RotalornGpu(LatentDecoder):
         lq1, lk1, lq2, lk2 = (get(p + n, D).double() for n in ("lq1", "lk1", "lq2", "lk2"))
         share = math.exp(float((lq1 * lk1).sum())) - math.exp(float((lq2 * lk2).sum())) + m.diff
         return _Layer(norm, w_in, self._out(get(p + "o", W, H * E), H, E, vp), dp, vp, share=share)
-
-    def _pairs(self, gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
-        """Rows (gate_0, up_0, gate_1, ...), padded."""
-        ff = gate.shape[0]
-        out = torch.zeros((up8(ff), 2, self.hp), dtype=self.dtype, device=self.device)
-        out[:ff, 0, :self.width], out[:ff, 1, :self.width] = gate.to(self.device, self.dtype), up.to(self.device, self.dtype)
-        return out.view(-1, self.hp)
 
     def _feed_forward(self, f: DenseSpec | ExpertsSpec, p: str, get) -> tuple[_FeedForward, torch.Tensor]:
         """(weights, the down projection that shares a GEMM with the mixer's output projection)."""

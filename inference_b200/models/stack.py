@@ -5,13 +5,19 @@ import torch
 
 from .. import ops
 from ..contracts.errors import LoadError, Unsupported
-from ..engine.kv_pool import LayeredKvPool
+from ..engine.kv_pool import LayeredKvPool, StateGeometry
 from ..parallel.comm import Communicator, single
-from .config import ModelConfig, rescale_frequencies
+from .config import ChannelDeltaSpec, ModelConfig, rescale_frequencies
 
 
 def up8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+def half_pairs(dim: int, rot: int) -> list[int]:
+    """Order of a head's dimensions that makes the partners (i, i + rot / 2) of a rotation neighbours; the kernels rotate neighbours, and
+    a head's scores do not depend on the order of its dimensions."""
+    return [j for i in range(rot // 2) for j in (i, i + rot // 2)] + list(range(rot, dim))
 
 
 class StackDecoder:
@@ -34,6 +40,7 @@ class StackDecoder:
         self.width, self.hp = cfg.hidden_size, up8(cfg.hidden_size)
         self.layers: list = []
         self.embed = self.final = None
+        self.head = None           # rows that give the logits, where they are not the embedding table
         self._rope: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
         self.max_positions = 0
         self.launches = 0
@@ -101,18 +108,39 @@ class StackDecoder:
         out[:self.width, :, :d] = o.to(self.device, self.dtype).reshape(self.width, heads, d)
         return out.reshape(self.hp, heads * dp)
 
+    def _pairs(self, gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+        """Rows (gate_0, up_0, gate_1, ...), padded."""
+        ff = gate.shape[0]
+        out = torch.zeros((up8(ff), 2, self.hp), dtype=self.dtype, device=self.device)
+        out[:ff, 0, :self.width], out[:ff, 1, :self.width] = gate.to(self.device, self.dtype), up.to(self.device, self.dtype)
+        return out.view(-1, self.hp)
+
+    def _delta_inputs(self, m: ChannelDeltaSpec, p: str, get) -> tuple[list[torch.Tensor], torch.Tensor]:
+        """Delta rule: (the projections q, k, v with every head padded, fp32 convolution weights [taps, their rows])."""
+        dp, vp = ops.delta_key_width(m.dim), up8(m.vdim)
+        parts = {"q": (m.kv_heads, m.dim, dp), "k": (m.kv_heads, m.dim, dp), "v": (m.heads, m.vdim, vp)}
+        rows = [self._heads(get(p + n, h * d, self.width), h, [(d, padded)]) for n, (h, d, padded) in parts.items()]
+        conv = torch.cat([torch.nn.functional.pad(self._fp32(get(f"{p}{n}.conv", h * d, m.conv)).view(h, d, m.conv),
+                                                  (0, 0, 0, padded - d)).reshape(-1, m.conv) for n, (h, d, padded) in parts.items()])
+        return rows, conv.t().contiguous()
+
+    @staticmethod
+    def _delta_geometry(m: ChannelDeltaSpec) -> StateGeometry:
+        dp, vp = ops.delta_key_width(m.dim), up8(m.vdim)
+        return StateGeometry((m.heads, vp, dp), (m.conv - 1, 2 * m.kv_heads * dp + m.heads * vp))
+
     # ---- forward ----------------------------------------------------------------------------------------------------
-    def _linear(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
-                out: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
+    def _linear(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None, out: torch.Tensor | None = None,
+                bias: torch.Tensor | None = None, act: str | None = None, act_params: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
         self.launches += 1
         if self.dtype == torch.float32:
-            return ops.gemm_f32(a, w, out=out, bias=bias)
-        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16, bias=bias)
+            return ops.gemm_f32(a, w, out=out, bias=bias, act=act, act_params=act_params)
+        return ops.gemm_bf16(a, w, out=out, out_dtype=out_dtype or torch.bfloat16, bias=bias, act=act, act_params=act_params)
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         if hidden.shape[0] == 0:
             return torch.empty((0, self.cfg.vocab_size), dtype=torch.float32, device=self.device)
-        return self._linear(hidden, self.embed, torch.float32)
+        return self._linear(hidden, self.embed if self.head is None else self.head, torch.float32)
 
     def greedy_tokens(self, hidden: torch.Tensor) -> torch.Tensor:
         self.launches += 1

@@ -149,7 +149,8 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                     kv_lens: torch.Tensor, *, cu_q: torch.Tensor | None, max_q_len: int, scale: float, chunk: int = 0,
                     sink: torch.Tensor | None = None, decode: bool = False, num_splits: int = 1, window: int = 0,
                     fresh_kv: tuple[torch.Tensor, torch.Tensor] | None = None, diff: Differential | None = None,
-                    out: torch.Tensor | None = None, kernel: str = "auto") -> torch.Tensor:
+                    out: torch.Tensor | None = None, kernel: str = "auto", all_values: bool = False,
+                    gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal paged attention with head widths of its own for q / k (D) and v (Dv), optional chunked or windowed masking and sinks.
 
     q [T, Hq, D] (heads contiguous), caches [blocks, Hkv, block_size, D] and [blocks, Hkv, block_size, Dv], block_table /
@@ -157,7 +158,9 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     run of `chunk` positions, counted from the start of the sequence. window > 0: position i sees only 0 <= i - j < window. sink
     fp32 [Hq]: exp(sink) joins each head's softmax denominator. diff: q [T, Hq, 2, D / 2], the two maps' keys side by side in each
     key row, the result combined. fresh_kv = (k [T, Hkv, D], v [T, Hkv, Dv]) strided views: every sequence starts in this step, so a
-    prefill reads its keys there instead of the pages.
+    prefill reads its keys there instead of the pages. all_values: the value cache has heads of its own number NV (and fresh values [T, NV,
+    Dv]), every query head's weights are applied to all of them -> [T, Hq * NV * Dv]. gate: logits in the shape of the result (strided
+    rows), which is scaled by their sigmoid.
     bf16 widths that are multiples of 8 up to 128 run on the tcgen05 kernel (prefill) or the TMA-fed decode kernel; other
     widths, fp32 and non-positive scales on the plain fp32-arithmetic kernel (kernel="simple" forces it)."""
     require_cuda(q, kcache, vcache, block_table, kv_lens, sink, out)
@@ -165,7 +168,10 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     T, Hq = q.shape[:2]
     nblk, Hkv, bs, D = kcache.shape
     Dv = vcache.shape[3]
-    assert vcache.shape[:3] == kcache.shape[:3] and kcache.is_contiguous() and vcache.is_contiguous()
+    NV = vcache.shape[1] if all_values else 0
+    assert vcache.shape[0] == nblk and vcache.shape[2] == bs and (all_values or vcache.shape[1] == Hkv)
+    assert kcache.is_contiguous() and vcache.is_contiguous() and not (diff is not None and (all_values or gate is not None))
+    problems = Hkv * max(NV, 1)          # of a sequence in decoding
     assert q.shape[2:] == ((D,) if diff is None else (2, D // 2)) and q.stride(-1) == 1 and q.stride(1) == D
     assert q.dtype == kcache.dtype == vcache.dtype and (diff is None or (D % 2 == 0 and q.stride(2) == D // 2))
     assert block_table.dtype == torch.int32 and kv_lens.dtype == torch.int32 and block_table.stride(1) == 1
@@ -174,13 +180,15 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     assert temp is None or (temp.is_cuda and temp.dtype == torch.float32 and temp.is_contiguous())
     num_seqs = kv_lens.numel()
     if out is None:
-        out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
-    assert out.shape == (T, Hq * Dv) and out.stride(1) == 1 and out.dtype == q.dtype
+        out = torch.empty((T, Hq * max(NV, 1) * Dv), dtype=q.dtype, device=q.device)
+    assert out.shape == (T, Hq * max(NV, 1) * Dv) and out.stride(1) == 1 and out.dtype == q.dtype
+    assert gate is None or (gate.shape == out.shape and gate.stride(1) == 1 and gate.dtype == q.dtype)
+    gate_args = (NV, ptr(gate), gate.stride(0) if gate is not None else 0)
     if q.dtype == torch.bfloat16 and kernel == "auto" and scale > 0 and max(D, Dv) <= 128 and D % (8 * maps) == 0 and Dv % 8 == 0:
         decode = decode and max_q_len * maps * (Hq // Hkv) <= 16 and bs == 16
         ws_ptr, ws_bytes, k, v, ks, vs, table = None, 0, kcache, vcache, 0, 0, block_table
         if decode and num_splits > 1:
-            ws = decode_workspace(q.device, kernels().swb_attn_decode_workspace_bytes(num_seqs, Hkv, num_splits))
+            ws = decode_workspace(q.device, kernels().swb_attn_decode_workspace_bytes(num_seqs, problems, num_splits))
             ws_ptr, ws_bytes = ws.data_ptr(), ws.numel()
         if not decode:
             if cu_q is None:
@@ -194,7 +202,7 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
                                     out.stride(0), ptr(table), block_table.stride(0), bs, nblk, ptr(cu_q),
                                     kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq, Hkv, D, Dv, scale, chunk, ptr(sink),
                                     1 if decode else 0, num_splits, ws_ptr, ws_bytes, window, 0 if diff is None else 1, d.share, d.eps, d.post,
-                                    d.softcap, ptr(temp), d.width, stream_ptr())
+                                    d.softcap, ptr(temp), d.width, *gate_args, stream_ptr())
         if rc != -3:
             check(rc, "swb_attn_ext")
             return out
@@ -202,7 +210,7 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
     rc = kernels().swb_attn_simple(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), res.data_ptr(),
                                    res.stride(0), block_table.data_ptr(), block_table.stride(0), bs, ptr(cu_q),
                                    kv_lens.data_ptr(), num_seqs, max_q_len, T, Hq * maps, Hkv, D // maps, Dv, 0, scale, chunk, ptr(sink),
-                                   window, diff.softcap if diff is not None else 0.0, ptr(temp), maps,
+                                   window, diff.softcap if diff is not None else 0.0, ptr(temp), maps, *gate_args,
                                    1 if q.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_attn_simple")
     if diff is not None:

@@ -6,8 +6,8 @@ import torch
 from .._native import kernels
 from .runtime import check, ptr, require_cuda, stream_ptr
 
-ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "swiglu_pairs": 3, "geglu_pairs": 4, "relu2": 5}
-_PAIRS = (3, 4)     # gated pairs halve the width
+ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "swiglu_pairs": 3, "geglu_pairs": 4, "relu2": 5, "xielu": 6, "clamped_pairs": 7}
+_PAIRS = (3, 4, 7)     # gated pairs halve the width
 _WORKSPACES: dict[tuple[int, int], torch.Tensor] = {}
 WORKSPACE_BYTES = 64 * 1024 + (96 << 20)
 
@@ -26,8 +26,9 @@ def gemm_workspace(device: torch.device, slot: int = 0) -> torch.Tensor:
 def gemm_bf16(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = None,
               residual: torch.Tensor | None = None, act: str | None = None, out: torch.Tensor | None = None,
               out_dtype: torch.dtype = torch.bfloat16, mode: int = -1, block_n: int = 0, ctas: int = 0,
-              workspace: torch.Tensor | None = None) -> torch.Tensor:
-    """out[T, N] = act(a[T, K] @ w[N, K]^T + bias) + residual. a and w are bf16 with contiguous rows."""
+              workspace: torch.Tensor | None = None, act_params: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
+    """out[T, N] = act(a[T, K] @ w[N, K]^T + bias) + residual. a and w are bf16 with contiguous rows. act_params: "xielu" (a, b): a z^2 +
+    z / 2 above zero, b (e^z - 1 - z) + z / 2 below; "clamped_pairs" (limit, -)."""
     require_cuda(a, w)
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert a.dim() == 2 and w.dim() == 2 and a.shape[1] == w.shape[1]
@@ -44,10 +45,10 @@ def gemm_bf16(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = N
         assert bias.dtype == torch.bfloat16 and bias.numel() == N and bias.is_contiguous()
     if workspace is None:
         workspace = gemm_workspace(a.device)
-    rc = kernels().swb_gemm_bf16(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0),
-                                 T, N, K, ptr(bias), ptr(residual), residual.stride(0) if residual is not None else 0,
-                                 ACT[act], 1 if out.dtype == torch.float32 else 0, workspace.data_ptr(),
-                                 workspace.numel(), mode, block_n, ctas, stream_ptr())
+    rc = kernels().swb_gemm_bf16_act(a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0),
+                                     T, N, K, ptr(bias), ptr(residual), residual.stride(0) if residual is not None else 0,
+                                     ACT[act], *act_params, 1 if out.dtype == torch.float32 else 0, workspace.data_ptr(),
+                                     workspace.numel(), mode, block_n, ctas, stream_ptr())
     check(rc, "swb_gemm_bf16")
     return out
 
@@ -148,7 +149,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *
 
 
 def gemm_f32(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = None, act: str | None = None, out: torch.Tensor | None = None,
-             offsets: torch.Tensor | None = None, src: torch.Tensor | None = None, rows: int | None = None) -> torch.Tensor:
+             offsets: torch.Tensor | None = None, src: torch.Tensor | None = None, rows: int | None = None,
+             act_params: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """True 32-bit product (no TF32): out[T, N] = act(a[T, K] @ w[N, K]^T + bias). Grouped: w [G, N, K], offsets int32 [G + 1] on
     the device, rows [offsets[g], offsets[g + 1]) use w[g] and read a[src[r]] (r itself without src); `rows` bounds them."""
     require_cuda(a, w)
@@ -162,6 +164,6 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None = No
         out = torch.empty((T, N), dtype=torch.float32, device=a.device)
     assert out.shape == (T, N) and out.dtype == torch.float32 and out.stride(1) == 1
     rc = kernels().swb_gemm_f32(a.data_ptr(), a.stride(0), ptr(src), ptr(offsets), G, w.data_ptr(), K, out.data_ptr(),
-                                out.stride(0), T, N, K, ACT[act], ptr(bias), stream_ptr())
+                                out.stride(0), T, N, K, ACT[act], *act_params, ptr(bias), stream_ptr())
     check(rc, "swb_gemm_f32")
     return out

@@ -185,6 +185,7 @@ def latent_attention_simple(q_abs: torch.Tensor, cache: torch.Tensor, block_tabl
     rc = kernels().swb_attn_simple(q_abs.data_ptr(), q_abs.stride(0), cache.data_ptr(), cache.data_ptr(), out.data_ptr(),
                                    out.stride(0), block_table.data_ptr(), block_table.stride(0), cache.shape[1], ptr(cu_q),
                                    kv_lens.data_ptr(), kv_lens.numel(), max_q_len, T, H, 1, D, w.rk, D, w.scale, 0, ptr(w.sink), w.window, 0.0, None, 1,
+                                   0, None, 0,
                                    1 if q_abs.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_attn_simple")
     return out

@@ -90,9 +90,10 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: torc
 
 
 def gated_act_mul(gate_up: torch.Tensor, act: str = "silu", out: torch.Tensor | None = None,
-                  paired: bool = False, row_gate: torch.Tensor | None = None) -> torch.Tensor:
+                  paired: bool = False, row_gate: torch.Tensor | None = None, limit: float = 0.0) -> torch.Tensor:
     """out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f] (SwiGLU / GeGLU, candle-llm models/llama.rs:1386-1391).
     paired: the projection's rows are interleaved (gate_0, up_0, gate_1, ...), out[t, f] = act(gu[t, 2f]) * gu[t, 2f+1].
+    act "clamped": g <- min(g, limit), u <- clamp(u, -limit, limit), out = g sigmoid(1.702 g) (u + 1).
     row_gate fp32 [T] logits (strided): row t is scaled by their sigmoid. bf16 or fp32."""
     require_cuda(gate_up, row_gate)
     g2 = gate_up.reshape(-1, gate_up.shape[-1])
@@ -103,7 +104,7 @@ def gated_act_mul(gate_up: torch.Tensor, act: str = "silu", out: torch.Tensor | 
     assert g2.stride(1) == 1 and out.stride(1) == 1 and out.shape == (T, F) and out.dtype == g2.dtype
     assert row_gate is None or (row_gate.dtype == torch.float32 and row_gate.shape == (T,))
     rc = kernels().swb_gated_act_mul_ex(g2.data_ptr(), g2.stride(0), out.data_ptr(), out.stride(0), T, F,
-                                        (2 if act in ("gelu", "gelu_tanh") else 1) + (2 if paired else 0), ptr(row_gate),
+                                        (5 + paired if act == "clamped" else (2 if act in ("gelu", "gelu_tanh") else 1) + 2 * paired), limit, ptr(row_gate),
                                         row_gate.stride(0) if row_gate is not None else 0, 1 if g2.dtype == torch.float32 else 0, stream_ptr())
     check(rc, "swb_gated_act_mul")
     return out.reshape(*gate_up.shape[:-1], F) if gate_up.dim() != 2 else out
@@ -112,12 +113,14 @@ def gated_act_mul(gate_up: torch.Tensor, act: str = "silu", out: torch.Tensor | 
 def row_rope_kv_write(buf: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, n_heads: int,
                       n_kv_heads: int, head_dim: int, *, v_col: int = 0, rope: tuple[torch.Tensor, torch.Tensor] | None = None,
                       q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, norm_counts: tuple[int, int] = (0, 0),
-                      eps: float = 0.0, v_from_k: bool = False, store_v: bool = False) -> None:
+                      eps: float = 0.0, v_from_k: bool = False, store_v: bool = False, unit: int = 0) -> None:
     """In place on buf [T, >= (Hq + Hkv) * D]: RMS norms over the whole q and the whole k of a token (fp32 weights q_norm [Hq * D] and
     k_norm [Hkv * D]; norm_counts: how many numbers enter each mean, the rest being zero padding), then rotation of the leading dimensions
     of every head in neighbouring pairs (rope = cos and sin tables fp32 [positions, rot / 2]). k and v go to the paged caches [blocks, Hkv,
     block_size, D | Dv] at `slots` (int64, -1 = skip). Values are the columns from v_col on, or with v_from_k the keys as projected, which
-    store_v also copies there. Without norm and rotation the queries are left alone. bf16 or fp32 throughout."""
+    store_v also copies there. vcache may have heads of its own (their columns then follow one another from v_col on). unit > 0: every q
+    and k head is divided by its own root mean square over `unit` columns (the rest being zero padding), without a weight. Without norm
+    and rotation the queries are left alone. bf16 or fp32 throughout."""
     require_cuda(buf, positions, slots, kcache, vcache, q_norm, k_norm)
     T, Dv = buf.shape[0], vcache.shape[-1]
     assert buf.stride(1) == 1 and kcache.dtype == vcache.dtype == buf.dtype and kcache.is_contiguous() and vcache.is_contiguous()
@@ -128,9 +131,35 @@ def row_rope_kv_write(buf: torch.Tensor, positions: torch.Tensor, slots: torch.T
     rc = kernels().swb_row_rope_kv_write(buf.data_ptr(), buf.stride(0), v_col, n_heads, n_kv_heads, head_dim, Dv,
                                          0 if cos is None else 2 * cos.shape[-1], ptr(q_norm), ptr(k_norm), norm_counts[0], norm_counts[1], eps,
                                          ptr(cos), ptr(sin), positions.data_ptr(), slots.data_ptr(), kcache.data_ptr(), vcache.data_ptr(),
-                                         kcache.shape[2], 1 if v_from_k else 0, 1 if store_v else 0, T, 1 if buf.dtype == torch.float32 else 0,
+                                         kcache.shape[2], 1 if v_from_k else 0, 1 if store_v else 0, vcache.shape[1], unit, T, 1 if buf.dtype == torch.float32 else 0,
                                          stream_ptr())
     check(rc, "swb_row_rope_kv_write")
+
+
+def head_mix_weights(talk: torch.Tensor, kv_heads: int) -> torch.Tensor:
+    """The mixing matrix [H (to), H (from)] in the layout of `head_mix`: fp32 [H (from), kv_heads, heads per group up to 8s]."""
+    H = talk.shape[0]
+    per = H // kv_heads
+    w = torch.zeros((H, kv_heads, (per + 7) // 8 * 8), dtype=torch.float32, device=talk.device)
+    w[:, :, :per] = talk.float().t().reshape(H, kv_heads, per)
+    return w
+
+
+def head_mix(a: torch.Tensor, talk: torch.Tensor, *, gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """Heads that exchange their attention weights. a [T, H, G, Dv]: the weights of each query head applied to the values of all G key/value
+    heads (`chunk_attention(all_values=True)`); talk from `head_mix_weights`; gate [T, H] logits (strided rows): head h is scaled by their
+    sigmoid. -> [T, H * Dv], out[t, h] = sigmoid(gate[t, h]) sum_g talk[h, g] a[t, g, h // (H / G)]. bf16 or fp32."""
+    require_cuda(a, talk, gate, out)
+    T, H, G, Dv = a.shape
+    assert a.stride()[1:] == (G * Dv, Dv, 1) and talk.shape[:2] == (H, G) and talk.dtype == torch.float32 and talk.is_contiguous()
+    assert gate is None or (gate.shape == (T, H) and gate.stride(1) == 1 and gate.dtype == a.dtype)
+    if out is None:
+        out = torch.empty((T, H * Dv), dtype=a.dtype, device=a.device)
+    assert out.shape == (T, H * Dv) and out.stride(1) == 1 and out.dtype == a.dtype
+    rc = kernels().swb_head_mix(a.data_ptr(), a.stride(0), talk.data_ptr(), ptr(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(),
+                                out.stride(0), T, H, G, Dv, 1 if a.dtype == torch.float32 else 0, stream_ptr())
+    check(rc, "swb_head_mix")
+    return out
 
 
 def diff_combine(maps: torch.Tensor, out: torch.Tensor, share: float, eps: float, post: float, width: int | None = None) -> torch.Tensor:

@@ -66,8 +66,10 @@ def _counters(device: torch.device) -> torch.Tensor:
     return _COUNTERS[idx]
 
 
-def logits_routing(logits: torch.Tensor, num_experts: int, top: int, *, rows: torch.Tensor | None = None) -> tuple[RoutingPlan, torch.Tensor | None]:
-    """Softmax router: the `top` experts of the largest scores per token, weighted by these scores as they are. logits fp32 [T, >=
+def logits_routing(logits: torch.Tensor, num_experts: int, top: int, *, rows: torch.Tensor | None = None,
+                   renorm: bool = False) -> tuple[RoutingPlan, torch.Tensor | None]:
+    """Softmax router: the `top` experts of the largest scores per token, weighted by these scores, as they are or (renorm) divided by
+    their sum. logits fp32 [T, >=
     num_experts]. Without `rows` a dense plan; with rows [T, H] a padded plan and the rows copied to their places in the expert-sorted
     buffer."""
     require_cuda(logits, rows)
@@ -84,7 +86,7 @@ def logits_routing(logits: torch.Tensor, num_experts: int, top: int, *, rows: to
     buf = torch.empty((cap, rows.shape[1]), dtype=rows.dtype, device=dev) if padded else None
     per = 16 // rows.element_size() if padded else 1
     assert not padded or (rows.stride(1) == 1 and rows.stride(0) % per == 0 and rows.shape[1] % per == 0)
-    rc = kernels().swb_moe_route(logits.data_ptr(), logits.stride(0), T, E, top, TILE if padded else 1, scratch[0].data_ptr(),
+    rc = kernels().swb_moe_route(logits.data_ptr(), logits.stride(0), T, E, top, 1 if renorm else 0, TILE if padded else 1, scratch[0].data_ptr(),
                                  scratch[1].data_ptr(), weights.data_ptr(), _counters(dev).data_ptr(), dest.data_ptr(), ptr(src),
                                  offsets.data_ptr(), ptr(active), ptr(tiles), cap, ptr(rows), rows.stride(0) // per if padded else 0, ptr(buf),
                                  rows.shape[1] // per if padded else 0, rows.shape[1] // per if padded else 0, stream_ptr())
@@ -92,16 +94,17 @@ def logits_routing(logits: torch.Tensor, num_experts: int, top: int, *, rows: to
     return RoutingPlan(dest, cap, src, offsets, active, tiles, weights), buf
 
 
-def gemm_grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: RoutingPlan, *, gather: bool, act: str | None = None) -> torch.Tensor:
+def gemm_grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: RoutingPlan, *, gather: bool, act: str | None = None,
+                      limit: float = 0.0) -> torch.Tensor:
     """out[r] = act(x[src[r] if gather else r] @ w[e]^T) for the rows r of each expert's dense segment; few rows per expert."""
     require_cuda(x, w)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and x.stride(1) == 1
     E, N, K = w.shape
     assert x.shape[1] == K and not plan.padded
-    out = torch.empty((plan.rows, N // 2 if act in ("swiglu_pairs", "geglu_pairs") else N), dtype=torch.bfloat16, device=x.device)
+    out = torch.empty((plan.rows, N // 2 if act in ("swiglu_pairs", "geglu_pairs", "clamped_pairs") else N), dtype=torch.bfloat16, device=x.device)
     rc = kernels().swb_gemm_grouped_rows(x.data_ptr(), x.stride(0), plan.src.data_ptr() if gather else None,
                                          plan.offsets.data_ptr(), plan.active.data_ptr(), plan.active.numel(), w.data_ptr(),
-                                         out.data_ptr(), out.stride(0), N, K, ACT[act], 1 if plan.ahead else 0, stream_ptr())
+                                         out.data_ptr(), out.stride(0), N, K, ACT[act], limit, 1 if plan.ahead else 0, stream_ptr())
     check(rc, "swb_gemm_grouped_rows")
     return out
 
@@ -117,15 +120,16 @@ def routed_ffn(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, plan: Rout
     return gemm_grouped_rows(gemm_grouped_rows(h, up, plan, gather=True, act=act), down, plan, gather=False)
 
 
-def routed_gated_ffn(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, plan: RoutingPlan, act: str) -> torch.Tensor:
-    """Expert outputs [plan.rows, H] in the plan's row order: down_e(act(gate_e x) * (up_e x)). gate_up [E, 2 F, H] with its rows in
+def routed_gated_ffn(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, plan: RoutingPlan, act: str, limit: float = 0.0) -> torch.Tensor:
+    """Expert outputs [plan.rows, H] in the plan's row order: down_e(act(gate_e x) * (up_e x)), or with act "clamped" the clamped unit of
+    `gated_act_mul`. gate_up [E, 2 F, H] with its rows in
     (gate, up) pairs, down [E, H, F]; h as in routed_ffn."""
     from .llm import gated_act_mul
 
     if h.dtype == torch.float32:
-        u = gated_act_mul(gemm_f32(h, gate_up, offsets=plan.offsets, src=plan.src, rows=plan.rows), act, paired=True)
+        u = gated_act_mul(gemm_f32(h, gate_up, offsets=plan.offsets, src=plan.src, rows=plan.rows), act, paired=True, limit=limit)
         return gemm_f32(u, down, offsets=plan.offsets, rows=plan.rows)
     if plan.padded:
-        return gemm_bf16_grouped(gated_act_mul(gemm_bf16_grouped(h, gate_up, plan.tile_group), act, paired=True), down, plan.tile_group)
-    pairs = "geglu_pairs" if act in ("gelu", "gelu_tanh") else "swiglu_pairs"
-    return gemm_grouped_rows(gemm_grouped_rows(h, gate_up, plan, gather=True, act=pairs), down, plan, gather=False)
+        return gemm_bf16_grouped(gated_act_mul(gemm_bf16_grouped(h, gate_up, plan.tile_group), act, paired=True, limit=limit), down, plan.tile_group)
+    pairs = "clamped_pairs" if act == "clamped" else "geglu_pairs" if act in ("gelu", "gelu_tanh") else "swiglu_pairs"
+    return gemm_grouped_rows(gemm_grouped_rows(h, gate_up, plan, gather=True, act=pairs, limit=limit), down, plan, gather=False)
