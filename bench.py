@@ -189,7 +189,7 @@ def main() -> int:
     ap.add_argument("--no-extra", action="store_true", help="skip the TTFT / batch-1 / batch-8 side measurements")
     ap.add_argument("--no-dit", action="store_true", help="skip the DiT 1024x1024 seconds-per-image section")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library-collective (NCCL, unfused) arm")
-    ap.add_argument("--design", default=None, choices=["zobunex", "gunedra", "rotalorn"],
+    ap.add_argument("--design", default=None, choices=["zobunex", "gunedra", "rotalorn", "nafelix"],
                     help="instead of the headline workload: prefill / decode throughput and kernel rooflines of this design "
                          "beside the closest Llama-family decoder at equal size (see benchmarks/bench_<design>.py)")
     args = ap.parse_args()
@@ -206,6 +206,10 @@ def main() -> int:
         from benchmarks.bench_rotalorn import main as bench_rotalorn
 
         return bench_rotalorn()
+    if args.design == "nafelix":
+        from benchmarks.bench_nafelix import main as bench_nafelix
+
+        return bench_nafelix()
     if args.impl == "reference":
         print(json.dumps(probe_reference()))
         return 0

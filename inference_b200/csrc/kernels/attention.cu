@@ -475,9 +475,10 @@ int attn_decode_tma_launch(const AttnParams& p, int num_blocks, cudaStream_t str
 extern "C" {
 
 // Bytes of fp32 scratch the decode path needs for `num_splits` KV splits.
-// Split-KV scratch: [ticket counters: num_seqs * Hkv ints, rounded up to 256 bytes][partial O][partial max / sum].
-// The counters must be zero before the first launch (the kernel leaves them zero).
-static size_t attn_counter_bytes(int num_seqs, int Hkv) { return (((size_t)num_seqs * Hkv * sizeof(int)) + 255) / 256 * 256; }
+// Split-KV scratch: [ticket counters: num_seqs * Hkv ints, rounded up to 64 KB][partial O][partial max / sum].
+// The counters must be zero before the first launch (the kernel leaves them zero); their area has one size for all but huge batches, so that
+// launches of different shapes may share the scratch.
+static size_t attn_counter_bytes(int num_seqs, int Hkv) { return (((size_t)num_seqs * Hkv * sizeof(int)) + 65535) / 65536 * 65536; }
 size_t swb_attn_decode_workspace_bytes(int num_seqs, int Hkv, int num_splits) {
   return attn_counter_bytes(num_seqs, Hkv) + (size_t)num_seqs * Hkv * num_splits * 16 * (swb::HD + 2) * sizeof(float);
 }

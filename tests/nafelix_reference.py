@@ -171,6 +171,12 @@ def route(h, router, top):
     return e[:, :top], s / (s.sum(-1, keepdim=True) + 1e-20)
 
 
+def margin(h, router, top):
+    """Distance between the last chosen expert's logit and the first one left out [T] (inf when none is)."""
+    z = torch.sort(h @ router.T, dim=-1, descending=True).values
+    return z[:, top - 1] - z[:, top] if top < z.shape[1] else torch.full((h.shape[0],), math.inf, dtype=F)
+
+
 def experts(h, W, p, f):
     e, s = route(h, W[p + "router"], f["router"]["top"])
     y = torch.zeros_like(h)
@@ -195,8 +201,8 @@ def runs(cfg):
     return [*range(lp["start"]), *(list(range(lp["start"], lp["stop"])) * lp["times"]), *range(lp["stop"], n)]
 
 
-def forward(cfg, weights, tokens, taps=None):
-    """Logits [T, vocab] of a whole sequence; `taps` collects the sum of the streams after every layer run."""
+def forward(cfg, weights, tokens, taps=None, margins=None):
+    """Logits [T, vocab] of a whole sequence; `taps` collects the sum of the streams after every layer run, `margins` those of the routers."""
     W = {k: v.to(F) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     x = W["embed"][torch.tensor(tokens)]
@@ -210,13 +216,17 @@ def forward(cfg, weights, tokens, taps=None):
         mixer = {"parallel": parallel, "attention": gated_attention}[lay["type"]]
         xs = sublayer(1, lambda h: mixer(h, W, L + "mix.", lay["mixer"], eps))
         if lay["mlp"] is not None:
-            xs = sublayer(2, lambda h: feed_forward(h, W, L + "mlp.", lay["mlp"]))
+            def ff(h):
+                if margins is not None and lay["mlp"]["kind"] == "moe":
+                    margins.append(margin(h, W[L + "mlp.router"], lay["mlp"]["router"]["top"]))
+                return feed_forward(h, W, L + "mlp.", lay["mlp"])
+            xs = sublayer(2, ff)
         if taps is not None:
             taps.append(xs.sum(0))
     return (rms(xs.sum(0), eps) * W["final.norm"]) @ W["head"].T
 
 
-def generate(cfg, weights, prompt, n):
+def greedy(cfg, weights, prompt, n):
     toks = list(prompt)
     for _ in range(n):
         toks.append(int(forward(cfg, weights, toks)[-1].argmax()))
@@ -263,7 +273,7 @@ def config(layers, width, vocab, streams, taps, loop=None, eps=1e-5):
 
 def model_a():
     """Every layer different; groups of two and three heads, a layer without a feed-forward inside the loop."""
-    return config([(par(talk(6, 3, 40, 24, 24, 24, 700.0), delta(6, 2, 24, 40, 3)), moe(7, 3, 24, 0.8)),
+    return config([(par(talk(6, 3, 40, 24, 24, 24, 700.0), delta(6, 2, 24, 40, 3)), moe(4, 4, 24, 0.8)),
                    (attn(6, 2, 24, 56, 33, 8, 500.0), None),
                    (par(talk(4, 1, 24, 40, 17, 24, 90.0, scale=0.3), delta(3, 3, 40, 24, 4)), dense(120)),
                    (attn(4, 4, 48, 32, 70, 48, 2000.0), moe(5, 2, 56, 1.5))], 144, 311, 4, 4, loop=(1, 3, 3), eps=1e-3)
