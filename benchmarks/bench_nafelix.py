@@ -10,6 +10,7 @@ Two parts, one JSON line per row:
           prompts against 128 fp32 lanes per SM at the maximum clock).
 CUDA events on the launching stream after warm-up; kernels with L2 flushed before every timed launch (a 512 MB write), models with weights and
 caches larger than L2. Run as `python bench.py --design nafelix` or directly (an argument selects rows by name)."""
+import dataclasses
 import json
 import statistics
 import sys
@@ -160,6 +161,8 @@ def kernel_rows(size, emit, only=""):
         m = min(n, window)
         return m * (m + 1) / 2 + (n - m) * m
     NV = G // 2                                           # value heads of 64, two to a tile
+    base = nafelix_config(size, "P")
+    model = NafelixGpu(ModelConfig.from_json({**base, "layers": [{**base["layers"][0], "mlp": None}]}), device=torch.device("cuda", 0)).init_random(seed=0)
     for n, B, win in ((1024, 8, 0), (8192, 1, 0), (8192, 1, 512)):
         cu = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
         pr = B * pairs_of(n, win or n)
@@ -193,15 +196,12 @@ def kernel_rows(size, emit, only=""):
         row(f"decode attention, sinks and element gates, {what} (like: the same without)",
             lambda: ops.chunk_attention(qq, lk, lv, tab, lens, num_splits=splits_for(B, G, reach), sink=sink, gate=g, **kw),
             B * keys * G * 512, "bytes", *like)
-        row(f"decode attention over all {G} value heads of 64, sinks, {what} (like: own values only, width 128)",
-            lambda: ops.chunk_attention(qq, lk, l2, tab, lens, num_splits=splits_for(B, G * NV, reach), sink=sink, all_values=True, **kw),
-            B * keys * G * 384, "bytes", *like)
+        gh, ns = rnd(B, H), model.decode_splits(B, reach)[0]
+        row(f"decode attention with exchanged weights, sinks and head gates, {what} (like: window attention, width 128)",
+            lambda: ops.exchange_attention(qq, lk, l2, tab, lens, num_splits=ns, sink=sink, talk=talk, gate=gh, **kw), B * keys * G * 384, "bytes", *like)
     # ---- delta rule ----------------------------------------------------------------------------------------------------------------
-    base = nafelix_config(size, "P")
-    model = NafelixGpu(ModelConfig.from_json({**base, "layers": [{**base["layers"][0], "mlp": None}]}), device=torch.device("cuda", 0)).init_random(seed=0)
     lay = model.layers[0]
     d = lay.delta.weights
-    import dataclasses
     dc = dataclasses.replace(d, head_decay=False, dt_bias=torch.zeros(H * d.dp, device=dev))
     for B, n in ((1, 1024), (8, 1024), (1, 1), (8, 1), (64, 1)):
         T = B * n

@@ -116,6 +116,11 @@ def _declare_kernels(lib: ctypes.CDLL) -> None:
                            c_void_p, c_void_p])
     sig("swb_short_conv", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                            c_int, c_void_p])
+    sig("swb_exchange_workspace_bytes", [c_int, c_int, c_int, c_int, c_int], c_size_t)
+    sig("swb_exchange_decode_stages", [c_int, c_int, c_int, c_int, c_int, c_int])
+    sig("swb_exchange_decode", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_ll, c_int, c_void_p, c_size_t,
+                                c_void_p])
     sig("swb_head_mix", [c_void_p, c_ll, c_void_p, c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_int, c_int, c_int, c_void_p])
     sig("swb_attn_simple", [c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float,

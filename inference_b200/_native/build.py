@@ -34,7 +34,7 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-I", str(CSRC / "include"),
 
 
 # kernel units of the paged text decoders (bf16 and 32-bit), their sampling and step metadata
-TEXT_UNITS = ("api_gemm", "argmax_static", "attention", "attention_decode_tma", "attention_tcgen05", "decode_meta", "delta_rule",
+TEXT_UNITS = ("api_gemm", "argmax_static", "attention", "attention_decode_tma", "attention_exchange", "attention_tcgen05", "decode_meta", "delta_rule",
               "f32_ops", "gemm_decode_cluster", "gemm_tcgen05", "hyper_stream", "latent_attention", "llm_ops", "moe_routed", "sample_device", "sampling", "status",
               "stream_ops")
 

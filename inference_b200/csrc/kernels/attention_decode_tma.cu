@@ -142,6 +142,15 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
     }
     *reinterpret_cast<uint4*>(sQp + q_off(row, c)) = val;
   }
+  if (EXT && !DIFF && p.gate) {          // the gates are read by the merge: have them near by then
+    for (int i = threadIdx.x; i < nrows * 2; i += blockDim.x) {
+      const int row = i >> 1, half = i & 1;
+      if (half * 64 < v_dim) {
+        const bf16* g = p.gate + (size_t)(q_start + row / p.G) * p.gate_stride + (size_t)(kvh * p.G + row % p.G) * v_dim + half * 64;
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(g));
+      }
+    }
+  }
   __syncthreads();
 
   float o[16][4];

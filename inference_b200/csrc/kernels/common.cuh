@@ -353,8 +353,9 @@ __device__ __forceinline__ float xielu_exact_f(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
 __device__ __forceinline__ float xielu_f(float z, float a, float b) {
-  const float low = z > -0.03f ? z * z * fmaf(z, 1.f / 6.f, 0.5f) : __expf(z) - 1.f - z;
-  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, low, 0.5f * z);
+  const float up = fmaxf(z, 0.f), down = fminf(z, 0.f);          // both sides are computed: no branch per element
+  const float far = __expf(down) - 1.f - down, near = down * down * fmaf(down, 1.f / 6.f, 0.5f);
+  return fmaf(a * up, up, fmaf(b, down > -0.03f ? near : far, 0.5f * z));
 }
 // Gated unit whose parts are clamped: g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1).
 template <bool EXACT>

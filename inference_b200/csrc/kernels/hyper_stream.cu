@@ -216,7 +216,7 @@ __global__ void __launch_bounds__(THREADS) hyper_step_kernel(const HyperParams p
   }
 }
 
-// out = h + conv(h) over a ragged batch of sequences: a thread owns four channels of up to `chunk` consecutive tokens. The first piece of
+// out = h + conv(h) over a ragged batch of sequences: a thread owns eight channels of up to `chunk` consecutive tokens. The first piece of
 // a sequence alone reads its window (chunk >= taps - 1), and moves it on.
 struct ShortConvParams {
   const void* h;              // [T, ldh]
@@ -234,44 +234,66 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const ShortConvParams p
   pdl_wait();
   const ConvParams& cv = p.conv;
   const int seq = blockIdx.z, start = p.cu_q ? p.cu_q[seq] : seq * p.uniform_q, n = p.cu_q ? p.cu_q[seq + 1] - start : p.uniform_q;
-  const int first = blockIdx.y * p.chunk, last = min(first + p.chunk, n), c4 = blockIdx.x * 128 + threadIdx.x, nvec = p.Hp / 4;
-  if (first >= n || c4 >= nvec) return;
+  const int first = blockIdx.y * p.chunk, last = min(first + p.chunk, n), c8 = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (first >= n || c8 >= p.Hp) return;
   const int taps = TAPS > 0 ? TAPS : cv.taps, keep = taps - 1, slot = cv.slots[seq];
-  E* win = slot >= 0 && keep > 0 ? reinterpret_cast<E*>(cv.window) + (size_t)slot * keep * p.Hp + c4 * 4 : nullptr;
+  E* win = slot >= 0 && keep > 0 ? reinterpret_cast<E*>(cv.window) + (size_t)slot * keep * p.Hp + c8 : nullptr;
   const bool carried = win && cv.positions[start] != 0;
-  const E* h = reinterpret_cast<const E*>(p.h) + (size_t)start * p.ldh + c4 * 4;
-  E* out = reinterpret_cast<E*>(p.out) + (size_t)start * p.ldo + c4 * 4;
-  const float4* wc = reinterpret_cast<const float4*>(cv.w) + c4;
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  auto input = [&](int r) {                    // input of token r of this step, r < 0: in front of it
-    if (r >= 0) return load_row4(h + (size_t)r * p.ldh);
-    return carried ? load_row4(win + (size_t)(keep + r) * p.Hp) : zero;
+  const E* h = reinterpret_cast<const E*>(p.h) + (size_t)start * p.ldh + c8;
+  E* out = reinterpret_cast<E*>(p.out) + (size_t)start * p.ldo + c8;
+  auto weights = [&](int j, float* w) { load_row8(cv.w + (size_t)j * p.Hp + c8, w); };
+  auto input = [&](int r, float* x) {          // input of token r of this step, r < 0: in front of it
+    if (r >= 0) load_row8(h + (size_t)r * p.ldh, x);
+    else if (carried) load_row8(win + (size_t)(keep + r) * p.Hp, x);
+    else
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[k] = 0.f;
   };
   if constexpr (TAPS > 0) {
-    float4 w[TAPS], past[TAPS];                // past[j]: input of token t - keep + j
+    constexpr int B = 4;                       // tokens whose loads are in flight together
+    float w[TAPS][8], x[TAPS - 1 + B][8];      // x[j]: input of token t - keep + j
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j] = __ldg(wc + (size_t)j * nvec);
+    for (int j = 0; j < TAPS; ++j) weights(j, w[j]);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) past[j] = input(first - keep + j);
-#pragma unroll 4
-    for (int t = first; t < last; ++t) {
-      past[TAPS - 1] = load_row4(h + (size_t)t * p.ldh);
-      float4 y = past[TAPS - 1];
+    for (int j = 0; j < TAPS - 1; ++j) input(first - keep + j, x[j]);
+    for (int t = first; t < last; t += B) {
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) y = fma4(w[j], past[j], y);
-      store_row4(out + (size_t)t * p.ldo, y);
+      for (int i = 0; i < B; ++i) load_row8(h + (size_t)min(t + i, last - 1) * p.ldh, x[TAPS - 1 + i]);
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) past[j] = past[j + 1];
+      for (int i = 0; i < B; ++i) {
+        if (t + i >= last) break;
+        float y[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          y[k] = x[TAPS - 1 + i][k];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) y[k] = fmaf(w[j][k], x[i + j][k], y[k]);
+        }
+        store_row8(out + (size_t)(t + i) * p.ldo, y);
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) x[j][k] = x[j + B][k];
     }
   } else {
     for (int t = first; t < last; ++t) {
-      float4 y = input(t);
-      for (int j = 0; j < taps; ++j) y = fma4(__ldg(wc + (size_t)j * nvec), input(t - keep + j), y);
-      store_row4(out + (size_t)t * p.ldo, y);
+      float y[8], x[8], w[8];
+      input(t, y);
+      for (int j = 0; j < taps; ++j) {
+        input(t - keep + j, x), weights(j, w);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) y[k] = fmaf(w[k], x[k], y[k]);
+      }
+      store_row8(out + (size_t)t * p.ldo, y);
     }
   }
   if (blockIdx.y == 0 && win)
-    for (int j = 0; j < keep; ++j) store_row4(win + (size_t)j * p.Hp, input(n - keep + j));     // ascending, as above
+    for (int j = 0; j < keep; ++j) {           // ascending, as above
+      float x[8];
+      input(n - keep + j, x);
+      store_row8(win + (size_t)j * p.Hp, x);
+    }
 }
 
 template <typename E, int THREADS, int VPT>
@@ -326,10 +348,10 @@ int swb_short_conv(const void* h, int ldh, void* out, int ldo, const float* conv
                    const int* positions, const int* cu_q, int num_seqs, int max_q, int Hp, int fp32, void* stream) {
   using namespace swb;
   if (num_seqs <= 0 || max_q <= 0) return 0;
-  if (Hp < 8 || (Hp % 8) || ((ldh | ldo) % 4) || taps < 1 || !conv_w || !slots || !positions || (taps > 1 && !window) || h == out) return -3;
+  if (Hp < 8 || (Hp % 8) || ((ldh | ldo) % 8) || taps < 1 || !conv_w || !slots || !positions || (taps > 1 && !window) || h == out) return -3;
   const int chunk = taps > 17 ? taps - 1 : 16;
   const ShortConvParams p{h, out, ldh, ldo, ConvParams{conv_w, taps, window, slots, positions}, cu_q, max_q, Hp, chunk};
-  const dim3 grid((Hp / 4 + 127) / 128, (max_q + chunk - 1) / chunk, num_seqs), block(128);
+  const dim3 grid((Hp / 8 + 127) / 128, (max_q + chunk - 1) / chunk, num_seqs), block(128);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto go = [&](auto bk, auto fk) { return fp32 ? launch_kernel(fk, grid, block, 0, s, p) : launch_kernel(bk, grid, block, 0, s, p); };
   switch (taps) {

@@ -518,13 +518,13 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(const E* __restrict__
 
 // Heads that exchange their attention weights: with a[t, g, c] the weights of query head g applied to the values of key/value head c,
 //     out[t, h] = sigmoid(gate[t, h]) sum_g talk[h, g] a[t, g, c(h)],   c(h) = h / (H / G)
-// because the weighted sum over the heads' weights passes through the (linear) application to the values. A thread owns two columns of
-// one c for TT tokens and up to HM of its query heads.
-constexpr int HM = 8;
+// because the weighted sum over the heads' weights passes through the (linear) application to the values. A thread owns four columns of
+// one c for TT tokens and HM of its query heads.
+constexpr int MIX_PAD = 8;
 struct HeadMixParams {
   const void* a;              // [T, H, G, Dv] (a token's part contiguous), a_tok apart
   long long a_tok;
-  const float* talk;          // [H (g), G (c), HP]: talk[c * H / G + i, g] at i, HP = H / G rounded up to HM, zeros behind
+  const float* talk;          // [H (g), G (c), HP]: talk[c * H / G + i, g] at i, HP = H / G rounded up to MIX_PAD, zeros behind
   const void* gate;           // optional logits [T, >= H], gate_tok apart
   long long gate_tok;
   void* out;                  // [T, H * Dv], out_tok apart
@@ -532,34 +532,35 @@ struct HeadMixParams {
   int T, H, G, Dv;
 };
 
-template <typename E, int TT>
+template <typename E, int TT, int HM>
 __global__ void __launch_bounds__(128) head_mix_kernel(const HeadMixParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int col = (blockIdx.x * 128 + threadIdx.x) * 2, width = p.G * p.Dv, t0 = blockIdx.y * TT;
+  const int col = (blockIdx.x * 128 + threadIdx.x) * 4, width = p.G * p.Dv, t0 = blockIdx.y * TT;
   if (col >= width) return;
-  const int c = col / p.Dv, per = p.H / p.G, hp = (per + HM - 1) / HM * HM, h0 = blockIdx.z * HM;
-  const E* a = reinterpret_cast<const E*>(p.a) + col;
+  const int c = col / p.Dv, per = p.H / p.G, hp = (per + MIX_PAD - 1) / MIX_PAD * MIX_PAD, h0 = blockIdx.z * HM;
+  const E* a[TT];
+#pragma unroll
+  for (int i = 0; i < TT; ++i) a[i] = reinterpret_cast<const E*>(p.a) + min(t0 + i, p.T - 1) * p.a_tok + col;
   const float* talk = p.talk + (size_t)c * hp + h0;
-  float acc[HM][TT][2] = {};
+  float4 acc[TT][HM];
+#pragma unroll
+  for (int i = 0; i < TT; ++i)
+#pragma unroll
+    for (int h = 0; h < HM; ++h) acc[i][h] = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
   for (int g = 0; g < p.H; ++g) {
-    const float4 w0 = __ldg(reinterpret_cast<const float4*>(talk + (size_t)g * p.G * hp)), w1 = __ldg(reinterpret_cast<const float4*>(talk + (size_t)g * p.G * hp) + 1);
-    const float w[HM] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+    float w[HM];
+#pragma unroll
+    for (int h = 0; h < HM; ++h) w[h] = __ldg(talk + (size_t)g * p.G * hp + h);
 #pragma unroll
     for (int i = 0; i < TT; ++i) {
-      if (t0 + i >= p.T) break;
-      const E* at = a + (t0 + i) * p.a_tok + (size_t)g * width;
-      float x, y;
-      if constexpr (sizeof(E) == 2) {
-        const uint32_t u = *reinterpret_cast<const uint32_t*>(at);
-        x = __uint_as_float(u << 16), y = __uint_as_float(u & 0xffff0000u);
-      } else {
-        const float2 u = *reinterpret_cast<const float2*>(at);
-        x = u.x, y = u.y;
-      }
+      const float4 x = load_row4(a[i] + (size_t)g * width);
 #pragma unroll
-      for (int h = 0; h < HM; ++h) acc[h][i][0] = fmaf(w[h], x, acc[h][i][0]), acc[h][i][1] = fmaf(w[h], y, acc[h][i][1]);
+      for (int h = 0; h < HM; ++h) {
+        acc[i][h].x = fmaf(w[h], x.x, acc[i][h].x), acc[i][h].y = fmaf(w[h], x.y, acc[i][h].y);
+        acc[i][h].z = fmaf(w[h], x.z, acc[i][h].z), acc[i][h].w = fmaf(w[h], x.w, acc[i][h].w);
+      }
     }
   }
 #pragma unroll
@@ -571,10 +572,24 @@ __global__ void __launch_bounds__(128) head_mix_kernel(const HeadMixParams p) {
       if (h0 + h >= per) break;
       const int head = c * per + h0 + h;
       const float s = p.gate ? 1.f / (1.f + expf(-to_f(reinterpret_cast<const E*>(p.gate)[t * p.gate_tok + head]))) : 1.f;
-      E* o = reinterpret_cast<E*>(p.out) + t * p.out_tok + (size_t)head * p.Dv + col % p.Dv;
-      from_f(o[0], acc[h][i][0] * s), from_f(o[1], acc[h][i][1] * s);
+      const float4 v = acc[i][h];
+      store_row4(reinterpret_cast<E*>(p.out) + t * p.out_tok + (size_t)head * p.Dv + col % p.Dv, make_float4(v.x * s, v.y * s, v.z * s, v.w * s));
     }
   }
+}
+
+template <typename E>
+int launch_head_mix(const HeadMixParams& p, cudaStream_t s) {
+  const int per = p.H / p.G;
+  const unsigned x = (p.G * p.Dv / 4 + 127) / 128;
+  auto go = [&](auto one, auto two, int hm) {
+    const unsigned z = (per + hm - 1) / hm;
+    return p.T < 512 ? launch_kernel(one, dim3(x, p.T, z), dim3(128), 0, s, p) : launch_kernel(two, dim3(x, (p.T + 1) / 2, z), dim3(128), 0, s, p);
+  };
+  if (per <= 1) return go(head_mix_kernel<E, 1, 1>, head_mix_kernel<E, 2, 1>, 1);
+  if (per <= 2) return go(head_mix_kernel<E, 1, 2>, head_mix_kernel<E, 2, 2>, 2);
+  if (per <= 4) return go(head_mix_kernel<E, 1, 4>, head_mix_kernel<E, 2, 4>, 4);
+  return go(head_mix_kernel<E, 1, 8>, head_mix_kernel<E, 2, 8>, 8);
 }
 
 __device__ __forceinline__ float gated_act(float g, bool gelu, bool exact) {
@@ -925,20 +940,15 @@ int swb_row_rope_kv_write(void* buf, int ld, int v_col, int H, int G, int D, int
   return fp32 ? launch_kernel(row_rope_kv_kernel<float>, grid, block, smem, s, p) : launch_kernel(row_rope_kv_kernel<bf16>, grid, block, smem, s, p);
 }
 
-// See HeadMixParams. Dv and the strides even, rows 8-byte aligned; talk 16-byte aligned.
+// See HeadMixParams. Dv and the strides multiples of 4, rows 8-byte (fp32: 16-byte) aligned.
 int swb_head_mix(const void* a, long long a_tok, const float* talk, const void* gate, long long gate_tok, void* out, long long out_tok, int T,
                  int H, int G, int Dv, int fp32, void* stream) {
   using namespace swb;
   if (T <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || Dv < 2 || ((Dv | a_tok | out_tok) % 2) || !talk) return -3;
+  if (H < 1 || G < 1 || H % G || Dv < 4 || ((Dv | a_tok | out_tok) % 4) || !talk) return -3;
   const HeadMixParams p{a, a_tok, talk, gate, gate_tok, out, out_tok, T, H, G, Dv};
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const unsigned x = (G * Dv / 2 + 127) / 128, z = (H / G + HM - 1) / HM;
-  if (T < 512)
-    return fp32 ? launch_kernel(head_mix_kernel<float, 1>, dim3(x, T, z), dim3(128), 0, s, p)
-                : launch_kernel(head_mix_kernel<bf16, 1>, dim3(x, T, z), dim3(128), 0, s, p);
-  return fp32 ? launch_kernel(head_mix_kernel<float, 4>, dim3(x, (T + 3) / 4, z), dim3(128), 0, s, p)
-              : launch_kernel(head_mix_kernel<bf16, 4>, dim3(x, (T + 3) / 4, z), dim3(128), 0, s, p);
+  return fp32 ? launch_head_mix<float>(p, s) : launch_head_mix<bf16>(p, s);
 }
 
 int swb_diff_combine(const void* in, long long in_tok, void* out, long long out_tok, int T, int H, int Dv, int N, float lambda, float eps,

@@ -17,7 +17,7 @@ mixer's two results, the weighted expert rows, the join of all streams, what the
 brings one token, its convolution, whose window is part of a sequence's state slot; prompts run the convolution as one more kernel. All
 projections of a mixer's input are one GEMM. Exchanged weights are never formed: a head's mixed weights applied to its values equal
 sum_g talk[h, g] (weights of head g applied to the values of h's group), so the attention kernels apply every head's weights to all value
-heads (cached side by side, up to 128 columns to a tile) and `ops.head_mix` combines and gates. Rotations pair i with i + dims / 2 in the
+heads (cached side by side, up to 128 columns to a tile) and their results are mixed and gated behind it (`ops.exchange_attention`). Rotations pair i with i + dims / 2 in the
 checkpoint; the weights' rows are reordered at load time so that partners are neighbours; the unit norms stand in front of the rotation,
 which does not change a head's length."""
 from __future__ import annotations
@@ -155,8 +155,13 @@ class NafelixGpu(StackDecoder):
         """KV splits per layer: a window (plus the rest of its first tile) is all that a layer reads."""
         def splits(m) -> int:
             a, par = (m.left, True) if isinstance(m, ParallelSpec) else (m, False)
-            per_seq = a.kv_heads * (self._value_heads(a, True)[0] if par else 1)
-            return splits_for(batch, per_seq, min(max_kv, a.window + 63) if a.window else max_kv)
+            keys, (nv, dv) = min(max_kv, a.window + 63) if a.window else max_kv, self._value_heads(a, par)
+            if par and self.dtype == torch.bfloat16 and ops.exchange_decode_fits(a.heads, a.kv_heads, up8(a.dim), nv, dv):
+                want, s = min(148 // batch, keys // 32, 32), 1       # one CTA per SM, two pages each at least
+                while s * 2 <= want:
+                    s *= 2
+                return s
+            return splits_for(batch, a.kv_heads * (nv if par else 1), keys)
         return tuple(splits(lay.mixer) for lay in self.stack.layers)
 
     @staticmethod
@@ -284,14 +289,13 @@ class NafelixGpu(StackDecoder):
         if inp.fresh_prefill and inp.cu_q is not None:
             fresh = (proj[:, nq:nq + nk].view(T, m.kv_heads, a.dk), proj[:, nq + nk:nq + nk + nv].view(T, a.value_heads, a.dv))
         self.launches += 2
-        mixed = a.talk is not None
-        out = ops.chunk_attention(proj[:, :nq].view(T, m.heads, a.dk), kc, vc, inp.block_table, inp.kv_lens, cu_q=inp.cu_q,
-                                  max_q_len=inp.max_q_len, scale=m.scale, window=m.window, sink=a.sink, decode=inp.decode, num_splits=splits,
-                                  fresh_kv=fresh, all_values=mixed, gate=None if mixed else gate)
-        if not mixed:
-            return out
+        kw = dict(cu_q=inp.cu_q, max_q_len=inp.max_q_len, scale=m.scale, window=m.window, sink=a.sink, gate=gate, decode=inp.decode,
+                  num_splits=splits, fresh_kv=fresh)
+        q = proj[:, :nq].view(T, m.heads, a.dk)
+        if a.talk is None:
+            return ops.chunk_attention(q, kc, vc, inp.block_table, inp.kv_lens, **kw)
         self.launches += 1
-        return ops.head_mix(out.view(T, m.heads, m.kv_heads, -1), a.talk, gate=gate)
+        return ops.exchange_attention(q, kc, vc, inp.block_table, inp.kv_lens, talk=a.talk, **kw)
 
     def _mixer(self, lay: _Layer, h: torch.Tensor, inp: StepInputs, kv: list, place: tuple[int, ...], splits: int) -> HyperBranch:
         a, m = lay.attention, lay.attention.spec

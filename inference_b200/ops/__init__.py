@@ -1,6 +1,6 @@
 """Python wrappers over the sm_100a kernel library (tensors in, tensors out, current CUDA stream)."""
-from .attention import (Differential, chunk_attention, dense_attention, dense_attention_padded, narrow_heads_on_kernel, paged_attention,  # noqa: F401
-                        varlen_causal_attention)
+from .attention import (Differential, chunk_attention, dense_attention, dense_attention_padded, exchange_attention, exchange_decode_fits,  # noqa: F401
+                        narrow_heads_on_kernel, paged_attention, varlen_causal_attention)
 from .gemm import SSQ_WORDS, ssq_buffer, ssq_values, gemm_bf16, gemm_bf16_grouped, gemm_bf16_normed, gemm_f32, gated_fused, gemm_workspace, linear, linear_gated  # noqa: F401
 from .llm import (argmax, sample_device, embedding, gated_act_mul, gated_residual, layernorm_mod, poly_norm, rmsnorm, rope_kv_write, row_rope_kv_write, diff_combine, head_mix, head_mix_weights,  # noqa: F401
                   spec_verify_greedy)

@@ -218,3 +218,50 @@ def chunk_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
 
         diff_combine(res, out, diff.share, diff.eps, diff.post, diff.width)
     return out
+
+
+def exchange_decode_fits(heads: int, kv_heads: int, dim: int, value_heads: int, v_dim: int, q_len: int = 1) -> bool:
+    """Whether decoding with exchanged weights runs on the kernel that takes all heads of a sequence in one CTA (the limits of
+    csrc/kernels/attention_exchange.cu): rows and value columns within its accumulators, two pages in shared memory."""
+    rows, cols = heads * q_len, value_heads * v_dim
+    page = 2048 * ((dim + 63) // 64 * kv_heads + (v_dim + 63) // 64 * value_heads)
+    fixed = (rows * ((dim + 15) // 16 * 32 + 16) + 15) // 16 * 16 + 2 * 64 * 52 + 1280
+    return (rows <= 64 and max(dim, v_dim) <= 128 and dim % 8 == 0 and v_dim % 8 == 0 and max(kv_heads, value_heads) <= 16
+            and cols <= (1024 if rows <= 16 else 512 if rows <= 32 else 256) and fixed + 2 * page <= 227 * 1024)
+
+
+def exchange_attention(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor, kv_lens: torch.Tensor, *,
+                       cu_q: torch.Tensor | None, max_q_len: int, scale: float, talk: torch.Tensor, sink: torch.Tensor | None = None,
+                       gate: torch.Tensor | None = None, window: int = 0, decode: bool = False, num_splits: int = 1,
+                       fresh_kv: tuple[torch.Tensor, torch.Tensor] | None = None, kernel: str = "auto") -> torch.Tensor:
+    """Attention whose heads exchange their weights: head h applies sum_g talk[h, g] (weights of head g) to the values of its own key/value
+    head and is scaled by the sigmoid of gate [T, Hq] logits. talk from `head_mix_weights`; vcache [blocks, NV, block_size, Dv] with NV Dv = Hkv
+    times the value width; the rest as in `chunk_attention` -> [T, Hq * width]. bf16 decode steps run on one kernel over all heads and a merge
+    that mixes and gates (`exchange_decode_fits`), everything else on chunk_attention over all values and `head_mix`."""
+    from .llm import head_mix
+
+    T, H, D = q.shape
+    nblk, G, bs, _ = kcache.shape
+    NV, Dv = vcache.shape[1], vcache.shape[3]
+    vp = NV * Dv // G
+    if (decode and cu_q is None and q.dtype == torch.bfloat16 and kernel == "auto" and bs == 16 and scale > 0
+            and exchange_decode_fits(H, G, D, NV, Dv, max_q_len)):
+        require_cuda(q, kcache, vcache, block_table, kv_lens, talk, sink, gate)
+        S = kv_lens.numel()
+        assert T == S * max_q_len and q.stride(2) == 1 and q.stride(1) == D and kcache.is_contiguous() and vcache.is_contiguous()
+        assert vcache.shape[0] == nblk and kcache.dtype == vcache.dtype == q.dtype and block_table.dtype == kv_lens.dtype == torch.int32
+        assert talk.shape[:2] == (H, G) and talk.dtype == torch.float32 and talk.is_contiguous() and block_table.stride(1) == 1
+        assert sink is None or (sink.dtype == torch.float32 and sink.numel() == H)
+        assert gate is None or (gate.shape == (T, H) and gate.stride(1) == 1 and gate.dtype == q.dtype)
+        n = max(1, min(32, num_splits))
+        ws = torch.empty(kernels().swb_exchange_workspace_bytes(S, H, max_q_len, NV * Dv, n), dtype=torch.uint8, device=q.device)
+        out = torch.empty((T, H * vp), dtype=q.dtype, device=q.device)
+        rc = kernels().swb_exchange_decode(q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), out.data_ptr(), out.stride(0),
+                                           block_table.data_ptr(), block_table.stride(0), nblk, kv_lens.data_ptr(), S, max_q_len, H, G, D, NV, Dv,
+                                           vp, scale, window, ptr(sink), talk.data_ptr(), ptr(gate), gate.stride(0) if gate is not None else 0, n,
+                                           ws.data_ptr(), ws.numel(), stream_ptr())
+        check(rc, "swb_exchange_decode")
+        return out
+    a = chunk_attention(q, kcache, vcache, block_table, kv_lens, cu_q=cu_q, max_q_len=max_q_len, scale=scale, window=window, sink=sink,
+                        decode=decode, num_splits=num_splits, fresh_kv=fresh_kv, kernel=kernel, all_values=True)
+    return head_mix(a.view(T, H, G, vp), talk, gate=gate)

@@ -227,6 +227,14 @@ def _attention_case(dtype, shape, lens, q_lens, how, window, *, mixed, splits=1,
         g = gate.to(dtype).cuda() if mixed else pad(gate.view(T, H, E), vp).reshape(T, -1).to(dtype).cuda()
         g = torch.nn.functional.pad(g, (0, 16))[:, :g.shape[1]]             # strided rows
     cols = H * G * vp if mixed else H * vp
+    if how == "exchange":                                                     # one kernel over all heads, and the merge
+        assert ops.exchange_decode_fits(H, G, dp, G // n, n * vp, max(q_lens)) and uniform
+        got = ops.exchange_attention(q, kc, vc, table, i32(lens), cu_q=None, max_q_len=max(q_lens), scale=scale, talk=ops.head_mix_weights(talk.cuda(), G),
+                                     sink=sink.cuda(), gate=g, window=window, decode=True, num_splits=splits)
+        ops.check_status()
+        got = got.view(T, H, vp)
+        assert (got[..., E:] == 0).all()
+        return rel(got[..., :E], want)
     out = torch.full((T, cols + 8), 3.0, dtype=dtype, device="cuda")
     ops.chunk_attention(q, kc, vc, table, i32(lens), cu_q=None if uniform else i32([0] + q_lens).cumsum(0).int(), max_q_len=max(q_lens), scale=scale,
                         window=window, sink=sink.cuda(), decode=how == "decode", num_splits=splits, fresh_kv=fresh, out=out[:, :cols],
@@ -266,6 +274,47 @@ def test_keys_at_the_edge_of_a_window(window, gap, how, mixed):
     q_lens = lens if how == "fresh" else [40, 1, 17] if how == "context" else [1, 2, 1]
     for dtype in DTYPES if how == "simple" else DTYPES[1:]:
         assert _attention_case(dtype, (4, 2, 48, 40), lens, q_lens, how, window, mixed=mixed, splits=3, plant=window - 1 + gap) < 1.5 * OP_TOL[dtype]
+
+
+EXCHANGE = SHAPES + [(1, 1, 8, 4), (8, 8, 128, 64), (16, 16, 24, 24), (32, 4, 64, 64), (64, 8, 32, 32), (32, 8, 128, 64), (16, 1, 128, 128)]
+
+
+@pytest.mark.parametrize("shape", EXCHANGE)
+@pytest.mark.parametrize("window", [0, 1, 2, 17, 129])
+def test_exchange_decode(shape, window):
+    """All heads of a sequence in one CTA: head counts from one to sixty-four, odd groups, several query tokens, any number of splits."""
+    lens = [401, 1, 130, 257, 37, 16]
+    for splits in (1, 2, 7, 32):
+        assert _attention_case(torch.bfloat16, shape, lens, [1] * 6, "exchange", window, mixed=True, splits=splits, uniform=True) < 1.5 * OP_TOL[torch.bfloat16]
+    if shape[0] * 3 <= 16:
+        for splits in (1, 5):
+            assert _attention_case(torch.bfloat16, shape, [401, 3, 130], [3] * 3, "exchange", window, mixed=True, splits=splits, uniform=True) < 1.5 * OP_TOL[torch.bfloat16]
+
+
+@pytest.mark.parametrize("window", [1, 15, 16, 17, 40, 64, 128, 200])
+@pytest.mark.parametrize("gap", [-1, 0, 1])
+def test_exchange_decode_at_the_edge_of_a_window(window, gap):
+    for q in (1, 2):
+        assert _attention_case(torch.bfloat16, (4, 2, 48, 40), [385, 130, 64], [q] * 3, "exchange", window, mixed=True, splits=3, plant=window - 1 + gap,
+                               uniform=True) < 1.5 * OP_TOL[torch.bfloat16]
+    for mean in (8.0, -30.0):
+        assert _attention_case(torch.bfloat16, (8, 4, 32, 64), [300, 70], [2, 2], "exchange", window, mixed=True, splits=4, uniform=True,
+                               sink_mean=mean, with_gate=gap > 0) < 2 * OP_TOL[torch.bfloat16]
+
+
+def test_exchange_decode_limits_agree():
+    from inference_b200 import ops
+    from inference_b200._native import kernels
+
+    g = torch.Generator().manual_seed(0)
+    yes = 0
+    for _ in range(3000):
+        G, D, NV, Dv, q = (int(torch.randint(1, n, (1,), generator=g)) for n in (18, 18, 18, 18, 4))
+        H = G * int(torch.randint(1, 9, (1,), generator=g))
+        fits = ops.exchange_decode_fits(H, G, D * 8, NV, Dv * 8, q)
+        assert fits == (kernels().swb_exchange_decode_stages(H, G, D * 8, NV, Dv * 8, q) > 0)
+        yes += fits
+    assert 100 < yes < 2900
 
 
 @pytest.mark.parametrize("mixed", [True, False])
