@@ -217,6 +217,14 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
 #pragma unroll
       for (int hr = 0; hr < 2; ++hr) row_scale[hr] *= p.diff.q_temp[min((g + hr * 8) / p.G, q_len - 1) + max(causal_shift, 0)];
     }
+    int first_key[2], last_key[2];         // visible keys of this lane's two rows
+#pragma unroll
+    for (int hr = 0; hr < 2; ++hr) {
+      const int qpos = (g + hr * 8) / p.G + causal_shift;
+      first_key[hr] = EXT && p.chunk > 0 ? qpos / p.chunk * p.chunk : 0;
+      if (EXT && p.window > 0) first_key[hr] = max(first_key[hr], qpos - p.window + 1);
+      last_key[hr] = p.causal ? min(kv_len - 1, qpos) : kv_len - 1;
+    }
     float row_cap[2] = {0.f, 0.f};         // 2 log2(e) scale / cap
     if (DIFF && p.diff.cap > 0.f) row_cap[0] = 2.8853900818f * row_scale[0] / p.diff.cap, row_cap[1] = 2.8853900818f * row_scale[1] / p.diff.cap;
     for (int j = 0; j < n_tiles; ++j) {
@@ -243,11 +251,7 @@ __global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(
         for (int e = 0; e < 4; ++e) {
           const float val = DIFF ? capped_score(s[nt][e], row_scale[e >> 1], row_cap[e >> 1], p.diff.cap) : score_transform(s[nt][e], p.scale, p.softcap);
           const int col = tok_base + nt * 8 + t4 * 2 + (e & 1);
-          const int row = g + ((e >> 1) ? 8 : 0);
-          const int qtok = row / p.G;
-          const int qpos = qtok + causal_shift;
-          const bool ok = (col < kv_len) && (!p.causal || col <= qpos) &&
-                          (!EXT || ((p.chunk <= 0 || col >= qpos / p.chunk * p.chunk) && (p.window <= 0 || col > qpos - p.window)));
+          const bool ok = col <= last_key[e >> 1] && (!EXT || col >= first_key[e >> 1]);
           s[nt][e] = ok ? val : -INFINITY;
         }
       }

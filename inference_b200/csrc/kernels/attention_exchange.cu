@@ -6,7 +6,8 @@
 // the eight compute warps first deal out tiles of eight query rows of one key head, S^T = K Q^T (16 keys by 8 rows) with the online softmax
 // along the fragment, and leave the weights and the rows' rescale factors in shared memory (two buffers, so one barrier per page); then each
 // warp takes an eighth of the value columns for all rows, O += P V. Per split the un-normalised O and (max, sum) go to the workspace.
-// exchange_merge_kernel: merges the splits, joins the sink, mixes the heads and applies the gates, one CTA per token and 128 columns.
+// exchange_merge_kernel: merges the splits, joins the sink, mixes the heads and applies the gates, one CTA per token and 128 columns (32 with
+// few tokens).
 #include "attention_common.cuh"
 #include "gemm_tcgen05.cuh"
 
@@ -273,45 +274,39 @@ struct MergeParams {
   int q_len, H, G, vp, num_splits;
 };
 
-constexpr int MERGE_SLICES = 4, MERGE_HEADS = 8;
+constexpr int MERGE_HEADS = 8, MERGE_THREADS = 256;
 
-// 64 column pairs by 4 slices of the query heads; blockIdx.z: which MERGE_HEADS of each group.
-__global__ void __launch_bounds__(64 * MERGE_SLICES) exchange_merge_kernel(const MergeParams p) {
+// PAIRS column pairs by MERGE_THREADS / PAIRS slices of the query heads; blockIdx.z: which MERGE_HEADS of each group.
+template <int PAIRS>
+__global__ void __launch_bounds__(MERGE_THREADS) exchange_merge_kernel(const MergeParams p) {
+  constexpr int SLICES = MERGE_THREADS / PAIRS;
   pdl_launch_dependents();
   pdl_wait(TL_ATTN_MERGE);
   __shared__ float weight[MAX_SPLITS * MAX_ROWS];             // [split][head]
-  __shared__ float sums[MERGE_SLICES][2 * MERGE_HEADS][64 + 1];
+  __shared__ float sums[SLICES][2 * MERGE_HEADS][PAIRS + 1];
   const int t = blockIdx.y, seq = t / p.q_len, qtok = t % p.q_len, per = p.H / p.G, rows = p.H * p.q_len, cols = p.G * p.vp;
   const int S = p.num_splits, h0 = blockIdx.z * MERGE_HEADS, hp = (per + MERGE_HEADS - 1) / MERGE_HEADS * MERGE_HEADS;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   auto row_of = [&](int h) { return h / per * per * p.q_len + qtok * per + h % per; };
   const size_t base = (size_t)seq * S * rows;
-  for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
+  for (int h = warp; h < p.H; h += MERGE_THREADS / 32) {      // a lane per split
     const float sink = p.sink ? p.sink[h] * 1.4426950408889634f : -INFINITY;
-    const float2* ml = p.part_ml + base + row_of(h);
-    float top = sink, den = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < S; ++s) top = fmaxf(top, __ldcg(ml + (size_t)s * rows).x);
-    for (int s = 0; s < S; ++s) {
-      const float2 x = __ldcg(ml + (size_t)s * rows);
-      const float e = x.x == -INFINITY ? 0.f : exp2f(x.x - top);
-      weight[s * p.H + h] = e;
-      den += e * x.y;
-    }
-    if (p.sink) den += exp2f(sink - top);
-    const float inv = den > 0.f ? 1.f / den : 0.f;
-    for (int s = 0; s < S; ++s) weight[s * p.H + h] *= inv;
+    const float2 ml = lane < S ? __ldcg(p.part_ml + base + (size_t)lane * rows + row_of(h)) : make_float2(-INFINITY, 0.f);
+    const float top = fmaxf(warp_max(ml.x), sink), e = ml.x == -INFINITY ? 0.f : exp2f(ml.x - top);
+    const float den = warp_sum(e * ml.y) + (p.sink ? exp2f(sink - top) : 0.f);
+    if (lane < S) weight[lane * p.H + h] = den > 0.f ? e / den : 0.f;
   }
   __syncthreads();
-  const int pair = threadIdx.x & 63, slice = threadIdx.x >> 6, col = blockIdx.x * 128 + pair * 2;
+  const int pair = threadIdx.x % PAIRS, slice = threadIdx.x / PAIRS, col = (blockIdx.x * PAIRS + pair) * 2;
   float acc[MERGE_HEADS][2] = {};
   if (col < cols) {
     const int c = col / p.vp;
     const float* talk = p.talk + (size_t)c * hp + h0;
 #pragma unroll 4
-    for (int h = slice; h < p.H; h += MERGE_SLICES) {
+    for (int h = slice; h < p.H; h += SLICES) {
       const float* o = p.part_o + (base + row_of(h)) * cols + col;
       float x = 0.f, y = 0.f;
-#pragma unroll 4
+#pragma unroll 8
       for (int s = 0; s < S; ++s) {
         const float2 v = __ldcg(reinterpret_cast<const float2*>(o + (size_t)s * rows * cols));
         const float w = weight[s * p.H + h];
@@ -326,12 +321,12 @@ __global__ void __launch_bounds__(64 * MERGE_SLICES) exchange_merge_kernel(const
 #pragma unroll
   for (int i = 0; i < MERGE_HEADS; ++i) sums[slice][2 * i][pair] = acc[i][0], sums[slice][2 * i + 1][pair] = acc[i][1];
   __syncthreads();
-  for (int i = threadIdx.x; i < MERGE_HEADS * 128; i += blockDim.x) {
-    const int head = i / 128, cc = i % 128, at = blockIdx.x * 128 + cc;
+  for (int i = threadIdx.x; i < MERGE_HEADS * PAIRS * 2; i += MERGE_THREADS) {
+    const int head = i / (PAIRS * 2), cc = i % (PAIRS * 2), at = blockIdx.x * PAIRS * 2 + cc;
     if (h0 + head >= per || at >= cols) continue;
     float x = 0.f;
 #pragma unroll
-    for (int s = 0; s < MERGE_SLICES; ++s) x += sums[s][2 * head + (cc & 1)][cc >> 1];
+    for (int s = 0; s < SLICES; ++s) x += sums[s][2 * head + (cc & 1)][cc >> 1];
     const int h = at / p.vp * per + h0 + head;
     if (p.gate) x /= 1.f + __expf(-__bfloat162float(p.gate[t * p.gate_stride + h]));
     p.out[t * p.out_stride + (size_t)h * p.vp + at % p.vp] = __float2bfloat16(x);
@@ -402,9 +397,10 @@ int swb_exchange_decode(const void* q, long long q_stride_tok, const void* kcach
   if (rc) return rc;
   const MergeParams m{part_o, part_ml, sink, talk, reinterpret_cast<const bf16*>(gate), gate_stride, reinterpret_cast<bf16*>(out), out_stride, q_len,
                       H, G, vp, num_splits};
-  const int per = H / G;
-  return launch_kernel(exchange_merge_kernel, dim3((cols + 127) / 128, num_seqs * q_len, (per + MERGE_HEADS - 1) / MERGE_HEADS),
-                       dim3(64 * MERGE_SLICES), 0, st, m);
+  const int tokens = num_seqs * q_len, z = (H / G + MERGE_HEADS - 1) / MERGE_HEADS;
+  if ((cols + 127) / 128 * tokens >= 148)
+    return launch_kernel(exchange_merge_kernel<64>, dim3((cols + 127) / 128, tokens, z), dim3(MERGE_THREADS), 0, st, m);
+  return launch_kernel(exchange_merge_kernel<16>, dim3((cols + 31) / 32, tokens, z), dim3(MERGE_THREADS), 0, st, m);
 }
 
 }  // extern "C"

@@ -612,10 +612,22 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
       }
       __syncwarp();
       const int row0 = q_base + q * TILE_STEP + (warp & 3) * 32;
-#pragma unroll 4
+      constexpr int AHEAD = 8;                                           // gates requested together
+      uint4 gates[AHEAD];
+#pragma unroll 8
       for (int it = 0; it < (DIFF && q ? 0 : CHUNKS); ++it) {            // CHUNKS lanes write one row: 32 / CHUNKS rows per pass
         const int r = (32 / CHUNKS) * it + lane / CHUNKS, ch = lane % CHUNKS;
         const int grow = row0 + r;
+        if constexpr (WIDE) {
+          if (p.out_gate && it % AHEAD == 0) {
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a) {
+              const int g2 = min(grow + (32 / CHUNKS) * a, q_len - 1);
+              gates[a] = __ldg(reinterpret_cast<const uint4*>(p.out_gate + (tok0 + g2) * p.out_gate_stride + (long long)blockIdx.y * p.v_dim +
+                                                              min(ch * 8, p.v_dim - 8)));
+            }
+          }
+        }
         if (grow < q_len) {
           uint4 val = *reinterpret_cast<const uint4*>(slab + r * ROW_BYTES + ((ch ^ (r & 7)) << 4));
           if (EXT && ch * 8 >= p.v_dim) continue;
@@ -624,7 +636,7 @@ attn_dense_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gr
             if (p.out_gate) {
               float x[8], z[8];
               load_row8(reinterpret_cast<const bf16*>(&val), x);
-              load_row8(p.out_gate + (tok0 + grow) * p.out_gate_stride + col + ch * 8, z);
+              load_row8(reinterpret_cast<const bf16*>(&gates[it % AHEAD]), z);
 #pragma unroll
               for (int i = 0; i < 8; ++i) x[i] *= rcp_approx(1.f + ex2(-1.4426950408889634f * z[i]));
               store_row8(reinterpret_cast<bf16*>(&val), x);

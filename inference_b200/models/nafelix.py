@@ -157,7 +157,7 @@ class NafelixGpu(StackDecoder):
             a, par = (m.left, True) if isinstance(m, ParallelSpec) else (m, False)
             keys, (nv, dv) = min(max_kv, a.window + 63) if a.window else max_kv, self._value_heads(a, par)
             if par and self.dtype == torch.bfloat16 and ops.exchange_decode_fits(a.heads, a.kv_heads, up8(a.dim), nv, dv):
-                want, s = min(148 // batch, keys // 32, 32), 1       # one CTA per SM, two pages each at least
+                want, s = min(148 // batch, keys // 64, 32), 1       # one CTA per SM, four pages each at least
                 while s * 2 <= want:
                     s *= 2
                 return s

@@ -246,10 +246,10 @@ def test_splits_follow_the_windows():
 
     m = gpu_model(_cfg("d"), device=torch.device("cpu"))
     long, short = m.decode_splits(1, 100000), m.decode_splits(1, 1)
-    assert long == m.decode_splits(1, 300) == (8, 2, 4) and short == (1, 1, 1)      # 263, 192 and 192 keys, two pages or one tile of 64 at least
+    assert long == m.decode_splits(1, 300) == (4, 2, 2) and short == (1, 1, 1)      # 263, 192 and 192 keys, 64 or 128 to a split at least
     assert m.decode_splits(500, 5000) == (1, 1, 1)
     plain = gpu_model(_cfg("d"), device=torch.device("cpu"), dtype=torch.float32)          # on the kernels with tiles of 64 keys
-    assert plain.decode_splits(1, 100000) == (4, 2, 2)
+    assert plain.decode_splits(1, 100000) == (4, 2, 2) and plain.decode_splits(64, 100000) != m.decode_splits(64, 100000)
 
 
 def test_exchange_behind_the_values():
