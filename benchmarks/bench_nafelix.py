@@ -4,7 +4,7 @@ Two parts, one JSON line per row:
   model   prefill and decode tokens/s through the model runner (random weights) at equal width, layers, heads, vocabulary and feed-forward
           parameters: routed layers beside Rotalorn's (grouped attention in a window, routed experts) and Qwen2-MoE layers, dense ones beside
           Gunedra's delta-rule layers and dense Llama. Nafelix stacks alternate both mixers; a stack of each alone is timed as well. Windows
-          are as long as the context, so that all read the same keys. Three streams, a convolution of three taps per sublayer.
+          are as long as the context, so that all read the same keys. Four streams, a convolution of four taps per sublayer.
   kernel  every kernel of a Nafelix layer beside its counterpart in the designs it shares the mechanism with: time, algorithmic bytes or
           FLOPs, and the fraction of the measured peak that is reached (MEASURED_PEAKS.json: copy bandwidth, bf16 GEMM; the delta rule in
           prompts against 128 fp32 lanes per SM at the maximum clock).
@@ -25,7 +25,7 @@ SIZES = {  # width, layers, heads, kv_heads, (experts, top, expert ff) or None, 
     "w2048_64x8": (2048, 12, 16, 4, (64, 8, 1024), 0, 32768),
     "w4096_dense": (4096, 6, 32, 8, None, 11264, 32768),
 }
-WINDOW, STREAMS, TAPS = 2048, 3, 3
+WINDOW, STREAMS, TAPS = 2048, 4, 4
 
 
 def nafelix_config(size, pattern="PA"):

@@ -24,9 +24,6 @@ namespace {
 #ifndef SWB_DEC_STAGES
 #define SWB_DEC_STAGES 3
 #endif
-#ifndef SWB_DEC_MIN_CTAS
-#define SWB_DEC_MIN_CTAS 1
-#endif
 constexpr int STAGES = SWB_DEC_STAGES;
 constexpr int STAGE_BYTES = 2 * TILE_BYTES;  // K tile + V tile = 32 KB
 constexpr int Q_BYTES = 16 * 256;            // 4 KB
@@ -75,11 +72,13 @@ __device__ __forceinline__ void sum_over_128(float* v, float* red, int n) {
     if (i < n) v[i] = (red[i * 4] + red[i * 4 + 1]) + (red[i * 4 + 2] + red[i * 4 + 3]);
 }
 
-// EXT: chunked and windowed masking, sinks, output gates, values of every head (blockIdx.y then runs over key head, value head). FULL: q / k and v are HD wide (their loop bounds are then constants). DIFF: the two maps
-// of a head are neighbouring query rows, each zero outside its own columns of the key row, so that both maps' scores come from one
-// product; the merge subtracts the second map and norms the difference.
+// EXT: chunked and windowed masking, sinks, output gates, values of every head (blockIdx.y then runs over key head, value head). FULL: q / k
+// and v are HD wide (their loop bounds are then constants). DIFF: the two maps of a head are neighbouring query rows, each zero outside its
+// own columns of the key row, so that both maps' scores come from one product; the merge subtracts the second map and norms the difference.
+// Two CTAs per SM put three warps on a scheduler's quarter of the registers, which leaves 168 for a thread: a bound of 192 threads asks the
+// compiler for that (160 are launched).
 template <bool EXT, bool FULL, bool DIFF>
-__global__ void __launch_bounds__(160, SWB_DEC_MIN_CTAS) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
+__global__ void __launch_bounds__(192, 2) attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                               const __grid_constant__ CUtensorMap tmap_v,
                                                               const AttnParams p) {
   pdl_launch_dependents();

@@ -37,7 +37,7 @@ def up8(n):
 
 # ---- streams -----------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("S,H,Hp", [(1, 90, 96), (2, 144, 144), (3, 256, 256), (4, 1030, 1032), (5, 600, 600), (8, 2048, 2048), (3, 4096, 4096),
+@pytest.mark.parametrize("S,H,Hp", [(1, 90, 96), (2, 144, 144), (3, 264, 264), (4, 1030, 1032), (5, 600, 600), (8, 2048, 2048), (3, 4096, 4096),
                                     (16, 520, 520), (2, 8200, 8200), (4, 3000, 3000)])
 def test_streams_are_read_and_joined(dtype, S, H, Hp):
     """Plain, doubly normed and routed branches; all streams alike at first; in place; chosen rows."""
@@ -249,7 +249,7 @@ def _attention_case(dtype, shape, lens, q_lens, how, window, *, mixed, splits=1,
     return rel(got[..., :E], want)
 
 
-SHAPES = [(8, 2, 64, 32), (6, 3, 40, 24), (4, 1, 128, 128), (16, 4, 72, 64), (12, 4, 32, 96), (3, 3, 10, 7), (24, 2, 16, 8), (5, 1, 64, 72)]
+SHAPES = [(8, 2, 56, 48), (6, 3, 40, 24), (4, 1, 128, 128), (16, 4, 72, 64), (12, 4, 32, 96), (3, 3, 10, 7), (24, 2, 16, 8), (5, 1, 64, 72)]
 
 
 @pytest.mark.parametrize("mixed", [True, False])
@@ -332,7 +332,7 @@ def test_sinks_far_above_and_below_the_scores(how, mixed):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,H,G,Dv", [(1, 1, 1, 8), (5, 6, 3, 24), (600, 8, 2, 32), (7, 40, 2, 64), (513, 24, 24, 8), (3, 32, 4, 128)])
+@pytest.mark.parametrize("T,H,G,Dv", [(1, 1, 1, 8), (5, 6, 3, 24), (600, 10, 2, 40), (7, 40, 2, 64), (513, 24, 24, 8), (3, 32, 4, 128)])
 def test_heads_exchange_weights(dtype, T, H, G, Dv):
     from inference_b200 import ops
 
@@ -345,7 +345,7 @@ def test_heads_exchange_weights(dtype, T, H, G, Dv):
 
 # ---- delta rule ----------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,D,E,taps", [(2, 1, 32, 64, 4), (6, 2, 24, 40, 3), (1, 1, 5, 9, 2), (3, 3, 100, 24, 1), (4, 2, 128, 128, 4), (2, 1, 200, 16, 6),
+@pytest.mark.parametrize("H,G,D,E,taps", [(4, 2, 32, 64, 4), (6, 2, 24, 40, 3), (1, 1, 5, 9, 2), (3, 3, 100, 24, 1), (4, 2, 128, 128, 4), (2, 1, 200, 16, 6),
                                           (2, 2, 300, 8, 4), (8, 4, 64, 136, 4)])
 def test_delta_rule_with_one_decay_per_head(dtype, H, G, D, E, taps):
     """Convolutions, decays, the recurrence, norm and gate over portions of two sequences (single tokens too), against the whole sequence;
